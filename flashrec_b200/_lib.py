@@ -62,6 +62,42 @@ class FrTrie(ctypes.Structure):
     ]
 
 
+class FrOutSegment(ctypes.Structure):
+    """Mirror of ``struct fr_out_segment``."""
+
+    _fields_ = [("kind", ctypes.c_int32), ("n0", ctypes.c_int32), ("n", ctypes.c_int32), ("pad_", ctypes.c_int32),
+                ("out", c_void_p), ("ldo", c_int64), ("row_map", c_void_p), ("bias", c_void_p)]
+
+
+class FrGatedPart(ctypes.Structure):
+    """Mirror of ``struct fr_gated_part``."""
+
+    _fields_ = [("a", c_void_p), ("w", c_void_p), ("gate", c_void_p), ("lda", c_int64), ("ldw", c_int64),
+                ("ldg", c_int64), ("K", ctypes.c_int32), ("pad_", ctypes.c_int32)]
+
+
+class FrConvOut(ctypes.Structure):
+    """Mirror of ``struct fr_conv_out``."""
+
+    _fields_ = [("out", c_void_p), ("ldo", c_int64), ("row_map", c_void_p), ("c0", ctypes.c_int32), ("c", ctypes.c_int32)]
+
+
+class FrMixAttn(ctypes.Structure):
+    """Mirror of ``struct fr_mix_attn``."""
+
+    _fields_ = ([(n, ctypes.c_int32) for n in ("dtype", "mix", "mask", "mask_size", "keep_first", "heads", "kv_heads",
+                                               "dim", "vdim", "vdim_true")]
+                + [(n, c_float) for n in ("scale", "lambda_", "eps", "out_scale")]
+                + [("coef", c_void_p), ("slopes", c_void_p), ("q", c_void_p), ("ldq", c_int64), ("k", c_void_p),
+                   ("v", c_void_p), ("ldk", c_int64), ("ldv", c_int64), ("out", c_void_p), ("ldo", c_int64),
+                   ("req_to_token", c_void_p), ("table_stride", c_int64), ("req_rows", c_void_p),
+                   ("tok_req", c_void_p), ("pos", c_void_p), ("num_slots", c_int64)])
+
+
+FR_SEG_STORE, FR_SEG_SWIGLU, FR_SEG_SIGMOID, FR_SEG_STORE_F32 = 0, 1, 2, 3
+FR_MIX_DIFF, FR_MIX_TALK = 0, 1
+FR_MASK_WINDOW, FR_MASK_CHUNK = 0, 1
+
 FR_TRIE_NONE, FR_TRIE_DENSE, FR_TRIE_CSR, FR_TRIE_BITMAP = 0, 1, 2, 3
 
 P = c_void_p
@@ -118,14 +154,34 @@ _SIGNATURES = {
     "fr_sid_head_topk_workspace_bytes": [_I, _I, _I, _I],
     "fr_sid_head_topk": [P] * 6 + [P, P, _L, P, P, _L, _I] + [P] * 8 + [_L] * 3 + [_I] * 8 + [P, P, P, _L, _I, P],
     "fr_topk_merge_shards": [P] * 16 + [_L] * 2 + [_I] * 7 + [P],
+    "fr_dense_proj": [_I, P, _L, P, _L, _I, _I, _I, P, _I, _I, P],
+    "fr_dense_gated_add": [_I, P, _I, P, _L, _I, _I, P, _I, _I, P],
+    "fr_dense_gated_add_splits": [_I] * 5,
+    "fr_lm_embed": [_I, P, _L, P, P, _L, _I, _I, _I, _F, P, _L, P, P, P, P],
+    "fr_lm_norm": [_I, P, _L, P, _F, _F, P, _I, _L, P, P, _L, _I, _I, P],
+    "fr_short_conv": [_I, P, _L, P, _I, _I, P, _I, P, P, P, P, P, _I, _I, _I, P],
+    "fr_mix_attn_rows": [P, _I, _I, _I, _I, P, _L, P, P],
+    "fr_mix_attn_rows_scratch": [_I] * 6,
+    "fr_mix_attn_tc": [P, P, _I, _I, P],
+    "fr_mix_attn_tc_fits": [_I] * 5,
 }
 _RESTYPES = {"fr_version": c_char_p, "fr_decode_attn_scratch_bytes": c_int64,
              "fr_sid_head_topk_workspace_bytes": c_int64, "fr_joint_select_workspace_bytes": c_int64,
-             "fr_trie_build_workspace_bytes": c_int64}
+             "fr_trie_build_workspace_bytes": c_int64, "fr_mix_attn_rows_scratch": c_int64}
 
 
 def lib_path() -> Path:
     return _LIB_PATH
+
+
+def use_library(path) -> None:
+    """Bind another build of the library (``flashrec_b200.build`` can compile a subset of the sources: the entry
+    points a model family needs). Must come before the first ``load()``; symbols the build lacks stay unbound."""
+    global _LIB_PATH
+    path = Path(path).resolve()
+    if _lib is not None and path != _LIB_PATH:
+        raise RuntimeError("use_library: a library is loaded already")
+    _LIB_PATH = path
 
 
 def load() -> ctypes.CDLL:

@@ -13,6 +13,7 @@ import subprocess
 import sys
 from concurrent.futures import ThreadPoolExecutor
 from pathlib import Path
+from typing import Optional, Sequence
 
 HERE = Path(__file__).resolve().parent
 CSRC = HERE / "csrc"
@@ -39,10 +40,24 @@ def _newest_header() -> float:
     return max(h.stat().st_mtime for h in hs)
 
 
-def build(verbose: bool = False, force: bool = False) -> Path:
+def is_current(lib: Path = LIB) -> bool:
+    """The library exists and no source or header is newer."""
+    srcs = list(CSRC.glob("*.cu"))
+    return lib.exists() and lib.stat().st_mtime >= max([_newest_header()] + [s.stat().st_mtime for s in srcs])
+
+
+def build_subset(name: str, stems: Sequence[str], verbose: bool = False) -> Path:
+    """``libflashrec_b200-<name>.so`` from some of the sources only (the entry points one model family calls), or
+    the complete library when it is up to date already."""
+    if is_current():
+        return LIB
+    return build(verbose=verbose, stems=stems, lib=HERE / f"libflashrec_b200-{name}.so")
+
+
+def build(verbose: bool = False, force: bool = False, stems: Optional[Sequence[str]] = None, lib: Path = LIB) -> Path:
     nvcc = _nvcc()
     OBJ.mkdir(exist_ok=True)
-    srcs = sorted(CSRC.glob("*.cu"))
+    srcs = sorted(CSRC.glob("*.cu")) if stems is None else [CSRC / f"{s}.cu" for s in stems]
     hdr_m = _newest_header()
     jobs = []
     for s in srcs:
@@ -65,13 +80,13 @@ def build(verbose: bool = False, force: bool = False) -> Path:
             if r.returncode != 0:
                 raise RuntimeError(f"nvcc failed on {s.name}")
     objs = [str(OBJ / (s.stem + ".o")) for s in srcs]
-    if jobs or not LIB.exists():
-        cmd = [nvcc, "-shared", "-o", str(LIB), *objs, "-gencode", "arch=compute_100a,code=sm_100a"]
+    if jobs or not lib.exists() or lib.stat().st_mtime < max(Path(o).stat().st_mtime for o in objs):
+        cmd = [nvcc, "-shared", "-o", str(lib), *objs, "-gencode", "arch=compute_100a,code=sm_100a"]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:
             sys.stderr.write(r.stdout + r.stderr)
             raise RuntimeError("link failed")
-    return LIB
+    return lib
 
 
 if __name__ == "__main__":

@@ -20,7 +20,8 @@ class ForwardBatch:
     that callers of this library may leave out what its kernels do not need (``seq_lens_cpu`` is only
     used to size the attention scratch without a device read). Two additions at the end:
     ``qo_indptr`` (int32, device, ``[n_rows + 1]``), the running sum of ``extend_seq_lens`` that the
-    prefill attention reads — derived from ``extend_seq_lens`` when absent.
+    prefill attention reads — derived from ``extend_seq_lens`` when absent; the fields after it are
+    described where they stand.
 
     Prefill (``is_prefill``): ``input_ids`` / ``positions`` / ``out_cache_loc`` hold one entry per
     extend token, ``seq_lens`` / ``kv_indptr`` one per request; ``extend_seq_lens`` and
@@ -40,6 +41,15 @@ class ForwardBatch:
     buffers_ready: bool = False  # decode graph static buffers already filled
     want_expand: bool = False
     qo_indptr: Optional[torch.Tensor] = None
+    # what the layers of ``flashrec_b200.lm_layers`` read besides (the slot table is indexed directly, so these
+    # batches carry no flat slot lists): request of every token and its slot-table row, the tokens whose
+    # attention runs row by row (the first ``n_row_tokens``) and the tensor-core tiles of the rest
+    tok_req: Optional[torch.Tensor] = None  # int32 [T]
+    tok_rows: Optional[torch.Tensor] = None  # int64 [T]
+    n_row_tokens: int = 0
+    tiles: Optional[torch.Tensor] = None  # int32 [n_tiles, 3] = request, first token, tokens
+    one_token: bool = False  # every request has exactly one token
+    max_pos: int = 0  # largest position of the batch (host bound)
 
     @property
     def n_rows(self) -> int:

@@ -1,0 +1,800 @@
+// Attention whose outputs are linear combinations of several softmax maps over the same values
+// (fr_mix_attn in the header): differential attention (two maps per head, weights 1 and -lambda, the result
+// divided by its root mean square) and talking heads (all heads' maps, one matrix row per output head), with
+// a sliding window that keeps the first tokens or with chunks, and an optional linear distance bias.
+//
+// Because the mixture is linear, sum_s coef[o, s] (P_s V) = (sum_s coef[o, s] P_s) V:
+//   * mix_scores_kernel + mix_values_kernel (fr_mix_attn_rows: decode, f32, any head size) write the scores of
+//     every visible key, mix the normalised weights and pass over V once; keys may be split over CTAs;
+//   * mix_tc_kernel (fr_mix_attn_tc: bf16 prompts, tcgen05) runs one flash pass per source map and adds
+//     coef[o, s] / l_s times its result to the outputs' accumulators, which stay in TMEM beside S and O.
+#include "fr_common.cuh"
+#include "sm100_ptx.cuh"
+
+namespace fr {
+
+int* device_status_ptr();  // capi.cu
+int make_tmap_bf16_box64(CUtensorMap* map, const void* ptr, uint64_t cols, uint64_t rows, int64_t pitch,
+                         uint32_t box_rows);  // dense_proj.cu
+
+namespace mix {
+
+constexpr float kLog2e = 1.4426950408889634f;
+
+template <typename T>
+__device__ __forceinline__ void load8(const T* p, float (&v)[8]);
+template <>
+__device__ __forceinline__ void load8<float>(const float* p, float (&v)[8]) {
+  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+  v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+template <>
+__device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, float (&v)[8]) {
+  const uint4 a = *reinterpret_cast<const uint4*>(p);
+  const uint32_t w[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    v[2 * i] = __uint_as_float(w[i] << 16);
+    v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+  }
+}
+template <typename T>
+__device__ __forceinline__ void st_f(T* p, float v) { *p = v; }
+template <>
+__device__ __forceinline__ void st_f<__nv_bfloat16>(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+
+// Visible keys of the query at position i: [0, n_first) and [lo, i].
+struct Visible {
+  int64_t lo;
+  int n_first, n;
+  __device__ __forceinline__ int64_t key(int idx) const { return idx < n_first ? idx : lo + (idx - n_first); }
+};
+__device__ __forceinline__ int64_t lowest_key(const fr_mix_attn& a, int64_t i) {
+  if (a.mask == FR_MASK_CHUNK) return i / a.mask_size * a.mask_size;
+  return i - a.mask_size + 1 > 0 ? i - a.mask_size + 1 : 0;
+}
+__device__ __forceinline__ Visible visible_keys(const fr_mix_attn& a, int64_t i, int max_keys) {
+  Visible v;
+  v.lo = lowest_key(a, i);
+  v.n_first = a.mask == FR_MASK_CHUNK ? 0 : static_cast<int>(a.keep_first < v.lo ? a.keep_first : v.lo);
+  const int64_t n = v.n_first + (i - v.lo + 1);
+  v.n = static_cast<int>(n < max_keys ? n : max_keys);
+  return v;
+}
+__device__ __forceinline__ int64_t slot_of(const fr_mix_attn& a, int64_t table_row, int64_t j) {
+  const int64_t s = a.req_to_token[table_row * a.table_stride + j];
+  return s < 0 ? 0 : (s >= a.num_slots ? a.num_slots - 1 : s);
+}
+// i-th source map that reads k head kh
+__device__ __forceinline__ int source_of(const fr_mix_attn& a, int kh, int i) {
+  const int rep = a.heads / a.kv_heads;
+  return a.mix == FR_MIX_DIFF ? 2 * ((kh >> 1) * rep + i) + (kh & 1) : kh * rep + i;
+}
+
+constexpr int kKeyBlock = 64;
+
+// ---------------------------------------------------------------------------
+// scores of one row, one k head and 64 keys for every source map that reads that k head; per block and map the
+// maximum and the sum of exponentials
+// ---------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(128)
+mix_scores_kernel(const __grid_constant__ fr_mix_attn a, int row0, int max_keys, int n_blocks, float* __restrict__ scores,
+                  float2* __restrict__ stats) {
+  extern __shared__ float sm[];
+  const int rep = a.heads / a.kv_heads;
+  const int n_src = a.mix == FR_MIX_DIFF ? 2 * a.heads : a.heads;
+  float* qs = sm;                       // [rep][dim]
+  float* sc = sm + rep * a.dim;         // [rep][64]
+  ptx::griddep_wait();
+  ptx::griddep_launch_dependents();
+  const int lrow = blockIdx.z, kh = blockIdx.y, blk = blockIdx.x;
+  const int64_t t = row0 + lrow;
+  const int64_t i = a.pos[t];
+  const Visible vis = visible_keys(a, i, max_keys);
+  const int k0 = blk * kKeyBlock;
+  if (k0 >= vis.n) return;
+  const int nk = min(kKeyBlock, vis.n - k0);
+  const T* q = static_cast<const T*>(a.q) + t * a.ldq;
+  for (int e = threadIdx.x; e < rep * (a.dim / 8); e += 128) {
+    const int s = e / (a.dim / 8), c = e % (a.dim / 8) * 8;
+    float v[8];
+    load8<T>(q + static_cast<int64_t>(source_of(a, kh, s)) * a.dim + c, v);
+#pragma unroll
+    for (int x = 0; x < 8; ++x) qs[s * a.dim + c + x] = v[x];
+  }
+  __syncthreads();
+  int lanes = 1;  // lanes per key
+  while (lanes < 32 && lanes * 8 < a.dim) lanes *= 2;
+  const int lane_k = threadIdx.x % lanes;
+  const int64_t table_row = a.req_rows[a.tok_req[t]];
+  const T* kc = static_cast<const T*>(a.k) + static_cast<int64_t>(kh) * a.dim;
+  const int keys_at_once = 128 / lanes;
+  for (int kb = 0; kb < kKeyBlock; kb += keys_at_once) {  // CTA-uniform trip count: shuffles below are whole-warp
+    const int kk = kb + threadIdx.x / lanes;
+    const bool live = kk < nk;
+    const int64_t j = vis.key(k0 + (live ? kk : 0));
+    const T* kr = kc + slot_of(a, table_row, j) * a.ldk;
+    for (int s0 = 0; s0 < rep; s0 += 4) {
+      float acc[4] = {};
+      for (int c = lane_k * 8; c < a.dim; c += lanes * 8) {
+        float v[8];
+        load8<T>(kr + c, v);
+#pragma unroll
+        for (int s = 0; s < 4; ++s)
+          if (s0 + s < rep) {
+#pragma unroll
+            for (int x = 0; x < 8; ++x) acc[s] = fmaf(v[x], qs[(s0 + s) * a.dim + c + x], acc[s]);
+          }
+      }
+#pragma unroll
+      for (int s = 0; s < 4; ++s) {
+        for (int o = lanes / 2; o > 0; o >>= 1) acc[s] += __shfl_xor_sync(0xffffffffu, acc[s], o);
+        if (lane_k == 0 && s0 + s < rep && kk < kKeyBlock) {
+          float v = acc[s] * a.scale;
+          if (a.slopes != nullptr) v -= a.slopes[source_of(a, kh, s0 + s)] * static_cast<float>(i - j);
+          sc[(s0 + s) * kKeyBlock + kk] = live ? v : -INFINITY;
+        }
+      }
+    }
+  }
+  __syncthreads();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int s = warp; s < rep; s += 4) {
+    const int64_t row = static_cast<int64_t>(lrow) * n_src + source_of(a, kh, s);
+    const float v0 = sc[s * kKeyBlock + lane], v1 = sc[s * kKeyBlock + 32 + lane];
+    const float m = warp_max(fmaxf(v0, v1));
+    const float l = warp_sum(expf(v0 - m) + expf(v1 - m));
+    if (k0 + lane < max_keys) scores[row * max_keys + k0 + lane] = v0;
+    if (k0 + 32 + lane < max_keys) scores[row * max_keys + k0 + 32 + lane] = v1;
+    if (lane == 0) stats[row * n_blocks + blk] = make_float2(m, l);
+  }
+}
+
+// ---------------------------------------------------------------------------
+// mixture of the maps and product with V for one row, one kv head and one share of the keys
+// ---------------------------------------------------------------------------
+constexpr int kValThreads = 256;
+constexpr int kOutBlock = 8;  // output heads accumulated per pass over the keys
+
+// Root-mean-square scaling (DIFF) and store of one output head; f [vdim] in shared memory.
+template <typename T>
+__device__ __forceinline__ void finish_head(const fr_mix_attn& a, int64_t t, int head, const float* f, float* red) {
+  float r = 1.0f;
+  if (a.mix == FR_MIX_DIFF) {
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < a.vdim; c += kValThreads) ss += f[c] * f[c];  // padded columns hold zero
+    ss = warp_sum(ss);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    float tot = 0.f;
+    for (int w = 0; w < kValThreads / 32; ++w) tot += red[w];
+    r = a.out_scale / sqrtf(tot / static_cast<float>(a.vdim_true) + a.eps);
+    __syncthreads();
+  }
+  T* out = static_cast<T*>(a.out) + t * a.ldo + static_cast<int64_t>(head) * a.vdim;
+  for (int c = threadIdx.x; c < a.vdim; c += kValThreads) st_f(out + c, f[c] * r);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kValThreads)
+mix_values_kernel(const __grid_constant__ fr_mix_attn a, int row0, int max_keys, int n_blocks, int splits,
+                  const float* __restrict__ scores, const float2* __restrict__ stats, float* __restrict__ partial,
+                  int32_t* __restrict__ counters) {
+  extern __shared__ float sm[];
+  const int rep = a.heads / a.kv_heads;
+  const bool diff = a.mix == FR_MIX_DIFF;
+  const int n_src = diff ? 2 * a.heads : a.heads;   // of the row
+  const int my_src = diff ? 2 * rep : a.heads;      // that this kv head's outputs mix
+  float* s_m = sm;                                  // [my_src]
+  float* s_il = s_m + my_src;                       // [my_src]
+  float* s_p = s_il + my_src;                       // [my_src][64]
+  float* s_w = s_p + my_src * kKeyBlock;            // [8][64]
+  float* s_red = s_w + kOutBlock * kKeyBlock;       // [256][8], afterwards [vdim]
+  int64_t* s_slot = reinterpret_cast<int64_t*>(s_red + kValThreads * 8 + 32);  // [64]
+  __shared__ float s_small[kValThreads / 32];
+  __shared__ int s_last;
+  ptx::griddep_wait();
+  ptx::griddep_launch_dependents();
+  const int split = blockIdx.x, g = blockIdx.y, lrow = blockIdx.z, tid = threadIdx.x;
+  const int64_t t = row0 + lrow;
+  const int64_t i = a.pos[t];
+  const Visible vis = visible_keys(a, i, max_keys);
+  const int blocks = (vis.n + kKeyBlock - 1) / kKeyBlock;
+  const int src0 = diff ? 2 * g * rep : 0;
+  const int64_t srow = static_cast<int64_t>(lrow) * n_src + src0;
+  for (int s = tid; s < my_src; s += kValThreads) {
+    const float2* st = stats + (srow + s) * n_blocks;
+    float m = -INFINITY, l = 0.f;
+    for (int b = 0; b < blocks; ++b) m = fmaxf(m, st[b].x);
+    for (int b = 0; b < blocks; ++b) l += st[b].y * expf(st[b].x - m);
+    s_m[s] = m;
+    s_il[s] = 1.0f / l;
+  }
+  const int b0 = static_cast<int>(static_cast<int64_t>(blocks) * split / splits);
+  const int b1 = static_cast<int>(static_cast<int64_t>(blocks) * (split + 1) / splits);
+  const int64_t table_row = a.req_rows[a.tok_req[t]];
+  const int vgroups = a.vdim / 8;
+  const int key_lanes = kValThreads / vgroups;
+  const int vg = tid % vgroups, kl = tid / vgroups;
+  const T* vc = static_cast<const T*>(a.v) + static_cast<int64_t>(g) * a.vdim + vg * 8;
+  const int64_t part_row = (static_cast<int64_t>(lrow) * splits + split) * a.heads;
+  for (int o0 = 0; o0 < rep; o0 += kOutBlock) {
+    const int no = min(kOutBlock, rep - o0);
+    float acc[kOutBlock][8] = {};
+    for (int b = b0; b < b1; ++b) {
+      const int k0 = b * kKeyBlock, nk = min(kKeyBlock, vis.n - k0);
+      __syncthreads();
+      for (int e = tid; e < my_src * kKeyBlock; e += kValThreads) {
+        const int s = e / kKeyBlock, kk = e % kKeyBlock;
+        s_p[e] = kk < nk ? expf(scores[(srow + s) * max_keys + k0 + kk] - s_m[s]) * s_il[s] : 0.f;
+      }
+      if (tid < kKeyBlock) s_slot[tid] = slot_of(a, table_row, vis.key(k0 + min(tid, nk - 1)));
+      __syncthreads();
+      for (int e = tid; e < no * kKeyBlock; e += kValThreads) {
+        const int o = e / kKeyBlock, kk = e % kKeyBlock;
+        float w = 0.f;
+        if (diff) {
+          w = s_p[2 * (o0 + o) * kKeyBlock + kk] - a.lambda * s_p[(2 * (o0 + o) + 1) * kKeyBlock + kk];
+        } else {
+          const float* cf = a.coef + static_cast<int64_t>(g * rep + o0 + o) * a.heads;
+          for (int s = 0; s < my_src; ++s) w = fmaf(__ldg(cf + s), s_p[s * kKeyBlock + kk], w);
+        }
+        s_w[e] = w;
+      }
+      __syncthreads();
+      if (kl < key_lanes) {
+#pragma unroll 2
+        for (int kk = kl; kk < nk; kk += key_lanes) {
+          float v[8];
+          load8<T>(vc + s_slot[kk] * a.ldv, v);
+#pragma unroll
+          for (int o = 0; o < kOutBlock; ++o)
+            if (o < no) {
+              const float w = s_w[o * kKeyBlock + kk];
+#pragma unroll
+              for (int x = 0; x < 8; ++x) acc[o][x] = fmaf(w, v[x], acc[o][x]);
+            }
+        }
+      }
+    }
+#pragma unroll
+    for (int o = 0; o < kOutBlock; ++o) {
+      if (o >= no) break;
+      const int head = g * rep + o0 + o;
+      __syncthreads();
+      if (kl < key_lanes) {
+#pragma unroll
+        for (int x = 0; x < 8; ++x) s_red[(kl * vgroups + vg) * 8 + x] = acc[o][x];
+      }
+      __syncthreads();
+      float f[4];  // vdim <= 4 * 256
+#pragma unroll
+      for (int n = 0; n < 4; ++n) {
+        const int c = tid + n * kValThreads;
+        f[n] = 0.f;
+        if (c < a.vdim)
+          for (int k = 0; k < key_lanes; ++k) f[n] += s_red[k * a.vdim + c];
+      }
+      if (splits > 1) {
+#pragma unroll
+        for (int n = 0; n < 4; ++n) {
+          const int c = tid + n * kValThreads;
+          if (c < a.vdim) partial[(part_row + head) * a.vdim + c] = f[n];
+        }
+      } else {
+        __syncthreads();
+#pragma unroll
+        for (int n = 0; n < 4; ++n) {
+          const int c = tid + n * kValThreads;
+          if (c < a.vdim) s_red[c] = f[n];
+        }
+        __syncthreads();
+        finish_head<T>(a, t, head, s_red, s_small);
+      }
+    }
+  }
+  if (splits <= 1) return;
+  // the CTA that finishes last adds the shares, in order
+  __threadfence();
+  __syncthreads();
+  if (tid == 0) {
+    int32_t* c = counters + static_cast<int64_t>(lrow) * a.kv_heads + g;
+    s_last = atomicAdd(c, 1) == splits - 1;
+    if (s_last) *c = 0;
+  }
+  __syncthreads();
+  if (!s_last) return;
+  __threadfence();
+  for (int o = 0; o < rep; ++o) {
+    const int head = g * rep + o;
+    __syncthreads();
+    for (int c = tid; c < a.vdim; c += kValThreads) {
+      float f = 0.f;
+      for (int s = 0; s < splits; ++s)
+        f += __ldcg(partial + ((static_cast<int64_t>(lrow) * splits + s) * a.heads + head) * a.vdim + c);
+      s_red[c] = f;
+    }
+    __syncthreads();
+    finish_head<T>(a, t, head, s_red, s_small);
+  }
+}
+
+static int values_smem(const fr_mix_attn& a) {
+  const int rep = a.heads / a.kv_heads;
+  const int my_src = a.mix == FR_MIX_DIFF ? 2 * rep : a.heads;
+  return (my_src * (2 + kKeyBlock) + kOutBlock * kKeyBlock + kValThreads * 8 + 32) * 4 + kKeyBlock * 8;
+}
+
+template <typename T>
+static int launch_rows(const fr_mix_attn& a, int row0, int n_rows, int max_keys, int splits, float* scores, float2* stats,
+                       float* partial, int32_t* counters, cudaStream_t stream) {
+  const int rep = a.heads / a.kv_heads;
+  const int n_blocks = ceil_div(max_keys, kKeyBlock);
+  const int k_heads = a.mix == FR_MIX_DIFF ? 2 * a.kv_heads : a.kv_heads;
+  const int s1 = rep * (a.dim + kKeyBlock) * 4, s2 = values_smem(a);
+  FR_CHECK_SUPPORTED(s1 <= 200 * 1024 && s2 <= 200 * 1024);
+  static PerDeviceFlag f1, f2;
+  if (ensure_dyn_smem(f1, mix_scores_kernel<T>, 200 * 1024) != FR_OK) return FR_ERR_CUDA;
+  if (ensure_dyn_smem(f2, mix_values_kernel<T>, 200 * 1024) != FR_OK) return FR_ERR_CUDA;
+  mix_scores_kernel<T><<<dim3(n_blocks, k_heads, n_rows), 128, s1, stream>>>(a, row0, max_keys, n_blocks, scores, stats);
+  if (launch_status() != FR_OK) return FR_ERR_CUDA;
+  mix_values_kernel<T><<<dim3(splits, a.kv_heads, n_rows), kValThreads, s2, stream>>>(a, row0, max_keys, n_blocks, splits,
+                                                                                     scores, stats, partial, counters);
+  return launch_status();
+}
+
+// ---------------------------------------------------------------------------
+// bf16 prompts on tcgen05. One CTA: up to 128 consecutive tokens of one request, one v head, the source maps its
+// outputs mix one after the other. Roles as in attn_tc.cu: warp 0 = TMA producer, warp 1 = TMEM allocation and
+// MMA issue, warps 2..5 = one token per thread (TMEM lane == token). Per key tile of 64 (one cache page):
+//     S = Q_s K_s^T (two TMEM buffers);  P = exp2(S - m) as bf16 over S;  O += P V, V as it lies in the cache
+// (token rows, so the B operand is MN-major). After a map's last tile the threads take O / l and add
+// coef[o, s] times it to the accumulators.
+// ---------------------------------------------------------------------------
+constexpr int kM = 128;
+constexpr int kTileN = 64;
+constexpr int kTcThreads = 192;
+constexpr float kRescaleThreshold = 8.0f;
+constexpr int kMaxOut = 8;
+
+struct TcPlan {
+  int q_boxes, v_boxes;   // 64-column boxes of a q / k row and of a v row
+  int v_cols;             // TMEM columns of O and of one accumulator
+  int n_out;              // outputs per CTA
+  int out_blocks;         // CTAs along y per v head (TALK) or per head (DIFF)
+  int tmem_cols, smem;
+};
+
+static bool plan_tc(int mix, int heads, int kv_heads, int dim, int vdim, TcPlan* pl) {
+  if (dim % 16 != 0 || vdim % 16 != 0 || dim <= 0 || vdim <= 0 || dim > 192 || vdim > 192) return false;
+  const int rep = heads / kv_heads;
+  pl->q_boxes = (dim + 63) / 64;
+  pl->v_boxes = (vdim + 63) / 64;
+  pl->v_cols = (vdim + 31) / 32 * 32;
+  int fit = (512 - 2 * kTileN - pl->v_cols) / pl->v_cols;
+  if (fit < 1) return false;
+  if (fit > kMaxOut) fit = kMaxOut;
+  const int outs = mix == FR_MIX_DIFF ? 1 : rep;
+  const int blocks = (outs + fit - 1) / fit;
+  pl->n_out = (outs + blocks - 1) / blocks;
+  pl->out_blocks = blocks;
+  const int need = 2 * kTileN + pl->v_cols * (1 + pl->n_out);
+  pl->tmem_cols = need <= 256 ? 256 : 512;
+  pl->smem = 1024 + 2 * pl->q_boxes * kM * 128 + 2 * (pl->q_boxes + pl->v_boxes) * kTileN * 128 + 256;
+  if (pl->tmem_cols == 512 && pl->smem < 116 * 1024) pl->smem = 116 * 1024;  // one CTA per SM owns all of TMEM
+  return pl->smem <= 227 * 1024;
+}
+
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// MN-major operand tile as TMA writes it with the 128-byte swizzle: rows of 64 values (128 bytes), one row per k;
+// 8-row groups 1024 bytes apart (stride), 64-value column blocks `lead` bytes apart (leading offset).
+__device__ __forceinline__ uint64_t smem_desc_mn(uint32_t addr, uint32_t lead) {
+  uint64_t d = ptx::smem_desc_sw128(addr) & ~(static_cast<uint64_t>(0x3fffu) << 16);
+  return d | static_cast<uint64_t>((lead >> 4) & 0x3fffu) << 16;
+}
+
+template <bool BIAS>
+__global__ void __launch_bounds__(kTcThreads, 2)
+mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tk,
+              const __grid_constant__ CUtensorMap tv, const __grid_constant__ fr_mix_attn a, const TcPlan pl,
+              const int32_t* __restrict__ tiles, int* status) {
+  extern __shared__ uint8_t smem_raw[];
+  const uint32_t raw = ptx::smem_u32(smem_raw);
+  const uint32_t base = (raw + 1023u) & ~1023u;
+  uint8_t* smem = smem_raw + (base - raw);
+  const int q_bytes = pl.q_boxes * kM * 128, k_bytes = pl.q_boxes * kTileN * 128, v_bytes = pl.v_boxes * kTileN * 128;
+  const uint32_t sm_q = base, sm_k = sm_q + 2 * q_bytes, sm_v = sm_k + 2 * k_bytes;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + 2 * q_bytes + 2 * k_bytes + 2 * v_bytes);
+  const uint32_t bar0 = ptx::smem_u32(bars);
+  const uint32_t bar_qfull = bar0, bar_qempty = bar0 + 16;    // [2] each
+  const uint32_t bar_kfull = bar0 + 32, bar_kempty = bar0 + 48;
+  const uint32_t bar_vfull = bar0 + 64, bar_vempty = bar0 + 80;
+  const uint32_t bar_sfull = bar0 + 96;                       // [2]
+  const uint32_t bar_pfull = bar0 + 112;                      // P written (128 arrivals), one phase per tile
+  const uint32_t bar_ofull = bar0 + 120;                      // P.V accumulated, one phase per tile
+  const uint32_t bar_done = bar0 + 128;                       // a map's last P.V, one phase per map
+  const uint32_t bar_oread = bar0 + 136;                      // O read out (128 arrivals), one phase per map
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 18);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+
+  const int rep = a.heads / a.kv_heads;
+  const bool diff = a.mix == FR_MIX_DIFF;
+  // y: DIFF head; TALK (v head, block of its outputs)
+  const int vh = diff ? static_cast<int>(blockIdx.y) / rep : static_cast<int>(blockIdx.y) / pl.out_blocks;
+  const int out0 = diff ? static_cast<int>(blockIdx.y)
+                        : vh * rep + static_cast<int>(blockIdx.y) % pl.out_blocks * pl.n_out;
+  const int n_out = diff ? 1 : min(pl.n_out, (vh + 1) * rep - out0);
+  const int n_src = diff ? 2 : a.heads;
+  const int src0 = diff ? 2 * out0 : 0;
+  const int req = tiles[3 * blockIdx.x], row0 = tiles[3 * blockIdx.x + 1], n_tok = tiles[3 * blockIdx.x + 2];
+  const int pos0 = static_cast<int>(a.pos[row0]);
+  const int pos_last = pos0 + n_tok - 1;
+  const int32_t* table = a.req_to_token + a.req_rows[req] * a.table_stride;
+  // key tiles: [0, n_keep) hold kept first tokens, [t_lo, t_hi] the rest (every role derives the same list)
+  const int t_lo = static_cast<int>(lowest_key(a, pos0)) / kTileN, t_hi = pos_last / kTileN;
+  const int n_keep = a.mask == FR_MASK_CHUNK ? 0 : min((min(a.keep_first, pos_last + 1) + kTileN - 1) / kTileN, t_lo);
+  const int n_tiles = n_keep + t_hi - t_lo + 1;
+  const int total = n_tiles * n_src;
+  auto tile_at = [&](int jj) { return jj < n_keep ? jj : t_lo + jj - n_keep; };
+  // key page of a tile: first slot of its 64 consecutive slots (clamped: a bad table entry reads a wrong page)
+  auto page_row = [&](int tile) {
+    const int s = table[static_cast<int64_t>(tile) * kTileN];
+    return s < 0 ? 0 : (s > static_cast<int>(a.num_slots) - kTileN ? static_cast<int>(a.num_slots) - kTileN : s);
+  };
+  auto k_head = [&](int s) { return diff ? 2 * vh + s : s / rep; };
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < 14; ++i) ptx::mbar_init(bar0 + 8 * i, 1);  // q, k, v full / empty and sfull
+    ptx::mbar_init(bar_pfull, 128);
+    ptx::mbar_init(bar_ofull, 1);
+    ptx::mbar_init(bar_done, 1);
+    ptx::mbar_init(bar_oread, 128);
+    *abort_flag = 0;
+    ptx::mbar_init_fence();
+    ptx::prefetch_tmap(&tq);
+    ptx::prefetch_tmap(&tk);
+    ptx::prefetch_tmap(&tv);
+  }
+  if (warp == 1) {
+    ptx::tmem_alloc(ptx::smem_u32(tmem_slot), pl.tmem_cols);
+    ptx::tmem_relinquish();
+  }
+  ptx::tc_fence_before();
+  __syncthreads();
+  ptx::tc_fence_after();
+  const uint32_t tmem_base = *tmem_slot;
+  const uint32_t col_o = tmem_base + 2 * kTileN;
+  const uint32_t col_acc = col_o + pl.v_cols;
+
+  if (warp == 0) {
+    if (lane == 0) {
+      bool ok = true;
+      auto load_q = [&](int s) -> bool {
+        const uint32_t st = s & 1;
+        if (!ptx::mbar_wait(bar_qempty + 8 * st, ((s >> 1) & 1) ^ 1u, abort_flag, status, 71)) return false;
+        ptx::mbar_expect_tx(bar_qfull + 8 * st, q_bytes);
+        for (int b = 0; b < pl.q_boxes; ++b)
+          ptx::tma_load_2d(sm_q + st * q_bytes + b * kM * 128, &tq, (src0 + s) * a.dim + b * 64, row0, bar_qfull + 8 * st);
+        return true;
+      };
+      auto load_k = [&](int it) -> bool {
+        const uint32_t st = it & 1;
+        if (!ptx::mbar_wait(bar_kempty + 8 * st, ((it >> 1) & 1) ^ 1u, abort_flag, status, 72)) return false;
+        ptx::mbar_expect_tx(bar_kfull + 8 * st, k_bytes);
+        const int row = page_row(tile_at(it % n_tiles));
+        for (int b = 0; b < pl.q_boxes; ++b)
+          ptx::tma_load_2d(sm_k + st * k_bytes + b * kTileN * 128, &tk, k_head(it / n_tiles) * a.dim + b * 64, row,
+                           bar_kfull + 8 * st);
+        return true;
+      };
+      ok = load_q(0) && load_k(0);
+      for (int it = 0; it < total && ok; ++it) {
+        if (it + 1 < total) {  // K (and at a map's end the next Q) runs one tile ahead of V
+          if ((it + 1) % n_tiles == 0) ok = load_q((it + 1) / n_tiles);
+          ok = ok && load_k(it + 1);
+          if (!ok) break;
+        }
+        const uint32_t st = it & 1;
+        ok = ptx::mbar_wait(bar_vempty + 8 * st, ((it >> 1) & 1) ^ 1u, abort_flag, status, 73);
+        if (!ok) break;
+        ptx::mbar_expect_tx(bar_vfull + 8 * st, v_bytes);
+        const int row = page_row(tile_at(it % n_tiles));
+        for (int b = 0; b < pl.v_boxes; ++b)
+          ptx::tma_load_2d(sm_v + st * v_bytes + b * kTileN * 128, &tv, vh * a.vdim + b * 64, row, bar_vfull + 8 * st);
+      }
+    }
+    __syncwarp();
+  } else if (warp == 1) {
+    if (lane == 0) {
+      const uint32_t idesc_s = ptx::make_idesc(1u, 1u, kM, kTileN);
+      const uint32_t idesc_o = ptx::make_idesc(1u, 1u, kM, a.vdim) | (1u << 16);  // B is MN-major
+      bool ok = true;
+      auto issue_s = [&](int it) -> bool {
+        const uint32_t st = it & 1;
+        const int s = it / n_tiles;
+        if (it % n_tiles == 0 && !ptx::mbar_wait(bar_qfull + 8 * (s & 1), (s >> 1) & 1, abort_flag, status, 74)) return false;
+        if (!ptx::mbar_wait(bar_kfull + 8 * st, (it >> 1) & 1, abort_flag, status, 75)) return false;
+        ptx::tc_fence_after();
+        for (int k = 0; k < a.dim / 16; ++k) {
+          const uint64_t a_desc = ptx::smem_desc_sw128(sm_q + (s & 1) * q_bytes + (k >> 2) * kM * 128) + 2u * (k & 3);
+          const uint64_t b_desc = ptx::smem_desc_sw128(sm_k + st * k_bytes + (k >> 2) * kTileN * 128) + 2u * (k & 3);
+          ptx::mma_f16(tmem_base + st * kTileN, a_desc, b_desc, idesc_s, k > 0 ? 1u : 0u);
+        }
+        ptx::tc_commit(bar_kempty + 8 * st);
+        if ((it + 1) % n_tiles == 0) ptx::tc_commit(bar_qempty + 8 * (s & 1));
+        ptx::tc_commit(bar_sfull + 8 * st);
+        return true;
+      };
+      ok = issue_s(0);
+      for (int it = 0; it < total && ok; ++it) {
+        // S of the next tile runs during the softmax of this one; its buffer held P of tile it - 1, whose P.V
+        // was issued before it
+        if (it + 1 < total) ok = issue_s(it + 1);
+        if (!ok) break;
+        const uint32_t st = it & 1;
+        const int s = it / n_tiles, j = it % n_tiles;
+        ok = ptx::mbar_wait(bar_pfull, it & 1, abort_flag, status, 76) &&
+             ptx::mbar_wait(bar_vfull + 8 * st, (it >> 1) & 1, abort_flag, status, 77);
+        // the first P.V of a map overwrites O: the previous map's must have been read
+        if (ok && j == 0 && s > 0) ok = ptx::mbar_wait(bar_oread, (s - 1) & 1, abort_flag, status, 78);
+        if (!ok) break;
+        ptx::tc_fence_after();
+        const uint64_t v_desc = smem_desc_mn(sm_v + st * v_bytes, kTileN * 128);
+        for (int k = 0; k < kTileN / 16; ++k)  // 16 keys = 8 columns of P, 16 rows of V
+          ptx::mma_f16_ts(col_o, tmem_base + st * kTileN + 8u * k, v_desc + static_cast<uint64_t>(k * 16 * 128 >> 4), idesc_o,
+                          (j | k) != 0 ? 1u : 0u);
+        ptx::tc_commit(bar_vempty + 8 * st);
+        ptx::tc_commit(bar_ofull);
+        if (j + 1 == n_tiles) ptx::tc_commit(bar_done);
+      }
+    }
+    __syncwarp();
+  } else {
+    const int quad = warp & 3;
+    const int r = quad * 32 + lane;
+    const bool live = r < n_tok;
+    const int i = pos0 + min(r, n_tok - 1);
+    const int lo = static_cast<int>(lowest_key(a, i));
+    const int keep = a.mask == FR_MASK_CHUNK ? 0 : a.keep_first;
+    const uint32_t lane_off = static_cast<uint32_t>(quad * 32) << 16;
+    const float scale = a.scale * kLog2e;
+    auto wait_all = [&](uint32_t bar, uint32_t parity, int site) -> bool {
+      int okw = 0;
+      if (lane == 0) okw = ptx::mbar_wait(bar, parity, abort_flag, status, site) ? 1 : 0;
+      okw = __shfl_sync(0xffffffffu, okw, 0);
+      ptx::tc_fence_after();
+      return okw != 0;
+    };
+    bool ok = true;
+    for (int s = 0; s < n_src && ok; ++s) {
+      float m_used = -INFINITY, l_sum = 0.f;
+      const float slope = BIAS ? a.slopes[src0 + s] * kLog2e : 0.f;
+      for (int j = 0; j < n_tiles; ++j) {
+        const int it = s * n_tiles + j;
+        const uint32_t st = it & 1;
+        ok = wait_all(bar_sfull + 8 * st, (it >> 1) & 1, 79);
+        if (!ok) break;
+        uint32_t s0[32], s1[32];
+        ptx::tmem_ld_32x32(tmem_base + lane_off + st * kTileN, s0);
+        ptx::tmem_ld_32x32(tmem_base + lane_off + st * kTileN + 32, s1);
+        ptx::tmem_ld_wait();
+        const int j0 = tile_at(j) * kTileN;
+        const float bias0 = slope * static_cast<float>(j0 - i);
+        auto sv = [&](int c) -> uint32_t& { return c < 32 ? s0[c & 31] : s1[c & 31]; };
+#pragma unroll
+        for (int c = 0; c < 64; ++c) {
+          float v = __uint_as_float(sv(c)) * scale;
+          if constexpr (BIAS) v += fmaf(slope, static_cast<float>(c), bias0);
+          sv(c) = __float_as_uint(v);
+        }
+        const bool partly = j0 + kTileN - 1 > i || (j0 < lo && j0 + kTileN > keep);
+        if (__any_sync(0xffffffffu, partly)) {
+          const int hi_c = i - j0, lo_c = lo - j0, keep_c = keep - j0;
+#pragma unroll
+          for (int c = 0; c < 64; ++c)
+            if (c > hi_c || (c < lo_c && c >= keep_c)) sv(c) = 0xff800000u;  // -inf
+        }
+        float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+#pragma unroll
+        for (int c = 0; c < 64; ++c) mx[c & 3] = fmaxf(mx[c & 3], __uint_as_float(sv(c)));
+        const float tmax = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
+        float factor = 1.0f;
+        if (tmax > m_used + kRescaleThreshold) {  // false while nothing is visible (both -inf)
+          factor = ex2(m_used - tmax);            // 0 at the first visible tile
+          m_used = tmax;
+        }
+        l_sum *= factor;
+        if (j > 0 && __any_sync(0xffffffffu, factor != 1.0f)) {
+          ok = wait_all(bar_ofull, (it - 1) & 1, 80);
+          if (!ok) break;
+#pragma unroll 1
+          for (int c = 0; c < pl.v_cols / 32; ++c) {
+            uint32_t o[32];
+            ptx::tmem_ld_32x32(col_o + lane_off + c * 32, o);
+            ptx::tmem_ld_wait();
+#pragma unroll
+            for (int x = 0; x < 32; ++x) o[x] = __float_as_uint(__uint_as_float(o[x]) * factor);
+            ptx::tmem_st_32x32(col_o + lane_off + c * 32, o);
+          }
+          ptx::tmem_st_wait();
+        }
+        const float m_ref = m_used == -INFINITY ? 0.f : m_used;  // nothing visible yet: every weight is 2^-inf = 0
+        float ps[4] = {0.f, 0.f, 0.f, 0.f};
+        uint32_t w[32];
+#pragma unroll
+        for (int x = 0; x < 32; ++x) {
+          const float p0 = ex2(__uint_as_float(sv(2 * x)) - m_ref), p1 = ex2(__uint_as_float(sv(2 * x + 1)) - m_ref);
+          ps[x & 3] += p0 + p1;
+          w[x] = pack_bf16(p0, p1);
+        }
+        l_sum += (ps[0] + ps[1]) + (ps[2] + ps[3]);
+        ptx::tmem_st_32x32(tmem_base + lane_off + st * kTileN, w);
+        ptx::tmem_st_wait();
+        ptx::tc_fence_before();
+        ptx::mbar_arrive(bar_pfull);
+      }
+      if (!ok) break;
+      ok = wait_all(bar_done, s & 1, 81);
+      if (!ok) break;
+      const float inv = 1.0f / l_sum;
+#pragma unroll 1
+      for (int c = 0; c < pl.v_cols / 32; ++c) {
+        uint32_t o[32];
+        ptx::tmem_ld_32x32(col_o + lane_off + c * 32, o);
+        ptx::tmem_ld_wait();
+#pragma unroll 1
+        for (int n = 0; n < n_out; ++n) {
+          const float cf = inv * (diff ? (s == 0 ? 1.0f : -a.lambda)
+                                       : __ldg(a.coef + static_cast<int64_t>(out0 + n) * a.heads + s));
+          uint32_t acc[32];
+          if (s > 0) {
+            ptx::tmem_ld_32x32(col_acc + lane_off + n * pl.v_cols + c * 32, acc);
+            ptx::tmem_ld_wait();
+          } else {
+#pragma unroll
+            for (int x = 0; x < 32; ++x) acc[x] = 0u;
+          }
+#pragma unroll
+          for (int x = 0; x < 32; ++x)
+            acc[x] = __float_as_uint(fmaf(cf, __uint_as_float(o[x]), __uint_as_float(acc[x])));
+          ptx::tmem_st_32x32(col_acc + lane_off + n * pl.v_cols + c * 32, acc);
+        }
+        ptx::tmem_st_wait();
+      }
+      ptx::tc_fence_before();
+      ptx::mbar_arrive(bar_oread);
+    }
+    if (ok) {
+      const int64_t t = row0 + min(r, n_tok - 1);
+      for (int n = 0; n < n_out; ++n) {
+        float scl = 1.0f;
+        if (diff) {
+          float ss = 0.f;
+#pragma unroll 1
+          for (int c = 0; c < pl.v_cols / 32; ++c) {
+            uint32_t o[32];
+            ptx::tmem_ld_32x32(col_acc + lane_off + n * pl.v_cols + c * 32, o);
+            ptx::tmem_ld_wait();
+#pragma unroll
+            for (int x = 0; x < 32; ++x)
+              if (c * 32 + x < a.vdim) ss = fmaf(__uint_as_float(o[x]), __uint_as_float(o[x]), ss);
+          }
+          scl = a.out_scale / sqrtf(ss / static_cast<float>(a.vdim_true) + a.eps);
+        }
+        __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(a.out) + t * a.ldo + static_cast<int64_t>(out0 + n) * a.vdim;
+#pragma unroll 1
+        for (int c = 0; c < pl.v_cols / 32; ++c) {
+          uint32_t o[32];
+          ptx::tmem_ld_32x32(col_acc + lane_off + n * pl.v_cols + c * 32, o);
+          ptx::tmem_ld_wait();
+          if (live) {
+            uint4* d4 = reinterpret_cast<uint4*>(dst + c * 32);
+#pragma unroll
+            for (int x = 0; x < 4; ++x)
+              if (c * 32 + x * 8 < a.vdim)
+                d4[x] = make_uint4(pack_bf16(__uint_as_float(o[8 * x]) * scl, __uint_as_float(o[8 * x + 1]) * scl),
+                                   pack_bf16(__uint_as_float(o[8 * x + 2]) * scl, __uint_as_float(o[8 * x + 3]) * scl),
+                                   pack_bf16(__uint_as_float(o[8 * x + 4]) * scl, __uint_as_float(o[8 * x + 5]) * scl),
+                                   pack_bf16(__uint_as_float(o[8 * x + 6]) * scl, __uint_as_float(o[8 * x + 7]) * scl));
+          }
+          __syncwarp();
+        }
+      }
+    }
+  }
+
+  ptx::tc_fence_before();
+  __syncthreads();
+  if (*abort_flag) {
+    for (int i = 0; i < 200; ++i) __nanosleep(1000);
+    __syncthreads();
+  }
+  if (warp == 1) {
+    ptx::tc_fence_after();
+    ptx::tmem_dealloc(tmem_base, pl.tmem_cols);
+  }
+}
+
+static int check_args(const fr_mix_attn* a) {
+  FR_CHECK_ARG(a && (a->dtype == 0 || a->dtype == 1) && (a->mix == FR_MIX_DIFF || a->mix == FR_MIX_TALK));
+  FR_CHECK_ARG((a->mask == FR_MASK_WINDOW || a->mask == FR_MASK_CHUNK) && a->mask_size > 0 && a->keep_first >= 0);
+  FR_CHECK_ARG(a->heads > 0 && a->kv_heads > 0 && a->heads % a->kv_heads == 0);
+  FR_CHECK_ARG(a->dim > 0 && a->dim % 16 == 0 && a->vdim > 0 && a->vdim % 16 == 0 && a->vdim_true > 0);
+  FR_CHECK_ARG(a->q && a->k && a->v && a->out && a->req_to_token && a->req_rows && a->tok_req && a->pos && a->num_slots > 0);
+  FR_CHECK_ARG(aligned16(a->q) && aligned16(a->k) && aligned16(a->v) && aligned16(a->out) && a->ldq % 8 == 0 &&
+               a->ldk % 8 == 0 && a->ldv % 8 == 0 && a->ldo % 8 == 0);
+  FR_CHECK_ARG(a->mix != FR_MIX_TALK || a->coef);
+  return FR_OK;
+}
+
+}  // namespace mix
+}  // namespace fr
+
+using namespace fr;
+
+extern "C" int64_t fr_mix_attn_rows_scratch(int mix_kind, int heads, int vdim, int n_rows, int max_keys, int splits) {
+  if (heads <= 0 || vdim <= 0 || n_rows < 0 || max_keys <= 0 || splits <= 0) return -1;
+  const int64_t src = static_cast<int64_t>(n_rows) * (mix_kind == FR_MIX_DIFF ? 2 * heads : heads);
+  const int64_t stats = src * ceil_div(max_keys, mix::kKeyBlock) * 8;
+  const int64_t part = splits > 1 ? static_cast<int64_t>(n_rows) * splits * heads * vdim * 4 : 0;
+  return stats + src * max_keys * 4 + part;
+}
+
+extern "C" int fr_mix_attn_rows(const fr_mix_attn* a, int row0, int n_rows, int max_keys, int splits, void* scratch,
+                                int64_t scratch_bytes, int32_t* counters, cudaStream_t stream) {
+  const int st = mix::check_args(a);
+  if (st != FR_OK) return st;
+  FR_CHECK_ARG(row0 >= 0 && n_rows >= 0 && max_keys > 0 && splits > 0);
+  if (n_rows == 0) return FR_OK;
+  FR_CHECK_ARG(scratch && aligned16(scratch) && (splits == 1 || counters));
+  FR_CHECK_ARG(scratch_bytes >= fr_mix_attn_rows_scratch(a->mix, a->heads, a->vdim, n_rows, max_keys, splits));
+  FR_CHECK_SUPPORTED(a->vdim <= 1024 && n_rows <= 65535);
+  const int64_t src = static_cast<int64_t>(n_rows) * (a->mix == FR_MIX_DIFF ? 2 * a->heads : a->heads);
+  float2* stats = static_cast<float2*>(scratch);
+  float* scores = reinterpret_cast<float*>(stats + src * ceil_div(max_keys, mix::kKeyBlock));
+  float* partial = scores + src * max_keys;
+  return a->dtype == 0 ? mix::launch_rows<__nv_bfloat16>(*a, row0, n_rows, max_keys, splits, scores, stats, partial, counters, stream)
+                       : mix::launch_rows<float>(*a, row0, n_rows, max_keys, splits, scores, stats, partial, counters, stream);
+}
+
+extern "C" int fr_mix_attn_tc_fits(int mix_kind, int heads, int kv_heads, int dim, int vdim) {
+  mix::TcPlan pl;
+  return heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && mix::plan_tc(mix_kind, heads, kv_heads, dim, vdim, &pl) ? 1 : 0;
+}
+
+extern "C" int fr_mix_attn_tc(const fr_mix_attn* a, const int32_t* tiles, int n_tiles, int n_rows, cudaStream_t stream) {
+  const int st = mix::check_args(a);
+  if (st != FR_OK) return st;
+  FR_CHECK_ARG(tiles && n_tiles >= 0 && n_rows >= 0);
+  if (n_tiles == 0 || n_rows == 0) return FR_OK;
+  mix::TcPlan pl;
+  FR_CHECK_SUPPORTED(a->dtype == 0 && a->num_slots >= mix::kTileN &&
+                     mix::plan_tc(a->mix, a->heads, a->kv_heads, a->dim, a->vdim, &pl));
+  const bool diff = a->mix == FR_MIX_DIFF;
+  const int n_src = diff ? 2 * a->heads : a->heads, k_heads = diff ? 2 * a->kv_heads : a->kv_heads;
+  CUtensorMap tq, tk, tv;
+  int r = make_tmap_bf16_box64(&tq, a->q, static_cast<uint64_t>(n_src) * a->dim, n_rows, a->ldq, mix::kM);
+  if (r == FR_OK) r = make_tmap_bf16_box64(&tk, a->k, static_cast<uint64_t>(k_heads) * a->dim, a->num_slots, a->ldk, mix::kTileN);
+  if (r == FR_OK) r = make_tmap_bf16_box64(&tv, a->v, static_cast<uint64_t>(a->kv_heads) * a->vdim, a->num_slots, a->ldv, mix::kTileN);
+  if (r != FR_OK) return r;
+  int* status = device_status_ptr();
+  if (!status) return FR_ERR_CUDA;
+  dim3 grid(n_tiles, diff ? a->heads : a->kv_heads * pl.out_blocks);
+  static PerDeviceFlag f0, f1;
+  if (a->slopes != nullptr) {
+    if (ensure_dyn_smem(f1, mix::mix_tc_kernel<true>, 227 * 1024) != FR_OK) return FR_ERR_CUDA;
+    mix::mix_tc_kernel<true><<<grid, mix::kTcThreads, pl.smem, stream>>>(tq, tk, tv, *a, pl, tiles, status);
+  } else {
+    if (ensure_dyn_smem(f0, mix::mix_tc_kernel<false>, 227 * 1024) != FR_OK) return FR_ERR_CUDA;
+    mix::mix_tc_kernel<false><<<grid, mix::kTcThreads, pl.smem, stream>>>(tq, tk, tv, *a, pl, tiles, status);
+  }
+  return launch_status();
+}

@@ -103,6 +103,11 @@ def iter_safetensors(model_path: str, key_filter: Optional[Callable[[str], bool]
                     yield key, f.get_tensor(key)
 
 
+def read_tensors(model_path: str, key_filter: Optional[Callable[[str], bool]] = None) -> Dict[str, torch.Tensor]:
+    """All tensors of a checkpoint directory on the CPU, in the checkpoint's types."""
+    return dict(iter_safetensors(model_path, key_filter))
+
+
 def _is_scale_key(key: str) -> bool:
     return key.endswith(".weight_scale") or key.endswith(".weight_scale_inv")
 

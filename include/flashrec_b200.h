@@ -512,6 +512,127 @@ int fr_topk_merge_shards(float* out_vals, int64_t* out_parents, int64_t* out_tok
 int fr_lse_combine_shards(const float* shard_max, const float* shard_logsum, float* row_max, float* row_logsum, int S,
                           int rows, int64_t shard_stride, cudaStream_t stream);
 
+/* ---- 16/32-bit decoder layers (fp32 residual stream) ---------------------------
+ * `dtype` of these entry points: the type of weights, activations and caches, 0 = bf16 (products accumulate
+ * in fp32), 1 = f32 (true fp32 arithmetic throughout). The residual stream `x` is always f32. Row pitches
+ * are in elements; pitches of matrix operands are multiples of 8 elements and their bases 16-byte aligned. */
+
+/* What happens to one range of output columns of fr_dense_proj. Column ranges start at multiples of 32. */
+enum fr_segment_kind {
+  FR_SEG_STORE = 0,   /* out[row, c] = z */
+  FR_SEG_SWIGLU = 1,  /* weight rows come in blocks of 64 = [32 gate | 32 up]; out[row, c] = silu(gate_c) * up_c */
+  FR_SEG_SIGMOID = 2, /* out[row, c] = sigmoid(z + bias[c]) */
+  FR_SEG_STORE_F32 = 3 /* out[row, c] = z, f32 whatever the dtype */
+};
+struct fr_out_segment {
+  int32_t kind;
+  int32_t n0;            /* first weight row of the range (a multiple of 32; of 64 for SWIGLU) */
+  int32_t n;             /* output columns written (SWIGLU: activation channels, half the weight rows) */
+  int32_t pad_;
+  void* out;
+  int64_t ldo;
+  const int64_t* row_map; /* output row per input row (KV-cache slots), or null */
+  const float* bias;      /* SIGMOID: [n], or null */
+};
+
+/* z = a . w^T for one merged weight matrix, each column range leaving through its segment. a [M, K], w [N, K].
+ * algo: 0 picks by shape; 1 = one warp per few weight rows (M <= 8); 2 = tcgen05 tiles (bf16), shared-memory
+ * tiles (f32). */
+int fr_dense_proj(int dtype, const void* a, int64_t lda, const void* w, int64_t ldw, int M, int N, int K,
+                  const struct fr_out_segment* segs, int n_segs, int algo, cudaStream_t stream);
+
+/* One term of fr_dense_gated_add. */
+struct fr_gated_part {
+  const void* a;   /* [M, K] */
+  const void* w;   /* [N, K] */
+  const void* gate; /* [M, N] elementwise factor, or null */
+  int64_t lda, ldw, ldg;
+  int32_t K;
+  int32_t pad_;
+};
+
+/* x[m, n] += sum_p gate_p[m, n] * (a_p . w_p^T)[m, n], one or two parts. With `partials` (f32
+ * [splits, M, N]) the K extent is split instead: partial s receives its share of the sum, x is left alone
+ * and fr_lm_norm adds the partials in order. n_splits: 0 without partials; else as returned by
+ * fr_dense_gated_add_splits for the same shape. */
+int fr_dense_gated_add(int dtype, const struct fr_gated_part* parts, int n_parts, float* x, int64_t ldx, int M, int N,
+                       float* partials, int n_splits, int algo, cudaStream_t stream);
+int fr_dense_gated_add_splits(int dtype, int M, int N, int K0, int K1);
+
+/* x[t, :] = table[ids[t], :] * scale, and the slot table entry of the token: req_to_token[rows[t], pos[t]] = loc[t]
+ * (skipped when req_to_token is null). */
+int fr_lm_embed(int dtype, const void* table, int64_t ldt, const int64_t* ids, float* x, int64_t ldx, int M, int W, int vocab,
+                float scale, int32_t* req_to_token, int64_t table_stride, const int64_t* rows, const int64_t* pos,
+                const int64_t* loc, cudaStream_t stream);
+
+/* RMS norm of the fp32 residual stream: x += sum of the partials (if any; written back unless
+ * row_idx is given), then out = x / sqrt(mean(x^2) + eps) * (offset + weight). row_idx (or null) picks the rows;
+ * columns [W, ldo) of out are zeroed up to a multiple of 8. */
+int fr_lm_norm(int dtype, float* x, int64_t ldx, const float* weight, float offset, float eps, const float* partials,
+               int n_partials, int64_t partial_stride, const int64_t* row_idx, void* out, int64_t ldo, int M, int W,
+               cudaStream_t stream);
+
+/* One channel range of fr_short_conv's output. */
+struct fr_conv_out {
+  void* out;
+  int64_t ldo;
+  const int64_t* row_map; /* output row per token, or null */
+  int32_t c0, c;          /* channels [c0, c0 + c) */
+};
+
+/* Depthwise causal convolution over time of a ragged batch: y_t = sum_j w[:, j] * u_(t - taps + 1 + j), zeros
+ * before position 0; values before the batch's tokens come from state [slots, taps - 1, C] (oldest first).
+ * u [T, C], w [C, taps] f32, tok_req [T] = index of the token's request in qo_indptr / state_slots. The state of
+ * every request is advanced past its tokens. one_token: every request has exactly one token. */
+int fr_short_conv(int dtype, const void* u, int64_t ldu, const float* w, int taps, int C, const struct fr_conv_out* outs,
+                  int n_outs, void* state, const int64_t* state_slots, const int32_t* tok_req, const int32_t* qo_indptr,
+                  const int64_t* pos, int T, int n_req, int one_token, cudaStream_t stream);
+
+/* Attention whose outputs are linear combinations of several softmax maps over the same values:
+ *     out_o(i) = sum_s coef[o, s] * sum_j softmax_j(scale * q_s(i) . k_s(j) - slope_s * (i - j)) v(j).
+ * FR_MIX_DIFF: output head h mixes its two maps with (1, -lambda) and is divided by its root mean square over
+ * vdim (eps inside the root), times out_scale. FR_MIX_TALK: output head h mixes all H heads' maps with row h of
+ * the matrix coef [H, H]. */
+enum fr_mix_kind { FR_MIX_DIFF = 0, FR_MIX_TALK = 1 };
+enum fr_mask_kind {
+  FR_MASK_WINDOW = 0, /* j <= i and (i - j < size or j < keep_first) */
+  FR_MASK_CHUNK = 1   /* j <= i and i / size == j / size */
+};
+struct fr_mix_attn {
+  int32_t dtype, mix, mask, mask_size, keep_first;
+  int32_t heads, kv_heads, dim, vdim; /* dim, vdim as laid out: multiples of 16, zero padded */
+  int32_t vdim_true;                  /* values the root mean square counts */
+  float scale, lambda, eps, out_scale;
+  const float* coef;    /* TALK: [heads, heads] */
+  const float* slopes;  /* one per source map, or null */
+  const void* q;        /* [T, sources * dim], pitch ldq */
+  int64_t ldq;
+  const void* k;        /* [slots, kv sources * dim], pitch ldk; DIFF: two maps per kv head */
+  const void* v;        /* [slots, kv_heads * vdim], pitch ldv */
+  int64_t ldk, ldv;
+  void* out;            /* [T, heads * vdim], pitch ldo */
+  int64_t ldo;
+  const int32_t* req_to_token; /* slot of (request row, position) */
+  int64_t table_stride;
+  const int64_t* req_rows; /* [n_req] slot-table row per request */
+  const int32_t* tok_req;  /* [T] */
+  const int64_t* pos;      /* [T] */
+  int64_t num_slots;
+};
+
+/* Any head sizes, bf16 or f32, prompts or decode: scores of every visible key, then the mixture over the values.
+ * Rows [row0, row0 + n_rows) of the batch. max_keys bounds the visible keys of a row; scratch holds
+ * fr_mix_attn_rows_scratch(...) bytes, counters n_rows * kv_heads zeroed words (left zeroed). */
+int fr_mix_attn_rows(const struct fr_mix_attn* a, int row0, int n_rows, int max_keys, int splits, void* scratch,
+                     int64_t scratch_bytes, int32_t* counters, cudaStream_t stream);
+int64_t fr_mix_attn_rows_scratch(int mix, int heads, int vdim, int n_rows, int max_keys, int splits);
+
+/* bf16 prompts on the tensor cores: tiles [n_tiles, 3] of {request, first row in the batch, rows} (at most 128
+ * rows). The cache is paged: positions [64 p, 64 p + 64) of a request occupy 64 consecutive slots that start at
+ * a multiple of 64. FR_ERR_UNSUPPORTED when the head sizes do not fit (fr_mix_attn_tc_fits tells). */
+int fr_mix_attn_tc(const struct fr_mix_attn* a, const int32_t* tiles, int n_tiles, int n_rows, cudaStream_t stream);
+int fr_mix_attn_tc_fits(int mix, int heads, int kv_heads, int dim, int vdim);
+
 #ifdef __cplusplus
 }
 #endif
