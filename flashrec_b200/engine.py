@@ -95,7 +95,7 @@ class LMEngine:
         # short portions first: their attention runs row by row, the rest in tiles
         order = sorted(range(len(entries)), key=lambda i: len(entries[i].tokens) > ROW_PORTION)
         start: Dict[int, int] = {}
-        toks, pos, loc, tok_req, rows, req_rows, qo = [], [], [], [], [], [], [0]
+        toks, pos, loc, tok_req, rows, req_rows, qo, pre, ext = [], [], [], [], [], [], [0], [], []
         tiles: List[Tuple[int, int, int]] = []
         n_row = 0
         for b, i in enumerate(order):
@@ -112,6 +112,8 @@ class LMEngine:
             rows += [seq.row] * n
             req_rows.append(seq.row)
             qo.append(t0 + n)
+            pre.append(first)
+            ext.append(n)
             if n <= ROW_PORTION:
                 n_row = t0 + n
             else:
@@ -121,7 +123,7 @@ class LMEngine:
         if one and self.use_graphs and on_layer is None and len(entries) <= self.GRAPH_SIZES[-1]:
             out = self._decode(toks, pos, loc, rows, want)
         else:
-            batch, want_d = self._stage(toks, pos, loc, rows, req_rows, want, tok_req, qo, tiles, n_row, one)
+            batch, want_d = self._stage(toks, pos, loc, rows, req_rows, want, tok_req, qo, pre, ext, tiles, n_row, one)
             x, partials = self.model.forward(batch, self.caches, self.seqs.req_to_token, self.counters, on_layer=on_layer)
             out = self.model.logits(x, partials, want_d) if want else \
                 torch.empty((0, vocab), dtype=torch.float32, device=self.device)
@@ -158,11 +160,12 @@ class LMEngine:
             p += n
         return out64, out32
 
-    def _stage(self, toks, pos, loc, rows, req_rows, want, tok_req, qo, tiles, n_row, one):
-        (d_tok, d_pos, d_loc, d_rows, d_req, d_want), (d_tr, d_qo, d_tiles) = self._upload(
-            [toks, pos, loc, rows, req_rows, want], [tok_req, qo, [v for t in tiles for v in t]])
-        batch = ForwardBatch(input_ids=d_tok, req_pool_indices=d_req, seq_lens=d_qo[1:], positions=d_pos,
-                             out_cache_loc=d_loc, is_prefill=not one, qo_indptr=d_qo, tok_req=d_tr, tok_rows=d_rows,
+    def _stage(self, toks, pos, loc, rows, req_rows, want, tok_req, qo, pre, ext, tiles, n_row, one):
+        (d_tok, d_pos, d_loc, d_rows, d_req, d_want), (d_tr, d_qo, d_tiles, d_len) = self._upload(
+            [toks, pos, loc, rows, req_rows, want],
+            [tok_req, qo, [v for t in tiles for v in t], [p + n for p, n in zip(pre, ext)]])
+        batch = ForwardBatch(input_ids=d_tok, req_pool_indices=d_req, seq_lens=d_len, positions=d_pos,
+                             out_cache_loc=d_loc, is_prefill=not one, extend_prefix_lens=pre, extend_seq_lens=ext, qo_indptr=d_qo, tok_req=d_tr, tok_rows=d_rows,
                              n_row_tokens=n_row, tiles=d_tiles.view(-1, 3), one_token=one, max_pos=max(pos))
         return batch, d_want
 
