@@ -162,12 +162,14 @@ _SIGNATURES = {
     "fr_short_conv": [_I, P, _L, P, _I, _I, P, _I, P, P, P, P, P, _I, _I, _I, P],
     "fr_mix_attn_rows": [P, _I, _I, _I, _I, P, _L, P, P],
     "fr_mix_attn_rows_scratch": [_I] * 6,
-    "fr_mix_attn_tc": [P, P, _I, _I, P],
+    "fr_mix_attn_tc": [P, P, _I, _I, _I, P, _L, P],
+    "fr_mix_attn_tc_scratch": [P, _I, _I, _L],
     "fr_mix_attn_tc_fits": [_I] * 5,
 }
 _RESTYPES = {"fr_version": c_char_p, "fr_decode_attn_scratch_bytes": c_int64,
              "fr_sid_head_topk_workspace_bytes": c_int64, "fr_joint_select_workspace_bytes": c_int64,
-             "fr_trie_build_workspace_bytes": c_int64, "fr_mix_attn_rows_scratch": c_int64}
+             "fr_trie_build_workspace_bytes": c_int64, "fr_mix_attn_rows_scratch": c_int64,
+             "fr_mix_attn_tc_scratch": c_int64}
 
 
 def lib_path() -> Path:

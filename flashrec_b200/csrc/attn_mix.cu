@@ -8,69 +8,15 @@
 //     every visible key, mix the normalised weights and pass over V once; keys may be split over CTAs;
 //   * mix_tc_kernel (fr_mix_attn_tc: bf16 prompts, tcgen05) runs one flash pass per source map and adds
 //     coef[o, s] / l_s times its result to the outputs' accumulators, which stay in TMEM beside S and O.
-#include "fr_common.cuh"
-#include "sm100_ptx.cuh"
+#include "attn_mix.cuh"
 
 namespace fr {
 
-int* device_status_ptr();  // capi.cu
-int make_tmap_bf16_box64(CUtensorMap* map, const void* ptr, uint64_t cols, uint64_t rows, int64_t pitch,
-                         uint32_t box_rows);  // dense_proj.cu
+int talk_tc(const fr_mix_attn& a, const int32_t* tiles, int n_tiles, int n_rows, int max_pos, void* scratch,
+            int64_t scratch_bytes, cudaStream_t stream);  // attn_talk.cu
+int64_t talk_tc_tile_bytes(const fr_mix_attn& a, int max_pos);
 
 namespace mix {
-
-constexpr float kLog2e = 1.4426950408889634f;
-
-template <typename T>
-__device__ __forceinline__ void load8(const T* p, float (&v)[8]);
-template <>
-__device__ __forceinline__ void load8<float>(const float* p, float (&v)[8]) {
-  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
-  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
-  v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
-}
-template <>
-__device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, float (&v)[8]) {
-  const uint4 a = *reinterpret_cast<const uint4*>(p);
-  const uint32_t w[4] = {a.x, a.y, a.z, a.w};
-#pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    v[2 * i] = __uint_as_float(w[i] << 16);
-    v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
-  }
-}
-template <typename T>
-__device__ __forceinline__ void st_f(T* p, float v) { *p = v; }
-template <>
-__device__ __forceinline__ void st_f<__nv_bfloat16>(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
-
-// Visible keys of the query at position i: [0, n_first) and [lo, i].
-struct Visible {
-  int64_t lo;
-  int n_first, n;
-  __device__ __forceinline__ int64_t key(int idx) const { return idx < n_first ? idx : lo + (idx - n_first); }
-};
-__device__ __forceinline__ int64_t lowest_key(const fr_mix_attn& a, int64_t i) {
-  if (a.mask == FR_MASK_CHUNK) return i / a.mask_size * a.mask_size;
-  return i - a.mask_size + 1 > 0 ? i - a.mask_size + 1 : 0;
-}
-__device__ __forceinline__ Visible visible_keys(const fr_mix_attn& a, int64_t i, int max_keys) {
-  Visible v;
-  v.lo = lowest_key(a, i);
-  v.n_first = a.mask == FR_MASK_CHUNK ? 0 : static_cast<int>(a.keep_first < v.lo ? a.keep_first : v.lo);
-  const int64_t n = v.n_first + (i - v.lo + 1);
-  v.n = static_cast<int>(n < max_keys ? n : max_keys);
-  return v;
-}
-__device__ __forceinline__ int64_t slot_of(const fr_mix_attn& a, int64_t table_row, int64_t j) {
-  const int64_t s = a.req_to_token[table_row * a.table_stride + j];
-  return s < 0 ? 0 : (s >= a.num_slots ? a.num_slots - 1 : s);
-}
-// i-th source map that reads k head kh
-__device__ __forceinline__ int source_of(const fr_mix_attn& a, int kh, int i) {
-  const int rep = a.heads / a.kv_heads;
-  return a.mix == FR_MIX_DIFF ? 2 * ((kh >> 1) * rep + i) + (kh & 1) : kh * rep + i;
-}
 
 constexpr int kKeyBlock = 64;
 
@@ -338,11 +284,12 @@ static int launch_rows(const fr_mix_attn& a, int row0, int n_rows, int max_keys,
   static PerDeviceFlag f1, f2;
   if (ensure_dyn_smem(f1, mix_scores_kernel<T>, 200 * 1024) != FR_OK) return FR_ERR_CUDA;
   if (ensure_dyn_smem(f2, mix_values_kernel<T>, 200 * 1024) != FR_OK) return FR_ERR_CUDA;
-  mix_scores_kernel<T><<<dim3(n_blocks, k_heads, n_rows), 128, s1, stream>>>(a, row0, max_keys, n_blocks, scores, stats);
-  if (launch_status() != FR_OK) return FR_ERR_CUDA;
-  mix_values_kernel<T><<<dim3(splits, a.kv_heads, n_rows), kValThreads, s2, stream>>>(a, row0, max_keys, n_blocks, splits,
-                                                                                     scores, stats, partial, counters);
-  return launch_status();
+  const bool pdl = n_rows <= kPdlRows;
+  if (launch_kernel(mix_scores_kernel<T>, dim3(n_blocks, k_heads, n_rows), 128, s1, stream, pdl, a, row0, max_keys, n_blocks,
+                    scores, stats) != FR_OK)
+    return FR_ERR_CUDA;
+  return launch_kernel(mix_values_kernel<T>, dim3(splits, a.kv_heads, n_rows), kValThreads, s2, stream, pdl, a, row0, max_keys,
+                       n_blocks, splits, scores, stats, partial, counters);
 }
 
 // ---------------------------------------------------------------------------
@@ -353,8 +300,6 @@ static int launch_rows(const fr_mix_attn& a, int row0, int n_rows, int max_keys,
 // (token rows, so the B operand is MN-major). After a map's last tile the threads take O / l and add
 // coef[o, s] times it to the accumulators.
 // ---------------------------------------------------------------------------
-constexpr int kM = 128;
-constexpr int kTileN = 64;
 constexpr int kTcThreads = 192;
 constexpr float kRescaleThreshold = 8.0f;
 constexpr int kMaxOut = 8;
@@ -364,6 +309,7 @@ struct TcPlan {
   int v_cols;             // TMEM columns of O and of one accumulator
   int n_out;              // outputs per CTA
   int out_blocks;         // CTAs along y per v head (TALK) or per head (DIFF)
+  int staged;             // DIFF: the first map's result waits in the output rows (fp16), not in TMEM
   int tmem_cols, smem;
 };
 
@@ -373,6 +319,7 @@ static bool plan_tc(int mix, int heads, int kv_heads, int dim, int vdim, TcPlan*
   pl->q_boxes = (dim + 63) / 64;
   pl->v_boxes = (vdim + 63) / 64;
   pl->v_cols = (vdim + 31) / 32 * 32;
+  pl->staged = 0;
   int fit = (512 - 2 * kTileN - pl->v_cols) / pl->v_cols;
   if (fit < 1) return false;
   if (fit > kMaxOut) fit = kMaxOut;
@@ -380,24 +327,15 @@ static bool plan_tc(int mix, int heads, int kv_heads, int dim, int vdim, TcPlan*
   const int blocks = (outs + fit - 1) / fit;
   pl->n_out = (outs + blocks - 1) / blocks;
   pl->out_blocks = blocks;
-  const int need = 2 * kTileN + pl->v_cols * (1 + pl->n_out);
+  int need = 2 * kTileN + pl->v_cols * (1 + pl->n_out);
+  if (mix == FR_MIX_DIFF && need > 256 && need - pl->v_cols <= 256) {  // without the accumulator two CTAs share an SM
+    pl->staged = 1;
+    need -= pl->v_cols;
+  }
   pl->tmem_cols = need <= 256 ? 256 : 512;
   pl->smem = 1024 + 2 * pl->q_boxes * kM * 128 + 2 * (pl->q_boxes + pl->v_boxes) * kTileN * 128 + 256;
   if (pl->tmem_cols == 512 && pl->smem < 116 * 1024) pl->smem = 116 * 1024;  // one CTA per SM owns all of TMEM
   return pl->smem <= 227 * 1024;
-}
-
-__device__ __forceinline__ float ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-
-// MN-major operand tile as TMA writes it with the 128-byte swizzle: rows of 64 values (128 bytes), one row per k;
-// 8-row groups 1024 bytes apart (stride), 64-value column blocks `lead` bytes apart (leading offset).
-__device__ __forceinline__ uint64_t smem_desc_mn(uint32_t addr, uint32_t lead) {
-  uint64_t d = ptx::smem_desc_sw128(addr) & ~(static_cast<uint64_t>(0x3fffu) << 16);
-  return d | static_cast<uint64_t>((lead >> 4) & 0x3fffu) << 16;
 }
 
 template <bool BIAS>
@@ -424,6 +362,8 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 18);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
+  ptx::griddep_wait();
+  ptx::griddep_launch_dependents();
   const int rep = a.heads / a.kv_heads;
   const bool diff = a.mix == FR_MIX_DIFF;
   // y: DIFF head; TALK (v head, block of its outputs)
@@ -437,17 +377,9 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
   const int pos0 = static_cast<int>(a.pos[row0]);
   const int pos_last = pos0 + n_tok - 1;
   const int32_t* table = a.req_to_token + a.req_rows[req] * a.table_stride;
-  // key tiles: [0, n_keep) hold kept first tokens, [t_lo, t_hi] the rest (every role derives the same list)
-  const int t_lo = static_cast<int>(lowest_key(a, pos0)) / kTileN, t_hi = pos_last / kTileN;
-  const int n_keep = a.mask == FR_MASK_CHUNK ? 0 : min((min(a.keep_first, pos_last + 1) + kTileN - 1) / kTileN, t_lo);
-  const int n_tiles = n_keep + t_hi - t_lo + 1;
+  const KeyTiles kt = key_tiles(a, pos0, pos_last);  // every role derives the same list
+  const int n_tiles = kt.n;
   const int total = n_tiles * n_src;
-  auto tile_at = [&](int jj) { return jj < n_keep ? jj : t_lo + jj - n_keep; };
-  // key page of a tile: first slot of its 64 consecutive slots (clamped: a bad table entry reads a wrong page)
-  auto page_row = [&](int tile) {
-    const int s = table[static_cast<int64_t>(tile) * kTileN];
-    return s < 0 ? 0 : (s > static_cast<int>(a.num_slots) - kTileN ? static_cast<int>(a.num_slots) - kTileN : s);
-  };
   auto k_head = [&](int s) { return diff ? 2 * vh + s : s / rep; };
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -489,7 +421,7 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
         const uint32_t st = it & 1;
         if (!ptx::mbar_wait(bar_kempty + 8 * st, ((it >> 1) & 1) ^ 1u, abort_flag, status, 72)) return false;
         ptx::mbar_expect_tx(bar_kfull + 8 * st, k_bytes);
-        const int row = page_row(tile_at(it % n_tiles));
+        const int row = page_row(a, table, kt.at(it % n_tiles));
         for (int b = 0; b < pl.q_boxes; ++b)
           ptx::tma_load_2d(sm_k + st * k_bytes + b * kTileN * 128, &tk, k_head(it / n_tiles) * a.dim + b * 64, row,
                            bar_kfull + 8 * st);
@@ -506,7 +438,7 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
         ok = ptx::mbar_wait(bar_vempty + 8 * st, ((it >> 1) & 1) ^ 1u, abort_flag, status, 73);
         if (!ok) break;
         ptx::mbar_expect_tx(bar_vfull + 8 * st, v_bytes);
-        const int row = page_row(tile_at(it % n_tiles));
+        const int row = page_row(a, table, kt.at(it % n_tiles));
         for (int b = 0; b < pl.v_boxes; ++b)
           ptx::tma_load_2d(sm_v + st * v_bytes + b * kTileN * 128, &tv, vh * a.vdim + b * 64, row, bar_vfull + 8 * st);
       }
@@ -574,9 +506,11 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
       return okw != 0;
     };
     bool ok = true;
+    __nv_bfloat16* out_row = static_cast<__nv_bfloat16*>(a.out) + (row0 + min(r, n_tok - 1)) * a.ldo +
+                             static_cast<int64_t>(out0) * a.vdim;
     for (int s = 0; s < n_src && ok; ++s) {
       float m_used = -INFINITY, l_sum = 0.f;
-      const float slope = BIAS ? a.slopes[src0 + s] * kLog2e : 0.f;
+      const float slope = BIAS && a.slopes != nullptr ? a.slopes[src0 + s] * kLog2e : 0.f;
       for (int j = 0; j < n_tiles; ++j) {
         const int it = s * n_tiles + j;
         const uint32_t st = it & 1;
@@ -586,14 +520,13 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
         ptx::tmem_ld_32x32(tmem_base + lane_off + st * kTileN, s0);
         ptx::tmem_ld_32x32(tmem_base + lane_off + st * kTileN + 32, s1);
         ptx::tmem_ld_wait();
-        const int j0 = tile_at(j) * kTileN;
+        const int j0 = kt.at(j) * kTileN;
         const float bias0 = slope * static_cast<float>(j0 - i);
         auto sv = [&](int c) -> uint32_t& { return c < 32 ? s0[c & 31] : s1[c & 31]; };
+        if constexpr (BIAS) {
 #pragma unroll
-        for (int c = 0; c < 64; ++c) {
-          float v = __uint_as_float(sv(c)) * scale;
-          if constexpr (BIAS) v += fmaf(slope, static_cast<float>(c), bias0);
-          sv(c) = __float_as_uint(v);
+          for (int c = 0; c < 64; ++c)
+            sv(c) = __float_as_uint(fmaf(__uint_as_float(sv(c)), scale, fmaf(slope, static_cast<float>(c), bias0)));
         }
         const bool partly = j0 + kTileN - 1 > i || (j0 < lo && j0 + kTileN > keep);
         if (__any_sync(0xffffffffu, partly)) {
@@ -605,7 +538,8 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
         float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
         for (int c = 0; c < 64; ++c) mx[c & 3] = fmaxf(mx[c & 3], __uint_as_float(sv(c)));
-        const float tmax = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
+        const float mraw = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
+        const float tmax = BIAS ? mraw : mraw * scale;  // without bias the scale (> 0) is applied with the maximum
         float factor = 1.0f;
         if (tmax > m_used + kRescaleThreshold) {  // false while nothing is visible (both -inf)
           factor = ex2(m_used - tmax);            // 0 at the first visible tile
@@ -631,7 +565,9 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
         uint32_t w[32];
 #pragma unroll
         for (int x = 0; x < 32; ++x) {
-          const float p0 = ex2(__uint_as_float(sv(2 * x)) - m_ref), p1 = ex2(__uint_as_float(sv(2 * x + 1)) - m_ref);
+          const float z0 = __uint_as_float(sv(2 * x)), z1 = __uint_as_float(sv(2 * x + 1));
+          const float p0 = ex2(BIAS ? z0 - m_ref : fmaf(z0, scale, -m_ref));
+          const float p1 = ex2(BIAS ? z1 - m_ref : fmaf(z1, scale, -m_ref));
           ps[x & 3] += p0 + p1;
           w[x] = pack_bf16(p0, p1);
         }
@@ -645,6 +581,51 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
       ok = wait_all(bar_done, s & 1, 81);
       if (!ok) break;
       const float inv = 1.0f / l_sum;
+      if (pl.staged) {
+        // first map: a1 as fp16 into this thread's own output row; second map: a1 - lambda a2, scaled by its root
+        // mean square, over it (two passes over O)
+        float ss = 0.f;
+        for (int pass = s == 0 ? 1 : 0; pass < 2; ++pass) {
+          const float scl = s == 0 ? inv : a.out_scale / sqrtf(ss / static_cast<float>(a.vdim_true) + a.eps);
+#pragma unroll 1
+          for (int c = 0; c < pl.v_cols / 32; ++c) {
+            uint32_t o[32];
+            ptx::tmem_ld_32x32(col_o + lane_off + c * 32, o);
+            ptx::tmem_ld_wait();
+            uint4* d4 = reinterpret_cast<uint4*>(out_row + c * 32);
+#pragma unroll
+            for (int x = 0; x < 4; ++x) {
+              if (c * 32 + x * 8 >= a.vdim) break;
+              uint32_t w4[4];
+              float f[8];
+              if (s == 0) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                  const __half2 h = __floats2half2_rn(__uint_as_float(o[8 * x + 2 * e]) * scl,
+                                                      __uint_as_float(o[8 * x + 2 * e + 1]) * scl);
+                  w4[e] = *reinterpret_cast<const uint32_t*>(&h);
+                }
+              } else {
+                const uint4 first = d4[x];
+                const uint32_t fw[4] = {first.x, first.y, first.z, first.w};
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                  const float2 a1 = __half22float2(*reinterpret_cast<const __half2*>(&fw[e]));
+                  f[2 * e] = fmaf(-a.lambda * inv, __uint_as_float(o[8 * x + 2 * e]), a1.x);
+                  f[2 * e + 1] = fmaf(-a.lambda * inv, __uint_as_float(o[8 * x + 2 * e + 1]), a1.y);
+                  ss = pass == 0 ? fmaf(f[2 * e], f[2 * e], fmaf(f[2 * e + 1], f[2 * e + 1], ss)) : ss;
+                  w4[e] = pack_bf16(f[2 * e] * scl, f[2 * e + 1] * scl);
+                }
+              }
+              if (live && pass == 1) d4[x] = make_uint4(w4[0], w4[1], w4[2], w4[3]);
+            }
+            __syncwarp();
+          }
+        }
+        ptx::tc_fence_before();
+        ptx::mbar_arrive(bar_oread);
+        continue;
+      }
 #pragma unroll 1
       for (int c = 0; c < pl.v_cols / 32; ++c) {
         uint32_t o[32];
@@ -672,8 +653,7 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
       ptx::tc_fence_before();
       ptx::mbar_arrive(bar_oread);
     }
-    if (ok) {
-      const int64_t t = row0 + min(r, n_tok - 1);
+    if (ok && !pl.staged) {
       for (int n = 0; n < n_out; ++n) {
         float scl = 1.0f;
         if (diff) {
@@ -689,7 +669,7 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
           }
           scl = a.out_scale / sqrtf(ss / static_cast<float>(a.vdim_true) + a.eps);
         }
-        __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(a.out) + t * a.ldo + static_cast<int64_t>(out0 + n) * a.vdim;
+        __nv_bfloat16* dst = out_row + static_cast<int64_t>(n) * a.vdim;
 #pragma unroll 1
         for (int c = 0; c < pl.v_cols / 32; ++c) {
           uint32_t o[32];
@@ -770,7 +750,20 @@ extern "C" int fr_mix_attn_tc_fits(int mix_kind, int heads, int kv_heads, int di
   return heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && mix::plan_tc(mix_kind, heads, kv_heads, dim, vdim, &pl) ? 1 : 0;
 }
 
-extern "C" int fr_mix_attn_tc(const fr_mix_attn* a, const int32_t* tiles, int n_tiles, int n_rows, cudaStream_t stream) {
+extern "C" int64_t fr_mix_attn_tc_scratch(const fr_mix_attn* a, int n_tiles, int max_pos, int64_t budget) {
+  if (a == nullptr || a->heads <= 0 || a->kv_heads <= 0 || a->mask_size <= 0 || n_tiles <= 0 || max_pos < 0) return 0;
+  mix::TcPlan pl;
+  if (a->mix != FR_MIX_TALK || !mix::plan_tc(a->mix, a->heads, a->kv_heads, a->dim, a->vdim, &pl)) return 0;
+  if (a->kv_heads * pl.out_blocks < 2) return 0;  // every map is computed once as it is
+  const int64_t per_tile = talk_tc_tile_bytes(*a, max_pos);
+  int64_t tiles = budget / per_tile;
+  if (tiles > n_tiles) tiles = n_tiles;
+  // too few tiles at a time leave SMs idle: the maps are recomputed per v head instead
+  return tiles < n_tiles && tiles * a->heads < 96 ? 0 : tiles * per_tile;
+}
+
+extern "C" int fr_mix_attn_tc(const fr_mix_attn* a, const int32_t* tiles, int n_tiles, int n_rows, int max_pos, void* scratch,
+                              int64_t scratch_bytes, cudaStream_t stream) {
   const int st = mix::check_args(a);
   if (st != FR_OK) return st;
   FR_CHECK_ARG(tiles && n_tiles >= 0 && n_rows >= 0);
@@ -778,6 +771,10 @@ extern "C" int fr_mix_attn_tc(const fr_mix_attn* a, const int32_t* tiles, int n_
   mix::TcPlan pl;
   FR_CHECK_SUPPORTED(a->dtype == 0 && a->num_slots >= mix::kTileN &&
                      mix::plan_tc(a->mix, a->heads, a->kv_heads, a->dim, a->vdim, &pl));
+  if (scratch != nullptr && scratch_bytes > 0) {
+    FR_CHECK_ARG(a->mix == FR_MIX_TALK && aligned16(scratch) && max_pos >= 0);
+    return talk_tc(*a, tiles, n_tiles, n_rows, max_pos, scratch, scratch_bytes, stream);
+  }
   const bool diff = a->mix == FR_MIX_DIFF;
   const int n_src = diff ? 2 * a->heads : a->heads, k_heads = diff ? 2 * a->kv_heads : a->kv_heads;
   CUtensorMap tq, tk, tv;
@@ -789,12 +786,13 @@ extern "C" int fr_mix_attn_tc(const fr_mix_attn* a, const int32_t* tiles, int n_
   if (!status) return FR_ERR_CUDA;
   dim3 grid(n_tiles, diff ? a->heads : a->kv_heads * pl.out_blocks);
   static PerDeviceFlag f0, f1;
-  if (a->slopes != nullptr) {
+  if (a->slopes != nullptr || !(a->scale > 0.f)) {
     if (ensure_dyn_smem(f1, mix::mix_tc_kernel<true>, 227 * 1024) != FR_OK) return FR_ERR_CUDA;
-    mix::mix_tc_kernel<true><<<grid, mix::kTcThreads, pl.smem, stream>>>(tq, tk, tv, *a, pl, tiles, status);
+    return launch_kernel(mix::mix_tc_kernel<true>, grid, mix::kTcThreads, pl.smem, stream, n_rows <= kPdlRows, tq, tk, tv, *a, pl,
+                         tiles, status);
   } else {
     if (ensure_dyn_smem(f0, mix::mix_tc_kernel<false>, 227 * 1024) != FR_OK) return FR_ERR_CUDA;
-    mix::mix_tc_kernel<false><<<grid, mix::kTcThreads, pl.smem, stream>>>(tq, tk, tv, *a, pl, tiles, status);
+    return launch_kernel(mix::mix_tc_kernel<false>, grid, mix::kTcThreads, pl.smem, stream, n_rows <= kPdlRows, tq, tk, tv, *a, pl,
+                         tiles, status);
   }
-  return launch_status();
 }

@@ -125,14 +125,24 @@ __device__ __forceinline__ void rows_dot(const T* __restrict__ a, int64_t lda, c
   }
 }
 
+// Start four weight rows on their way into L2 (weights never change: this may run before griddepcontrol.wait, while
+// the previous kernel is still working).
+template <typename T>
+__device__ __forceinline__ void prefetch_rows(const T* const (&w)[4], int K, int kwarp, int ks) {
+  constexpr int kLine = 128 / sizeof(T);
+  const int lane = threadIdx.x & 31;
+#pragma unroll
+  for (int r = 0; r < 4; ++r)
+    for (int k = (kwarp * 32 + lane) * kLine; k < K; k += ks * 32 * kLine)
+      asm volatile("prefetch.global.L2 [%0];" ::"l"(w[r] + k));
+}
+
 template <typename T, int MB>
 __global__ void __launch_bounds__(kRowsThreads)
 dense_rows_proj_kernel(const T* __restrict__ a, int64_t lda, const T* __restrict__ w, int64_t ldw, int M, int N, int K,
                        const __grid_constant__ Segs sg, int ks) {
   constexpr bool kFast = sizeof(T) == 2;
   __shared__ float red[8][4 * MB];
-  ptx::griddep_wait();
-  ptx::griddep_launch_dependents();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int groups_per_cta = (kRowsThreads / 32) / ks;
   const int grp = blockIdx.x * groups_per_cta + warp / ks;  // group of four weight rows
@@ -140,11 +150,11 @@ dense_rows_proj_kernel(const T* __restrict__ a, int64_t lda, const T* __restrict
   const bool live = grp * 4 < N;
   int si = 0, c0 = 0;
   float acc[4][MB] = {};
+  const T* wr[4] = {};
   if (live) {
     si = seg_of(sg, grp * 4);
     const fr_out_segment& s = sg.s[si];
     const int local = grp * 4 - s.n0;
-    const T* wr[4];
     if (s.kind == FR_SEG_SWIGLU) {  // two channels: rows {gate c, gate c + 1, up c, up c + 1}
       c0 = local / 2;
       const int64_t g = s.n0 + (c0 / 32) * 64 + c0 % 32;
@@ -157,8 +167,11 @@ dense_rows_proj_kernel(const T* __restrict__ a, int64_t lda, const T* __restrict
 #pragma unroll
       for (int r = 0; r < 4; ++r) wr[r] = w + static_cast<int64_t>(grp * 4 + r) * ldw;
     }
-    rows_dot<T, MB>(a, lda, wr, K, kwarp, ks, M, acc);
+    prefetch_rows<T>(wr, K, kwarp, ks);
   }
+  ptx::griddep_wait();
+  ptx::griddep_launch_dependents();
+  if (live) rows_dot<T, MB>(a, lda, wr, K, kwarp, ks, M, acc);
 #pragma unroll
   for (int r = 0; r < 4; ++r)
 #pragma unroll
@@ -191,21 +204,31 @@ template <typename T, int MB>
 __global__ void __launch_bounds__(kRowsThreads)
 dense_rows_gated_kernel(const __grid_constant__ Parts pt, float* __restrict__ x, int64_t ldx, int M, int N, int ks) {
   __shared__ float red[8][2][4 * MB];
-  ptx::griddep_wait();
-  ptx::griddep_launch_dependents();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int groups_per_cta = (kRowsThreads / 32) / ks;
   const int grp = blockIdx.x * groups_per_cta + warp / ks;
   const int kwarp = warp % ks;
   const bool live = grp * 4 < N;
+  auto weight_rows = [&](const fr_gated_part& part, const T* (&wr)[4]) {
+#pragma unroll
+    for (int r = 0; r < 4; ++r)
+      wr[r] = static_cast<const T*>(part.w) + static_cast<int64_t>(min(grp * 4 + r, N - 1)) * part.ldw;
+  };
+  if (live) {
+    for (int p = 0; p < pt.n; ++p) {
+      const T* wr[4];
+      weight_rows(pt.p[p], wr);
+      prefetch_rows<T>(wr, pt.p[p].K, kwarp, ks);
+    }
+  }
+  ptx::griddep_wait();
+  ptx::griddep_launch_dependents();
   for (int p = 0; p < pt.n; ++p) {
     const fr_gated_part& part = pt.p[p];
     float acc[4][MB] = {};
     if (live) {
       const T* wr[4];
-#pragma unroll
-      for (int r = 0; r < 4; ++r)
-        wr[r] = static_cast<const T*>(part.w) + static_cast<int64_t>(min(grp * 4 + r, N - 1)) * part.ldw;
+      weight_rows(part, wr);
       rows_dot<T, MB>(static_cast<const T*>(part.a), part.lda, wr, part.K, kwarp, ks, M, acc);
     }
 #pragma unroll
@@ -713,8 +736,8 @@ static int launch_tc(const TcArgs& g, const fr_gated_part* parts, cudaStream_t s
   const int64_t units = static_cast<int64_t>(ceil_div(g.M, kBlockM)) * ceil_div(g.N, BLOCK_N) *
                         (EPI == kEpiPartial ? g.splits[0] + g.splits[1] : 1);
   const int grid = static_cast<int>(units < device_sm_count() ? units : device_sm_count());
-  kern<<<grid, kThreads, Cfg<BLOCK_N>::kSmemBytes, stream>>>(ta[0], tb[0], ta[1], tb[1], g, status);
-  return launch_status();
+  return launch_kernel(kern, grid, kThreads, Cfg<BLOCK_N>::kSmemBytes, stream, g.M <= kPdlRows, ta[0], tb[0], ta[1], tb[1], g,
+                       status);
 }
 
 // Widest tile that still gives every SM one.
@@ -741,11 +764,10 @@ static int launch_rows_proj(const void* a, int64_t lda, const void* w, int64_t l
   const int grid = ceil_div(ceil_div(N, 4), (kRowsThreads / 32) / ks);
   const T* A = static_cast<const T*>(a);
   const T* W = static_cast<const T*>(w);
-  if (M == 1) dense_rows_proj_kernel<T, 1><<<grid, kRowsThreads, 0, stream>>>(A, lda, W, ldw, M, N, K, sg, ks);
-  else if (M == 2) dense_rows_proj_kernel<T, 2><<<grid, kRowsThreads, 0, stream>>>(A, lda, W, ldw, M, N, K, sg, ks);
-  else if (M <= 4) dense_rows_proj_kernel<T, 4><<<grid, kRowsThreads, 0, stream>>>(A, lda, W, ldw, M, N, K, sg, ks);
-  else dense_rows_proj_kernel<T, 8><<<grid, kRowsThreads, 0, stream>>>(A, lda, W, ldw, M, N, K, sg, ks);
-  return launch_status();
+  if (M == 1) return launch_kernel(dense_rows_proj_kernel<T, 1>, grid, kRowsThreads, 0, stream, true, A, lda, W, ldw, M, N, K, sg, ks);
+  if (M == 2) return launch_kernel(dense_rows_proj_kernel<T, 2>, grid, kRowsThreads, 0, stream, true, A, lda, W, ldw, M, N, K, sg, ks);
+  if (M <= 4) return launch_kernel(dense_rows_proj_kernel<T, 4>, grid, kRowsThreads, 0, stream, true, A, lda, W, ldw, M, N, K, sg, ks);
+  return launch_kernel(dense_rows_proj_kernel<T, 8>, grid, kRowsThreads, 0, stream, true, A, lda, W, ldw, M, N, K, sg, ks);
 }
 
 template <typename T>
@@ -754,11 +776,10 @@ static int launch_rows_gated(const Parts& pt, float* x, int64_t ldx, int M, int 
   for (int p = 0; p < pt.n; ++p) K = K > pt.p[p].K ? K : pt.p[p].K;
   const int ks = rows_ks(N, K);
   const int grid = ceil_div(ceil_div(N, 4), (kRowsThreads / 32) / ks);
-  if (M == 1) dense_rows_gated_kernel<T, 1><<<grid, kRowsThreads, 0, stream>>>(pt, x, ldx, M, N, ks);
-  else if (M == 2) dense_rows_gated_kernel<T, 2><<<grid, kRowsThreads, 0, stream>>>(pt, x, ldx, M, N, ks);
-  else if (M <= 4) dense_rows_gated_kernel<T, 4><<<grid, kRowsThreads, 0, stream>>>(pt, x, ldx, M, N, ks);
-  else dense_rows_gated_kernel<T, 8><<<grid, kRowsThreads, 0, stream>>>(pt, x, ldx, M, N, ks);
-  return launch_status();
+  if (M == 1) return launch_kernel(dense_rows_gated_kernel<T, 1>, grid, kRowsThreads, 0, stream, true, pt, x, ldx, M, N, ks);
+  if (M == 2) return launch_kernel(dense_rows_gated_kernel<T, 2>, grid, kRowsThreads, 0, stream, true, pt, x, ldx, M, N, ks);
+  if (M <= 4) return launch_kernel(dense_rows_gated_kernel<T, 4>, grid, kRowsThreads, 0, stream, true, pt, x, ldx, M, N, ks);
+  return launch_kernel(dense_rows_gated_kernel<T, 8>, grid, kRowsThreads, 0, stream, true, pt, x, ldx, M, N, ks);
 }
 
 static bool operand_ok(const void* p, int64_t ld, int K) {

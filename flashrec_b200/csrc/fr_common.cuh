@@ -79,6 +79,29 @@ static inline int device_sm_count() {
   return cache[d];
 }
 
+// Launch with or without programmatic dependence on the previous kernel of the stream: with it the kernel may start
+// while its predecessor is finishing and must execute griddepcontrol.wait before it touches what others write.
+template <class... KArgs, class... Args>
+static inline int launch_kernel(void (*kern)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream, bool pdl,
+                                Args... args) {
+  cudaLaunchConfig_t cfg{};
+  cfg.gridDim = grid;
+  cfg.blockDim = block;
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = stream;
+  cudaLaunchAttribute attr[1];
+  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[0].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = pdl ? 1 : 0;
+  if (cudaLaunchKernelEx(&cfg, kern, static_cast<KArgs>(args)...) != cudaSuccess) {
+    cudaGetLastError();
+    return FR_ERR_CUDA;
+  }
+  return FR_OK;
+}
+constexpr int kPdlRows = 2048;  // batches up to this many rows launch their kernels with the dependence
+
 static inline bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; }
 
 static inline int ceil_div(int64_t a, int64_t b) { return static_cast<int>((a + b - 1) / b); }

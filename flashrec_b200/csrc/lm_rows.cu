@@ -125,6 +125,115 @@ __device__ __forceinline__ float conv_tap(const T* __restrict__ u, int64_t ldu, 
   return ld_f(st + static_cast<int64_t>(taps - 1 + e - back) * C + c);
 }
 
+// Eight channels per thread, 16-byte accesses. ONE: one token per request (and per blockIdx.x). Otherwise a thread
+// walks up to kConvRun consecutive tokens with the window of past values in registers; it reloads the window where
+// another request begins.
+constexpr int kConvRun = 16;
+
+template <typename T>
+__device__ __forceinline__ void conv_load8(const T* p, float (&v)[8]) {
+  if constexpr (sizeof(T) == 2) {
+    const uint4 a = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      v[2 * i] = __uint_as_float(w[i] << 16);
+      v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+    }
+  } else {
+    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+    v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+  }
+}
+template <typename T>
+__device__ __forceinline__ void conv_store8(T* p, const float (&v)[8]) {
+  if constexpr (sizeof(T) == 2) {
+    *reinterpret_cast<uint4*>(p) =
+        make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
+  } else {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+  }
+}
+
+template <typename T, int TAPS, bool ONE>
+__global__ void __launch_bounds__(128)
+conv_vec_kernel(const T* __restrict__ u, int64_t ldu, const float* __restrict__ w, int C, const __grid_constant__ ConvOuts outs,
+                T* __restrict__ state, const int64_t* __restrict__ state_slots, const int32_t* __restrict__ tok_req,
+                const int32_t* __restrict__ qo_indptr, const int64_t* __restrict__ pos, int n_tok) {
+  constexpr int P = TAPS - 1;
+  const int c = (blockIdx.y * 128 + threadIdx.x) * 8;
+  float wr[TAPS][8];
+  if (c < C) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+      for (int k = 0; k < TAPS; ++k) wr[k][i] = __ldg(w + static_cast<int64_t>(c + i) * TAPS + k);
+  }
+  ptx::griddep_wait();
+  ptx::griddep_launch_dependents();
+  if (c >= C) return;
+  int oi = 0;
+  while (oi + 1 < outs.n && !(c >= outs.o[oi].c0 && c < outs.o[oi].c0 + outs.o[oi].c)) ++oi;
+  const fr_conv_out& o = outs.o[oi];
+  const bool keep = c >= o.c0 && c < o.c0 + o.c;
+  T* out = static_cast<T*>(o.out) + (c - o.c0);
+  float win[P > 0 ? P : 1][8] = {};
+  const int t0 = ONE ? blockIdx.x : blockIdx.x * kConvRun;
+  const int t1 = ONE ? t0 + 1 : min(t0 + kConvRun, n_tok);
+  int cur = -1;
+  for (int t = t0; t < t1; t += 4) {
+    float v[4][8];
+#pragma unroll
+    for (int x = 0; x < (ONE ? 1 : 4); ++x)
+      if (t + x < t1) conv_load8<T>(u + static_cast<int64_t>(t + x) * ldu + c, v[x]);
+#pragma unroll
+    for (int x = 0; x < (ONE ? 1 : 4); ++x) {
+      if (t + x >= t1) break;
+      const int b = tok_req[t + x];
+      if (b != cur) {  // fill the window: earlier tokens of the batch, then the state, zeros before position 0
+        cur = b;
+        const int64_t p = pos[t + x];
+        const int e = ONE ? 0 : t + x - qo_indptr[b];
+        const T* st = state + state_slots[b] * P * C + c;
+#pragma unroll
+        for (int k = 0; k < P; ++k) {
+          const int back = P - k;
+          if (p < back) {
+#pragma unroll
+            for (int i = 0; i < 8; ++i) win[k][i] = 0.f;
+          } else if (e >= back) {
+            conv_load8<T>(u + static_cast<int64_t>(t + x - back) * ldu + c, win[k]);
+          } else {
+            conv_load8<T>(st + static_cast<int64_t>(k + e) * C, win[k]);
+          }
+        }
+      }
+      float y[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        y[i] = 0.f;
+#pragma unroll
+        for (int k = 0; k < P; ++k) y[i] = fmaf(wr[k][i], win[k][i], y[i]);
+        y[i] = fmaf(wr[P][i], v[x][i], y[i]);
+      }
+      if (keep) conv_store8<T>(out + (o.row_map != nullptr ? o.row_map[t + x] : t + x) * o.ldo, y);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+#pragma unroll
+        for (int k = 0; k + 1 < P; ++k) win[k][i] = win[k + 1][i];
+        if (P > 0) win[P - 1][i] = v[x][i];
+      }
+      if (ONE && P > 0) {  // the window is the request's new state
+        T* st = state + state_slots[b] * P * C + c;
+#pragma unroll
+        for (int k = 0; k < P; ++k) conv_store8<T>(st + static_cast<int64_t>(k) * C, win[k]);
+      }
+    }
+  }
+}
+
 // One token and 256 channels per CTA. ONE: every request has one token, so the thread that has read a channel's
 // state also advances it.
 template <typename T, bool ONE>
@@ -184,6 +293,23 @@ static int launch_conv(const void* u, int64_t ldu, const float* w, int taps, int
                        int one, cudaStream_t stream) {
   const T* up = static_cast<const T*>(u);
   T* st = static_cast<T*>(state);
+  bool vec = C % 8 == 0 && ldu % 8 == 0 && aligned16(u) && aligned16(state) && taps >= 2 && taps <= 4;
+  for (int i = 0; i < outs.n; ++i)
+    vec = vec && outs.o[i].c0 % 8 == 0 && outs.o[i].c % 8 == 0 && outs.o[i].ldo % 8 == 0 && aligned16(outs.o[i].out);
+  if (vec) {
+    auto go = [&](auto one_kern, auto run_kern) -> int {
+      const dim3 g(one ? Tn : ceil_div(Tn, kConvRun), ceil_div(C, 1024));
+      return launch_kernel(one ? one_kern : run_kern, g, 128, 0, stream, Tn <= kPdlRows, up, ldu, w, C, outs, st, slots, tok_req,
+                           qo, pos, Tn);
+    };
+    int r = FR_OK;
+    if (taps == 2) r = go(&conv_vec_kernel<T, 2, true>, &conv_vec_kernel<T, 2, false>);
+    if (taps == 3) r = go(&conv_vec_kernel<T, 3, true>, &conv_vec_kernel<T, 3, false>);
+    if (taps == 4) r = go(&conv_vec_kernel<T, 4, true>, &conv_vec_kernel<T, 4, false>);
+    if (r != FR_OK || one) return r;
+    conv_state_kernel<T><<<dim3(n_req, ceil_div(C, 256)), 256, 0, stream>>>(up, ldu, taps, C, st, slots, qo);
+    return launch_status();
+  }
   dim3 grid(Tn, ceil_div(C, 256));
   if (one) {
     short_conv_kernel<T, true><<<grid, 256, 0, stream>>>(up, ldu, w, taps, C, outs, st, slots, tok_req, qo, pos);
@@ -202,13 +328,8 @@ static int launch_norm(float* x, int64_t ldx, const float* weight, float offset,
   const bool vec = W % 4 == 0 && W <= kNormThreads * 4 * kNormVec && ldx % 4 == 0 && ldo % 4 == 0 && aligned16(x) &&
                    aligned16(weight) && aligned16(out) && (partials == nullptr || (aligned16(partials) && ps % 4 == 0));
   T* o = static_cast<T*>(out);
-  if (vec)
-    norm_kernel<T, true><<<M, kNormThreads, 0, stream>>>(x, ldx, weight, offset, eps, partials, n_partials, ps, row_idx, o,
-                                                         ldo, W);
-  else
-    norm_kernel<T, false><<<M, kNormThreads, 0, stream>>>(x, ldx, weight, offset, eps, partials, n_partials, ps, row_idx, o,
-                                                          ldo, W);
-  return launch_status();
+  return launch_kernel(vec ? norm_kernel<T, true> : norm_kernel<T, false>, M, kNormThreads, 0, stream, M <= kPdlRows, x, ldx,
+                       weight, offset, eps, partials, n_partials, ps, row_idx, o, ldo, W);
 }
 
 }  // namespace lm

@@ -205,7 +205,7 @@ class DibepelForCausalLM:
     """Embedding -> layer runs -> final norm -> logits. ``forward`` returns the residual stream (and the last
     layer's pending partials); ``logits`` turns chosen rows of it into fp32 logits."""
 
-    SOURCES = ("capi", "dense_proj", "lm_rows", "attn_mix")  # what a build of this family alone compiles
+    SOURCES = ("capi", "dense_proj", "lm_rows", "attn_mix", "attn_talk")  # what a build of this family alone compiles
 
     def __init__(self, cfg: DibepelConfig, tensors: Dict[str, torch.Tensor], dtype: torch.dtype, device):
         self.cfg, self.dtype, self.device = cfg, dtype, torch.device(device)

@@ -8,6 +8,7 @@ both. bfloat16 runs on the tensor cores, float32 is true 32-bit arithmetic throu
 from __future__ import annotations
 
 import ctypes
+import os
 from dataclasses import dataclass
 from typing import List, Optional, Sequence, Tuple
 
@@ -21,6 +22,7 @@ from flashrec_b200.kvcache import CacheSpec
 SEG = {"store": _lib.FR_SEG_STORE, "swiglu": _lib.FR_SEG_SWIGLU, "sigmoid": _lib.FR_SEG_SIGMOID,
        "store_f32": _lib.FR_SEG_STORE_F32}
 _SCORE_SCRATCH_BYTES = 256 << 20
+_MAP_SCRATCH_BYTES = int(os.environ.get("FR_MAP_SCRATCH_MB", "224")) << 20  # maps of talking heads between their kernels
 
 
 def ceil_to(n: int, m: int) -> int:
@@ -251,7 +253,10 @@ class MixAttention:
             keys = self.cache.max_keys(batch.max_pos) if max_keys is None else max_keys
             self._rows(a, n_row, keys, counters, s, q.device)
         if n_row < t:
-            call("fr_mix_attn_tc", ctypes.byref(a), ptr(batch.tiles), int(batch.tiles.shape[0]), t, s)
+            n_tiles = int(batch.tiles.shape[0])
+            size = _lib.load().fr_mix_attn_tc_scratch(ctypes.byref(a), n_tiles, batch.max_pos, _MAP_SCRATCH_BYTES)
+            scratch = torch.empty(size, dtype=torch.uint8, device=q.device) if size > 0 else None
+            call("fr_mix_attn_tc", ctypes.byref(a), ptr(batch.tiles), n_tiles, t, batch.max_pos, ptr(scratch), max(size, 0), s)
         return out
 
     def _rows(self, a: FrMixAttn, n_row: int, keys: int, counters: torch.Tensor, stream, device) -> None:

@@ -42,7 +42,7 @@ def _load_dibepel(path: str, cfg: dict, dtype: torch.dtype, device):
 FAMILIES: List[ModelFamily] = [
     ModelFamily("qwen3-fp8", _is_qwen3, _load_qwen3, (torch.bfloat16,)),
     ModelFamily("dibepel", lambda c: c.get("architecture") == "Dibepel", _load_dibepel, (torch.bfloat16, torch.float32),
-                ("capi", "dense_proj", "lm_rows", "attn_mix")),
+                ("capi", "dense_proj", "lm_rows", "attn_mix", "attn_talk")),
 ]
 
 

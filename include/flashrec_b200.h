@@ -629,8 +629,13 @@ int64_t fr_mix_attn_rows_scratch(int mix, int heads, int vdim, int n_rows, int m
 
 /* bf16 prompts on the tensor cores: tiles [n_tiles, 3] of {request, first row in the batch, rows} (at most 128
  * rows). The cache is paged: positions [64 p, 64 p + 64) of a request occupy 64 consecutive slots that start at
- * a multiple of 64. FR_ERR_UNSUPPORTED when the head sizes do not fit (fr_mix_attn_tc_fits tells). */
-int fr_mix_attn_tc(const struct fr_mix_attn* a, const int32_t* tiles, int n_tiles, int n_rows, cudaStream_t stream);
+ * a multiple of 64. FR_ERR_UNSUPPORTED when the head sizes do not fit (fr_mix_attn_tc_fits tells). scratch (may be
+ * null): fr_mix_attn_tc_scratch(...) bytes, or any smaller multiple of its value for one tile; with it TALK
+ * writes the maps once, mixes them in place of recomputing them per v head, and works through the tiles in as many
+ * blocks as the scratch takes. max_pos: largest position of the batch. */
+int fr_mix_attn_tc(const struct fr_mix_attn* a, const int32_t* tiles, int n_tiles, int n_rows, int max_pos, void* scratch,
+                   int64_t scratch_bytes, cudaStream_t stream);
+int64_t fr_mix_attn_tc_scratch(const struct fr_mix_attn* a, int n_tiles, int max_pos, int64_t budget);
 int fr_mix_attn_tc_fits(int mix, int heads, int kv_heads, int dim, int vdim);
 
 #ifdef __cplusplus
