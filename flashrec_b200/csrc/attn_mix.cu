@@ -19,29 +19,32 @@ int64_t talk_tc_tile_bytes(const fr_mix_attn& a, int max_pos);
 namespace mix {
 
 constexpr int kKeyBlock = 64;
+constexpr int kMaxPer = 4;  // key blocks per CTA of the scores kernel when the batch fills the GPU anyway
 
 // ---------------------------------------------------------------------------
-// scores of one row, one k head and 64 keys for every source map that reads that k head; per block and map the
+// scores of one row, one k head and `per` blocks of 64 keys for every source map that reads that k head; per block and map the
 // maximum and the sum of exponentials
 // ---------------------------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(128)
-mix_scores_kernel(const __grid_constant__ fr_mix_attn a, int row0, int max_keys, int n_blocks, float* __restrict__ scores,
-                  float2* __restrict__ stats) {
+mix_scores_kernel(const __grid_constant__ fr_mix_attn a, int row0, int max_keys, int n_blocks, int per,
+                  float* __restrict__ scores, float2* __restrict__ stats) {
   extern __shared__ float sm[];
   const int rep = a.heads / a.kv_heads;
   const int n_src = a.mix == FR_MIX_DIFF ? 2 * a.heads : a.heads;
   float* qs = sm;                       // [rep][dim]
-  float* sc = sm + rep * a.dim;         // [rep][64]
+  float* sc = sm + rep * a.dim;         // [rep][64 per]
+  __shared__ int64_t slots[kMaxPer * kKeyBlock];
   ptx::griddep_wait();
   ptx::griddep_launch_dependents();
   const int lrow = blockIdx.z, kh = blockIdx.y, blk = blockIdx.x;
   const int64_t t = row0 + lrow;
   const int64_t i = a.pos[t];
   const Visible vis = visible_keys(a, i, max_keys);
-  const int k0 = blk * kKeyBlock;
+  const int span = per * kKeyBlock;
+  const int k0 = blk * span;
   if (k0 >= vis.n) return;
-  const int nk = min(kKeyBlock, vis.n - k0);
+  const int nk = min(span, vis.n - k0);
   const T* q = static_cast<const T*>(a.q) + t * a.ldq;
   for (int e = threadIdx.x; e < rep * (a.dim / 8); e += 128) {
     const int s = e / (a.dim / 8), c = e % (a.dim / 8) * 8;
@@ -50,51 +53,73 @@ mix_scores_kernel(const __grid_constant__ fr_mix_attn a, int row0, int max_keys,
 #pragma unroll
     for (int x = 0; x < 8; ++x) qs[s * a.dim + c + x] = v[x];
   }
+  const int64_t table_row = a.req_rows[a.tok_req[t]];
+  for (int e = threadIdx.x; e < nk; e += 128) slots[e] = slot_of(a, table_row, vis.key(k0 + e));
   __syncthreads();
   int lanes = 1;  // lanes per key
   while (lanes < 32 && lanes * 8 < a.dim) lanes *= 2;
   const int lane_k = threadIdx.x % lanes;
-  const int64_t table_row = a.req_rows[a.tok_req[t]];
   const T* kc = static_cast<const T*>(a.k) + static_cast<int64_t>(kh) * a.dim;
   const int keys_at_once = 128 / lanes;
-  for (int kb = 0; kb < kKeyBlock; kb += keys_at_once) {  // CTA-uniform trip count: shuffles below are whole-warp
-    const int kk = kb + threadIdx.x / lanes;
-    const bool live = kk < nk;
-    const int64_t j = vis.key(k0 + (live ? kk : 0));
-    const T* kr = kc + slot_of(a, table_row, j) * a.ldk;
-    for (int s0 = 0; s0 < rep; s0 += 4) {
-      float acc[4] = {};
-      for (int c = lane_k * 8; c < a.dim; c += lanes * 8) {
-        float v[8];
-        load8<T>(kr + c, v);
+  const bool one_chunk = lanes * 8 >= a.dim;  // a lane holds its share of a key in registers
+  const bool in_dim = lane_k * 8 < a.dim;
+  // groups of up to four keys per thread, their rows in flight together; trip counts are CTA-uniform (the shuffles
+  // are whole-warp)
+  for (int kb = 0; kb < span; kb += 4 * keys_at_once) {
+    float kv[4][8] = {};
+    const T* kr[4];
 #pragma unroll
-        for (int s = 0; s < 4; ++s)
-          if (s0 + s < rep) {
+    for (int x = 0; x < 4; ++x) {
+      const int kk = kb + x * keys_at_once + threadIdx.x / lanes;
+      kr[x] = kc + slots[min(kk, nk - 1)] * a.ldk;
+      if (one_chunk && in_dim && kk < nk) load8<T>(kr[x] + lane_k * 8, kv[x]);
+    }
 #pragma unroll
-            for (int x = 0; x < 8; ++x) acc[s] = fmaf(v[x], qs[(s0 + s) * a.dim + c + x], acc[s]);
+    for (int x = 0; x < 4; ++x) {
+      if (kb + x * keys_at_once >= span) break;
+      const int kk = kb + x * keys_at_once + threadIdx.x / lanes;
+      const bool live = kk < nk;
+      const float dist = static_cast<float>(i - vis.key(k0 + (live ? kk : 0)));
+      for (int s = 0; s < rep; ++s) {
+        const float* qr = qs + s * a.dim;
+        float acc = 0.f;
+        if (one_chunk) {
+          if (in_dim) {
+            const float4 q0 = *reinterpret_cast<const float4*>(qr + lane_k * 8);
+            const float4 q1 = *reinterpret_cast<const float4*>(qr + lane_k * 8 + 4);
+            acc = kv[x][0] * q0.x + kv[x][1] * q0.y + kv[x][2] * q0.z + kv[x][3] * q0.w + kv[x][4] * q1.x + kv[x][5] * q1.y +
+                  kv[x][6] * q1.z + kv[x][7] * q1.w;
           }
-      }
+        } else {
+          for (int c = lane_k * 8; c < a.dim; c += lanes * 8) {
+            float v[8];
+            load8<T>(kr[x] + c, v);
 #pragma unroll
-      for (int s = 0; s < 4; ++s) {
-        for (int o = lanes / 2; o > 0; o >>= 1) acc[s] += __shfl_xor_sync(0xffffffffu, acc[s], o);
-        if (lane_k == 0 && s0 + s < rep && kk < kKeyBlock) {
-          float v = acc[s] * a.scale;
-          if (a.slopes != nullptr) v -= a.slopes[source_of(a, kh, s0 + s)] * static_cast<float>(i - j);
-          sc[(s0 + s) * kKeyBlock + kk] = live ? v : -INFINITY;
+            for (int y = 0; y < 8; ++y) acc = fmaf(v[y], qr[c + y], acc);
+          }
+        }
+        for (int o = lanes / 2; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+        if (lane_k == 0 && kk < span) {
+          float v = acc * a.scale;
+          if (a.slopes != nullptr) v -= a.slopes[source_of(a, kh, s)] * dist;
+          sc[s * span + kk] = live ? v : -INFINITY;
         }
       }
     }
   }
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int s = warp; s < rep; s += 4) {
+  for (int e = warp; e < rep * per; e += 4) {  // (map, block of 64)
+    const int s = e / per, sub = e % per, c0 = sub * kKeyBlock;
+    if (c0 >= nk) continue;
     const int64_t row = static_cast<int64_t>(lrow) * n_src + source_of(a, kh, s);
-    const float v0 = sc[s * kKeyBlock + lane], v1 = sc[s * kKeyBlock + 32 + lane];
+    const float v0 = sc[s * span + c0 + lane], v1 = sc[s * span + c0 + 32 + lane];
     const float m = warp_max(fmaxf(v0, v1));
     const float l = warp_sum(expf(v0 - m) + expf(v1 - m));
-    if (k0 + lane < max_keys) scores[row * max_keys + k0 + lane] = v0;
-    if (k0 + 32 + lane < max_keys) scores[row * max_keys + k0 + 32 + lane] = v1;
-    if (lane == 0) stats[row * n_blocks + blk] = make_float2(m, l);
+    const int k1 = k0 + c0;
+    if (k1 + lane < max_keys) scores[row * max_keys + k1 + lane] = v0;
+    if (k1 + 32 + lane < max_keys) scores[row * max_keys + k1 + 32 + lane] = v1;
+    if (lane == 0) stats[row * n_blocks + blk * per + sub] = make_float2(m, l);
   }
 }
 
@@ -102,7 +127,7 @@ mix_scores_kernel(const __grid_constant__ fr_mix_attn a, int row0, int max_keys,
 // mixture of the maps and product with V for one row, one kv head and one share of the keys
 // ---------------------------------------------------------------------------
 constexpr int kValThreads = 256;
-constexpr int kOutBlock = 8;  // output heads accumulated per pass over the keys
+constexpr int kValKeys = 256;  // keys per pass (weights of all maps in shared memory)
 
 // Root-mean-square scaling (DIFF) and store of one output head; f [vdim] in shared memory.
 template <typename T>
@@ -123,9 +148,10 @@ __device__ __forceinline__ void finish_head(const fr_mix_attn& a, int64_t t, int
   for (int c = threadIdx.x; c < a.vdim; c += kValThreads) st_f(out + c, f[c] * r);
 }
 
-template <typename T>
-__global__ void __launch_bounds__(kValThreads)
-mix_values_kernel(const __grid_constant__ fr_mix_attn a, int row0, int max_keys, int n_blocks, int splits,
+// OB: output heads accumulated per pass over the keys
+template <typename T, int OB>
+__global__ void __launch_bounds__(kValThreads, OB <= 2 ? 4 : (OB == 4 ? 3 : 2))
+mix_values_kernel(const __grid_constant__ fr_mix_attn a, int row0, int max_keys, int n_blocks, int splits, int pass_keys,
                   const float* __restrict__ scores, const float2* __restrict__ stats, float* __restrict__ partial,
                   int32_t* __restrict__ counters) {
   extern __shared__ float sm[];
@@ -135,10 +161,10 @@ mix_values_kernel(const __grid_constant__ fr_mix_attn a, int row0, int max_keys,
   const int my_src = diff ? 2 * rep : a.heads;      // that this kv head's outputs mix
   float* s_m = sm;                                  // [my_src]
   float* s_il = s_m + my_src;                       // [my_src]
-  float* s_p = s_il + my_src;                       // [my_src][64]
-  float* s_w = s_p + my_src * kKeyBlock;            // [8][64]
-  float* s_red = s_w + kOutBlock * kKeyBlock;       // [256][8], afterwards [vdim]
-  int64_t* s_slot = reinterpret_cast<int64_t*>(s_red + kValThreads * 8 + 32);  // [64]
+  float* s_p = s_il + my_src;                       // [my_src][keys per pass]
+  float* s_w = s_p + my_src * pass_keys;            // [OB][keys per pass]
+  float* s_red = s_w + OB * pass_keys;              // [256][8], afterwards [vdim]
+  int64_t* s_slot = reinterpret_cast<int64_t*>(s_red + kValThreads * 8 + 32);
   __shared__ float s_small[kValThreads / 32];
   __shared__ int s_last;
   ptx::griddep_wait();
@@ -150,13 +176,21 @@ mix_values_kernel(const __grid_constant__ fr_mix_attn a, int row0, int max_keys,
   const int blocks = (vis.n + kKeyBlock - 1) / kKeyBlock;
   const int src0 = diff ? 2 * g * rep : 0;
   const int64_t srow = static_cast<int64_t>(lrow) * n_src + src0;
-  for (int s = tid; s < my_src; s += kValThreads) {
+  for (int s = tid >> 5; s < my_src; s += kValThreads / 32) {
     const float2* st = stats + (srow + s) * n_blocks;
     float m = -INFINITY, l = 0.f;
-    for (int b = 0; b < blocks; ++b) m = fmaxf(m, st[b].x);
-    for (int b = 0; b < blocks; ++b) l += st[b].y * expf(st[b].x - m);
-    s_m[s] = m;
-    s_il[s] = 1.0f / l;
+    for (int b = tid & 31; b < blocks; b += 32) {
+      const float2 v = st[b];
+      const float mn = fmaxf(m, v.x);
+      l = l * expf(m - mn) + v.y * expf(v.x - mn);  // the block maxima are finite
+      m = mn;
+    }
+    const float mw = warp_max(m);
+    l = warp_sum(m == -INFINITY ? 0.f : l * expf(m - mw));
+    if ((tid & 31) == 0) {
+      s_m[s] = mw;
+      s_il[s] = 1.0f / l;
+    }
   }
   const int b0 = static_cast<int>(static_cast<int64_t>(blocks) * split / splits);
   const int b1 = static_cast<int>(static_cast<int64_t>(blocks) * (split + 1) / splits);
@@ -166,39 +200,38 @@ mix_values_kernel(const __grid_constant__ fr_mix_attn a, int row0, int max_keys,
   const int vg = tid % vgroups, kl = tid / vgroups;
   const T* vc = static_cast<const T*>(a.v) + static_cast<int64_t>(g) * a.vdim + vg * 8;
   const int64_t part_row = (static_cast<int64_t>(lrow) * splits + split) * a.heads;
-  for (int o0 = 0; o0 < rep; o0 += kOutBlock) {
-    const int no = min(kOutBlock, rep - o0);
-    float acc[kOutBlock][8] = {};
-    for (int b = b0; b < b1; ++b) {
-      const int k0 = b * kKeyBlock, nk = min(kKeyBlock, vis.n - k0);
+  for (int o0 = 0; o0 < rep; o0 += OB) {
+    const int no = min(OB, rep - o0);
+    float acc[OB][8] = {};
+    for (int k0 = b0 * kKeyBlock; k0 < min(b1 * kKeyBlock, vis.n); k0 += pass_keys) {
+      const int nk = min(pass_keys, min(b1 * kKeyBlock, vis.n) - k0);
       __syncthreads();
-      for (int e = tid; e < my_src * kKeyBlock; e += kValThreads) {
-        const int s = e / kKeyBlock, kk = e % kKeyBlock;
-        s_p[e] = kk < nk ? expf(scores[(srow + s) * max_keys + k0 + kk] - s_m[s]) * s_il[s] : 0.f;
-      }
-      if (tid < kKeyBlock) s_slot[tid] = slot_of(a, table_row, vis.key(k0 + min(tid, nk - 1)));
+      for (int s = tid / 64; s < my_src; s += kValThreads / 64)
+        for (int kk = tid % 64; kk < nk; kk += 64)
+          s_p[s * pass_keys + kk] = expf(scores[(srow + s) * max_keys + k0 + kk] - s_m[s]) * s_il[s];
+      if (tid < nk) s_slot[tid] = slot_of(a, table_row, vis.key(k0 + tid));
       __syncthreads();
-      for (int e = tid; e < no * kKeyBlock; e += kValThreads) {
-        const int o = e / kKeyBlock, kk = e % kKeyBlock;
-        float w = 0.f;
-        if (diff) {
-          w = s_p[2 * (o0 + o) * kKeyBlock + kk] - a.lambda * s_p[(2 * (o0 + o) + 1) * kKeyBlock + kk];
-        } else {
-          const float* cf = a.coef + static_cast<int64_t>(g * rep + o0 + o) * a.heads;
-          for (int s = 0; s < my_src; ++s) w = fmaf(__ldg(cf + s), s_p[s * kKeyBlock + kk], w);
+      for (int o = tid / 64; o < no; o += kValThreads / 64)
+        for (int kk = tid % 64; kk < nk; kk += 64) {
+          float w = 0.f;
+          if (diff) {
+            w = s_p[2 * (o0 + o) * pass_keys + kk] - a.lambda * s_p[(2 * (o0 + o) + 1) * pass_keys + kk];
+          } else {
+            const float* cf = a.coef + static_cast<int64_t>(g * rep + o0 + o) * a.heads;
+            for (int s = 0; s < my_src; ++s) w = fmaf(__ldg(cf + s), s_p[s * pass_keys + kk], w);
+          }
+          s_w[o * pass_keys + kk] = w;
         }
-        s_w[e] = w;
-      }
       __syncthreads();
       if (kl < key_lanes) {
-#pragma unroll 2
+#pragma unroll 4
         for (int kk = kl; kk < nk; kk += key_lanes) {
           float v[8];
           load8<T>(vc + s_slot[kk] * a.ldv, v);
 #pragma unroll
-          for (int o = 0; o < kOutBlock; ++o)
+          for (int o = 0; o < OB; ++o)
             if (o < no) {
-              const float w = s_w[o * kKeyBlock + kk];
+              const float w = s_w[o * pass_keys + kk];
 #pragma unroll
               for (int x = 0; x < 8; ++x) acc[o][x] = fmaf(w, v[x], acc[o][x]);
             }
@@ -206,7 +239,7 @@ mix_values_kernel(const __grid_constant__ fr_mix_attn a, int row0, int max_keys,
       }
     }
 #pragma unroll
-    for (int o = 0; o < kOutBlock; ++o) {
+    for (int o = 0; o < OB; ++o) {
       if (o >= no) break;
       const int head = g * rep + o0 + o;
       __syncthreads();
@@ -267,10 +300,24 @@ mix_values_kernel(const __grid_constant__ fr_mix_attn a, int row0, int max_keys,
   }
 }
 
-static int values_smem(const fr_mix_attn& a) {
+static int values_smem(const fr_mix_attn& a, int ob, int pass_keys) {
   const int rep = a.heads / a.kv_heads;
   const int my_src = a.mix == FR_MIX_DIFF ? 2 * rep : a.heads;
-  return (my_src * (2 + kKeyBlock) + kOutBlock * kKeyBlock + kValThreads * 8 + 32) * 4 + kKeyBlock * 8;
+  return (my_src * (2 + pass_keys) + ob * pass_keys + kValThreads * 8 + 32) * 4 + pass_keys * 8;
+}
+
+template <typename T, int OB>
+static int launch_values(const fr_mix_attn& a, int row0, int n_rows, int max_keys, int n_blocks, int splits, const float* scores,
+                         const float2* stats, float* partial, int32_t* counters, bool pdl, cudaStream_t stream) {
+  int pass_keys = kValKeys;  // no more than a split has, and what leaves several CTAs per SM their shared memory
+  const int share = ceil_div(n_blocks, splits) * kKeyBlock;
+  while (pass_keys > kKeyBlock && (pass_keys / 2 >= share || values_smem(a, OB, pass_keys) > 56 * 1024)) pass_keys /= 2;
+  const int smem = values_smem(a, OB, pass_keys);
+  FR_CHECK_SUPPORTED(smem <= 200 * 1024);
+  static PerDeviceFlag f;
+  if (ensure_dyn_smem(f, mix_values_kernel<T, OB>, 200 * 1024) != FR_OK) return FR_ERR_CUDA;
+  return launch_kernel(mix_values_kernel<T, OB>, dim3(splits, a.kv_heads, n_rows), kValThreads, smem, stream, pdl, a, row0, max_keys,
+                       n_blocks, splits, pass_keys, scores, stats, partial, counters);
 }
 
 template <typename T>
@@ -279,17 +326,21 @@ static int launch_rows(const fr_mix_attn& a, int row0, int n_rows, int max_keys,
   const int rep = a.heads / a.kv_heads;
   const int n_blocks = ceil_div(max_keys, kKeyBlock);
   const int k_heads = a.mix == FR_MIX_DIFF ? 2 * a.kv_heads : a.kv_heads;
-  const int s1 = rep * (a.dim + kKeyBlock) * 4, s2 = values_smem(a);
-  FR_CHECK_SUPPORTED(s1 <= 200 * 1024 && s2 <= 200 * 1024);
-  static PerDeviceFlag f1, f2;
+  const int64_t ctas = static_cast<int64_t>(n_blocks) * k_heads * n_rows;
+  int per = ctas > device_sm_count() * 32 ? kMaxPer : 1;
+  if (rep * (a.dim + per * kKeyBlock) * 4 > 40 * 1024) per = 1;
+  const int s1 = rep * (a.dim + per * kKeyBlock) * 4;
+  FR_CHECK_SUPPORTED(s1 <= 200 * 1024);
+  static PerDeviceFlag f1;
   if (ensure_dyn_smem(f1, mix_scores_kernel<T>, 200 * 1024) != FR_OK) return FR_ERR_CUDA;
-  if (ensure_dyn_smem(f2, mix_values_kernel<T>, 200 * 1024) != FR_OK) return FR_ERR_CUDA;
   const bool pdl = n_rows <= kPdlRows;
-  if (launch_kernel(mix_scores_kernel<T>, dim3(n_blocks, k_heads, n_rows), 128, s1, stream, pdl, a, row0, max_keys, n_blocks,
-                    scores, stats) != FR_OK)
+  if (launch_kernel(mix_scores_kernel<T>, dim3(ceil_div(n_blocks, per), k_heads, n_rows), 128, s1, stream, pdl, a, row0, max_keys,
+                    n_blocks, per, scores, stats) != FR_OK)
     return FR_ERR_CUDA;
-  return launch_kernel(mix_values_kernel<T>, dim3(splits, a.kv_heads, n_rows), kValThreads, s2, stream, pdl, a, row0, max_keys,
-                       n_blocks, splits, scores, stats, partial, counters);
+  if (rep == 1) return launch_values<T, 1>(a, row0, n_rows, max_keys, n_blocks, splits, scores, stats, partial, counters, pdl, stream);
+  if (rep == 2) return launch_values<T, 2>(a, row0, n_rows, max_keys, n_blocks, splits, scores, stats, partial, counters, pdl, stream);
+  if (rep <= 4) return launch_values<T, 4>(a, row0, n_rows, max_keys, n_blocks, splits, scores, stats, partial, counters, pdl, stream);
+  return launch_values<T, 8>(a, row0, n_rows, max_keys, n_blocks, splits, scores, stats, partial, counters, pdl, stream);
 }
 
 // ---------------------------------------------------------------------------
@@ -303,6 +354,7 @@ static int launch_rows(const fr_mix_attn& a, int row0, int n_rows, int max_keys,
 constexpr int kTcThreads = 192;
 constexpr float kRescaleThreshold = 8.0f;
 constexpr int kMaxOut = 8;
+constexpr int kTcBarBytes = 256 + kPageList * 4;
 
 struct TcPlan {
   int q_boxes, v_boxes;   // 64-column boxes of a q / k row and of a v row
@@ -310,6 +362,7 @@ struct TcPlan {
   int n_out;              // outputs per CTA
   int out_blocks;         // CTAs along y per v head (TALK) or per head (DIFF)
   int staged;             // DIFF: the first map's result waits in the output rows (fp16), not in TMEM
+  int stages;             // K and V stages
   int tmem_cols, smem;
 };
 
@@ -333,7 +386,10 @@ static bool plan_tc(int mix, int heads, int kv_heads, int dim, int vdim, TcPlan*
     need -= pl->v_cols;
   }
   pl->tmem_cols = need <= 256 ? 256 : 512;
-  pl->smem = 1024 + 2 * pl->q_boxes * kM * 128 + 2 * (pl->q_boxes + pl->v_boxes) * kTileN * 128 + 256;
+  for (pl->stages = 4;; --pl->stages) {
+    pl->smem = 1024 + 2 * pl->q_boxes * kM * 128 + pl->stages * (pl->q_boxes + pl->v_boxes) * kTileN * 128 + kTcBarBytes;
+    if (pl->stages == 2 || pl->smem <= (pl->tmem_cols == 256 ? 112 : 227) * 1024) break;
+  }
   if (pl->tmem_cols == 512 && pl->smem < 116 * 1024) pl->smem = 116 * 1024;  // one CTA per SM owns all of TMEM
   return pl->smem <= 227 * 1024;
 }
@@ -348,20 +404,23 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
   const uint32_t base = (raw + 1023u) & ~1023u;
   uint8_t* smem = smem_raw + (base - raw);
   const int q_bytes = pl.q_boxes * kM * 128, k_bytes = pl.q_boxes * kTileN * 128, v_bytes = pl.v_boxes * kTileN * 128;
-  const uint32_t sm_q = base, sm_k = sm_q + 2 * q_bytes, sm_v = sm_k + 2 * k_bytes;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + 2 * q_bytes + 2 * k_bytes + 2 * v_bytes);
+  const int n_st = pl.stages;
+  const uint32_t sm_q = base, sm_k = sm_q + 2 * q_bytes, sm_v = sm_k + n_st * k_bytes;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + 2 * q_bytes + n_st * (k_bytes + v_bytes));
   const uint32_t bar0 = ptx::smem_u32(bars);
   const uint32_t bar_qfull = bar0, bar_qempty = bar0 + 16;    // [2] each
-  const uint32_t bar_kfull = bar0 + 32, bar_kempty = bar0 + 48;
-  const uint32_t bar_vfull = bar0 + 64, bar_vempty = bar0 + 80;
-  const uint32_t bar_sfull = bar0 + 96;                       // [2]
-  const uint32_t bar_pfull = bar0 + 112;                      // P written (128 arrivals), one phase per tile
-  const uint32_t bar_ofull = bar0 + 120;                      // P.V accumulated, one phase per tile
-  const uint32_t bar_done = bar0 + 128;                       // a map's last P.V, one phase per map
-  const uint32_t bar_oread = bar0 + 136;                      // O read out (128 arrivals), one phase per map
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 18);
+  const uint32_t bar_sfull = bar0 + 32;                       // [2]
+  const uint32_t bar_kfull = bar0 + 48, bar_kempty = bar0 + 80;   // [stages <= 4] each
+  const uint32_t bar_vfull = bar0 + 112, bar_vempty = bar0 + 144;
+  const uint32_t bar_ofull = bar0 + 176;                      // P.V accumulated, one phase per tile
+  const uint32_t bar_done = bar0 + 184;                       // a map's last P.V, one phase per map
+  // P written (128 arrivals), one per S buffer: the softmax threads may finish two tiles while the issuing thread
+  // still waits for V, and a single barrier would then be two phases ahead of its parity wait
+  const uint32_t bar_pfull = bar0 + 192;                      // [2]
+  const uint32_t bar_oread = bar0 + 208;                      // O read out (128 arrivals), one phase per map
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 27);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
-
+  int* pages = reinterpret_cast<int*>(bars + 32);
   ptx::griddep_wait();
   ptx::griddep_launch_dependents();
   const int rep = a.heads / a.kv_heads;
@@ -384,10 +443,9 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
-    for (int i = 0; i < 14; ++i) ptx::mbar_init(bar0 + 8 * i, 1);  // q, k, v full / empty and sfull
+    for (int i = 0; i < 24; ++i) ptx::mbar_init(bar0 + 8 * i, 1);
     ptx::mbar_init(bar_pfull, 128);
-    ptx::mbar_init(bar_ofull, 1);
-    ptx::mbar_init(bar_done, 1);
+    ptx::mbar_init(bar_pfull + 8, 128);
     ptx::mbar_init(bar_oread, 128);
     *abort_flag = 0;
     ptx::mbar_init_fence();
@@ -395,7 +453,9 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
     ptx::prefetch_tmap(&tk);
     ptx::prefetch_tmap(&tv);
   }
+  load_pages(a, table, kt, pages);
   if (warp == 1) {
+    __syncwarp();
     ptx::tmem_alloc(ptx::smem_u32(tmem_slot), pl.tmem_cols);
     ptx::tmem_relinquish();
   }
@@ -417,30 +477,33 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
           ptx::tma_load_2d(sm_q + st * q_bytes + b * kM * 128, &tq, (src0 + s) * a.dim + b * 64, row0, bar_qfull + 8 * st);
         return true;
       };
-      auto load_k = [&](int it) -> bool {
-        const uint32_t st = it & 1;
-        if (!ptx::mbar_wait(bar_kempty + 8 * st, ((it >> 1) & 1) ^ 1u, abort_flag, status, 72)) return false;
-        ptx::mbar_expect_tx(bar_kfull + 8 * st, k_bytes);
-        const int row = page_row(a, table, kt.at(it % n_tiles));
+      // stage and parity of the next K and V tile, position of the next K tile (map, tile): counted, not divided
+      int k_st = 0, k_ph = 0, k_j = 0, k_s = 0, next_k = 0;
+      auto load_k = [&]() -> bool {
+        if (k_j == 0 && !load_q(k_s)) return false;
+        if (!ptx::mbar_wait(bar_kempty + 8 * k_st, k_ph ^ 1u, abort_flag, status, 72)) return false;
+        ptx::mbar_expect_tx(bar_kfull + 8 * k_st, k_bytes);
+        const int row = page_at(a, table, kt, pages, k_j), col = k_head(k_s) * a.dim;
         for (int b = 0; b < pl.q_boxes; ++b)
-          ptx::tma_load_2d(sm_k + st * k_bytes + b * kTileN * 128, &tk, k_head(it / n_tiles) * a.dim + b * 64, row,
-                           bar_kfull + 8 * st);
+          ptx::tma_load_2d(sm_k + k_st * k_bytes + b * kTileN * 128, &tk, col + b * 64, row, bar_kfull + 8 * k_st);
+        if (++k_st == n_st) { k_st = 0; k_ph ^= 1; }
+        if (++k_j == n_tiles) { k_j = 0; ++k_s; }
+        ++next_k;
         return true;
       };
-      ok = load_q(0) && load_k(0);
+      // K (and at a map's start its Q) runs up to n_st - 1 tiles ahead of V
+      int v_st = 0, v_ph = 0, v_j = 0;
       for (int it = 0; it < total && ok; ++it) {
-        if (it + 1 < total) {  // K (and at a map's end the next Q) runs one tile ahead of V
-          if ((it + 1) % n_tiles == 0) ok = load_q((it + 1) / n_tiles);
-          ok = ok && load_k(it + 1);
-          if (!ok) break;
-        }
-        const uint32_t st = it & 1;
-        ok = ptx::mbar_wait(bar_vempty + 8 * st, ((it >> 1) & 1) ^ 1u, abort_flag, status, 73);
+        while (ok && next_k < total && next_k < it + n_st) ok = load_k();
         if (!ok) break;
-        ptx::mbar_expect_tx(bar_vfull + 8 * st, v_bytes);
-        const int row = page_row(a, table, kt.at(it % n_tiles));
+        ok = ptx::mbar_wait(bar_vempty + 8 * v_st, v_ph ^ 1u, abort_flag, status, 73);
+        if (!ok) break;
+        ptx::mbar_expect_tx(bar_vfull + 8 * v_st, v_bytes);
+        const int row = page_at(a, table, kt, pages, v_j);
         for (int b = 0; b < pl.v_boxes; ++b)
-          ptx::tma_load_2d(sm_v + st * v_bytes + b * kTileN * 128, &tv, vh * a.vdim + b * 64, row, bar_vfull + 8 * st);
+          ptx::tma_load_2d(sm_v + v_st * v_bytes + b * kTileN * 128, &tv, vh * a.vdim + b * 64, row, bar_vfull + 8 * v_st);
+        if (++v_st == n_st) { v_st = 0; v_ph ^= 1; }
+        if (++v_j == n_tiles) v_j = 0;
       }
     }
     __syncwarp();
@@ -449,43 +512,56 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
       const uint32_t idesc_s = ptx::make_idesc(1u, 1u, kM, kTileN);
       const uint32_t idesc_o = ptx::make_idesc(1u, 1u, kM, a.vdim) | (1u << 16);  // B is MN-major
       bool ok = true;
-      auto issue_s = [&](int it) -> bool {
-        const uint32_t st = it & 1;
-        const int s = it / n_tiles;
-        if (it % n_tiles == 0 && !ptx::mbar_wait(bar_qfull + 8 * (s & 1), (s >> 1) & 1, abort_flag, status, 74)) return false;
-        if (!ptx::mbar_wait(bar_kfull + 8 * st, (it >> 1) & 1, abort_flag, status, 75)) return false;
+      const int k_steps = a.dim / 16;
+      int s_st = 0, s_ph = 0, s_j = 0, s_s = 0, s_it = 0;  // next S tile
+      auto issue_s = [&]() -> bool {
+        const uint32_t sb = s_it & 1;
+        if (s_j == 0 && !ptx::mbar_wait(bar_qfull + 8 * (s_s & 1), (s_s >> 1) & 1, abort_flag, status, 74)) return false;
+        if (!ptx::mbar_wait(bar_kfull + 8 * s_st, s_ph, abort_flag, status, 75)) return false;
         ptx::tc_fence_after();
-        for (int k = 0; k < a.dim / 16; ++k) {
-          const uint64_t a_desc = ptx::smem_desc_sw128(sm_q + (s & 1) * q_bytes + (k >> 2) * kM * 128) + 2u * (k & 3);
-          const uint64_t b_desc = ptx::smem_desc_sw128(sm_k + st * k_bytes + (k >> 2) * kTileN * 128) + 2u * (k & 3);
-          ptx::mma_f16(tmem_base + st * kTileN, a_desc, b_desc, idesc_s, k > 0 ? 1u : 0u);
+        const uint64_t a_desc = ptx::smem_desc_sw128(sm_q + (s_s & 1) * q_bytes);
+        const uint64_t b_desc = ptx::smem_desc_sw128(sm_k + s_st * k_bytes);
+        for (int k = 0; k < k_steps; ++k)  // descriptor addresses count 16-byte units
+          ptx::mma_f16(tmem_base + sb * kTileN, a_desc + (k >> 2) * (kM * 128 / 16) + 2u * (k & 3),
+                       b_desc + (k >> 2) * (kTileN * 128 / 16) + 2u * (k & 3), idesc_s, k > 0 ? 1u : 0u);
+        ptx::tc_commit(bar_sfull + 8 * sb);
+        ptx::tc_commit(bar_kempty + 8 * s_st);
+        if (++s_st == n_st) { s_st = 0; s_ph ^= 1; }
+        if (++s_j == n_tiles) {
+          ptx::tc_commit(bar_qempty + 8 * (s_s & 1));
+          s_j = 0;
+          ++s_s;
         }
-        ptx::tc_commit(bar_kempty + 8 * st);
-        if ((it + 1) % n_tiles == 0) ptx::tc_commit(bar_qempty + 8 * (s & 1));
-        ptx::tc_commit(bar_sfull + 8 * st);
+        ++s_it;
         return true;
       };
-      ok = issue_s(0);
+      ok = issue_s();
+      int v_st = 0, v_ph = 0, j = 0, s = 0;
       for (int it = 0; it < total && ok; ++it) {
         // S of the next tile runs during the softmax of this one; its buffer held P of tile it - 1, whose P.V
         // was issued before it
-        if (it + 1 < total) ok = issue_s(it + 1);
+        if (it + 1 < total) ok = issue_s();
         if (!ok) break;
-        const uint32_t st = it & 1;
-        const int s = it / n_tiles, j = it % n_tiles;
-        ok = ptx::mbar_wait(bar_pfull, it & 1, abort_flag, status, 76) &&
-             ptx::mbar_wait(bar_vfull + 8 * st, (it >> 1) & 1, abort_flag, status, 77);
+        const uint32_t sb = it & 1;
+        ok = ptx::mbar_wait(bar_vfull + 8 * v_st, v_ph, abort_flag, status, 77) &&
+             ptx::mbar_wait(bar_pfull + 8 * sb, (it >> 1) & 1, abort_flag, status, 76);
         // the first P.V of a map overwrites O: the previous map's must have been read
         if (ok && j == 0 && s > 0) ok = ptx::mbar_wait(bar_oread, (s - 1) & 1, abort_flag, status, 78);
         if (!ok) break;
         ptx::tc_fence_after();
-        const uint64_t v_desc = smem_desc_mn(sm_v + st * v_bytes, kTileN * 128);
+        const uint64_t v_desc = smem_desc_mn(sm_v + v_st * v_bytes, kTileN * 128);
+#pragma unroll
         for (int k = 0; k < kTileN / 16; ++k)  // 16 keys = 8 columns of P, 16 rows of V
-          ptx::mma_f16_ts(col_o, tmem_base + st * kTileN + 8u * k, v_desc + static_cast<uint64_t>(k * 16 * 128 >> 4), idesc_o,
+          ptx::mma_f16_ts(col_o, tmem_base + sb * kTileN + 8u * k, v_desc + static_cast<uint64_t>(k * 16 * 128 >> 4), idesc_o,
                           (j | k) != 0 ? 1u : 0u);
-        ptx::tc_commit(bar_vempty + 8 * st);
         ptx::tc_commit(bar_ofull);
-        if (j + 1 == n_tiles) ptx::tc_commit(bar_done);
+        ptx::tc_commit(bar_vempty + 8 * v_st);
+        if (++v_st == n_st) { v_st = 0; v_ph ^= 1; }
+        if (++j == n_tiles) {
+          ptx::tc_commit(bar_done);
+          j = 0;
+          ++s;
+        }
       }
     }
     __syncwarp();
@@ -575,7 +651,7 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
         ptx::tmem_st_32x32(tmem_base + lane_off + st * kTileN, w);
         ptx::tmem_st_wait();
         ptx::tc_fence_before();
-        ptx::mbar_arrive(bar_pfull);
+        ptx::mbar_arrive(bar_pfull + 8 * st);
       }
       if (!ok) break;
       ok = wait_all(bar_done, s & 1, 81);

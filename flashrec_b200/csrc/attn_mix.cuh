@@ -100,5 +100,15 @@ __device__ __forceinline__ int page_row(const fr_mix_attn& a, const int32_t* tab
   return s < 0 ? 0 : (s > last ? last : s);
 }
 
+// The tiles' page rows, read once by all threads (before a __syncthreads) so that the TMA producer does not wait for
+// a table entry per tile.
+constexpr int kPageList = 512;
+__device__ __forceinline__ void load_pages(const fr_mix_attn& a, const int32_t* table, const KeyTiles& kt, int* pages) {
+  for (int j = threadIdx.x; j < kt.n && j < kPageList; j += blockDim.x) pages[j] = page_row(a, table, kt.at(j));
+}
+__device__ __forceinline__ int page_at(const fr_mix_attn& a, const int32_t* table, const KeyTiles& kt, const int* pages, int j) {
+  return j < kPageList ? pages[j] : page_row(a, table, kt.at(j));
+}
+
 }  // namespace mix
 }  // namespace fr

@@ -1,11 +1,11 @@
 // Talking heads for bf16 prompts (the TALK side of fr_mix_attn_tc with scratch). Every output head mixes all H softmax
 // maps, and an SM's tensor memory cannot hold the accumulators of all heads, so a kernel that keeps its maps on chip
 // has to recompute them for every v head. Here the maps are computed once, in blocks of token tiles:
-//   1. talk_maps_kernel   (tile, head): one pass over the keys for the row maxima and sums, a second one that
-//                         writes the normalised fp32 weights P_h [128, keys]
-//   2. talk_mix_kernel    M_h = sum_g T[h, g] P_g in fp32, written as bf16 (the MMA operand)
+//   1. talk_maps_kernel   (tile, head): one pass over the keys; writes fp32 exponentials E_h [128, keys] relative to
+//                         the running row maximum and, per key tile, the factor that turns them into weights
+//   2. talk_mix_kernel    M_h = sum_g T[h, g] factor_g E_g in fp32, written as bf16 (the MMA operand)
 //   3. talk_values_kernel (tile, head): O_h = M_h V, a plain tcgen05 product with V as it lies in the cache
-// Scratch per tile: H x 128 x keys x (4 + 2) bytes; the caller's budget keeps a block of tiles near the L2.
+// Scratch per tile: H x 128 x keys x (4 + 2 + 1/16) bytes.
 #include "attn_mix.cuh"
 
 namespace fr {
@@ -34,7 +34,7 @@ constexpr int kKStages = 3;
 __global__ void __launch_bounds__(kThreads, 2)
 talk_maps_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tk,
                  const __grid_constant__ fr_mix_attn a, int boxes, const int32_t* __restrict__ tiles, float* __restrict__ maps,
-                 int ldp, int* status) {
+                 float* __restrict__ factors, int ldp, int* status) {
   extern __shared__ uint8_t smem_raw[];
   const uint32_t raw = ptx::smem_u32(smem_raw);
   const uint32_t base = (raw + 1023u) & ~1023u;
@@ -47,6 +47,7 @@ talk_maps_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
   const uint32_t bar_sfull = bar_kempty + 8 * kKStages, bar_sempty = bar_sfull + 8 * kSBufs;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 1 + 2 * kKStages + 2 * kSBufs);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  int* pages = reinterpret_cast<int*>(bars + 32);
   ptx::griddep_wait();
   ptx::griddep_launch_dependents();
   const int head = blockIdx.y, kvh = head / (a.heads / a.kv_heads);
@@ -54,7 +55,7 @@ talk_maps_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
   const int pos0 = static_cast<int>(a.pos[row0]);
   const int32_t* table = a.req_to_token + a.req_rows[req] * a.table_stride;
   const mix::KeyTiles kt = mix::key_tiles(a, pos0, pos0 + n_tok - 1);
-  const int total = 2 * kt.n;  // every key tile twice
+  const int total = kt.n;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
     ptx::mbar_init(bar_q, 1);
@@ -71,7 +72,9 @@ talk_maps_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
     ptx::prefetch_tmap(&tq);
     ptx::prefetch_tmap(&tk);
   }
+  mix::load_pages(a, table, kt, pages);
   if (warp == 1) {
+    __syncwarp();
     ptx::tmem_alloc(ptx::smem_u32(tmem_slot), kSBufs * kTileN);
     ptx::tmem_relinquish();
   }
@@ -90,7 +93,7 @@ talk_maps_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
         ok = ptx::mbar_wait(bar_kempty + 8 * st, ((it / kKStages) & 1) ^ 1u, abort_flag, status, 91);
         if (!ok) break;
         ptx::mbar_expect_tx(bar_kfull + 8 * st, k_bytes);
-        const int row = mix::page_row(a, table, kt.at(it < kt.n ? it : it - kt.n));
+        const int row = mix::page_at(a, table, kt, pages, it);
         for (int b = 0; b < boxes; ++b)
           ptx::tma_load_2d(sm_k + st * k_bytes + b * kTileN * 128, &tk, kvh * a.dim + b * 64, row, bar_kfull + 8 * st);
       }
@@ -124,13 +127,15 @@ talk_maps_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
     const float scale = a.scale * kLog2e;
     const float slope = a.slopes != nullptr ? a.slopes[head] * kLog2e : 0.f;
     float* out = maps + ((static_cast<int64_t>(blockIdx.x) * a.heads + head) * kM + r) * ldp;
-    float m = -INFINITY, l = 0.f, inv = 0.f;
+    float* fac = factors + (static_cast<int64_t>(blockIdx.x) * a.heads + head) * (ldp / kTileN) * kM + r;
+    float m = -INFINITY, l = 0.f;
+    bool ok = true;
     for (int it = 0; it < total; ++it) {
       const int sb = it % kSBufs;
       int okw = 0;
       if (lane == 0) okw = ptx::mbar_wait(bar_sfull + 8 * sb, (it / kSBufs) & 1, abort_flag, status, 95) ? 1 : 0;
       okw = __shfl_sync(0xffffffffu, okw, 0);
-      if (!okw) break;
+      if (!okw) { ok = false; break; }
       ptx::tc_fence_after();
       uint32_t s0[32], s1[32];
       ptx::tmem_ld_32x32(tmem_base + lane_off + sb * kTileN, s0);
@@ -138,8 +143,7 @@ talk_maps_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
       ptx::tmem_ld_wait();
       ptx::tc_fence_before();
       ptx::mbar_arrive(bar_sempty + 8 * sb);
-      const int j = it < kt.n ? it : it - kt.n;
-      const int j0 = kt.at(j) * kTileN;
+      const int j0 = kt.at(it) * kTileN;
       const float bias0 = slope * static_cast<float>(j0 - i);
       auto sv = [&](int c) -> uint32_t& { return c < 32 ? s0[c & 31] : s1[c & 31]; };
 #pragma unroll
@@ -151,30 +155,33 @@ talk_maps_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
         for (int c = 0; c < 64; ++c)
           if (c > hi_c || (c < lo_c && c >= keep_c)) sv(c) = 0xff800000u;  // -inf
       }
-      if (it < kt.n) {
-        float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+      float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
-        for (int c = 0; c < 64; ++c) mx[c & 3] = fmaxf(mx[c & 3], __uint_as_float(sv(c)));
-        const float mn = fmaxf(m, fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])));
-        if (mn > m) {
-          l *= mix::ex2(m - mn);
-          m = mn;
-        }
-        const float ref = m == -INFINITY ? 0.f : m;
-        float ps[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-        for (int c = 0; c < 64; ++c) ps[c & 3] += mix::ex2(__uint_as_float(sv(c)) - ref);
-        l += (ps[0] + ps[1]) + (ps[2] + ps[3]);
-        if (it + 1 == kt.n) inv = 1.0f / l;
-      } else {
-#pragma unroll
-        for (int x = 0; x < 8; ++x) {
-          uint32_t w[8];
-#pragma unroll
-          for (int e = 0; e < 8; ++e) w[e] = __float_as_uint(mix::ex2(__uint_as_float(sv(8 * x + e)) - m) * inv);
-          ptx::st_global_v8(out + j * kTileN + 8 * x, w);
-        }
+      for (int c = 0; c < 64; ++c) mx[c & 3] = fmaxf(mx[c & 3], __uint_as_float(sv(c)));
+      const float mn = fmaxf(m, fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])));
+      if (mn > m) {
+        l *= mix::ex2(m - mn);
+        m = mn;
       }
+      const float ref = m == -INFINITY ? 0.f : m;
+      float ps[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int x = 0; x < 8; ++x) {
+        uint32_t w[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          const float p = mix::ex2(__uint_as_float(sv(8 * x + e)) - ref);
+          ps[e & 3] += p;
+          w[e] = __float_as_uint(p);
+        }
+        ptx::st_global_v8(out + it * kTileN + 8 * x, w);
+      }
+      l += (ps[0] + ps[1]) + (ps[2] + ps[3]);
+      fac[it * kM] = m;
+    }
+    if (ok) {
+      const float inv = 1.0f / l;
+      for (int j = 0; j < total; ++j) fac[j * kM] = mix::ex2(fac[j * kM] - m) * inv;  // 0 where nothing was visible yet
     }
   }
   ptx::tc_fence_before();
@@ -190,48 +197,100 @@ talk_maps_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
 }
 
 // ---------------------------------------------------------------------------
-// 2. M_h = sum_g T[h, g] P_g. A thread holds four keys of one row for kHeadBlock output heads.
+// 2. M_h = sum_g T[h, g] factor_g E_g. A thread holds four keys of one row for kHeadBlock output heads; the products
+//    run two to an instruction.
 // ---------------------------------------------------------------------------
 constexpr int kHeadBlock = 16;
 
-__global__ void __launch_bounds__(256)
+__device__ __forceinline__ uint64_t pack_f32x2(float lo, float hi) {
+  uint64_t d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+  return d;
+}
+__device__ __forceinline__ void unpack_f32x2(uint64_t v, float& lo, float& hi) {
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
+}
+__device__ __forceinline__ void fma_f32x2(uint64_t& d, uint64_t a, uint64_t b) {
+  asm("fma.rn.f32x2 %0, %1, %2, %0;" : "+l"(d) : "l"(a), "l"(b));
+}
+
+constexpr int kMixThreads = 128;
+constexpr int kMixAhead = 8;  // maps on their way while as many are used
+
+__global__ void __launch_bounds__(kMixThreads, 3)
 talk_mix_kernel(const __grid_constant__ fr_mix_attn a, const int32_t* __restrict__ tiles, const float* __restrict__ maps,
-                __nv_bfloat16* __restrict__ mixed, int ldp) {
-  extern __shared__ float coef[];  // [heads (source)][kHeadBlock]
+                const float* __restrict__ factors, __nv_bfloat16* __restrict__ mixed, int ldp) {
+  extern __shared__ uint64_t coef[];  // [heads (source)][kHeadBlock], every value twice
   ptx::griddep_wait();
   ptx::griddep_launch_dependents();
   const int tile = blockIdx.y, h0 = blockIdx.z * kHeadBlock;
-  for (int e = threadIdx.x; e < a.heads * kHeadBlock; e += 256) {
-    const int g = e / kHeadBlock, h = h0 + e % kHeadBlock;
-    coef[e] = h < a.heads ? a.coef[static_cast<int64_t>(h) * a.heads + g] : 0.f;
-  }
-  __syncthreads();
   const int row0 = tiles[3 * tile + 1], n_tok = tiles[3 * tile + 2];
   const int pos0 = static_cast<int>(a.pos[row0]);
   const int keys = mix::key_tiles(a, pos0, pos0 + n_tok - 1).n * kTileN;
   const int quads = keys / 4;
-  for (int e = blockIdx.x * 256 + threadIdx.x; e < kM * quads; e += gridDim.x * 256) {
+  if (static_cast<int>(blockIdx.x) * kMixThreads >= kM * quads) return;
+  for (int e = threadIdx.x; e < a.heads * kHeadBlock; e += kMixThreads) {
+    const int g = e / kHeadBlock, h = h0 + e % kHeadBlock;
+    const float t = h < a.heads ? a.coef[static_cast<int64_t>(h) * a.heads + g] : 0.f;
+    coef[e] = pack_f32x2(t, t);
+  }
+  __syncthreads();
+  const int64_t head_stride = static_cast<int64_t>(kM) * ldp;
+  const int64_t fac_stride = static_cast<int64_t>(ldp / kTileN) * kM;
+  for (int e = blockIdx.x * kMixThreads + threadIdx.x; e < kM * quads; e += gridDim.x * kMixThreads) {
     const int r = e / quads, c = e % quads * 4;
     const int64_t off = (static_cast<int64_t>(tile) * a.heads * kM + r) * ldp + c;
-    const int64_t head_stride = static_cast<int64_t>(kM) * ldp;
-    float acc[kHeadBlock][4] = {};
-#pragma unroll 4
-    for (int g = 0; g < a.heads; ++g) {
-      const float4 p = __ldcs(reinterpret_cast<const float4*>(maps + off + g * head_stride));
+    const float* fac = factors + static_cast<int64_t>(tile) * a.heads * fac_stride + (c / kTileN) * kM + r;
+    uint64_t acc[kHeadBlock][2] = {};
+    float4 nxt[kMixAhead];
+    float nf[kMixAhead];
 #pragma unroll
-      for (int h = 0; h < kHeadBlock; ++h) {
-        const float t = coef[g * kHeadBlock + h];
-        acc[h][0] = fmaf(t, p.x, acc[h][0]);
-        acc[h][1] = fmaf(t, p.y, acc[h][1]);
-        acc[h][2] = fmaf(t, p.z, acc[h][2]);
-        acc[h][3] = fmaf(t, p.w, acc[h][3]);
+    for (int x = 0; x < kMixAhead; ++x) {
+      nxt[x] = make_float4(0, 0, 0, 0);
+      nf[x] = 0.f;
+      if (x < a.heads) {
+        nxt[x] = __ldcs(reinterpret_cast<const float4*>(maps + off + x * head_stride));
+        nf[x] = __ldg(fac + x * fac_stride);
+      }
+    }
+    for (int g0 = 0; g0 < a.heads; g0 += kMixAhead) {
+      uint64_t p[kMixAhead][2];
+#pragma unroll
+      for (int x = 0; x < kMixAhead; ++x) {
+        p[x][0] = pack_f32x2(nxt[x].x * nf[x], nxt[x].y * nf[x]);
+        p[x][1] = pack_f32x2(nxt[x].z * nf[x], nxt[x].w * nf[x]);
+      }
+#pragma unroll
+      for (int x = 0; x < kMixAhead; ++x) {
+        if (g0 + kMixAhead + x < a.heads) {  // the next maps are on their way while these are used
+          nxt[x] = __ldcs(reinterpret_cast<const float4*>(maps + off + (g0 + kMixAhead + x) * head_stride));
+          nf[x] = __ldg(fac + (g0 + kMixAhead + x) * fac_stride);
+        }
+      }
+#pragma unroll
+      for (int x = 0; x < kMixAhead; ++x) {
+        if (g0 + x < a.heads) {
+          const uint64_t* cf = coef + (g0 + x) * kHeadBlock;
+#pragma unroll
+          for (int h = 0; h < kHeadBlock; h += 2) {
+            const ulonglong2 t = *reinterpret_cast<const ulonglong2*>(cf + h);
+            fma_f32x2(acc[h][0], t.x, p[x][0]);
+            fma_f32x2(acc[h][1], t.x, p[x][1]);
+            fma_f32x2(acc[h + 1][0], t.y, p[x][0]);
+            fma_f32x2(acc[h + 1][1], t.y, p[x][1]);
+          }
+        }
       }
     }
 #pragma unroll
     for (int h = 0; h < kHeadBlock; ++h)
-      if (h0 + h < a.heads)
+      if (h0 + h < a.heads) {
+        float f[4];
+        unpack_f32x2(acc[h][0], f[0], f[1]);
+        unpack_f32x2(acc[h][1], f[2], f[3]);
         *reinterpret_cast<uint2*>(mixed + off + (h0 + h) * head_stride) =
-            make_uint2(pack_bf16(acc[h][0], acc[h][1]), pack_bf16(acc[h][2], acc[h][3]));
+            make_uint2(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]));
+      }
   }
 }
 
@@ -253,6 +312,7 @@ talk_values_kernel(const __grid_constant__ CUtensorMap tm, const __grid_constant
   const uint32_t bar_full = ptx::smem_u32(bars), bar_empty = bar_full + 8 * kStages, bar_done = bar_empty + 8 * kStages;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 2 * kStages + 1);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  int* pages = reinterpret_cast<int*>(bars + 32);
   ptx::griddep_wait();
   ptx::griddep_launch_dependents();
   const int head = blockIdx.y, vh = head / (a.heads / a.kv_heads);
@@ -272,7 +332,9 @@ talk_values_kernel(const __grid_constant__ CUtensorMap tm, const __grid_constant
     ptx::prefetch_tmap(&tm);
     ptx::prefetch_tmap(&tv);
   }
+  mix::load_pages(a, table, kt, pages);
   if (warp == 1) {
+    __syncwarp();
     ptx::tmem_alloc(ptx::smem_u32(tmem_slot), tmem_cols);
     ptx::tmem_relinquish();
   }
@@ -289,7 +351,7 @@ talk_values_kernel(const __grid_constant__ CUtensorMap tm, const __grid_constant
         if (!ok) break;
         ptx::mbar_expect_tx(bar_full + 8 * st, stage);
         ptx::tma_load_2d(base + st * stage, &tm, it * kTileN, (static_cast<int>(blockIdx.x) * a.heads + head) * kM, bar_full + 8 * st);
-        const int row = mix::page_row(a, table, kt.at(it));
+        const int row = mix::page_at(a, table, kt, pages, it);
         for (int b = 0; b < v_boxes; ++b)
           ptx::tma_load_2d(base + st * stage + m_bytes + b * kTileN * 128, &tv, vh * a.vdim + b * 64, row, bar_full + 8 * st);
       }
@@ -357,7 +419,7 @@ talk_values_kernel(const __grid_constant__ CUtensorMap tm, const __grid_constant
 }  // namespace talk
 
 int64_t talk_tc_tile_bytes(const fr_mix_attn& a, int max_pos) {
-  return static_cast<int64_t>(a.heads) * talk::kM * talk::tile_keys(a, max_pos) * 6;
+  return static_cast<int64_t>(a.heads) * talk::kM * (talk::tile_keys(a, max_pos) / 16 * 97);  // E, M, factors
 }
 
 int talk_tc(const fr_mix_attn& a, const int32_t* tiles, int n_tiles, int n_rows, int max_pos, void* scratch,
@@ -369,13 +431,15 @@ int talk_tc(const fr_mix_attn& a, const int32_t* tiles, int n_tiles, int n_rows,
   if (block < 1) return FR_ERR_BAD_ARG;
   if (block > 32768 / a.heads) block = 32768 / a.heads;
   float* maps = static_cast<float*>(scratch);
-  __nv_bfloat16* mixed = reinterpret_cast<__nv_bfloat16*>(maps + static_cast<int64_t>(block) * a.heads * kM * ldp);
+  const int64_t values = static_cast<int64_t>(block) * a.heads * kM * ldp;
+  float* factors = maps + values;
+  __nv_bfloat16* mixed = reinterpret_cast<__nv_bfloat16*>(factors + values / kTileN);
   const int boxes = (a.dim + 63) / 64, v_boxes = (a.vdim + 63) / 64, v_cols = (a.vdim + 31) / 32 * 32;
   int tmem_cols = 32;
   while (tmem_cols < v_cols) tmem_cols *= 2;
-  const int smem_maps = 1024 + boxes * (kM + kKStages * kTileN) * 128 + 256;
-  const int smem_values = 1024 + kStages * (kM + v_boxes * kTileN) * 128 + 256;
-  const int smem_mix = a.heads * kHeadBlock * 4;
+  const int smem_maps = 1024 + boxes * (kM + kKStages * kTileN) * 128 + 256 + mix::kPageList * 4;
+  const int smem_values = 1024 + kStages * (kM + v_boxes * kTileN) * 128 + 256 + mix::kPageList * 4;
+  const int smem_mix = a.heads * kHeadBlock * 8;
   FR_CHECK_SUPPORTED(smem_mix <= 48 * 1024 && smem_maps <= 227 * 1024 && smem_values <= 227 * 1024);
   static PerDeviceFlag f0, f1;
   if (ensure_dyn_smem(f0, talk_maps_kernel, 227 * 1024) != FR_OK) return FR_ERR_CUDA;
@@ -392,10 +456,11 @@ int talk_tc(const fr_mix_attn& a, const int32_t* tiles, int n_tiles, int n_rows,
   for (int t0 = 0; t0 < n_tiles; t0 += block) {
     const int n = n_tiles - t0 < block ? n_tiles - t0 : block;
     const int32_t* tl = tiles + 3 * static_cast<int64_t>(t0);
-    r = launch_kernel(talk_maps_kernel, dim3(n, a.heads), kThreads, smem_maps, stream, pdl, tq, tk, a, boxes, tl, maps, ldp, status);
+    r = launch_kernel(talk_maps_kernel, dim3(n, a.heads), kThreads, smem_maps, stream, pdl, tq, tk, a, boxes, tl, maps,
+                      factors, ldp, status);
     if (r == FR_OK)
-      r = launch_kernel(talk_mix_kernel, dim3(ceil_div(static_cast<int64_t>(kM) * ldp / 4, 256), n, ceil_div(a.heads, kHeadBlock)), 256,
-                        smem_mix, stream, pdl, a, tl, maps, mixed, ldp);
+      r = launch_kernel(talk_mix_kernel, dim3(ceil_div(static_cast<int64_t>(kM) * ldp / 4, kMixThreads), n, ceil_div(a.heads, kHeadBlock)), kMixThreads,
+                        smem_mix, stream, pdl, a, tl, maps, factors, mixed, ldp);
     if (r == FR_OK)
       r = launch_kernel(talk_values_kernel, dim3(n, a.heads), kThreads, smem_values, stream, pdl, tm, tv, a, v_boxes, v_cols, tmem_cols,
                         tl, status);

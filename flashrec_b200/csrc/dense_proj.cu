@@ -750,10 +750,11 @@ static int pick_block_n(int M, int N) {
 }
 
 static int rows_ks(int N, int K) {
-  // warps per CTA that share a group of four rows along K: enough warps in flight for narrow matrices
+  // warps per CTA that share a group of four rows along K: several waves of small CTAs, so that the last one is
+  // short, as long as a warp keeps two steps of 256 columns
   const int64_t warps = ceil_div(N, 4);
   int ks = 1;
-  while (ks < 8 && warps * ks < 148 * 16 && K / (ks * 2) >= 256) ks *= 2;
+  while (ks < 8 && ((warps * ks < 148 * 16 && K / (ks * 2) >= 256) || (warps * ks < 148 * 96 && K / (ks * 2) >= 512))) ks *= 2;
   return ks;
 }
 

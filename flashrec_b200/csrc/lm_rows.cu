@@ -130,20 +130,41 @@ __device__ __forceinline__ float conv_tap(const T* __restrict__ u, int64_t ldu, 
 // another request begins.
 constexpr int kConvRun = 16;
 
+// eight consecutive values as they lie in memory
 template <typename T>
-__device__ __forceinline__ void conv_load8(const T* p, float (&v)[8]) {
-  if constexpr (sizeof(T) == 2) {
-    const uint4 a = *reinterpret_cast<const uint4*>(p);
-    const uint32_t w[4] = {a.x, a.y, a.z, a.w};
+struct Raw8 {
+  uint4 q[sizeof(T) / 2];
+};
+template <typename T>
+__device__ __forceinline__ Raw8<T> raw_load(const T* p) {
+  Raw8<T> r;
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      v[2 * i] = __uint_as_float(w[i] << 16);
-      v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
-    }
-  } else {
-    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
-    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
-    v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+  for (int i = 0; i < static_cast<int>(sizeof(T)) / 2; ++i) r.q[i] = reinterpret_cast<const uint4*>(p)[i];
+  return r;
+}
+template <typename T>
+__device__ __forceinline__ void raw_store(T* p, const Raw8<T>& r) {
+#pragma unroll
+  for (int i = 0; i < static_cast<int>(sizeof(T)) / 2; ++i) reinterpret_cast<uint4*>(p)[i] = r.q[i];
+}
+template <typename T>
+__device__ __forceinline__ Raw8<T> raw_zero() {
+  Raw8<T> r;
+#pragma unroll
+  for (int i = 0; i < static_cast<int>(sizeof(T)) / 2; ++i) r.q[i] = make_uint4(0, 0, 0, 0);
+  return r;
+}
+__device__ __forceinline__ void raw_unpack(const Raw8<float>& r, float (&v)[8]) {
+  const uint32_t w[8] = {r.q[0].x, r.q[0].y, r.q[0].z, r.q[0].w, r.q[1].x, r.q[1].y, r.q[1].z, r.q[1].w};
+#pragma unroll
+  for (int i = 0; i < 8; ++i) v[i] = __uint_as_float(w[i]);
+}
+__device__ __forceinline__ void raw_unpack(const Raw8<__nv_bfloat16>& r, float (&v)[8]) {
+  const uint32_t w[4] = {r.q[0].x, r.q[0].y, r.q[0].z, r.q[0].w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    v[2 * i] = __uint_as_float(w[i] << 16);
+    v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
   }
 }
 template <typename T>
@@ -166,10 +187,16 @@ conv_vec_kernel(const T* __restrict__ u, int64_t ldu, const float* __restrict__ 
   const int c = (blockIdx.y * 128 + threadIdx.x) * 8;
   float wr[TAPS][8];
   if (c < C) {
+    float flat[8 * TAPS];  // TAPS * 8 consecutive values
+#pragma unroll
+    for (int i = 0; i < 2 * TAPS; ++i) {
+      const float4 q = __ldg(reinterpret_cast<const float4*>(w + static_cast<int64_t>(c) * TAPS) + i);
+      flat[4 * i] = q.x; flat[4 * i + 1] = q.y; flat[4 * i + 2] = q.z; flat[4 * i + 3] = q.w;
+    }
 #pragma unroll
     for (int i = 0; i < 8; ++i)
 #pragma unroll
-      for (int k = 0; k < TAPS; ++k) wr[k][i] = __ldg(w + static_cast<int64_t>(c + i) * TAPS + k);
+      for (int k = 0; k < TAPS; ++k) wr[k][i] = flat[i * TAPS + k];
   }
   ptx::griddep_wait();
   ptx::griddep_launch_dependents();
@@ -179,19 +206,50 @@ conv_vec_kernel(const T* __restrict__ u, int64_t ldu, const float* __restrict__ 
   const fr_conv_out& o = outs.o[oi];
   const bool keep = c >= o.c0 && c < o.c0 + o.c;
   T* out = static_cast<T*>(o.out) + (c - o.c0);
-  float win[P > 0 ? P : 1][8] = {};
+  Raw8<T> win[P];
   const int t0 = ONE ? blockIdx.x : blockIdx.x * kConvRun;
   const int t1 = ONE ? t0 + 1 : min(t0 + kConvRun, n_tok);
+  constexpr int B = ONE ? 1 : 4;  // tokens loaded together, the next ones while these are worked on
+  Raw8<T> v[B], nv[B];
+  int req[B], nreq[B];
+  int64_t dst[B], ndst[B];
+  auto fetch = [&](int t) {
+#pragma unroll
+    for (int i = 0; i < B; ++i)
+      if (t + i < t1) {
+        nv[i] = raw_load<T>(u + static_cast<int64_t>(t + i) * ldu + c);
+        nreq[i] = tok_req[t + i];
+        ndst[i] = o.row_map != nullptr ? o.row_map[t + i] : t + i;
+      }
+  };
   int cur = -1;
-  for (int t = t0; t < t1; t += 4) {
-    float v[4][8];
+  fetch(t0);
 #pragma unroll
-    for (int x = 0; x < (ONE ? 1 : 4); ++x)
-      if (t + x < t1) conv_load8<T>(u + static_cast<int64_t>(t + x) * ldu + c, v[x]);
+  for (int k = 0; k < P; ++k) win[k] = raw_zero<T>();
+  if (!ONE) {  // the tokens just before the run are the window when they belong to the same request
+    bool same = t0 >= P;
+    if (same) {
+      const int b0 = tok_req[t0];
 #pragma unroll
-    for (int x = 0; x < (ONE ? 1 : 4); ++x) {
+      for (int k = 0; k < P; ++k) {
+        win[k] = raw_load<T>(u + static_cast<int64_t>(t0 - (P - k)) * ldu + c);
+        same = same && tok_req[t0 - (P - k)] == b0;
+      }
+      if (same) cur = b0;
+    }
+  }
+  for (int t = t0; t < t1; t += B) {
+#pragma unroll
+    for (int x = 0; x < B; ++x) {
+      v[x] = nv[x];
+      req[x] = nreq[x];
+      dst[x] = ndst[x];
+    }
+    if (t + B < t1) fetch(t + B);
+#pragma unroll
+    for (int x = 0; x < B; ++x) {
       if (t + x >= t1) break;
-      const int b = tok_req[t + x];
+      const int b = req[x];
       if (b != cur) {  // fill the window: earlier tokens of the batch, then the state, zeros before position 0
         cur = b;
         const int64_t p = pos[t + x];
@@ -201,34 +259,30 @@ conv_vec_kernel(const T* __restrict__ u, int64_t ldu, const float* __restrict__ 
         for (int k = 0; k < P; ++k) {
           const int back = P - k;
           if (p < back) {
-#pragma unroll
-            for (int i = 0; i < 8; ++i) win[k][i] = 0.f;
+            win[k] = raw_zero<T>();
           } else if (e >= back) {
-            conv_load8<T>(u + static_cast<int64_t>(t + x - back) * ldu + c, win[k]);
+            win[k] = raw_load<T>(u + static_cast<int64_t>(t + x - back) * ldu + c);
           } else {
-            conv_load8<T>(st + static_cast<int64_t>(k + e) * C, win[k]);
+            win[k] = raw_load<T>(st + static_cast<int64_t>(k + e) * C);
           }
         }
       }
-      float y[8];
+      float y[8] = {};
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        y[i] = 0.f;
+      for (int k = 0; k < TAPS; ++k) {
+        float f[8];
+        raw_unpack(k < P ? win[k < P ? k : 0] : v[x], f);
 #pragma unroll
-        for (int k = 0; k < P; ++k) y[i] = fmaf(wr[k][i], win[k][i], y[i]);
-        y[i] = fmaf(wr[P][i], v[x][i], y[i]);
+        for (int i = 0; i < 8; ++i) y[i] = fmaf(wr[k][i], f[i], y[i]);
       }
-      if (keep) conv_store8<T>(out + (o.row_map != nullptr ? o.row_map[t + x] : t + x) * o.ldo, y);
+      if (keep) conv_store8<T>(out + dst[x] * o.ldo, y);
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
-#pragma unroll
-        for (int k = 0; k + 1 < P; ++k) win[k][i] = win[k + 1][i];
-        if (P > 0) win[P - 1][i] = v[x][i];
-      }
-      if (ONE && P > 0) {  // the window is the request's new state
+      for (int k = 0; k + 1 < P; ++k) win[k] = win[k + 1];
+      win[P - 1] = v[x];
+      if (ONE) {  // the window is the request's new state
         T* st = state + state_slots[b] * P * C + c;
 #pragma unroll
-        for (int k = 0; k < P; ++k) conv_store8<T>(st + static_cast<int64_t>(k) * C, win[k]);
+        for (int k = 0; k < P; ++k) raw_store<T>(st + static_cast<int64_t>(k) * C, win[k]);
       }
     }
   }
@@ -293,7 +347,7 @@ static int launch_conv(const void* u, int64_t ldu, const float* w, int taps, int
                        int one, cudaStream_t stream) {
   const T* up = static_cast<const T*>(u);
   T* st = static_cast<T*>(state);
-  bool vec = C % 8 == 0 && ldu % 8 == 0 && aligned16(u) && aligned16(state) && taps >= 2 && taps <= 4;
+  bool vec = C % 8 == 0 && ldu % 8 == 0 && aligned16(u) && aligned16(state) && aligned16(w) && taps >= 2 && taps <= 4;
   for (int i = 0; i < outs.n; ++i)
     vec = vec && outs.o[i].c0 % 8 == 0 && outs.o[i].c % 8 == 0 && outs.o[i].ldo % 8 == 0 && aligned16(outs.o[i].out);
   if (vec) {

@@ -8,7 +8,6 @@ both. bfloat16 runs on the tensor cores, float32 is true 32-bit arithmetic throu
 from __future__ import annotations
 
 import ctypes
-import os
 from dataclasses import dataclass
 from typing import List, Optional, Sequence, Tuple
 
@@ -22,7 +21,7 @@ from flashrec_b200.kvcache import CacheSpec
 SEG = {"store": _lib.FR_SEG_STORE, "swiglu": _lib.FR_SEG_SWIGLU, "sigmoid": _lib.FR_SEG_SIGMOID,
        "store_f32": _lib.FR_SEG_STORE_F32}
 _SCORE_SCRATCH_BYTES = 256 << 20
-_MAP_SCRATCH_BYTES = int(os.environ.get("FR_MAP_SCRATCH_MB", "224")) << 20  # maps of talking heads between their kernels
+_MAP_SCRATCH_BYTES = 1 << 30  # maps of talking heads between their kernels: every token tile of a large step at once
 
 
 def ceil_to(n: int, m: int) -> int:
