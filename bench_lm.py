@@ -8,6 +8,7 @@ from __future__ import annotations
 
 import json
 import statistics
+import time
 from pathlib import Path
 
 ROOT = Path(__file__).resolve().parent
@@ -27,8 +28,12 @@ def dibepel_config(width, heads, kv_heads, ff, layers):
                 layers=entries)
 
 
-def event_time(torch, fn, iters: int, warmup: int = 3) -> float:
-    """Median milliseconds of ``fn(i)``; the caller's working set exceeds L2 or rotates through buffers."""
+def event_time(torch, fn, iters: int, warmup: int = 3, rest: float = 0.0) -> float:
+    """Median milliseconds of ``fn(i)``; the caller's working set exceeds L2 or rotates through buffers. ``rest``: seconds of
+    idling first, for single kernels that are set against the burst peak (the clocks recover from the power cap)."""
+    if rest > 0:
+        torch.cuda.synchronize()
+        time.sleep(rest)
     for i in range(warmup):
         fn(i)
     torch.cuda.synchronize()
@@ -114,19 +119,19 @@ def kernel_times(torch, model, n_tok, peaks, iters=10):
         w = cfg.width
         x = torch.randn((n_tok, w), device=dev)
         h = torch.empty((n_tok, w), **bf)
-        put(f"{kind}.norm", event_time(torch, lambda i: rms_norm(x, l.norm_w, 1.0, cfg.eps, h), iters), byts=n_tok * w * 6)
+        put(f"{kind}.norm", event_time(torch, lambda i: rms_norm(x, l.norm_w, 1.0, cfg.eps, h), iters, rest=0.4), byts=n_tok * w * 6)
         outs, maps = [], []
         for r in l.proj.ranges:
             outs.append(torch.empty((n_tok, r.n), **bf))
             maps.append(None)
         n = sum(r.n * (2 if r.kind == "swiglu" else 1) for r in l.proj.ranges)
-        put(f"{kind}.projections", event_time(torch, lambda i: layers[i % len(layers)].proj(h, outs, maps), iters),
+        put(f"{kind}.projections", event_time(torch, lambda i: layers[i % len(layers)].proj(h, outs, maps), iters, rest=0.4),
             flops=2 * n_tok * n * w)
         q = torch.randn((n_tok, l.attn.q_cols), device=dev).bfloat16()
         a = l.attn
         hsum = a.heads * (a.maps * a.dim_p + a.maps * a.vdim_p) if kind == "diff" else a.heads * (a.dim_p + a.vdim_p)
         put(f"{kind}.attention", event_time(
-            torch, lambda i: a.forward(q, caches.k[li], caches.v[li], table, batch, eng.counters), iters),
+            torch, lambda i: a.forward(q, caches.k[li], caches.v[li], table, batch, eng.counters), iters, rest=0.4),
             flops=2 * visible[kind] * hsum)
         if l.conv_w is not None:
             u = outs[0]
@@ -134,12 +139,12 @@ def kernel_times(torch, model, n_tok, peaks, iters=10):
             put(f"{kind}.conv", event_time(torch, lambda i: short_conv(
                 u, l.conv_w, [(q, None, 0, a.q_cols), (caches.k[li], batch.out_cache_loc, a.q_cols, l.spec.k_cols),
                               (caches.v[li], batch.out_cache_loc, a.q_cols + l.spec.k_cols, l.spec.v_cols)],
-                caches.conv[li], batch), iters), byts=n_tok * c * 4)
+                caches.conv[li], batch), iters, rest=0.4), byts=n_tok * c * 4)
         o = torch.randn((n_tok, a.heads * a.vdim_p), device=dev).bfloat16()
         act = torch.randn((n_tok, l.ff_cols), device=dev).bfloat16()
         g1, g2 = torch.rand((n_tok, w), device=dev).bfloat16(), torch.rand((n_tok, w), device=dev).bfloat16()
         put(f"{kind}.update", event_time(torch, lambda i: gated_add(
-            x, [(o, layers[i % len(layers)].o_w, g1), (act, layers[i % len(layers)].down_w, g2)]), iters),
+            x, [(o, layers[i % len(layers)].o_w, g1), (act, layers[i % len(layers)].down_w, g2)]), iters, rest=0.4),
             flops=2 * n_tok * w * (a.heads * a.vdim_p + l.ff_cols))
     return res
 
@@ -162,13 +167,13 @@ def qwen3_kernel_times(torch, lm, n_tok, peaks, iters=10):
 
     qkv = l.self_attn.qkv_proj
     put("qkv", event_time(torch, lambda i: lm.model.layers[i % len(lm.model.layers)].self_attn.qkv_proj.forward_fp8(
-        q8, s, (n_tok, c.hidden_size), torch.bfloat16), iters), 2 * n_tok * qkv.out_features * c.hidden_size, peak8)
+        q8, s, (n_tok, c.hidden_size), torch.bfloat16), iters, rest=0.4), 2 * n_tok * qkv.out_features * c.hidden_size, peak8)
     put("gate_up", event_time(torch, lambda i: fp8_scaled_mm_silu_mul(
-        q8, lm.model.layers[i % len(lm.model.layers)].mlp._gu_w, s, lm.model.layers[i % len(lm.model.layers)].mlp._gu_s), iters),
+        q8, lm.model.layers[i % len(lm.model.layers)].mlp._gu_w, s, lm.model.layers[i % len(lm.model.layers)].mlp._gu_s), iters, rest=0.4),
         4 * n_tok * c.intermediate_size * c.hidden_size, peak8)
     y8, ys = per_token_quant_fp8(torch.randn((n_tok, c.intermediate_size), device=dev).bfloat16())
     r = torch.zeros((n_tok, c.hidden_size), **dict(dtype=torch.bfloat16, device=dev))
-    put("down", event_time(torch, lambda i: lm.model.layers[i % len(lm.model.layers)].mlp.down_proj.forward_fp8_add_(y8, ys, r), iters),
+    put("down", event_time(torch, lambda i: lm.model.layers[i % len(lm.model.layers)].mlp.down_proj.forward_fp8_add_(y8, ys, r), iters, rest=0.4),
         2 * n_tok * c.intermediate_size * c.hidden_size, peak8)
     pool = lm.new_caches(n_tok // 64 + 2, 2)
     q = torch.randn((n_tok, c.num_attention_heads, c.head_dim), device=dev).bfloat16()
@@ -176,7 +181,7 @@ def qwen3_kernel_times(torch, lm, n_tok, peaks, iters=10):
                      is_prefill=True, kv_indices=torch.arange(64, 64 + n_tok, dtype=torch.int32, device=dev),
                      kv_indptr=torch.tensor([0, n_tok], dtype=torch.int32, device=dev), extend_prefix_lens=[0],
                      extend_seq_lens=[n_tok], qo_indptr=torch.tensor([0, n_tok], dtype=torch.int32, device=dev))
-    put("attention", event_time(torch, lambda i: lm.attn.forward(q, None, None, 0, b, skip_store=True), iters),
+    put("attention", event_time(torch, lambda i: lm.attn.forward(q, None, None, 0, b, skip_store=True), iters, rest=0.4),
         4 * c.num_attention_heads * c.head_dim * n_tok * (n_tok + 1) // 2, peaks["bf16_tflops"])
     del pool
     return res

@@ -346,23 +346,24 @@ static int launch_rows(const fr_mix_attn& a, int row0, int n_rows, int max_keys,
 // ---------------------------------------------------------------------------
 // bf16 prompts on tcgen05. One CTA: up to 128 consecutive tokens of one request, one v head, the source maps its
 // outputs mix one after the other. Roles as in attn_tc.cu: warp 0 = TMA producer, warp 1 = TMEM allocation and
-// MMA issue, warps 2..5 = one token per thread (TMEM lane == token). Per key tile of 64 (one cache page):
+// issue of S = Q K^T, warp 6 = issue of P V (one thread issuing both paced the tiles), warps 2..5 = one token per thread (TMEM lane == token). Per key tile of 64 (one cache page):
 //     S = Q_s K_s^T (two TMEM buffers);  P = exp2(S - m) as bf16 over S;  O += P V, V as it lies in the cache
 // (token rows, so the B operand is MN-major). After a map's last tile the threads take O / l and add
 // coef[o, s] times it to the accumulators.
 // ---------------------------------------------------------------------------
-constexpr int kTcThreads = 192;
+constexpr int kTcThreads = 224;
 constexpr float kRescaleThreshold = 8.0f;
 constexpr int kMaxOut = 8;
-constexpr int kTcBarBytes = 256 + kPageList * 4;
+constexpr int kTcBarBytes = 288 + kPageList * 4;
 
 struct TcPlan {
   int q_boxes, v_boxes;   // 64-column boxes of a q / k row and of a v row
   int v_cols;             // TMEM columns of O and of one accumulator
   int n_out;              // outputs per CTA
   int out_blocks;         // CTAs along y per v head (TALK) or per head (DIFF)
-  int staged;             // DIFF: the first map's result waits in the output rows (fp16), not in TMEM
+  int staged;             // DIFF: the first map's result waits in shared memory (fp16), not in TMEM
   int stages;             // K and V stages
+  int extra;              // bytes before Q that the staged rows need besides Q's first buffer (a multiple of 1024)
   int tmem_cols, smem;
 };
 
@@ -388,6 +389,8 @@ static bool plan_tc(int mix, int heads, int kv_heads, int dim, int vdim, TcPlan*
   pl->tmem_cols = need <= 256 ? 256 : 512;
   for (pl->stages = 4;; --pl->stages) {
     pl->smem = 1024 + 2 * pl->q_boxes * kM * 128 + pl->stages * (pl->q_boxes + pl->v_boxes) * kTileN * 128 + kTcBarBytes;
+    pl->extra = pl->staged && kM * pl->v_cols * 2 > pl->q_boxes * kM * 128 ? kM * pl->v_cols * 2 - pl->q_boxes * kM * 128 : 0;
+    pl->smem += pl->extra;
     if (pl->stages == 2 || pl->smem <= (pl->tmem_cols == 256 ? 112 : 227) * 1024) break;
   }
   if (pl->tmem_cols == 512 && pl->smem < 116 * 1024) pl->smem = 116 * 1024;  // one CTA per SM owns all of TMEM
@@ -405,22 +408,25 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
   uint8_t* smem = smem_raw + (base - raw);
   const int q_bytes = pl.q_boxes * kM * 128, k_bytes = pl.q_boxes * kTileN * 128, v_bytes = pl.v_boxes * kTileN * 128;
   const int n_st = pl.stages;
-  const uint32_t sm_q = base, sm_k = sm_q + 2 * q_bytes, sm_v = sm_k + n_st * k_bytes;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + 2 * q_bytes + n_st * (k_bytes + v_bytes));
+  const uint32_t sm_q = base + pl.extra, sm_k = sm_q + 2 * q_bytes, sm_v = sm_k + n_st * k_bytes;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + pl.extra + 2 * q_bytes + n_st * (k_bytes + v_bytes));
   const uint32_t bar0 = ptx::smem_u32(bars);
   const uint32_t bar_qfull = bar0, bar_qempty = bar0 + 16;    // [2] each
   const uint32_t bar_sfull = bar0 + 32;                       // [2]
   const uint32_t bar_kfull = bar0 + 48, bar_kempty = bar0 + 80;   // [stages <= 4] each
   const uint32_t bar_vfull = bar0 + 112, bar_vempty = bar0 + 144;
-  const uint32_t bar_ofull = bar0 + 176;                      // P.V accumulated, one phase per tile
-  const uint32_t bar_done = bar0 + 184;                       // a map's last P.V, one phase per map
+  const uint32_t bar_ofull = bar0 + 176;                      // [2] P.V accumulated, by S buffer
   // P written (128 arrivals), one per S buffer: the softmax threads may finish two tiles while the issuing thread
   // still waits for V, and a single barrier would then be two phases ahead of its parity wait
   const uint32_t bar_pfull = bar0 + 192;                      // [2]
   const uint32_t bar_oread = bar0 + 208;                      // O read out (128 arrivals), one phase per map
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 27);
+  const uint32_t bar_done = bar0 + 216;                       // a map's last P.V, one phase per map
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 32);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
-  int* pages = reinterpret_cast<int*>(bars + 32);
+  int* pages = reinterpret_cast<int*>(bars + 36);
+  // staged: [128 rows][v_cols] fp16, 16-byte chunks swizzled by row, in `extra` bytes and Q's first buffer behind them,
+  // which the first map is done with
+  uint8_t* stage_rows = smem;
   ptx::griddep_wait();
   ptx::griddep_launch_dependents();
   const int rep = a.heads / a.kv_heads;
@@ -447,6 +453,7 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
     ptx::mbar_init(bar_pfull, 128);
     ptx::mbar_init(bar_pfull + 8, 128);
     ptx::mbar_init(bar_oread, 128);
+    ptx::mbar_init(bar_done, 1);
     *abort_flag = 0;
     ptx::mbar_init_fence();
     ptx::prefetch_tmap(&tq);
@@ -510,53 +517,59 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
   } else if (warp == 1) {
     if (lane == 0) {
       const uint32_t idesc_s = ptx::make_idesc(1u, 1u, kM, kTileN);
+      const int k_steps = a.dim / 16;
+      bool ok = true;
+      int st = 0, ph = 0, j = 0, s = 0;
+      for (int it = 0; it < total && ok; ++it) {
+        const uint32_t sb = it & 1;
+        if (j == 0) ok = ptx::mbar_wait(bar_qfull + 8 * (s & 1), (s >> 1) & 1, abort_flag, status, 74);
+        ok = ok && ptx::mbar_wait(bar_kfull + 8 * st, ph, abort_flag, status, 75);
+        // the buffer held P of tile it - 2
+        if (ok && it >= 2) ok = ptx::mbar_wait(bar_ofull + 8 * sb, ((it >> 1) - 1) & 1, abort_flag, status, 83);
+        if (!ok) break;
+        ptx::tc_fence_after();
+        const uint64_t a_desc = ptx::smem_desc_sw128(sm_q + (s & 1) * q_bytes);
+        const uint64_t b_desc = ptx::smem_desc_sw128(sm_k + st * k_bytes);
+        const uint32_t d = tmem_base + sb * kTileN;
+#pragma unroll 1
+        for (int kb = 0; kb < k_steps; kb += 4) {  // 64 columns per box; descriptor addresses count 16-byte units
+          const uint64_t ad = a_desc + (kb >> 2) * (kM * 128 / 16), bd = b_desc + (kb >> 2) * (kTileN * 128 / 16);
+#pragma unroll
+          for (int k = 0; k < 4; ++k)
+            if (kb + k < k_steps) ptx::mma_f16(d, ad + 2u * k, bd + 2u * k, idesc_s, (kb | k) != 0 ? 1u : 0u);
+        }
+        ptx::tc_commit(bar_sfull + 8 * sb);
+        ptx::tc_commit(bar_kempty + 8 * st);
+        if (++st == n_st) { st = 0; ph ^= 1; }
+        if (++j == n_tiles) {
+          ptx::tc_commit(bar_qempty + 8 * (s & 1));
+          j = 0;
+          ++s;
+        }
+      }
+    }
+    __syncwarp();
+  } else if (warp == 6) {
+    if (lane == 0) {
       const uint32_t idesc_o = ptx::make_idesc(1u, 1u, kM, a.vdim) | (1u << 16);  // B is MN-major
       bool ok = true;
-      const int k_steps = a.dim / 16;
-      int s_st = 0, s_ph = 0, s_j = 0, s_s = 0, s_it = 0;  // next S tile
-      auto issue_s = [&]() -> bool {
-        const uint32_t sb = s_it & 1;
-        if (s_j == 0 && !ptx::mbar_wait(bar_qfull + 8 * (s_s & 1), (s_s >> 1) & 1, abort_flag, status, 74)) return false;
-        if (!ptx::mbar_wait(bar_kfull + 8 * s_st, s_ph, abort_flag, status, 75)) return false;
-        ptx::tc_fence_after();
-        const uint64_t a_desc = ptx::smem_desc_sw128(sm_q + (s_s & 1) * q_bytes);
-        const uint64_t b_desc = ptx::smem_desc_sw128(sm_k + s_st * k_bytes);
-        for (int k = 0; k < k_steps; ++k)  // descriptor addresses count 16-byte units
-          ptx::mma_f16(tmem_base + sb * kTileN, a_desc + (k >> 2) * (kM * 128 / 16) + 2u * (k & 3),
-                       b_desc + (k >> 2) * (kTileN * 128 / 16) + 2u * (k & 3), idesc_s, k > 0 ? 1u : 0u);
-        ptx::tc_commit(bar_sfull + 8 * sb);
-        ptx::tc_commit(bar_kempty + 8 * s_st);
-        if (++s_st == n_st) { s_st = 0; s_ph ^= 1; }
-        if (++s_j == n_tiles) {
-          ptx::tc_commit(bar_qempty + 8 * (s_s & 1));
-          s_j = 0;
-          ++s_s;
-        }
-        ++s_it;
-        return true;
-      };
-      ok = issue_s();
-      int v_st = 0, v_ph = 0, j = 0, s = 0;
+      int st = 0, ph = 0, j = 0, s = 0;
       for (int it = 0; it < total && ok; ++it) {
-        // S of the next tile runs during the softmax of this one; its buffer held P of tile it - 1, whose P.V
-        // was issued before it
-        if (it + 1 < total) ok = issue_s();
-        if (!ok) break;
         const uint32_t sb = it & 1;
-        ok = ptx::mbar_wait(bar_vfull + 8 * v_st, v_ph, abort_flag, status, 77) &&
+        ok = ptx::mbar_wait(bar_vfull + 8 * st, ph, abort_flag, status, 77) &&
              ptx::mbar_wait(bar_pfull + 8 * sb, (it >> 1) & 1, abort_flag, status, 76);
         // the first P.V of a map overwrites O: the previous map's must have been read
         if (ok && j == 0 && s > 0) ok = ptx::mbar_wait(bar_oread, (s - 1) & 1, abort_flag, status, 78);
         if (!ok) break;
         ptx::tc_fence_after();
-        const uint64_t v_desc = smem_desc_mn(sm_v + v_st * v_bytes, kTileN * 128);
+        const uint64_t v_desc = smem_desc_mn(sm_v + st * v_bytes, kTileN * 128);
 #pragma unroll
         for (int k = 0; k < kTileN / 16; ++k)  // 16 keys = 8 columns of P, 16 rows of V
           ptx::mma_f16_ts(col_o, tmem_base + sb * kTileN + 8u * k, v_desc + static_cast<uint64_t>(k * 16 * 128 >> 4), idesc_o,
                           (j | k) != 0 ? 1u : 0u);
-        ptx::tc_commit(bar_ofull);
-        ptx::tc_commit(bar_vempty + 8 * v_st);
-        if (++v_st == n_st) { v_st = 0; v_ph ^= 1; }
+        ptx::tc_commit(bar_ofull + 8 * sb);
+        ptx::tc_commit(bar_vempty + 8 * st);
+        if (++st == n_st) { st = 0; ph ^= 1; }
         if (++j == n_tiles) {
           ptx::tc_commit(bar_done);
           j = 0;
@@ -582,6 +595,7 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
       return okw != 0;
     };
     bool ok = true;
+    const int chunk_mask = pl.v_cols % 64 == 0 ? 7 : 3;  // swizzle within 128 (or 64) bytes of a row
     __nv_bfloat16* out_row = static_cast<__nv_bfloat16*>(a.out) + (row0 + min(r, n_tok - 1)) * a.ldo +
                              static_cast<int64_t>(out0) * a.vdim;
     for (int s = 0; s < n_src && ok; ++s) {
@@ -623,7 +637,7 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
         }
         l_sum *= factor;
         if (j > 0 && __any_sync(0xffffffffu, factor != 1.0f)) {
-          ok = wait_all(bar_ofull, (it - 1) & 1, 80);
+          ok = wait_all(bar_ofull + 8 * (st ^ 1u), ((it - 1) >> 1) & 1, 80);
           if (!ok) break;
 #pragma unroll 1
           for (int c = 0; c < pl.v_cols / 32; ++c) {
@@ -658,8 +672,10 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
       if (!ok) break;
       const float inv = 1.0f / l_sum;
       if (pl.staged) {
-        // first map: a1 as fp16 into this thread's own output row; second map: a1 - lambda a2, scaled by its root
-        // mean square, over it (two passes over O)
+        // first map: a1 as fp16 into this thread's own row of shared memory; second map: a1 - lambda a2, scaled by its
+        // root mean square, into the output (two passes over O)
+        uint8_t* row = stage_rows + r * pl.v_cols * 2;
+        auto chunk = [&](int c) { return reinterpret_cast<uint4*>(row + (((c & ~chunk_mask) | ((c ^ r) & chunk_mask)) << 4)); };
         float ss = 0.f;
         for (int pass = s == 0 ? 1 : 0; pass < 2; ++pass) {
           const float scl = s == 0 ? inv : a.out_scale / sqrtf(ss / static_cast<float>(a.vdim_true) + a.eps);
@@ -668,32 +684,39 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
             uint32_t o[32];
             ptx::tmem_ld_32x32(col_o + lane_off + c * 32, o);
             ptx::tmem_ld_wait();
-            uint4* d4 = reinterpret_cast<uint4*>(out_row + c * 32);
+            if (s == 0) {
 #pragma unroll
-            for (int x = 0; x < 4; ++x) {
-              if (c * 32 + x * 8 >= a.vdim) break;
-              uint32_t w4[4];
-              float f[8];
-              if (s == 0) {
+              for (int x = 0; x < 4; ++x) {
+                uint32_t w4[4];
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                   const __half2 h = __floats2half2_rn(__uint_as_float(o[8 * x + 2 * e]) * scl,
                                                       __uint_as_float(o[8 * x + 2 * e + 1]) * scl);
                   w4[e] = *reinterpret_cast<const uint32_t*>(&h);
                 }
-              } else {
-                const uint4 first = d4[x];
-                const uint32_t fw[4] = {first.x, first.y, first.z, first.w};
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                  const float2 a1 = __half22float2(*reinterpret_cast<const __half2*>(&fw[e]));
-                  f[2 * e] = fmaf(-a.lambda * inv, __uint_as_float(o[8 * x + 2 * e]), a1.x);
-                  f[2 * e + 1] = fmaf(-a.lambda * inv, __uint_as_float(o[8 * x + 2 * e + 1]), a1.y);
-                  ss = pass == 0 ? fmaf(f[2 * e], f[2 * e], fmaf(f[2 * e + 1], f[2 * e + 1], ss)) : ss;
-                  w4[e] = pack_bf16(f[2 * e] * scl, f[2 * e + 1] * scl);
-                }
+                *chunk(c * 4 + x) = make_uint4(w4[0], w4[1], w4[2], w4[3]);
               }
-              if (live && pass == 1) d4[x] = make_uint4(w4[0], w4[1], w4[2], w4[3]);
+            } else {
+#pragma unroll
+              for (int x = 0; x < 2; ++x) {  // 16 columns: one 32-byte store
+                uint32_t w8[8];
+                const bool valid = c * 32 + x * 16 < a.vdim;
+#pragma unroll
+                for (int y = 0; y < 2; ++y) {
+                  const uint4 first = *chunk(c * 4 + 2 * x + y);
+                  const uint32_t fw[4] = {first.x, first.y, first.z, first.w};
+#pragma unroll
+                  for (int e = 0; e < 4; ++e) {
+                    const int q = 16 * x + 8 * y + 2 * e;
+                    const float2 a1 = __half22float2(*reinterpret_cast<const __half2*>(&fw[e]));
+                    const float f0 = fmaf(-a.lambda * inv, __uint_as_float(o[q]), a1.x);
+                    const float f1 = fmaf(-a.lambda * inv, __uint_as_float(o[q + 1]), a1.y);
+                    if (valid) ss = pass == 0 ? fmaf(f0, f0, fmaf(f1, f1, ss)) : ss;
+                    w8[4 * y + e] = pack_bf16(f0 * scl, f1 * scl);
+                  }
+                }
+                if (live && valid && pass == 1) ptx::st_global_v8(out_row + c * 32 + x * 16, w8);
+              }
             }
             __syncwarp();
           }
@@ -843,6 +866,7 @@ extern "C" int fr_mix_attn_tc(const fr_mix_attn* a, const int32_t* tiles, int n_
   const int st = mix::check_args(a);
   if (st != FR_OK) return st;
   FR_CHECK_ARG(tiles && n_tiles >= 0 && n_rows >= 0);
+  FR_CHECK_ARG((reinterpret_cast<uintptr_t>(a->out) & 31u) == 0 && a->ldo % 16 == 0);  // 32-byte stores
   if (n_tiles == 0 || n_rows == 0) return FR_OK;
   mix::TcPlan pl;
   FR_CHECK_SUPPORTED(a->dtype == 0 && a->num_slots >= mix::kTileN &&

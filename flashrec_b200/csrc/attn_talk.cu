@@ -2,10 +2,10 @@
 // maps, and an SM's tensor memory cannot hold the accumulators of all heads, so a kernel that keeps its maps on chip
 // has to recompute them for every v head. Here the maps are computed once, in blocks of token tiles:
 //   1. talk_maps_kernel   (tile, head): one pass over the keys; writes fp32 exponentials E_h [128, keys] relative to
-//                         the running row maximum and, per key tile, the factor that turns them into weights
+//                         a running row maximum and, per 32 keys, the factor that turns them into weights
 //   2. talk_mix_kernel    M_h = sum_g T[h, g] factor_g E_g in fp32, written as bf16 (the MMA operand)
 //   3. talk_values_kernel (tile, head): O_h = M_h V, a plain tcgen05 product with V as it lies in the cache
-// Scratch per tile: H x 128 x keys x (4 + 2 + 1/16) bytes.
+// Scratch per tile: H x 128 x keys x (4 + 2 + 1/8) bytes.
 #include "attn_mix.cuh"
 
 namespace fr {
@@ -25,13 +25,16 @@ static int tile_keys(const fr_mix_attn& a, int max_pos) {
 }
 
 // ---------------------------------------------------------------------------
-// 1. maps. warp 0 = TMA, warp 1 = MMA, warps 2..5 = one token per thread. S has four TMEM buffers, so the product
+// 1. maps. warp 0 = TMA, warp 1 = MMA, warps 2..9 = two threads per token, 32 keys of a tile each (own running maximum;
+//    they meet at the end). S has four TMEM buffers, so the product
 //    runs up to three key tiles ahead of the softmax threads.
 // ---------------------------------------------------------------------------
 constexpr int kSBufs = 4;
 constexpr int kKStages = 3;
+constexpr int kMapThreads = 64 + 8 * 32;
+constexpr int kFactorKeys = 32;  // keys that share a factor
 
-__global__ void __launch_bounds__(kThreads, 2)
+__global__ void __launch_bounds__(kMapThreads, 2)
 talk_maps_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tk,
                  const __grid_constant__ fr_mix_attn a, int boxes, const int32_t* __restrict__ tiles, float* __restrict__ maps,
                  float* __restrict__ factors, int ldp, int* status) {
@@ -45,9 +48,11 @@ talk_maps_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
   const uint32_t bar_q = ptx::smem_u32(bars);
   const uint32_t bar_kfull = bar_q + 8, bar_kempty = bar_kfull + 8 * kKStages;
   const uint32_t bar_sfull = bar_kempty + 8 * kKStages, bar_sempty = bar_sfull + 8 * kSBufs;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 1 + 2 * kKStages + 2 * kSBufs);
+  const uint32_t bar_pair = bar_sempty + 8 * kSBufs;  // [4] a warp and its partner
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 5 + 2 * kKStages + 2 * kSBufs);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
   int* pages = reinterpret_cast<int*>(bars + 32);
+  float2* pair_buf = reinterpret_cast<float2*>(pages + mix::kPageList);  // [2 halves][128 rows] maximum, sum
   ptx::griddep_wait();
   ptx::griddep_launch_dependents();
   const int head = blockIdx.y, kvh = head / (a.heads / a.kv_heads);
@@ -65,8 +70,9 @@ talk_maps_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
     }
     for (int i = 0; i < kSBufs; ++i) {
       ptx::mbar_init(bar_sfull + 8 * i, 1);
-      ptx::mbar_init(bar_sempty + 8 * i, 128);
+      ptx::mbar_init(bar_sempty + 8 * i, 8);
     }
+    for (int i = 0; i < 4; ++i) ptx::mbar_init(bar_pair + 8 * i, 2);
     *abort_flag = 0;
     ptx::mbar_init_fence();
     ptx::prefetch_tmap(&tq);
@@ -119,45 +125,49 @@ talk_maps_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
     }
     __syncwarp();
   } else {
-    const int quad = warp & 3, r = quad * 32 + lane;
+    const int quad = warp & 3, half = (warp - 2) >> 2, r = quad * 32 + lane;
     const int i = pos0 + min(r, n_tok - 1);
     const int lo = static_cast<int>(mix::lowest_key(a, i));
     const int keep = a.mask == FR_MASK_CHUNK ? 0 : a.keep_first;
     const uint32_t lane_off = static_cast<uint32_t>(quad * 32) << 16;
     const float scale = a.scale * kLog2e;
     const float slope = a.slopes != nullptr ? a.slopes[head] * kLog2e : 0.f;
-    float* out = maps + ((static_cast<int64_t>(blockIdx.x) * a.heads + head) * kM + r) * ldp;
-    float* fac = factors + (static_cast<int64_t>(blockIdx.x) * a.heads + head) * (ldp / kTileN) * kM + r;
+    float* out = maps + ((static_cast<int64_t>(blockIdx.x) * a.heads + head) * kM + r) * ldp + half * kFactorKeys;
+    float* fac = factors + ((static_cast<int64_t>(blockIdx.x) * a.heads + head) * (ldp / kFactorKeys) + half) * kM + r;
+    auto wait_all = [&](uint32_t bar, uint32_t parity, int site) -> bool {
+      int okw = 0;
+      if (lane == 0) okw = ptx::mbar_wait(bar, parity, abort_flag, status, site) ? 1 : 0;
+      okw = __shfl_sync(0xffffffffu, okw, 0);
+      __syncwarp();
+      return okw != 0;
+    };
     float m = -INFINITY, l = 0.f;
     bool ok = true;
     for (int it = 0; it < total; ++it) {
       const int sb = it % kSBufs;
-      int okw = 0;
-      if (lane == 0) okw = ptx::mbar_wait(bar_sfull + 8 * sb, (it / kSBufs) & 1, abort_flag, status, 95) ? 1 : 0;
-      okw = __shfl_sync(0xffffffffu, okw, 0);
-      if (!okw) { ok = false; break; }
+      ok = wait_all(bar_sfull + 8 * sb, (it / kSBufs) & 1, 95);
+      if (!ok) break;
       ptx::tc_fence_after();
-      uint32_t s0[32], s1[32];
-      ptx::tmem_ld_32x32(tmem_base + lane_off + sb * kTileN, s0);
-      ptx::tmem_ld_32x32(tmem_base + lane_off + sb * kTileN + 32, s1);
+      uint32_t sv[32];
+      ptx::tmem_ld_32x32(tmem_base + lane_off + sb * kTileN + half * kFactorKeys, sv);
       ptx::tmem_ld_wait();
       ptx::tc_fence_before();
-      ptx::mbar_arrive(bar_sempty + 8 * sb);
-      const int j0 = kt.at(it) * kTileN;
+      __syncwarp();
+      if (lane == 0) ptx::mbar_arrive(bar_sempty + 8 * sb);
+      const int j0 = kt.at(it) * kTileN + half * kFactorKeys;
       const float bias0 = slope * static_cast<float>(j0 - i);
-      auto sv = [&](int c) -> uint32_t& { return c < 32 ? s0[c & 31] : s1[c & 31]; };
 #pragma unroll
-      for (int c = 0; c < 64; ++c)
-        sv(c) = __float_as_uint(fmaf(__uint_as_float(sv(c)), scale, fmaf(slope, static_cast<float>(c), bias0)));
-      if (__any_sync(0xffffffffu, j0 + kTileN - 1 > i || (j0 < lo && j0 + kTileN > keep))) {
+      for (int c = 0; c < 32; ++c)
+        sv[c] = __float_as_uint(fmaf(__uint_as_float(sv[c]), scale, fmaf(slope, static_cast<float>(c), bias0)));
+      if (__any_sync(0xffffffffu, j0 + 31 > i || (j0 < lo && j0 + 32 > keep))) {
         const int hi_c = i - j0, lo_c = lo - j0, keep_c = keep - j0;
 #pragma unroll
-        for (int c = 0; c < 64; ++c)
-          if (c > hi_c || (c < lo_c && c >= keep_c)) sv(c) = 0xff800000u;  // -inf
+        for (int c = 0; c < 32; ++c)
+          if (c > hi_c || (c < lo_c && c >= keep_c)) sv[c] = 0xff800000u;  // -inf
       }
       float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
-      for (int c = 0; c < 64; ++c) mx[c & 3] = fmaxf(mx[c & 3], __uint_as_float(sv(c)));
+      for (int c = 0; c < 32; ++c) mx[c & 3] = fmaxf(mx[c & 3], __uint_as_float(sv[c]));
       const float mn = fmaxf(m, fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])));
       if (mn > m) {
         l *= mix::ex2(m - mn);
@@ -166,22 +176,30 @@ talk_maps_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
       const float ref = m == -INFINITY ? 0.f : m;
       float ps[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-      for (int x = 0; x < 8; ++x) {
+      for (int x = 0; x < 4; ++x) {
         uint32_t w[8];
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
-          const float p = mix::ex2(__uint_as_float(sv(8 * x + e)) - ref);
+          const float p = mix::ex2(__uint_as_float(sv[8 * x + e]) - ref);
           ps[e & 3] += p;
           w[e] = __float_as_uint(p);
         }
         ptx::st_global_v8(out + it * kTileN + 8 * x, w);
       }
       l += (ps[0] + ps[1]) + (ps[2] + ps[3]);
-      fac[it * kM] = m;
+      fac[it * 2 * kM] = m;
     }
     if (ok) {
-      const float inv = 1.0f / l;
-      for (int j = 0; j < total; ++j) fac[j * kM] = mix::ex2(fac[j * kM] - m) * inv;  // 0 where nothing was visible yet
+      pair_buf[half * kM + r] = make_float2(m, l);
+      __syncwarp();
+      if (lane == 0) ptx::mbar_arrive(bar_pair + 8 * quad);
+      ok = wait_all(bar_pair + 8 * quad, 0, 99);
+    }
+    if (ok) {
+      const float2 other = pair_buf[(half ^ 1) * kM + r];
+      const float mt = fmaxf(m, other.x);  // finite: a token sees itself
+      const float inv = 1.0f / (l * mix::ex2(m - mt) + other.y * mix::ex2(other.x - mt));
+      for (int j = 0; j < total; ++j) fac[j * 2 * kM] = mix::ex2(fac[j * 2 * kM] - mt) * inv;  // 0 where nothing was visible yet
     }
   }
   ptx::tc_fence_before();
@@ -236,11 +254,11 @@ talk_mix_kernel(const __grid_constant__ fr_mix_attn a, const int32_t* __restrict
   }
   __syncthreads();
   const int64_t head_stride = static_cast<int64_t>(kM) * ldp;
-  const int64_t fac_stride = static_cast<int64_t>(ldp / kTileN) * kM;
+  const int64_t fac_stride = static_cast<int64_t>(ldp / kFactorKeys) * kM;
   for (int e = blockIdx.x * kMixThreads + threadIdx.x; e < kM * quads; e += gridDim.x * kMixThreads) {
     const int r = e / quads, c = e % quads * 4;
     const int64_t off = (static_cast<int64_t>(tile) * a.heads * kM + r) * ldp + c;
-    const float* fac = factors + static_cast<int64_t>(tile) * a.heads * fac_stride + (c / kTileN) * kM + r;
+    const float* fac = factors + static_cast<int64_t>(tile) * a.heads * fac_stride + (c / kFactorKeys) * kM + r;
     uint64_t acc[kHeadBlock][2] = {};
     float4 nxt[kMixAhead];
     float nf[kMixAhead];
@@ -419,7 +437,7 @@ talk_values_kernel(const __grid_constant__ CUtensorMap tm, const __grid_constant
 }  // namespace talk
 
 int64_t talk_tc_tile_bytes(const fr_mix_attn& a, int max_pos) {
-  return static_cast<int64_t>(a.heads) * talk::kM * (talk::tile_keys(a, max_pos) / 16 * 97);  // E, M, factors
+  return static_cast<int64_t>(a.heads) * talk::kM * (talk::tile_keys(a, max_pos) / 8 * 49);  // E, M, factors
 }
 
 int talk_tc(const fr_mix_attn& a, const int32_t* tiles, int n_tiles, int n_rows, int max_pos, void* scratch,
@@ -433,11 +451,11 @@ int talk_tc(const fr_mix_attn& a, const int32_t* tiles, int n_tiles, int n_rows,
   float* maps = static_cast<float*>(scratch);
   const int64_t values = static_cast<int64_t>(block) * a.heads * kM * ldp;
   float* factors = maps + values;
-  __nv_bfloat16* mixed = reinterpret_cast<__nv_bfloat16*>(factors + values / kTileN);
+  __nv_bfloat16* mixed = reinterpret_cast<__nv_bfloat16*>(factors + values / kFactorKeys);
   const int boxes = (a.dim + 63) / 64, v_boxes = (a.vdim + 63) / 64, v_cols = (a.vdim + 31) / 32 * 32;
   int tmem_cols = 32;
   while (tmem_cols < v_cols) tmem_cols *= 2;
-  const int smem_maps = 1024 + boxes * (kM + kKStages * kTileN) * 128 + 256 + mix::kPageList * 4;
+  const int smem_maps = 1024 + boxes * (kM + kKStages * kTileN) * 128 + 256 + mix::kPageList * 4 + 2 * kM * 8;
   const int smem_values = 1024 + kStages * (kM + v_boxes * kTileN) * 128 + 256 + mix::kPageList * 4;
   const int smem_mix = a.heads * kHeadBlock * 8;
   FR_CHECK_SUPPORTED(smem_mix <= 48 * 1024 && smem_maps <= 227 * 1024 && smem_values <= 227 * 1024);
@@ -456,7 +474,7 @@ int talk_tc(const fr_mix_attn& a, const int32_t* tiles, int n_tiles, int n_rows,
   for (int t0 = 0; t0 < n_tiles; t0 += block) {
     const int n = n_tiles - t0 < block ? n_tiles - t0 : block;
     const int32_t* tl = tiles + 3 * static_cast<int64_t>(t0);
-    r = launch_kernel(talk_maps_kernel, dim3(n, a.heads), kThreads, smem_maps, stream, pdl, tq, tk, a, boxes, tl, maps,
+    r = launch_kernel(talk_maps_kernel, dim3(n, a.heads), kMapThreads, smem_maps, stream, pdl, tq, tk, a, boxes, tl, maps,
                       factors, ldp, status);
     if (r == FR_OK)
       r = launch_kernel(talk_mix_kernel, dim3(ceil_div(static_cast<int64_t>(kM) * ldp / 4, kMixThreads), n, ceil_div(a.heads, kHeadBlock)), kMixThreads,
