@@ -620,14 +620,17 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
         }
         const bool partly = j0 + kTileN - 1 > i || (j0 < lo && j0 + kTileN > keep);
         if (__any_sync(0xffffffffu, partly)) {
-          const int hi_c = i - j0, lo_c = lo - j0, keep_c = keep - j0;
+          const uint64_t vis = visible_bits(j0, i, lo, keep);
+          const uint32_t v0 = static_cast<uint32_t>(vis), v1 = static_cast<uint32_t>(vis >> 32);
 #pragma unroll
-          for (int c = 0; c < 64; ++c)
-            if (c > hi_c || (c < lo_c && c >= keep_c)) sv(c) = 0xff800000u;  // -inf
+          for (int c = 0; c < 32; ++c) {
+            if (!((v0 >> c) & 1u)) s0[c] = 0xff800000u;  // -inf
+            if (!((v1 >> c) & 1u)) s1[c] = 0xff800000u;
+          }
         }
         float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
-        for (int c = 0; c < 64; ++c) mx[c & 3] = fmaxf(mx[c & 3], __uint_as_float(sv(c)));
+        for (int c = 0; c < 32; ++c) mx[c & 3] = max3(mx[c & 3], __uint_as_float(s0[c]), __uint_as_float(s1[c]));
         const float mraw = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
         const float tmax = BIAS ? mraw : mraw * scale;  // without bias the scale (> 0) is applied with the maximum
         float factor = 1.0f;
@@ -651,17 +654,22 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
           ptx::tmem_st_wait();
         }
         const float m_ref = m_used == -INFINITY ? 0.f : m_used;  // nothing visible yet: every weight is 2^-inf = 0
-        float ps[4] = {0.f, 0.f, 0.f, 0.f};
+        uint64_t ps[4] = {0ull, 0ull, 0ull, 0ull};
+        const uint64_t scale2 = pack_f32x2(scale, scale), neg_m2 = pack_f32x2(-m_ref, -m_ref);
         uint32_t w[32];
 #pragma unroll
         for (int x = 0; x < 32; ++x) {
-          const float z0 = __uint_as_float(sv(2 * x)), z1 = __uint_as_float(sv(2 * x + 1));
-          const float p0 = ex2(BIAS ? z0 - m_ref : fmaf(z0, scale, -m_ref));
-          const float p1 = ex2(BIAS ? z1 - m_ref : fmaf(z1, scale, -m_ref));
-          ps[x & 3] += p0 + p1;
+          const uint64_t z = pack_f32x2(__uint_as_float(sv(2 * x)), __uint_as_float(sv(2 * x + 1)));
+          float p0, p1;
+          unpack_f32x2(BIAS ? add_f32x2(z, neg_m2) : fma_f32x2(z, scale2, neg_m2), p0, p1);
+          p0 = ex2(p0);
+          p1 = ex2(p1);
+          ps[x & 3] = add_f32x2(ps[x & 3], pack_f32x2(p0, p1));
           w[x] = pack_bf16(p0, p1);
         }
-        l_sum += (ps[0] + ps[1]) + (ps[2] + ps[3]);
+        float ps0, ps1;
+        unpack_f32x2(add_f32x2(add_f32x2(ps[0], ps[1]), add_f32x2(ps[2], ps[3])), ps0, ps1);
+        l_sum += ps0 + ps1;
         ptx::tmem_st_32x32(tmem_base + lane_off + st * kTileN, w);
         ptx::tmem_st_wait();
         ptx::tc_fence_before();

@@ -74,6 +74,37 @@ __device__ __forceinline__ float ex2(float x) {
   return y;
 }
 
+__device__ __forceinline__ float max3(float a, float b, float c) {
+  float d;
+  asm("max.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
+  return d;
+}
+// two fp32 operations per instruction
+__device__ __forceinline__ uint64_t pack_f32x2(float lo, float hi) {
+  uint64_t d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+  return d;
+}
+__device__ __forceinline__ void unpack_f32x2(uint64_t v, float& lo, float& hi) {
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
+}
+__device__ __forceinline__ uint64_t fma_f32x2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ uint64_t add_f32x2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+
+// Bit c: the query at i, whose window or chunk begins at lo, sees the key j0 + c.
+__device__ __forceinline__ uint64_t low_bits(int n) { return n <= 0 ? 0ull : (n >= 64 ? ~0ull : (1ull << n) - 1ull); }
+__device__ __forceinline__ uint64_t visible_bits(int j0, int i, int lo, int keep) {
+  return low_bits(i - j0 + 1) & (~low_bits(lo - j0) | low_bits(keep - j0));
+}
+
 // MN-major operand tile as TMA writes it with the 128-byte swizzle: rows of 64 values (128 bytes), one row per k;
 // 8-row groups 1024 bytes apart (stride), 64-value column blocks `lead` bytes apart (leading offset).
 __device__ __forceinline__ uint64_t smem_desc_mn(uint32_t addr, uint32_t lead) {

@@ -160,10 +160,10 @@ talk_maps_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
       for (int c = 0; c < 32; ++c)
         sv[c] = __float_as_uint(fmaf(__uint_as_float(sv[c]), scale, fmaf(slope, static_cast<float>(c), bias0)));
       if (__any_sync(0xffffffffu, j0 + 31 > i || (j0 < lo && j0 + 32 > keep))) {
-        const int hi_c = i - j0, lo_c = lo - j0, keep_c = keep - j0;
+        const uint32_t vis = static_cast<uint32_t>(mix::visible_bits(j0, i, lo, keep));
 #pragma unroll
         for (int c = 0; c < 32; ++c)
-          if (c > hi_c || (c < lo_c && c >= keep_c)) sv[c] = 0xff800000u;  // -inf
+          if (!((vis >> c) & 1u)) sv[c] = 0xff800000u;  // -inf
       }
       float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -220,18 +220,6 @@ talk_maps_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
 // ---------------------------------------------------------------------------
 constexpr int kHeadBlock = 16;
 
-__device__ __forceinline__ uint64_t pack_f32x2(float lo, float hi) {
-  uint64_t d;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
-  return d;
-}
-__device__ __forceinline__ void unpack_f32x2(uint64_t v, float& lo, float& hi) {
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
-}
-__device__ __forceinline__ void fma_f32x2(uint64_t& d, uint64_t a, uint64_t b) {
-  asm("fma.rn.f32x2 %0, %1, %2, %0;" : "+l"(d) : "l"(a), "l"(b));
-}
-
 constexpr int kMixThreads = 128;
 constexpr int kMixAhead = 8;  // maps on their way while as many are used
 
@@ -250,7 +238,7 @@ talk_mix_kernel(const __grid_constant__ fr_mix_attn a, const int32_t* __restrict
   for (int e = threadIdx.x; e < a.heads * kHeadBlock; e += kMixThreads) {
     const int g = e / kHeadBlock, h = h0 + e % kHeadBlock;
     const float t = h < a.heads ? a.coef[static_cast<int64_t>(h) * a.heads + g] : 0.f;
-    coef[e] = pack_f32x2(t, t);
+    coef[e] = mix::pack_f32x2(t, t);
   }
   __syncthreads();
   const int64_t head_stride = static_cast<int64_t>(kM) * ldp;
@@ -275,8 +263,8 @@ talk_mix_kernel(const __grid_constant__ fr_mix_attn a, const int32_t* __restrict
       uint64_t p[kMixAhead][2];
 #pragma unroll
       for (int x = 0; x < kMixAhead; ++x) {
-        p[x][0] = pack_f32x2(nxt[x].x * nf[x], nxt[x].y * nf[x]);
-        p[x][1] = pack_f32x2(nxt[x].z * nf[x], nxt[x].w * nf[x]);
+        p[x][0] = mix::pack_f32x2(nxt[x].x * nf[x], nxt[x].y * nf[x]);
+        p[x][1] = mix::pack_f32x2(nxt[x].z * nf[x], nxt[x].w * nf[x]);
       }
 #pragma unroll
       for (int x = 0; x < kMixAhead; ++x) {
@@ -292,10 +280,10 @@ talk_mix_kernel(const __grid_constant__ fr_mix_attn a, const int32_t* __restrict
 #pragma unroll
           for (int h = 0; h < kHeadBlock; h += 2) {
             const ulonglong2 t = *reinterpret_cast<const ulonglong2*>(cf + h);
-            fma_f32x2(acc[h][0], t.x, p[x][0]);
-            fma_f32x2(acc[h][1], t.x, p[x][1]);
-            fma_f32x2(acc[h + 1][0], t.y, p[x][0]);
-            fma_f32x2(acc[h + 1][1], t.y, p[x][1]);
+            acc[h][0] = mix::fma_f32x2(t.x, p[x][0], acc[h][0]);
+            acc[h][1] = mix::fma_f32x2(t.x, p[x][1], acc[h][1]);
+            acc[h + 1][0] = mix::fma_f32x2(t.y, p[x][0], acc[h + 1][0]);
+            acc[h + 1][1] = mix::fma_f32x2(t.y, p[x][1], acc[h + 1][1]);
           }
         }
       }
@@ -304,8 +292,8 @@ talk_mix_kernel(const __grid_constant__ fr_mix_attn a, const int32_t* __restrict
     for (int h = 0; h < kHeadBlock; ++h)
       if (h0 + h < a.heads) {
         float f[4];
-        unpack_f32x2(acc[h][0], f[0], f[1]);
-        unpack_f32x2(acc[h][1], f[2], f[3]);
+        mix::unpack_f32x2(acc[h][0], f[0], f[1]);
+        mix::unpack_f32x2(acc[h][1], f[2], f[3]);
         *reinterpret_cast<uint2*>(mixed + off + (h0 + h) * head_stride) =
             make_uint2(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]));
       }
