@@ -2,8 +2,7 @@
 weights it is given (float32 or float64). Whole sequences only: no cache, no state, no batching. It is written
 from the equations and shares no code with ``flashrec_b200``.
 
-Notation: ``x [T, width]`` residual stream, ``h = norm1(x)``, positions ``i`` (query) and ``j`` (key) count from 0.
-``faults`` (tests only) plants one mistake in the oracle, to show that a comparison would notice it."""
+Notation: ``x [T, width]`` residual stream, ``h = norm1(x)``, positions ``i`` (query) and ``j`` (key) count from 0."""
 
 from __future__ import annotations
 

@@ -230,11 +230,12 @@ def _mix_run(kind, q, k, v, mixer, dtype, coef, lam, eps, portions, tensor_cores
 DIFF_SHAPES = [  # heads, kv, dim, vdim, window, keep, tokens
     (4, 2, 64, 128, 100, 5, 300), (3, 3, 20, 24, 64, 0, 200), (8, 1, 96, 112, 33, 70, 270), (1, 1, 128, 192, 1000, 1, 150),
     (2, 1, 16, 16, 1, 0, 100), (2, 2, 192, 64, 65, 64, 260), (6, 2, 40, 80, 63, 65, 210), (2, 1, 208, 48, 50, 3, 140),
-    (2, 2, 32, 256, 80, 2, 130),
+    (2, 2, 32, 256, 80, 2, 130), (4, 2, 64, 128, 900, 4, 1500),
 ]
 TALK_SHAPES = [  # heads, kv, dim, vdim, chunk, tokens
     (4, 2, 64, 64, 100, 300), (8, 2, 128, 128, 128, 300), (6, 6, 24, 40, 64, 200), (5, 1, 48, 96, 63, 200),
     (1, 1, 16, 192, 65, 150), (3, 1, 192, 176, 1000, 140), (16, 8, 32, 128, 1, 70), (2, 1, 200, 200, 90, 150), (12, 4, 80, 32, 70, 210),
+    (4, 2, 128, 128, 700, 1300),
 ]
 
 
