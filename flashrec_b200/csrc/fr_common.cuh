@@ -268,8 +268,9 @@ __device__ __forceinline__ float ex2_approx(float x) {
 // Fast path only: returns the approximate silu(g) and sets `hard` when its bf16 rounding cannot
 // be trusted. Branch-free.
 __device__ __forceinline__ float silu_fast(float g, bool& hard) {
-  constexpr float kL2eHi = 1.44269502162933349609375f;  // fp32(log2 e)
-  constexpr float kL2eLo = 1.925963033500e-8f;          // log2 e - fp32(log2 e)
+  constexpr double kLog2e = 1.4426950408889634074;  // log2 e, split into its fp32 rounding and the rest
+  constexpr float kL2eHi = static_cast<float>(kLog2e);
+  constexpr float kL2eLo = static_cast<float>(kLog2e - static_cast<double>(kL2eHi));
   const float th = __fmul_rn(g, -kL2eHi);
   const float tl = __fmaf_rn(g, -kL2eLo, __fmaf_rn(g, -kL2eHi, -th));
   float e = ex2_approx(th);
