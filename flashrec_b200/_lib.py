@@ -66,7 +66,9 @@ class FrOutSegment(ctypes.Structure):
     """Mirror of ``struct fr_out_segment``."""
 
     _fields_ = [("kind", ctypes.c_int32), ("n0", ctypes.c_int32), ("n", ctypes.c_int32), ("pad_", ctypes.c_int32),
-                ("out", c_void_p), ("ldo", c_int64), ("row_map", c_void_p), ("bias", c_void_p)]
+                ("out", c_void_p), ("ldo", c_int64), ("row_map", c_void_p), ("bias", c_void_p), ("limit", c_float),
+                ("alpha", c_float), ("up_bias", c_float), ("pad2_", ctypes.c_int32), ("mul", c_void_p), ("ld_mul", c_int64),
+                ("mul_map", c_void_p)]
 
 
 class FrGatedPart(ctypes.Structure):
@@ -91,11 +93,58 @@ class FrMixAttn(ctypes.Structure):
                 + [("coef", c_void_p), ("slopes", c_void_p), ("q", c_void_p), ("ldq", c_int64), ("k", c_void_p),
                    ("v", c_void_p), ("ldk", c_int64), ("ldv", c_int64), ("out", c_void_p), ("ldo", c_int64),
                    ("req_to_token", c_void_p), ("table_stride", c_int64), ("req_rows", c_void_p),
-                   ("tok_req", c_void_p), ("pos", c_void_p), ("num_slots", c_int64)])
+                   ("tok_req", c_void_p), ("pos", c_void_p), ("num_slots", c_int64), ("head_gate", c_void_p),
+                   ("ld_gate", c_int64)])
 
 
-FR_SEG_STORE, FR_SEG_SWIGLU, FR_SEG_SIGMOID, FR_SEG_STORE_F32 = 0, 1, 2, 3
-FR_MIX_DIFF, FR_MIX_TALK = 0, 1
+class FrNormPart(ctypes.Structure):
+    """Mirror of ``struct fr_norm_part``."""
+
+    _fields_ = [("y", c_void_p), ("ldy", c_int64), ("weight", c_void_p), ("coef", c_float), ("pad_", ctypes.c_int32)]
+
+
+class FrNormUpdate(ctypes.Structure):
+    """Mirror of ``struct fr_norm_update``."""
+
+    _fields_ = ([(n, ctypes.c_int32) for n in ("dtype", "n_parts", "n_partials")] + [("eps", c_float), ("offset", c_float),
+                ("pad_", ctypes.c_int32), ("x", c_void_p), ("ldx", c_int64), ("partials", c_void_p), ("partial_stride", c_int64),
+                ("parts", FrNormPart * 2), ("add", c_void_p), ("row_idx", c_void_p), ("weight", c_void_p), ("out", c_void_p),
+                ("ldo", c_int64)])
+
+
+class FrGroupNorm(ctypes.Structure):
+    """Mirror of ``struct fr_group_norm``."""
+
+    _fields_ = ([(n, ctypes.c_int32) for n in ("dtype", "gate_mode", "groups", "size", "weight_per_group")] + [("eps", c_float),
+                ("y", c_void_p), ("ldy", c_int64), ("gate", c_void_p), ("ldg", c_int64), ("weight", c_void_p), ("out", c_void_p),
+                ("ldo", c_int64)])
+
+
+class FrQkRope(ctypes.Structure):
+    """Mirror of ``struct fr_qk_rope``."""
+
+    _fields_ = ([(n, ctypes.c_int32) for n in ("dtype", "heads", "kv_heads", "dim", "dim_true", "rot_dims")] + [("eps", c_float),
+                ("pad_", ctypes.c_int32), ("q", c_void_p), ("ldq", c_int64), ("k", c_void_p), ("ldk", c_int64),
+                ("q_weight", c_void_p), ("k_weight", c_void_p), ("inv_freq", c_void_p), ("pos", c_void_p), ("loc", c_void_p),
+                ("k_cache", c_void_p), ("ldkc", c_int64)])
+
+
+class FrLinearScan(ctypes.Structure):
+    """Mirror of ``struct fr_linear_scan``."""
+
+    _fields_ = ([(n, ctypes.c_int32) for n in ("dtype", "decay", "heads", "key_heads", "dim", "vdim", "rank")]
+                + [("scale", c_float), ("inv_tau", c_float), ("pad_", ctypes.c_int32), ("q", c_void_p), ("ldq", c_int64),
+                   ("k", c_void_p), ("ldk", c_int64), ("v", c_void_p), ("ldv", c_int64), ("out", c_void_p), ("ldo", c_int64),
+                   ("step", c_void_p), ("ldstep", c_int64), ("step_bias", c_void_p), ("rate", c_void_p), ("up", c_void_p),
+                   ("skip", c_void_p), ("state", c_void_p), ("state_slots", c_void_p), ("qo_indptr", c_void_p),
+                   ("pos", c_void_p)])
+
+
+FR_SEG_STORE, FR_SEG_SWIGLU, FR_SEG_SIGMOID, FR_SEG_STORE_F32, FR_SEG_GLU_CLAMP, FR_SEG_GELU_MUL = 0, 1, 2, 3, 4, 5
+FR_MIX_DIFF, FR_MIX_TALK, FR_MIX_PLAIN = 0, 1, 2
+FR_CONV_LINEAR, FR_CONV_SILU = 0, 1
+FR_GATE_NONE, FR_GATE_BEFORE, FR_GATE_AFTER = 0, 1, 2
+FR_DECAY_CHANNEL, FR_DECAY_HEAD = 0, 1
 FR_MASK_WINDOW, FR_MASK_CHUNK = 0, 1
 
 FR_TRIE_NONE, FR_TRIE_DENSE, FR_TRIE_CSR, FR_TRIE_BITMAP = 0, 1, 2, 3
@@ -159,7 +208,12 @@ _SIGNATURES = {
     "fr_dense_gated_add_splits": [_I] * 5,
     "fr_lm_embed": [_I, P, _L, P, P, _L, _I, _I, _I, _F, P, _L, P, P, P, P],
     "fr_lm_norm": [_I, P, _L, P, _F, _F, P, _I, _L, P, P, _L, _I, _I, P],
-    "fr_short_conv": [_I, P, _L, P, _I, _I, P, _I, P, P, P, P, P, _I, _I, _I, P],
+    "fr_lm_update_norm": [P, _I, _I, P],
+    "fr_lm_group_norm": [P, _I, P],
+    "fr_lm_qk_norm_rope": [P, _I, P],
+    "fr_linear_state_floats": [_I, _I],
+    "fr_linear_scan_rows": [P, _I, _I, _I, P],
+    "fr_short_conv": [_I, P, _L, P, P, _I, _I, _I, P, _I, P, P, P, P, P, _I, _I, _I, P],
     "fr_mix_attn_rows": [P, _I, _I, _I, _I, P, _L, P, P],
     "fr_mix_attn_rows_scratch": [_I] * 6,
     "fr_mix_attn_tc": [P, P, _I, _I, _I, P, _L, P],
@@ -169,7 +223,7 @@ _SIGNATURES = {
 _RESTYPES = {"fr_version": c_char_p, "fr_decode_attn_scratch_bytes": c_int64,
              "fr_sid_head_topk_workspace_bytes": c_int64, "fr_joint_select_workspace_bytes": c_int64,
              "fr_trie_build_workspace_bytes": c_int64, "fr_mix_attn_rows_scratch": c_int64,
-             "fr_mix_attn_tc_scratch": c_int64}
+             "fr_mix_attn_tc_scratch": c_int64, "fr_linear_state_floats": c_int64}
 
 
 def lib_path() -> Path:

@@ -1,6 +1,7 @@
 // Attention whose outputs are linear combinations of several softmax maps over the same values
 // (fr_mix_attn in the header): differential attention (two maps per head, weights 1 and -lambda, the result
-// divided by its root mean square) and talking heads (all heads' maps, one matrix row per output head), with
+// divided by its root mean square), talking heads (all heads' maps, one matrix row per output head) and ordinary
+// attention (one map per head, optionally times a sigmoid per head), with
 // a sliding window that keeps the first tokens or with chunks, and an optional linear distance bias.
 //
 // Because the mixture is linear, sum_s coef[o, s] (P_s V) = (sum_s coef[o, s] P_s) V:
@@ -129,7 +130,12 @@ mix_scores_kernel(const __grid_constant__ fr_mix_attn a, int row0, int max_keys,
 constexpr int kValThreads = 256;
 constexpr int kValKeys = 256;  // keys per pass (weights of all maps in shared memory)
 
-// Root-mean-square scaling (DIFF) and store of one output head; f [vdim] in shared memory.
+// sigmoid(head_gate) of one output head, 1 without a gate
+__device__ __forceinline__ float head_gate_of(const fr_mix_attn& a, int64_t t, int head) {
+  return a.head_gate != nullptr ? 1.0f / (1.0f + expf(-a.head_gate[t * a.ld_gate + head])) : 1.0f;
+}
+
+// Root-mean-square scaling (DIFF) or head gate, and store of one output head; f [vdim] in shared memory.
 template <typename T>
 __device__ __forceinline__ void finish_head(const fr_mix_attn& a, int64_t t, int head, const float* f, float* red) {
   float r = 1.0f;
@@ -143,6 +149,8 @@ __device__ __forceinline__ void finish_head(const fr_mix_attn& a, int64_t t, int
     for (int w = 0; w < kValThreads / 32; ++w) tot += red[w];
     r = a.out_scale / sqrtf(tot / static_cast<float>(a.vdim_true) + a.eps);
     __syncthreads();
+  } else {
+    r = head_gate_of(a, t, head);
   }
   T* out = static_cast<T*>(a.out) + t * a.ldo + static_cast<int64_t>(head) * a.vdim;
   for (int c = threadIdx.x; c < a.vdim; c += kValThreads) st_f(out + c, f[c] * r);
@@ -158,7 +166,8 @@ mix_values_kernel(const __grid_constant__ fr_mix_attn a, int row0, int max_keys,
   const int rep = a.heads / a.kv_heads;
   const bool diff = a.mix == FR_MIX_DIFF;
   const int n_src = diff ? 2 * a.heads : a.heads;   // of the row
-  const int my_src = diff ? 2 * rep : a.heads;      // that this kv head's outputs mix
+  const bool plain = a.mix == FR_MIX_PLAIN;
+  const int my_src = diff ? 2 * rep : (plain ? rep : a.heads);  // that this kv head's outputs mix
   float* s_m = sm;                                  // [my_src]
   float* s_il = s_m + my_src;                       // [my_src]
   float* s_p = s_il + my_src;                       // [my_src][keys per pass]
@@ -174,7 +183,7 @@ mix_values_kernel(const __grid_constant__ fr_mix_attn a, int row0, int max_keys,
   const int64_t i = a.pos[t];
   const Visible vis = visible_keys(a, i, max_keys);
   const int blocks = (vis.n + kKeyBlock - 1) / kKeyBlock;
-  const int src0 = diff ? 2 * g * rep : 0;
+  const int src0 = diff ? 2 * g * rep : (plain ? g * rep : 0);
   const int64_t srow = static_cast<int64_t>(lrow) * n_src + src0;
   for (int s = tid >> 5; s < my_src; s += kValThreads / 32) {
     const float2* st = stats + (srow + s) * n_blocks;
@@ -216,6 +225,8 @@ mix_values_kernel(const __grid_constant__ fr_mix_attn a, int row0, int max_keys,
           float w = 0.f;
           if (diff) {
             w = s_p[2 * (o0 + o) * pass_keys + kk] - a.lambda * s_p[(2 * (o0 + o) + 1) * pass_keys + kk];
+          } else if (plain) {
+            w = s_p[(o0 + o) * pass_keys + kk];
           } else {
             const float* cf = a.coef + static_cast<int64_t>(g * rep + o0 + o) * a.heads;
             for (int s = 0; s < my_src; ++s) w = fmaf(__ldg(cf + s), s_p[s * pass_keys + kk], w);
@@ -302,7 +313,7 @@ mix_values_kernel(const __grid_constant__ fr_mix_attn a, int row0, int max_keys,
 
 static int values_smem(const fr_mix_attn& a, int ob, int pass_keys) {
   const int rep = a.heads / a.kv_heads;
-  const int my_src = a.mix == FR_MIX_DIFF ? 2 * rep : a.heads;
+  const int my_src = a.mix == FR_MIX_DIFF ? 2 * rep : (a.mix == FR_MIX_PLAIN ? rep : a.heads);
   return (my_src * (2 + pass_keys) + ob * pass_keys + kValThreads * 8 + 32) * 4 + pass_keys * 8;
 }
 
@@ -359,7 +370,7 @@ constexpr int kTcBarBytes = 288 + kPageList * 4;
 struct TcPlan {
   int q_boxes, v_boxes;   // 64-column boxes of a q / k row and of a v row
   int v_cols;             // TMEM columns of O and of one accumulator
-  int n_out;              // outputs per CTA
+  int n_out;              // outputs per CTA (PLAIN: 1, which needs no accumulator)
   int out_blocks;         // CTAs along y per v head (TALK) or per head (DIFF)
   int staged;             // DIFF: the first map's result waits in shared memory (fp16), not in TMEM
   int stages;             // K and V stages
@@ -377,11 +388,11 @@ static bool plan_tc(int mix, int heads, int kv_heads, int dim, int vdim, TcPlan*
   int fit = (512 - 2 * kTileN - pl->v_cols) / pl->v_cols;
   if (fit < 1) return false;
   if (fit > kMaxOut) fit = kMaxOut;
-  const int outs = mix == FR_MIX_DIFF ? 1 : rep;
+  const int outs = mix == FR_MIX_TALK ? rep : 1;
   const int blocks = (outs + fit - 1) / fit;
   pl->n_out = (outs + blocks - 1) / blocks;
   pl->out_blocks = blocks;
-  int need = 2 * kTileN + pl->v_cols * (1 + pl->n_out);
+  int need = 2 * kTileN + pl->v_cols * (mix == FR_MIX_PLAIN ? 1 : 1 + pl->n_out);
   if (mix == FR_MIX_DIFF && need > 256 && need - pl->v_cols <= 256) {  // without the accumulator two CTAs share an SM
     pl->staged = 1;
     need -= pl->v_cols;
@@ -430,22 +441,28 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
   ptx::griddep_wait();
   ptx::griddep_launch_dependents();
   const int rep = a.heads / a.kv_heads;
-  const bool diff = a.mix == FR_MIX_DIFF;
-  // y: DIFF head; TALK (v head, block of its outputs)
-  const int vh = diff ? static_cast<int>(blockIdx.y) / rep : static_cast<int>(blockIdx.y) / pl.out_blocks;
-  const int out0 = diff ? static_cast<int>(blockIdx.y)
-                        : vh * rep + static_cast<int>(blockIdx.y) % pl.out_blocks * pl.n_out;
-  const int n_out = diff ? 1 : min(pl.n_out, (vh + 1) * rep - out0);
-  const int n_src = diff ? 2 : a.heads;
-  const int src0 = diff ? 2 * out0 : 0;
-  const int req = tiles[3 * blockIdx.x], row0 = tiles[3 * blockIdx.x + 1], n_tok = tiles[3 * blockIdx.x + 2];
+  const bool diff = a.mix == FR_MIX_DIFF, plain = a.mix == FR_MIX_PLAIN;
+  // x: tile, y: DIFF head; TALK (v head, block of its outputs). PLAIN: the heads of a tile side by side, the last
+  // tiles (with the most keys below the causal edge) first
+  int tile = blockIdx.x, by = blockIdx.y;
+  if (plain) {
+    const int id = static_cast<int>(blockIdx.y * gridDim.x + blockIdx.x);
+    tile = static_cast<int>(gridDim.x) - 1 - id / a.heads;
+    by = id % a.heads;
+  }
+  const int vh = diff || plain ? by / rep : by / pl.out_blocks;
+  const int out0 = diff || plain ? by : vh * rep + by % pl.out_blocks * pl.n_out;
+  const int n_out = diff || plain ? 1 : min(pl.n_out, (vh + 1) * rep - out0);
+  const int n_src = diff ? 2 : (plain ? 1 : a.heads);
+  const int src0 = diff ? 2 * out0 : (plain ? out0 : 0);
+  const int req = tiles[3 * tile], row0 = tiles[3 * tile + 1], n_tok = tiles[3 * tile + 2];
   const int pos0 = static_cast<int>(a.pos[row0]);
   const int pos_last = pos0 + n_tok - 1;
   const int32_t* table = a.req_to_token + a.req_rows[req] * a.table_stride;
   const KeyTiles kt = key_tiles(a, pos0, pos_last);  // every role derives the same list
   const int n_tiles = kt.n;
   const int total = n_tiles * n_src;
-  auto k_head = [&](int s) { return diff ? 2 * vh + s : s / rep; };
+  auto k_head = [&](int s) { return diff ? 2 * vh + s : (plain ? vh : s / rep); };
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
@@ -679,6 +696,26 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
       ok = wait_all(bar_done, s & 1, 81);
       if (!ok) break;
       const float inv = 1.0f / l_sum;
+      if (plain) {
+        const float scl = inv * head_gate_of(a, row0 + min(r, n_tok - 1), out0);
+#pragma unroll 1
+        for (int c = 0; c < pl.v_cols / 32; ++c) {
+          uint32_t o[32];
+          ptx::tmem_ld_32x32(col_o + lane_off + c * 32, o);
+          ptx::tmem_ld_wait();
+#pragma unroll
+          for (int x = 0; x < 2; ++x) {  // 16 columns: one 32-byte store
+            uint32_t w8[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e)
+              w8[e] = pack_bf16(__uint_as_float(o[16 * x + 2 * e]) * scl, __uint_as_float(o[16 * x + 2 * e + 1]) * scl);
+            if (live && c * 32 + x * 16 < a.vdim) ptx::st_global_v8(out_row + c * 32 + x * 16, w8);
+          }
+          __syncwarp();
+        }
+        ptx::tc_fence_before();
+        continue;
+      }
       if (pl.staged) {
         // first map: a1 as fp16 into this thread's own row of shared memory; second map: a1 - lambda a2, scaled by its
         // root mean square, into the output (two passes over O)
@@ -760,7 +797,7 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
       ptx::tc_fence_before();
       ptx::mbar_arrive(bar_oread);
     }
-    if (ok && !pl.staged) {
+    if (ok && !pl.staged && !plain) {
       for (int n = 0; n < n_out; ++n) {
         float scl = 1.0f;
         if (diff) {
@@ -811,7 +848,7 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
 }
 
 static int check_args(const fr_mix_attn* a) {
-  FR_CHECK_ARG(a && (a->dtype == 0 || a->dtype == 1) && (a->mix == FR_MIX_DIFF || a->mix == FR_MIX_TALK));
+  FR_CHECK_ARG(a && (a->dtype == 0 || a->dtype == 1) && a->mix >= FR_MIX_DIFF && a->mix <= FR_MIX_PLAIN);
   FR_CHECK_ARG((a->mask == FR_MASK_WINDOW || a->mask == FR_MASK_CHUNK) && a->mask_size > 0 && a->keep_first >= 0);
   FR_CHECK_ARG(a->heads > 0 && a->kv_heads > 0 && a->heads % a->kv_heads == 0);
   FR_CHECK_ARG(a->dim > 0 && a->dim % 16 == 0 && a->vdim > 0 && a->vdim % 16 == 0 && a->vdim_true > 0);
@@ -819,6 +856,7 @@ static int check_args(const fr_mix_attn* a) {
   FR_CHECK_ARG(aligned16(a->q) && aligned16(a->k) && aligned16(a->v) && aligned16(a->out) && a->ldq % 8 == 0 &&
                a->ldk % 8 == 0 && a->ldv % 8 == 0 && a->ldo % 8 == 0);
   FR_CHECK_ARG(a->mix != FR_MIX_TALK || a->coef);
+  FR_CHECK_ARG(a->head_gate == nullptr || (a->mix == FR_MIX_PLAIN && a->ld_gate >= a->heads));
   return FR_OK;
 }
 
@@ -892,7 +930,7 @@ extern "C" int fr_mix_attn_tc(const fr_mix_attn* a, const int32_t* tiles, int n_
   if (r != FR_OK) return r;
   int* status = device_status_ptr();
   if (!status) return FR_ERR_CUDA;
-  dim3 grid(n_tiles, diff ? a->heads : a->kv_heads * pl.out_blocks);
+  dim3 grid(n_tiles, a->mix == FR_MIX_TALK ? a->kv_heads * pl.out_blocks : a->heads);
   static PerDeviceFlag f0, f1;
   if (a->slopes != nullptr || !(a->scale > 0.f)) {
     if (ensure_dyn_smem(f1, mix::mix_tc_kernel<true>, 227 * 1024) != FR_OK) return FR_ERR_CUDA;

@@ -2,7 +2,8 @@
 //
 //   fr_dense_proj       every projection of the normalised input h as ONE product with the merged weight; the
 //                       column ranges leave through their own epilogues (plain store, store into KV-cache
-//                       slots, SwiGLU of interleaved gate / up rows, sigmoid with bias)
+//                       slots, SwiGLU or clamped GLU of interleaved gate / up rows, sigmoid with bias, GELU
+//                       times a looked-up row)
 //   fr_dense_gated_add  x += g1 * (A1 W1^T) + g2 * (A2 W2^T) on the fp32 residual stream
 //
 // Three implementations behind each:
@@ -21,7 +22,7 @@ int* device_status_ptr();  // capi.cu
 
 namespace dense {
 
-constexpr int kMaxSegs = 8;
+constexpr int kMaxSegs = 12;
 struct Segs {
   fr_out_segment s[kMaxSegs];
   int n;
@@ -70,6 +71,25 @@ __device__ __forceinline__ float sigmoid_f(float z) {
 template <bool FAST>
 __device__ __forceinline__ float silu_f(float z) { return z * sigmoid_f<FAST>(z); }
 
+// gelu with the tanh approximation: 0.5 z (1 + tanh(u)) = z sigmoid(2 u)
+template <bool FAST>
+__device__ __forceinline__ float gelu_tanh_f(float z) {
+  constexpr float kRoot = 0.7978845608028654f;  // sqrt(2 / pi)
+  return z * sigmoid_f<FAST>(2.0f * kRoot * (z + 0.044715f * z * z * z));
+}
+
+// Ranges whose weight rows come in [32 gate | 32 up] blocks, and the activation of a pair.
+__host__ __device__ __forceinline__ bool paired(const fr_out_segment& s) {
+  return s.kind == FR_SEG_SWIGLU || s.kind == FR_SEG_GLU_CLAMP;
+}
+template <bool FAST>
+__device__ __forceinline__ float pair_act(const fr_out_segment& s, float g, float u) {
+  if (s.kind == FR_SEG_SWIGLU) return silu_f<FAST>(g) * u;
+  g = fminf(g, s.limit);
+  u = fminf(fmaxf(u, -s.limit), s.limit);
+  return g * sigmoid_f<FAST>(s.alpha * g) * (u + s.up_bias);
+}
+
 __device__ __forceinline__ int seg_of(const Segs& sg, int col) {
   int i = 0;
 #pragma unroll 1
@@ -87,6 +107,8 @@ __device__ __forceinline__ void seg_write(const fr_out_segment& s, int64_t row, 
     return;
   }
   if (s.kind == FR_SEG_SIGMOID) z = sigmoid_f<FAST>(z + (s.bias != nullptr ? s.bias[c] : 0.f));
+  if (s.kind == FR_SEG_GELU_MUL)
+    z = gelu_tanh_f<FAST>(z) * to_f<T>(static_cast<const T*>(s.mul)[(s.mul_map != nullptr ? s.mul_map[row] : row) * s.ld_mul + c]);
   static_cast<T*>(s.out)[r * s.ldo + c] = from_f<T>(z);
 }
 
@@ -155,7 +177,7 @@ dense_rows_proj_kernel(const T* __restrict__ a, int64_t lda, const T* __restrict
     si = seg_of(sg, grp * 4);
     const fr_out_segment& s = sg.s[si];
     const int local = grp * 4 - s.n0;
-    if (s.kind == FR_SEG_SWIGLU) {  // two channels: rows {gate c, gate c + 1, up c, up c + 1}
+    if (paired(s)) {  // two channels: rows {gate c, gate c + 1, up c, up c + 1}
       c0 = local / 2;
       const int64_t g = s.n0 + (c0 / 32) * 64 + c0 % 32;
       wr[0] = w + g * ldw;
@@ -182,7 +204,7 @@ dense_rows_proj_kernel(const T* __restrict__ a, int64_t lda, const T* __restrict
   __syncthreads();
   if (!live || kwarp != 0) return;
   const fr_out_segment& s = sg.s[si];
-  if (s.kind == FR_SEG_SWIGLU) {
+  if (paired(s)) {
     if (lane < 2 * MB) {
       const int r = lane / MB, m = lane % MB;
       float g = 0.f, u = 0.f;
@@ -190,7 +212,7 @@ dense_rows_proj_kernel(const T* __restrict__ a, int64_t lda, const T* __restrict
         g += red[warp + k][r * MB + m];
         u += red[warp + k][(r + 2) * MB + m];
       }
-      if (m < M) seg_write<T, kFast>(s, m, c0 + r, silu_f<kFast>(g) * u);
+      if (m < M) seg_write<T, kFast>(s, m, c0 + r, pair_act<kFast>(s, g, u));
     }
   } else if (lane < 4 * MB) {
     const int r = lane / MB, m = lane % MB;
@@ -301,13 +323,13 @@ dense_simt_proj_kernel(const float* __restrict__ a, int64_t lda, const float* __
     const int col0 = n0 + half * 32;  // a 32-column chunk lies in one range
     if (col0 >= N) break;
     const fr_out_segment& s = sg.s[seg_of(sg, col0)];
-    if (s.kind == FR_SEG_SWIGLU) {
+    if (paired(s)) {
       if (half == 1) continue;
       const int ch = (col0 - s.n0) / 2 + tx * 2;
       for (int i = 0; i < 4; ++i) {
         const int row = m0 + ty * 4 + i;
         if (row >= M) break;
-        for (int j = 0; j < 2; ++j) seg_write<float, false>(s, row, ch + j, silu_f<false>(acc[i][j]) * acc[i][2 + j]);
+        for (int j = 0; j < 2; ++j) seg_write<float, false>(s, row, ch + j, pair_act<false>(s, acc[i][j], acc[i][2 + j]));
       }
     } else {
       for (int i = 0; i < 4; ++i) {
@@ -579,11 +601,11 @@ dense_tc_kernel(const __grid_constant__ CUtensorMap ta0, const __grid_constant__
             ptx::tmem_ld_wait();
             if (row < g.M) {
             const fr_out_segment& s0 = g.segs.s[seg_of(g.segs, col)];
-            if (s0.kind == FR_SEG_SWIGLU) {
+            if (paired(s0)) {
               const int ch = (col - s0.n0) / 2;
               float v[32];
 #pragma unroll
-              for (int i = 0; i < 32; ++i) v[i] = silu_f<true>(__uint_as_float(r0[i])) * __uint_as_float(r1[i]);
+              for (int i = 0; i < 32; ++i) v[i] = pair_act<true>(s0, __uint_as_float(r0[i]), __uint_as_float(r1[i]));
               const int64_t r = s0.row_map != nullptr ? s0.row_map[row] : row;
               store32_bf16(static_cast<__nv_bfloat16*>(s0.out) + r * s0.ldo + ch, v, s0.n - ch);
             } else {
@@ -607,6 +629,13 @@ dense_tc_kernel(const __grid_constant__ CUtensorMap ta0, const __grid_constant__
                           const float b = (s.bias != nullptr && i < nvalid) ? __ldg(s.bias + lc + i) : 0.f;
                           v[i] = sigmoid_f<true>(v[i] + b);
                         }
+                      }
+                      if (s.kind == FR_SEG_GELU_MUL) {
+                        const __nv_bfloat16* mul = static_cast<const __nv_bfloat16*>(s.mul) +
+                                                   (s.mul_map != nullptr ? s.mul_map[row] : row) * s.ld_mul + lc;
+#pragma unroll
+                        for (int i = 0; i < 32; ++i)
+                          if (i < nvalid) v[i] = gelu_tanh_f<true>(v[i]) * __bfloat162float(__ldg(mul + i));
                       }
                       store32_bf16(static_cast<__nv_bfloat16*>(s.out) + r * s.ldo + lc, v, nvalid);
                     }
@@ -826,9 +855,10 @@ extern "C" int fr_dense_proj(int dtype, const void* a, int64_t lda, const void* 
   for (int i = 0; i < n_segs; ++i) {
     const fr_out_segment& s = segs[i];
     const int end = i + 1 < n_segs ? segs[i + 1].n0 : N;
-    FR_CHECK_ARG(s.out && s.n0 % 32 == 0 && s.n > 0 && s.kind >= 0 && s.kind <= FR_SEG_STORE_F32);
+    FR_CHECK_ARG(s.out && s.n0 % 32 == 0 && s.n > 0 && s.kind >= 0 && s.kind <= FR_SEG_GELU_MUL);
     FR_CHECK_ARG(s.n0 < end && (i > 0 || s.n0 == 0));
-    if (s.kind == FR_SEG_SWIGLU)
+    FR_CHECK_ARG(s.kind != FR_SEG_GELU_MUL || s.mul);
+    if (dense::paired(s))
       FR_CHECK_ARG(s.n0 % 64 == 0 && (end - s.n0) % 64 == 0 && 2 * s.n <= end - s.n0);
     else
       FR_CHECK_ARG(s.n <= end - s.n0);

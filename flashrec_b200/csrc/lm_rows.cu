@@ -1,5 +1,7 @@
 // Row kernels of the 16/32-bit decoder layers: embedding lookup into the fp32 residual stream (with the slot
-// table entry of every new token), RMS norm of the fp32 stream, and the short causal convolution with its state.
+// table entry of every new token), RMS norm of the fp32 stream, updates of the stream by normalised vectors fused with
+// the norm that follows, gated norms over groups of columns, norm and rotation of queries and keys, and the short
+// causal convolution with its state.
 #include "fr_common.cuh"
 #include "sm100_ptx.cuh"
 
@@ -114,7 +116,15 @@ norm_kernel(float* __restrict__ x, int64_t ldx, const float* __restrict__ weight
 struct ConvOuts {
   fr_conv_out o[4];
   int n;
+  const float* bias;
+  int act;  // fr_conv_act
 };
+
+// silu; the 16-bit results leave through a fast exponential
+template <typename T>
+__device__ __forceinline__ float silu_t(float z) {
+  return sizeof(T) == 2 ? __fdividef(z, 1.0f + __expf(-z)) : z / (1.0f + expf(-z));
+}
 
 // Value of channel c at `back` tokens before token t of the batch (e = index of t within its request).
 template <typename T>
@@ -198,6 +208,10 @@ conv_vec_kernel(const T* __restrict__ u, int64_t ldu, const float* __restrict__ 
 #pragma unroll
       for (int k = 0; k < TAPS; ++k) wr[k][i] = flat[i * TAPS + k];
   }
+  float b0[8] = {};
+  if (c < C && outs.bias != nullptr)
+#pragma unroll
+    for (int i = 0; i < 8; ++i) b0[i] = outs.bias[c + i];
   ptx::griddep_wait();
   ptx::griddep_launch_dependents();
   if (c >= C) return;
@@ -267,7 +281,9 @@ conv_vec_kernel(const T* __restrict__ u, int64_t ldu, const float* __restrict__ 
           }
         }
       }
-      float y[8] = {};
+      float y[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) y[i] = b0[i];
 #pragma unroll
       for (int k = 0; k < TAPS; ++k) {
         float f[8];
@@ -275,6 +291,9 @@ conv_vec_kernel(const T* __restrict__ u, int64_t ldu, const float* __restrict__ 
 #pragma unroll
         for (int i = 0; i < 8; ++i) y[i] = fmaf(wr[k][i], f[i], y[i]);
       }
+      if (outs.act == FR_CONV_SILU)
+#pragma unroll
+        for (int i = 0; i < 8; ++i) y[i] = silu_t<T>(y[i]);
       if (keep) conv_store8<T>(out + dst[x] * o.ldo, y);
 #pragma unroll
       for (int k = 0; k + 1 < P; ++k) win[k] = win[k + 1];
@@ -306,9 +325,10 @@ short_conv_kernel(const T* __restrict__ u, int64_t ldu, const float* __restrict_
   const int64_t p = pos[t];
   T* st = state + state_slots[b] * (taps - 1) * C;
   const float* wc = w + static_cast<int64_t>(c) * taps;
-  float y = 0.f;
+  float y = outs.bias != nullptr ? outs.bias[c] : 0.f;
   for (int back = taps - 1; back >= 0; --back)
     y = fmaf(wc[taps - 1 - back], conv_tap(u, ldu, st, C, taps, t, e, p, c, back), y);
+  if (outs.act == FR_CONV_SILU) y = silu_t<T>(y);
   for (int i = 0; i < outs.n; ++i) {
     const fr_conv_out& o = outs.o[i];
     if (c >= o.c0 && c < o.c0 + o.c) {
@@ -386,6 +406,319 @@ static int launch_norm(float* x, int64_t ldx, const float* weight, float offset,
                        weight, offset, eps, partials, n_partials, ps, row_idx, o, ldo, W);
 }
 
+// ---------------------------------------------------------------------------
+// x += partials, += coef * rms(y) * w per part, += a vector; then the norm of the result (or the result itself)
+// ---------------------------------------------------------------------------
+template <typename T>
+__device__ __forceinline__ float4 ld4(const T* p);
+template <>
+__device__ __forceinline__ float4 ld4<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
+template <>
+__device__ __forceinline__ float4 ld4<__nv_bfloat16>(const __nv_bfloat16* p) {
+  const uint2 q = *reinterpret_cast<const uint2*>(p);
+  return make_float4(bf16lo(q.x), bf16hi(q.x), bf16lo(q.y), bf16hi(q.y));
+}
+template <typename T>
+__device__ __forceinline__ void st4(T* p, const float4& v) {
+  if constexpr (sizeof(T) == 2) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+  } else {
+    *reinterpret_cast<float4*>(p) = v;
+  }
+}
+__device__ __forceinline__ float sq4(const float4& v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+
+// Sum of a value over a CTA of NT threads (every thread gets it); `sums` is scratch that the next call may reuse only
+// after another barrier, so callers alternate between two.
+template <int NT>
+__device__ __forceinline__ float cta_sum(float v, float* sums) {
+  v = warp_sum(v);
+  if ((threadIdx.x & 31) == 0) sums[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float tot = 0.f;
+#pragma unroll
+  for (int i = 0; i < NT / 32; ++i) tot += sums[i];
+  return tot;
+}
+
+// NV: float4 values per thread; 0: any width, re-reading what does not fit into registers
+template <typename T, int NV>
+__global__ void __launch_bounds__(kNormThreads)
+update_norm_kernel(const __grid_constant__ fr_norm_update u, int W) {
+  __shared__ float sums[4][kNormThreads / 32];
+  ptx::griddep_wait();
+  ptx::griddep_launch_dependents();
+  const int64_t t = blockIdx.x;
+  const int64_t src = u.row_idx != nullptr ? u.row_idx[t] : t;
+  float* xr = u.x + src * u.ldx;
+  T* o = static_cast<T*>(u.out) + t * u.ldo;
+  const float* pr = u.n_partials > 0 ? u.partials + src * W : nullptr;
+  const bool write_x = u.row_idx == nullptr && (pr != nullptr || u.n_parts > 0 || u.add != nullptr);
+  if constexpr (NV > 0) {
+    float4 v[NV], y[2][NV];
+    float ss[2] = {0.f, 0.f};
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * kNormThreads + threadIdx.x) * 4;
+      v[i] = y[0][i] = y[1][i] = make_float4(0, 0, 0, 0);
+      if (c >= W) continue;
+      v[i] = *reinterpret_cast<const float4*>(xr + c);
+#pragma unroll
+      for (int p = 0; p < 2; ++p)
+        if (p < u.n_parts) {
+          y[p][i] = ld4<T>(static_cast<const T*>(u.parts[p].y) + src * u.parts[p].ldy + c);
+          ss[p] += sq4(y[p][i]);
+        }
+      if (pr != nullptr)
+        for (int s = 0; s < u.n_partials; ++s) {
+          const float4 q = *reinterpret_cast<const float4*>(pr + s * u.partial_stride + c);
+          v[i].x += q.x; v[i].y += q.y; v[i].z += q.z; v[i].w += q.w;
+        }
+    }
+    float r[2] = {0.f, 0.f};
+#pragma unroll
+    for (int p = 0; p < 2; ++p)
+      if (p < u.n_parts)
+        r[p] = u.parts[p].coef / sqrtf(cta_sum<kNormThreads>(ss[p], sums[p]) / static_cast<float>(W) + u.eps);
+    float sx = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * kNormThreads + threadIdx.x) * 4;
+      if (c >= W) continue;
+#pragma unroll
+      for (int p = 0; p < 2; ++p)
+        if (p < u.n_parts) {
+          const float4 w = *reinterpret_cast<const float4*>(u.parts[p].weight + c);
+          v[i].x += y[p][i].x * r[p] * w.x; v[i].y += y[p][i].y * r[p] * w.y;
+          v[i].z += y[p][i].z * r[p] * w.z; v[i].w += y[p][i].w * r[p] * w.w;
+        }
+      if (u.add != nullptr) {
+        const float4 a = *reinterpret_cast<const float4*>(u.add + c);
+        v[i].x += a.x; v[i].y += a.y; v[i].z += a.z; v[i].w += a.w;
+      }
+      if (write_x) *reinterpret_cast<float4*>(xr + c) = v[i];
+      sx += sq4(v[i]);
+    }
+    if (u.out == nullptr) return;
+    float rx = 1.0f;
+    if (u.weight != nullptr) rx = 1.0f / sqrtf(cta_sum<kNormThreads>(sx, sums[2]) / static_cast<float>(W) + u.eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * kNormThreads + threadIdx.x) * 4;
+      if (c >= W) continue;
+      float4 w = make_float4(1, 1, 1, 1);
+      if (u.weight != nullptr) {
+        w = *reinterpret_cast<const float4*>(u.weight + c);
+        w.x += u.offset; w.y += u.offset; w.z += u.offset; w.w += u.offset;
+      }
+      st4(o + c, make_float4(v[i].x * rx * w.x, v[i].y * rx * w.y, v[i].z * rx * w.z, v[i].w * rx * w.w));
+    }
+  } else {
+    float r[2] = {0.f, 0.f};
+    for (int p = 0; p < u.n_parts; ++p) {
+      float ss = 0.f;
+      const T* y = static_cast<const T*>(u.parts[p].y) + src * u.parts[p].ldy;
+      for (int c = threadIdx.x; c < W; c += kNormThreads) {
+        const float f = ld_f(y + c);
+        ss += f * f;
+      }
+      r[p] = u.parts[p].coef / sqrtf(cta_sum<kNormThreads>(ss, sums[p]) / static_cast<float>(W) + u.eps);
+    }
+    auto value = [&](int c) {
+      float f = xr[c];
+      if (pr != nullptr)
+        for (int s = 0; s < u.n_partials; ++s) f += pr[s * u.partial_stride + c];
+      for (int p = 0; p < u.n_parts; ++p)
+        f += ld_f(static_cast<const T*>(u.parts[p].y) + src * u.parts[p].ldy + c) * r[p] * u.parts[p].weight[c];
+      if (u.add != nullptr) f += u.add[c];
+      return f;
+    };
+    float rx = 1.0f;
+    if (u.weight != nullptr && u.out != nullptr) {
+      float sx = 0.f;
+      for (int c = threadIdx.x; c < W; c += kNormThreads) {
+        const float f = value(c);
+        sx += f * f;
+      }
+      rx = 1.0f / sqrtf(cta_sum<kNormThreads>(sx, sums[2]) / static_cast<float>(W) + u.eps);
+    }
+    for (int c = threadIdx.x; c < W; c += kNormThreads) {  // a thread writes what only it reads
+      const float f = value(c);
+      if (write_x) xr[c] = f;
+      if (u.out != nullptr) st_f(o + c, u.weight != nullptr ? f * rx * (u.offset + u.weight[c]) : f);
+    }
+  }
+  if (u.out == nullptr) return;
+  const int wpad = (W + 7) / 8 * 8;
+  for (int c = W + threadIdx.x; c < wpad && c < u.ldo; c += kNormThreads) st_f(o + c, 0.f);
+}
+
+template <typename T>
+static int launch_update_norm(const fr_norm_update& u, int M, int W, cudaStream_t stream) {
+  bool vec = W % 4 == 0 && W <= kNormThreads * 4 * kNormVec && u.ldx % 4 == 0 && aligned16(u.x) && aligned16(u.weight) &&
+             aligned16(u.add) && u.ldo % 4 == 0 && aligned16(u.out) &&
+             (u.n_partials == 0 || (aligned16(u.partials) && u.partial_stride % 4 == 0));
+  for (int p = 0; p < u.n_parts; ++p)
+    vec = vec && u.parts[p].ldy % 4 == 0 && aligned16(u.parts[p].y) && aligned16(u.parts[p].weight);
+  auto kern = update_norm_kernel<T, 0>;
+  if (vec) kern = W <= kNormThreads * 8 ? update_norm_kernel<T, 2> : (W <= kNormThreads * 16 ? update_norm_kernel<T, 4> : update_norm_kernel<T, 8>);
+  return launch_kernel(kern, M, kNormThreads, 0, stream, M <= kPdlRows, u, W);
+}
+
+// ---------------------------------------------------------------------------
+// out = norm over groups of `size` columns, each by its own root mean square, with a silu gate before or after
+// ---------------------------------------------------------------------------
+constexpr int kGroupThreads = 256;
+
+// NT threads per (row, group); eight columns at a time, NV of them per thread in registers
+template <typename T, int NT, int NV>
+__global__ void __launch_bounds__(kGroupThreads)
+group_norm_kernel(const __grid_constant__ fr_group_norm a, int M) {
+  __shared__ float sums[kGroupThreads / 32];
+  ptx::griddep_wait();
+  ptx::griddep_launch_dependents();
+  const int64_t job = static_cast<int64_t>(blockIdx.x) * (kGroupThreads / NT) + threadIdx.x / NT;
+  if (job >= static_cast<int64_t>(M) * a.groups) return;  // whole warps (NT is 32 or the CTA)
+  const int64_t t = job / a.groups;
+  const int g = static_cast<int>(job % a.groups), c0 = g * a.size, l = threadIdx.x % NT;
+  const T* y = static_cast<const T*>(a.y) + t * a.ldy + c0;
+  const T* z = a.gate_mode != FR_GATE_NONE ? static_cast<const T*>(a.gate) + t * a.ldg + c0 : nullptr;
+  const float* w = a.weight + (a.weight_per_group ? c0 : 0);
+  T* o = static_cast<T*>(a.out) + t * a.ldo + c0;
+  float ss = 0.f;
+  if constexpr (NV > 0) {
+    float v[NV][8];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * NT + l) * 8;
+      if (c >= a.size) continue;
+      raw_unpack(raw_load<T>(y + c), v[i]);
+      if (a.gate_mode == FR_GATE_BEFORE) {
+        float zv[8];
+        raw_unpack(raw_load<T>(z + c), zv);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[i][e] *= silu_t<T>(zv[e]);
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss = fmaf(v[i][e], v[i][e], ss);
+    }
+    ss = NT == 32 ? warp_sum(ss) : cta_sum<kGroupThreads>(ss, sums);
+    const float r = 1.0f / sqrtf(ss / static_cast<float>(a.size) + a.eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * NT + l) * 8;
+      if (c >= a.size) continue;
+      float wv[8], f[8];
+      *reinterpret_cast<float4*>(wv) = *reinterpret_cast<const float4*>(w + c);
+      *reinterpret_cast<float4*>(wv + 4) = *reinterpret_cast<const float4*>(w + c + 4);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) f[e] = v[i][e] * r * wv[e];
+      if (a.gate_mode == FR_GATE_AFTER) {
+        float zv[8];
+        raw_unpack(raw_load<T>(z + c), zv);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] *= silu_t<T>(zv[e]);
+      }
+      conv_store8<T>(o + c, f);
+    }
+  } else {
+    auto value = [&](int c) { return ld_f(y + c) * (a.gate_mode == FR_GATE_BEFORE ? silu_t<T>(ld_f(z + c)) : 1.0f); };
+    for (int c = l; c < a.size; c += NT) {
+      const float f = value(c);
+      ss = fmaf(f, f, ss);
+    }
+    ss = NT == 32 ? warp_sum(ss) : cta_sum<kGroupThreads>(ss, sums);
+    const float r = 1.0f / sqrtf(ss / static_cast<float>(a.size) + a.eps);
+    for (int c = l; c < a.size; c += NT) {
+      float f = value(c) * r * w[c];
+      if (a.gate_mode == FR_GATE_AFTER) f *= silu_t<T>(ld_f(z + c));
+      st_f(o + c, f);
+    }
+  }
+  // columns up to the next multiple of eight: a matrix operand's padding
+  const int n = a.groups * a.size, npad = (n + 7) / 8 * 8;
+  if (g == a.groups - 1)
+    for (int c = n + l; c < npad && c < a.ldo; c += NT) st_f(static_cast<T*>(a.out) + t * a.ldo + c, 0.f);
+}
+
+template <typename T>
+static int launch_group_norm(const fr_group_norm& a, int M, cudaStream_t stream) {
+  const bool vec = a.size % 8 == 0 && a.ldy % 8 == 0 && a.ldo % 8 == 0 && aligned16(a.y) && aligned16(a.out) && aligned16(a.weight) &&
+                   (a.gate_mode == FR_GATE_NONE || (a.ldg % 8 == 0 && aligned16(a.gate)));
+  const int64_t jobs = static_cast<int64_t>(M) * a.groups;
+  const bool warp = a.size <= 1024;
+  auto kern = warp ? group_norm_kernel<T, 32, 0> : group_norm_kernel<T, kGroupThreads, 0>;
+  if (vec && warp) kern = a.size <= 256 ? group_norm_kernel<T, 32, 1> : group_norm_kernel<T, 32, 4>;
+  if (vec && !warp && a.size <= kGroupThreads * 32)
+    kern = a.size <= kGroupThreads * 16 ? group_norm_kernel<T, kGroupThreads, 2> : group_norm_kernel<T, kGroupThreads, 4>;
+  return launch_kernel(kern, ceil_div(jobs, warp ? kGroupThreads / 32 : 1), kGroupThreads, 0, stream, M <= kPdlRows, a, M);
+}
+
+// ---------------------------------------------------------------------------
+// queries and keys of one token: RMS norm over all heads at once, rotation, keys into the cache
+// ---------------------------------------------------------------------------
+constexpr int kRopeThreads = 256;
+
+template <typename T>
+__global__ void __launch_bounds__(kRopeThreads)
+qk_norm_rope_kernel(const __grid_constant__ fr_qk_rope a) {
+  extern __shared__ float sm[];
+  __shared__ float sums[2][kRopeThreads / 32];
+  const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim, half = a.rot_dims / 2;
+  float* s_q = sm;
+  float* s_k = s_q + nq;
+  float* s_cos = s_k + nk;
+  float* s_sin = s_cos + half;
+  ptx::griddep_wait();
+  ptx::griddep_launch_dependents();
+  const int64_t t = blockIdx.x;
+  const float p = static_cast<float>(a.pos[t]);
+  T* q = static_cast<T*>(a.q) + t * a.ldq;
+  const T* k = static_cast<const T*>(a.k) + t * a.ldk;
+  float sq = 0.f, sk = 0.f;
+  for (int c = threadIdx.x * 8; c < nq + nk; c += kRopeThreads * 8) {
+    float v[8];
+    raw_unpack(raw_load<T>(c < nq ? q + c : k + (c - nq)), v);
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss = fmaf(v[e], v[e], ss);
+    if (c < nq) sq += ss; else sk += ss;
+    *reinterpret_cast<float4*>(sm + c) = make_float4(v[0], v[1], v[2], v[3]);
+    *reinterpret_cast<float4*>(sm + c + 4) = make_float4(v[4], v[5], v[6], v[7]);
+  }
+  for (int i = threadIdx.x; i < half; i += kRopeThreads) {
+    float s, c;
+    sincosf(p * a.inv_freq[i], &s, &c);
+    s_cos[i] = c;
+    s_sin[i] = s;
+  }
+  sq = cta_sum<kRopeThreads>(sq, sums[0]);
+  sk = cta_sum<kRopeThreads>(sk, sums[1]);
+  const float rq = 1.0f / sqrtf(sq / static_cast<float>(a.heads * a.dim_true) + a.eps);
+  const float rk = 1.0f / sqrtf(sk / static_cast<float>(a.kv_heads * a.dim_true) + a.eps);
+  T* kc = static_cast<T*>(a.k_cache) + a.loc[t] * a.ldkc;
+  for (int c = threadIdx.x * 8; c < nq + nk; c += kRopeThreads * 8) {
+    const bool is_q = c < nq;
+    const float* src = is_q ? s_q : s_k;
+    const float* w = is_q ? a.q_weight : a.k_weight;
+    const int b = is_q ? c : c - nq, d0 = b % a.dim;
+    const float rr = is_q ? rq : rk;
+    float v[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      const int d = d0 + e;
+      const float me = src[b + e] * rr * w[b + e];
+      v[e] = me;
+      if (d < a.rot_dims) {
+        const int pair = d < half ? d : d - half, other = d < half ? b + e + half : b + e - half;
+        const float it = src[other] * rr * w[other];
+        v[e] = d < half ? me * s_cos[pair] - it * s_sin[pair] : me * s_cos[pair] + it * s_sin[pair];
+      }
+    }
+    conv_store8<T>(is_q ? q + b : kc + b, v);
+  }
+}
+
 }  // namespace lm
 }  // namespace fr
 
@@ -419,15 +752,18 @@ extern "C" int fr_lm_norm(int dtype, float* x, int64_t ldx, const float* weight,
                                              ldo, M, W, stream);
 }
 
-extern "C" int fr_short_conv(int dtype, const void* u, int64_t ldu, const float* w, int taps, int C, const fr_conv_out* outs,
-                             int n_outs, void* state, const int64_t* state_slots, const int32_t* tok_req,
+extern "C" int fr_short_conv(int dtype, const void* u, int64_t ldu, const float* w, const float* bias, int act, int taps, int C,
+                             const fr_conv_out* outs, int n_outs, void* state, const int64_t* state_slots, const int32_t* tok_req,
                              const int32_t* qo_indptr, const int64_t* pos, int T, int n_req, int one_token,
                              cudaStream_t stream) {
+  FR_CHECK_ARG((act == FR_CONV_LINEAR || act == FR_CONV_SILU));
   FR_CHECK_ARG((dtype == 0 || dtype == 1) && T >= 0 && n_req >= 0 && taps >= 1 && C > 0 && ldu >= C && n_outs > 0 && n_outs <= 4);
   if (T == 0 || n_req == 0) return FR_OK;
   FR_CHECK_ARG(u && w && outs && state && state_slots && tok_req && qo_indptr && pos && (!one_token || T == n_req));
   lm::ConvOuts co{};
   co.n = n_outs;
+  co.bias = bias;
+  co.act = act;
   for (int i = 0; i < n_outs; ++i) {
     FR_CHECK_ARG(outs[i].out && outs[i].c0 >= 0 && outs[i].c > 0 && outs[i].c0 + outs[i].c <= C);
     co.o[i] = outs[i];
@@ -436,4 +772,38 @@ extern "C" int fr_short_conv(int dtype, const void* u, int64_t ldu, const float*
                                                      n_req, one_token, stream)
                     : lm::launch_conv<float>(u, ldu, w, taps, C, co, state, state_slots, tok_req, qo_indptr, pos, T, n_req,
                                              one_token, stream);
+}
+
+extern "C" int fr_lm_update_norm(const fr_norm_update* u, int M, int W, cudaStream_t stream) {
+  FR_CHECK_ARG(u && (u->dtype == 0 || u->dtype == 1) && M >= 0 && W > 0 && u->ldx >= W && u->n_parts >= 0 && u->n_parts <= 2);
+  if (M == 0) return FR_OK;
+  FR_CHECK_ARG(u->x && (u->out == nullptr || u->ldo >= W) && u->n_partials >= 0 && (u->n_partials == 0 || u->partials));
+  for (int p = 0; p < u->n_parts; ++p) FR_CHECK_ARG(u->parts[p].y && u->parts[p].weight && u->parts[p].ldy >= W);
+  return u->dtype == 0 ? lm::launch_update_norm<__nv_bfloat16>(*u, M, W, stream) : lm::launch_update_norm<float>(*u, M, W, stream);
+}
+
+extern "C" int fr_lm_group_norm(const fr_group_norm* a, int M, cudaStream_t stream) {
+  FR_CHECK_ARG(a && (a->dtype == 0 || a->dtype == 1) && M >= 0 && a->groups > 0 && a->size > 0);
+  if (M == 0) return FR_OK;
+  const int64_t n = static_cast<int64_t>(a->groups) * a->size;
+  FR_CHECK_ARG(a->y && a->out && a->weight && a->ldy >= n && a->ldo >= n);
+  FR_CHECK_ARG(a->gate_mode >= FR_GATE_NONE && a->gate_mode <= FR_GATE_AFTER && (a->gate_mode == FR_GATE_NONE || (a->gate && a->ldg >= n)));
+  return a->dtype == 0 ? lm::launch_group_norm<__nv_bfloat16>(*a, M, stream) : lm::launch_group_norm<float>(*a, M, stream);
+}
+
+extern "C" int fr_lm_qk_norm_rope(const fr_qk_rope* a, int M, cudaStream_t stream) {
+  FR_CHECK_ARG(a && (a->dtype == 0 || a->dtype == 1) && M >= 0 && a->heads > 0 && a->kv_heads > 0 && a->dim > 0 && a->dim % 8 == 0);
+  if (M == 0) return FR_OK;
+  FR_CHECK_ARG(a->dim_true > 0 && a->dim_true <= a->dim && a->rot_dims >= 0 && a->rot_dims % 2 == 0 && a->rot_dims <= a->dim_true);
+  FR_CHECK_ARG(a->q && a->k && a->k_cache && a->q_weight && a->k_weight && a->pos && a->loc && (a->rot_dims == 0 || a->inv_freq));
+  FR_CHECK_ARG(aligned16(a->q) && aligned16(a->k) && aligned16(a->k_cache) && a->ldq % 8 == 0 && a->ldk % 8 == 0 && a->ldkc % 8 == 0);
+  const int smem = ((a->heads + a->kv_heads) * a->dim + a->rot_dims) * 4;
+  FR_CHECK_SUPPORTED(smem <= 200 * 1024);
+  static PerDeviceFlag f0, f1;
+  if (a->dtype == 0) {
+    if (ensure_dyn_smem(f0, lm::qk_norm_rope_kernel<__nv_bfloat16>, 200 * 1024) != FR_OK) return FR_ERR_CUDA;
+    return launch_kernel(lm::qk_norm_rope_kernel<__nv_bfloat16>, M, lm::kRopeThreads, smem, stream, M <= kPdlRows, *a);
+  }
+  if (ensure_dyn_smem(f1, lm::qk_norm_rope_kernel<float>, 200 * 1024) != FR_OK) return FR_ERR_CUDA;
+  return launch_kernel(lm::qk_norm_rope_kernel<float>, M, lm::kRopeThreads, smem, stream, M <= kPdlRows, *a);
 }

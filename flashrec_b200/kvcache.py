@@ -1,5 +1,5 @@
 """Cache and state of the 16/32-bit decoder models: paged K/V per layer run, the slot table, the short
-convolutions' state, and the host-side manager that hands pages and rows to requests.
+convolutions' and the recurrences' state, and the host-side manager that hands pages and rows to requests.
 
 A page is 64 consecutive slots and holds positions ``[64 p, 64 p + 64)`` of one request (the tensor-core
 attention loads a page as one tile). The slot table has the layout of ``ReqToTokenPool.req_to_token``
@@ -18,29 +18,44 @@ PAGE = 64
 
 @dataclass(frozen=True)
 class CacheSpec:
-    """What one layer run keeps per sequence: cache columns, convolution state, and which keys stay visible."""
+    """What one layer run keeps per sequence: cache columns, convolution state, a recurrent state matrix per head, and
+    which keys stay visible."""
 
     k_cols: int
     v_cols: int
     conv_channels: int = 0
     conv_taps: int = 1
-    mask: str = "window"  # "window": the last `size` positions and the first `keep_first`; "chunk": the own chunk
+    # "window": the last `size` positions and the first `keep_first`; "chunk": the own chunk; "none": no keys at all
+    mask: str = "window"
     size: int = 0
     keep_first: int = 0
+    state_heads: int = 0  # recurrent state [state_dim, state_vdim] per head, fp32
+    state_dim: int = 0
+    state_vdim: int = 0
+
+    @property
+    def state_floats(self) -> int:
+        """Per sequence; rows and columns are padded as the scan kernels lay them out."""
+        return self.state_heads * ((self.state_dim + 7) // 8 * 8) * ((self.state_vdim + 15) // 16 * 16)
 
     def lowest_key(self, pos: int) -> int:
         """Lowest visible position (besides the kept first ones) of a query at ``pos``."""
+        if self.mask == "none":
+            return pos
         if self.mask == "chunk":
             return pos // self.size * self.size
         return max(0, pos - self.size + 1)
 
     def max_keys(self, pos: int) -> int:
         """Upper bound of the keys that any query at a position <= ``pos`` sees."""
+        if self.mask == "none":
+            return 0
         return min(self.size + (self.keep_first if self.mask == "window" else 0), pos + 1)
 
 
 class LayerCaches:
-    """Device memory of every layer run: ``k[i]``, ``v[i]`` [slots, cols] and ``conv[i]`` [rows, taps - 1, C].
+    """Device memory of every layer run: ``k[i]``, ``v[i]`` [slots, cols], ``conv[i]`` [rows, taps - 1, C] and
+    ``state[i]`` [rows, state floats], fp32 whatever the dtype.
     Zero-initialised: the tensor-core kernel multiplies unused slots of a page by zero weights."""
 
     def __init__(self, specs: Sequence[CacheSpec], n_pages: int, n_rows: int, dtype: torch.dtype, device):
@@ -50,6 +65,7 @@ class LayerCaches:
         self.k = [torch.zeros((self.num_slots, s.k_cols), **kw) for s in specs]
         self.v = [torch.zeros((self.num_slots, s.v_cols), **kw) for s in specs]
         self.conv = [torch.zeros(max(1, n_rows * (s.conv_taps - 1) * s.conv_channels), **kw) for s in specs]
+        self.state = [torch.zeros((n_rows, s.state_floats), dtype=torch.float32, device=device) for s in specs]
 
 
 @dataclass

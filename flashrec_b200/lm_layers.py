@@ -1,6 +1,8 @@
 """Building blocks of the 16/32-bit decoder models, each a thin wrapper around one C-ABI entry point with its
 constants as parameters: merged projections with per-range epilogues, the gated two-part residual update, RMS norm
-of the fp32 residual stream, the short causal convolution, and attention that mixes several softmax maps.
+of the fp32 residual stream (also fused with an update of the stream by normalised vectors), gated norms over groups,
+norm and rotation of queries and keys, the short causal convolution, attention that mixes several softmax maps, and
+recurrences with a matrix state per head.
 
 ``dtype`` (bfloat16 or float32) is the type of weights, activations and caches; the residual stream is fp32 in
 both. bfloat16 runs on the tensor cores, float32 is true 32-bit arithmetic throughout."""
@@ -8,18 +10,22 @@ both. bfloat16 runs on the tensor cores, float32 is true 32-bit arithmetic throu
 from __future__ import annotations
 
 import ctypes
-from dataclasses import dataclass
+import math
+from dataclasses import dataclass, field
 from typing import List, Optional, Sequence, Tuple
 
 import torch
 
 from flashrec_b200 import _lib
-from flashrec_b200._lib import FrConvOut, FrGatedPart, FrMixAttn, FrOutSegment, call, ptr, require_cuda, stream_ptr
+from flashrec_b200._lib import (FrConvOut, FrGatedPart, FrGroupNorm, FrLinearScan, FrMixAttn, FrNormPart, FrNormUpdate,
+                                FrOutSegment, FrQkRope, call, ptr, require_cuda, stream_ptr)
 from flashrec_b200.core import ForwardBatch
 from flashrec_b200.kvcache import CacheSpec
 
 SEG = {"store": _lib.FR_SEG_STORE, "swiglu": _lib.FR_SEG_SWIGLU, "sigmoid": _lib.FR_SEG_SIGMOID,
-       "store_f32": _lib.FR_SEG_STORE_F32}
+       "store_f32": _lib.FR_SEG_STORE_F32, "glu_clamp": _lib.FR_SEG_GLU_CLAMP, "gelu_mul": _lib.FR_SEG_GELU_MUL}
+_PAIRED = ("swiglu", "glu_clamp")  # weight rows in [32 gate | 32 up] blocks
+MIX = {"diff": _lib.FR_MIX_DIFF, "talk": _lib.FR_MIX_TALK, "plain": _lib.FR_MIX_PLAIN}
 _SCORE_SCRATCH_BYTES = 256 << 20
 _MAP_SCRATCH_BYTES = 1 << 30  # maps of talking heads between their kernels: every token tile of a large step at once
 
@@ -68,6 +74,9 @@ class ColumnRange:
     rows: int
     n: int
     bias: Optional[torch.Tensor] = None
+    limit: float = 0.0
+    alpha: float = 0.0
+    up_bias: float = 0.0
 
 
 class MergedProjection:
@@ -81,9 +90,10 @@ class MergedProjection:
         self.weight: Optional[torch.Tensor] = None
 
     def add(self, kind: str, weight: torch.Tensor, n: Optional[int] = None, bias: Optional[torch.Tensor] = None,
-            align: int = 32) -> int:
-        """Append a range; returns its index. ``swiglu`` takes an interleaved weight and must stay 64-aligned."""
-        if kind == "swiglu":
+            align: int = 32, limit: float = 0.0, alpha: float = 0.0, up_bias: float = 0.0) -> int:
+        """Append a range; returns its index. ``swiglu`` and ``glu_clamp`` (with ``limit``, ``alpha``, ``up_bias``) take
+        an interleaved weight and must stay 64-aligned."""
+        if kind in _PAIRED:
             start = sum(r.rows for r in self.ranges)
             if start % 64:  # start the interleaved blocks on a 64-row boundary: widen the range before
                 self._parts[-1] = pad_rows(self._parts[-1], 32)
@@ -96,7 +106,7 @@ class MergedProjection:
             weight = pad_rows(weight, align)
             rows = weight.shape[0]
         self._parts.append(weight)
-        self.ranges.append(ColumnRange(kind, rows, int(n), bias))
+        self.ranges.append(ColumnRange(kind, rows, int(n), bias, float(limit), float(alpha), float(up_bias)))
         return len(self.ranges) - 1
 
     def finish(self, dtype: torch.dtype, device) -> None:
@@ -108,15 +118,19 @@ class MergedProjection:
         self._parts = []
 
     def __call__(self, a: torch.Tensor, outs: Sequence[torch.Tensor],
-                 row_maps: Optional[Sequence[Optional[torch.Tensor]]] = None, algo: int = 0) -> None:
-        """``a`` [M, lda >= K padded]; ``outs`` one 2-D tensor per range (rows are ``row_maps[i][m]`` if given)."""
+                 row_maps: Optional[Sequence[Optional[torch.Tensor]]] = None, algo: int = 0,
+                 mul: Optional[Tuple[torch.Tensor, torch.Tensor]] = None) -> None:
+        """``a`` [M, lda >= K padded]; ``outs`` one 2-D tensor per range (rows are ``row_maps[i][m]`` if given);
+        ``mul`` = (table [rows, n], row of each m) of the ``gelu_mul`` ranges."""
         require_cuda(a)
         segs = (FrOutSegment * len(self.ranges))()
         n0 = 0
         for i, r in enumerate(self.ranges):
             o = outs[i]
             rm = row_maps[i] if row_maps is not None else None
-            segs[i] = FrOutSegment(SEG[r.kind], n0, r.n, 0, ptr(o), o.stride(0), ptr(rm), ptr(r.bias))
+            segs[i] = FrOutSegment(SEG[r.kind], n0, r.n, 0, ptr(o), o.stride(0), ptr(rm), ptr(r.bias), r.limit, r.alpha, r.up_bias)
+            if r.kind == "gelu_mul":
+                segs[i].mul, segs[i].ld_mul, segs[i].mul_map = ptr(mul[0]), mul[0].stride(0), ptr(mul[1])
             n0 += r.rows
         w = self.weight
         call("fr_dense_proj", dtype_code(w.dtype), ptr(a), a.stride(0), ptr(w), w.stride(0), int(a.shape[0]), n0,
@@ -163,6 +177,79 @@ def rms_norm(x: torch.Tensor, weight: torch.Tensor, offset: float, eps: float, o
     return out
 
 
+@dataclass
+class Pending:
+    """What still has to be added to the residual stream: K shares of a product, and vectors that are divided by their
+    root mean square, weighted and scaled, ``(y [M, W], weight [W], coefficient)``."""
+
+    partials: Optional[Partials] = None
+    parts: List[Tuple[torch.Tensor, torch.Tensor, float]] = field(default_factory=list)
+
+    @property
+    def empty(self) -> bool:
+        return self.partials is None and not self.parts
+
+
+def update_norm(x: torch.Tensor, eps: float, out: Optional[torch.Tensor], weight: Optional[torch.Tensor] = None,
+                offset: float = 0.0, pending: Optional[Pending] = None, add: Optional[torch.Tensor] = None,
+                row_idx: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """Adds ``pending`` and the vector ``add`` to the stream, then ``out`` = its norm (its rounded copy without a
+    weight). With ``row_idx`` only those rows are read and the stream itself stays."""
+    require_cuda(x)
+    pending = pending or Pending()
+    dtype = out.dtype if out is not None else (pending.parts[0][0].dtype if pending.parts else torch.float32)
+    u = FrNormUpdate(dtype=dtype_code(dtype), n_parts=len(pending.parts), eps=eps, offset=offset, x=ptr(x), ldx=x.stride(0),
+                     add=ptr(add), row_idx=ptr(row_idx), weight=ptr(weight), out=ptr(out),
+                     ldo=out.stride(0) if out is not None else 0)
+    if pending.partials is not None:
+        u.n_partials, u.partials = pending.partials.n, ptr(pending.partials.buf)
+        u.partial_stride = pending.partials.buf.stride(0)
+    for i, (y, w, coef) in enumerate(pending.parts):
+        u.parts[i] = FrNormPart(ptr(y), y.stride(0), ptr(w), coef, 0)
+    m = int(x.shape[0]) if row_idx is None else int(row_idx.numel())
+    call("fr_lm_update_norm", ctypes.byref(u), m, int(x.shape[1]), stream_ptr(x.device))
+    return out
+
+
+def group_norm(y: torch.Tensor, groups: int, size: int, weight: torch.Tensor, eps: float, out: torch.Tensor,
+               gate: Optional[torch.Tensor] = None, gate_first: bool = False) -> torch.Tensor:
+    """RMS norm over each of ``groups`` runs of ``size`` columns; ``gate``: times its silu, before or after. ``weight``
+    has ``size`` values (every group the same) or one per column."""
+    require_cuda(y)
+    mode = _lib.FR_GATE_NONE if gate is None else (_lib.FR_GATE_BEFORE if gate_first else _lib.FR_GATE_AFTER)
+    a = FrGroupNorm(dtype=dtype_code(y.dtype), gate_mode=mode, groups=groups, size=size,
+                    weight_per_group=0 if weight.numel() == size else 1, eps=eps, y=ptr(y), ldy=y.stride(0), gate=ptr(gate),
+                    ldg=gate.stride(0) if gate is not None else 0, weight=ptr(weight), out=ptr(out), ldo=out.stride(0))
+    call("fr_lm_group_norm", ctypes.byref(a), int(y.shape[0]), stream_ptr(y.device))
+    return out
+
+
+def rotary_frequencies(dims: int, base: float, scaling: Optional[dict] = None) -> torch.Tensor:
+    """Angle per position of each rotated pair (fp32 [dims / 2]). ``scaling`` (factor, low, high, original): pairs whose
+    wavelength exceeds original / low turn ``factor`` times slower, those below original / high as they are, and a
+    linear blend in original / wavelength between."""
+    f = float(base) ** (-torch.arange(0, dims, 2, dtype=torch.float64) / dims)
+    if scaling is not None:
+        turns = float(scaling["original"]) * f / (2 * math.pi)  # within the original length
+        low, high = float(scaling["low"]), float(scaling["high"])
+        slow = f / float(scaling["factor"])
+        s = (turns - low) / (high - low) if high != low else torch.zeros_like(f)
+        f = torch.where(turns > high, f, torch.where(turns < low, slow, (1 - s) * slow + s * f))
+    return f.float()
+
+
+def qk_norm_rope(q: torch.Tensor, k: torch.Tensor, heads: int, kv_heads: int, dim: int, q_weight: torch.Tensor,
+                 k_weight: torch.Tensor, eps: float, inv_freq: torch.Tensor, batch: ForwardBatch, k_cache: torch.Tensor) -> None:
+    """Norms over all heads at once and rotation by ``positions * inv_freq``; ``q`` in place, ``k`` into its cache slots.
+    Heads are padded as the weights are."""
+    require_cuda(q, k, k_cache)
+    a = FrQkRope(dtype=dtype_code(q.dtype), heads=heads, kv_heads=kv_heads, dim=int(q_weight.numel()) // heads, dim_true=dim,
+                 rot_dims=2 * int(inv_freq.numel()), eps=eps, q=ptr(q), ldq=q.stride(0), k=ptr(k), ldk=k.stride(0),
+                 q_weight=ptr(q_weight), k_weight=ptr(k_weight), inv_freq=ptr(inv_freq), pos=ptr(batch.positions),
+                 loc=ptr(batch.out_cache_loc), k_cache=ptr(k_cache), ldkc=k_cache.stride(0))
+    call("fr_lm_qk_norm_rope", ctypes.byref(a), int(q.shape[0]), stream_ptr(q.device))
+
+
 def embed(table: torch.Tensor, width: int, batch: ForwardBatch, scale: float, req_to_token: Optional[torch.Tensor],
           ) -> torch.Tensor:
     """fp32 residual stream ``table[id] * scale``; also enters the batch's new slots into the slot table."""
@@ -175,14 +262,17 @@ def embed(table: torch.Tensor, width: int, batch: ForwardBatch, scale: float, re
     return x
 
 
-def short_conv(u: torch.Tensor, weight: torch.Tensor, outs, state: torch.Tensor, batch: ForwardBatch) -> None:
-    """Causal depthwise convolution of ``u`` [T, C] with ``weight`` [C, taps] fp32; ``outs`` = list of
-    ``(tensor, row_map or None, first channel, channels)``; ``state`` [rows, taps - 1, C] is read and advanced."""
+def short_conv(u: torch.Tensor, weight: torch.Tensor, outs, state: torch.Tensor, batch: ForwardBatch,
+               bias: Optional[torch.Tensor] = None, silu: bool = False) -> None:
+    """Causal depthwise convolution of ``u`` [T, C] with ``weight`` [C, taps] fp32, plus ``bias``, through a silu;
+    ``outs`` = list of ``(tensor, row_map or None, first channel, channels)``; ``state`` [rows, taps - 1, C] is read and
+    advanced."""
     require_cuda(u)
     arr = (FrConvOut * len(outs))()
     for i, (o, rm, c0, c) in enumerate(outs):
         arr[i] = FrConvOut(ptr(o), o.stride(0), ptr(rm), c0, c)
-    call("fr_short_conv", dtype_code(u.dtype), ptr(u), u.stride(0), ptr(weight), int(weight.shape[1]),
+    call("fr_short_conv", dtype_code(u.dtype), ptr(u), u.stride(0), ptr(weight), ptr(bias),
+         _lib.FR_CONV_SILU if silu else _lib.FR_CONV_LINEAR, int(weight.shape[1]),
          int(weight.shape[0]), arr, len(outs), ptr(state), ptr(batch.req_pool_indices), ptr(batch.tok_req),
          ptr(batch.qo_indptr), ptr(batch.positions), int(u.shape[0]), int(batch.req_pool_indices.numel()),
          1 if batch.one_token else 0, stream_ptr(u.device))
@@ -196,7 +286,8 @@ def alibi_slopes(heads: int) -> List[float]:
 class MixAttention:
     """Attention whose outputs are linear combinations of several softmax maps over the same values
     (``fr_mix_attn`` in the header). ``mix``: "diff" (two maps per head, second one subtracted ``lam`` times, output
-    divided by its root mean square, times ``out_scale``) or "talk" (all heads' maps through the matrix ``coef``).
+    divided by its root mean square, times ``out_scale``), "talk" (all heads' maps through the matrix ``coef``) or "plain"
+    (ordinary attention; ``forward`` may get a gate per head).
     ``dim`` / ``vdim`` are the model's sizes; caches and buffers use ``dim_p`` / ``vdim_p`` (multiples of 16)."""
 
     def __init__(self, mix: str, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, cache: CacheSpec, *,
@@ -210,7 +301,7 @@ class MixAttention:
         self.cache = cache
         self.coef, self.slopes = coef, slopes
         big = (1 << 31) - 1
-        self._args = FrMixAttn(mix=_lib.FR_MIX_DIFF if mix == "diff" else _lib.FR_MIX_TALK,
+        self._args = FrMixAttn(mix=MIX[mix],
                                mask=_lib.FR_MASK_CHUNK if cache.mask == "chunk" else _lib.FR_MASK_WINDOW,
                                mask_size=min(cache.size, big), keep_first=min(cache.keep_first, big), heads=self.heads,
                                kv_heads=self.kv_heads, dim=self.dim_p, vdim=self.vdim_p, vdim_true=int(vdim),
@@ -232,8 +323,9 @@ class MixAttention:
                                                                 self.vdim_p))
 
     def forward(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, req_to_token: torch.Tensor,
-                batch: ForwardBatch, counters: torch.Tensor, max_keys: Optional[int] = None) -> torch.Tensor:
-        """q [T, q_cols]; ``k`` / ``v`` the layer's caches (the batch's own keys are in already). bf16 prompts take
+                batch: ForwardBatch, counters: torch.Tensor, max_keys: Optional[int] = None,
+                head_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """q [T, q_cols]; ``head_gate`` fp32 [T, heads], whose sigmoid multiplies the heads ("plain"); ``k`` / ``v`` the layer's caches (the batch's own keys are in already). bf16 prompts take
         the tensor-core kernel, short portions, decode steps and fp32 the row kernels."""
         require_cuda(q, k, v)
         t = int(q.shape[0])
@@ -245,6 +337,8 @@ class MixAttention:
         a.req_to_token, a.table_stride = ptr(req_to_token), req_to_token.stride(0)
         a.req_rows, a.tok_req, a.pos = ptr(batch.req_pool_indices), ptr(batch.tok_req), ptr(batch.positions)
         a.num_slots = int(k.shape[0])
+        if head_gate is not None:
+            a.head_gate, a.ld_gate = ptr(head_gate), head_gate.stride(0)
         s = stream_ptr(q.device)
         tc = self.tensor_cores and a.dtype == 0
         n_row = batch.n_row_tokens if tc else t
@@ -270,3 +364,37 @@ class MixAttention:
         for r0 in range(0, n_row, step):
             call("fr_mix_attn_rows", ctypes.byref(a), r0, min(step, n_row - r0), keys, splits, ptr(scratch),
                  int(scratch.numel()), ptr(counters), stream)
+
+
+class LinearScan:
+    """Recurrence ``S <- diag(a_t) S + k_t u_t^T``, ``o_t = S^T (scale q_t) + skip v_t`` per head, fp32 state and decays
+    (``fr_linear_scan`` in the header). ``decay`` "channel": ``a_t = sigmoid(up . step_t + step_bias) ^ (1 / tau)`` per row
+    of S, u = v; "head": step size ``d_t = softplus(step_t + step_bias)``, ``a_t = exp(-rate d_t)``, ``u = d_t v``."""
+
+    def __init__(self, decay: str, heads: int, key_heads: int, dim: int, vdim: int, step_bias: torch.Tensor, *,
+                 scale: float = 1.0, tau: float = 1.0, rate: Optional[torch.Tensor] = None, up: Optional[torch.Tensor] = None,
+                 skip: Optional[torch.Tensor] = None, device=None):
+        if heads % key_heads:
+            raise ValueError("heads must be a multiple of key_heads")
+        f32 = lambda t: None if t is None else t.to(device=device, dtype=torch.float32).contiguous()
+        self.heads, self.vdim = int(heads), int(vdim)
+        self.step_bias, self.rate, self.up, self.skip = f32(step_bias), f32(rate), f32(up), f32(skip)
+        self._args = FrLinearScan(decay=_lib.FR_DECAY_CHANNEL if decay == "channel" else _lib.FR_DECAY_HEAD, heads=heads,
+                                  key_heads=key_heads, dim=dim, vdim=vdim, rank=0 if up is None else int(up.shape[1]),
+                                  scale=scale, inv_tau=1.0 / tau, step_bias=ptr(self.step_bias), rate=ptr(self.rate),
+                                  up=ptr(self.up), skip=ptr(self.skip))
+
+    def forward(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, step: torch.Tensor, state: torch.Tensor,
+                batch: ForwardBatch, out: torch.Tensor) -> torch.Tensor:
+        """q, k [T, key_heads * dim], v and out [T, heads * vdim], step fp32; ``state`` [rows, state floats]."""
+        require_cuda(q, k, v, step, state)
+        a = FrLinearScan.from_buffer_copy(self._args)
+        a.dtype = dtype_code(q.dtype)
+        a.q, a.ldq, a.k, a.ldk, a.v, a.ldv = ptr(q), q.stride(0), ptr(k), k.stride(0), ptr(v), v.stride(0)
+        a.out, a.ldo, a.step, a.ldstep = ptr(out), out.stride(0), ptr(step), step.stride(0)
+        a.state, a.state_slots = ptr(state), ptr(batch.req_pool_indices)
+        a.qo_indptr, a.pos = ptr(batch.qo_indptr), ptr(batch.positions)
+        longest = 1 if batch.one_token else max(batch.extend_seq_lens)
+        call("fr_linear_scan_rows", ctypes.byref(a), int(batch.req_pool_indices.numel()), longest, int(q.shape[0]),
+             stream_ptr(q.device))
+        return out

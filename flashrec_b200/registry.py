@@ -39,10 +39,19 @@ def _load_dibepel(path: str, cfg: dict, dtype: torch.dtype, device):
     return DibepelForCausalLM(DibepelConfig.from_json(cfg), read_tensors(path), dtype, device)
 
 
+def _load_kotipel(path: str, cfg: dict, dtype: torch.dtype, device):
+    from flashrec_b200.kotipel import KotipelConfig, KotipelForCausalLM
+    from flashrec_b200.weights import read_tensors
+
+    return KotipelForCausalLM(KotipelConfig.from_json(cfg), read_tensors(path), dtype, device)
+
+
 FAMILIES: List[ModelFamily] = [
     ModelFamily("qwen3-fp8", _is_qwen3, _load_qwen3, (torch.bfloat16,)),
     ModelFamily("dibepel", lambda c: c.get("architecture") == "Dibepel", _load_dibepel, (torch.bfloat16, torch.float32),
                 ("capi", "dense_proj", "lm_rows", "attn_mix", "attn_talk")),
+    ModelFamily("kotipel", lambda c: c.get("architecture") == "Kotipel", _load_kotipel, (torch.bfloat16, torch.float32),
+                ("capi", "dense_proj", "lm_rows", "attn_mix", "attn_talk", "linear_scan")),
 ]
 
 

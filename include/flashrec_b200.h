@@ -522,17 +522,25 @@ enum fr_segment_kind {
   FR_SEG_STORE = 0,   /* out[row, c] = z */
   FR_SEG_SWIGLU = 1,  /* weight rows come in blocks of 64 = [32 gate | 32 up]; out[row, c] = silu(gate_c) * up_c */
   FR_SEG_SIGMOID = 2, /* out[row, c] = sigmoid(z + bias[c]) */
-  FR_SEG_STORE_F32 = 3 /* out[row, c] = z, f32 whatever the dtype */
+  FR_SEG_STORE_F32 = 3, /* out[row, c] = z, f32 whatever the dtype */
+  FR_SEG_GLU_CLAMP = 4, /* rows as for SWIGLU; g = min(gate_c, limit), u = clamp(up_c, -limit, limit);
+                           out[row, c] = g * sigmoid(alpha * g) * (u + up_bias) */
+  FR_SEG_GELU_MUL = 5   /* out[row, c] = gelu_tanh(z) * mul[mul_map[row], c] */
 };
 struct fr_out_segment {
   int32_t kind;
-  int32_t n0;            /* first weight row of the range (a multiple of 32; of 64 for SWIGLU) */
-  int32_t n;             /* output columns written (SWIGLU: activation channels, half the weight rows) */
+  int32_t n0;            /* first weight row of the range (a multiple of 32; of 64 for SWIGLU and GLU_CLAMP) */
+  int32_t n;             /* output columns written (SWIGLU, GLU_CLAMP: activation channels, half the weight rows) */
   int32_t pad_;
   void* out;
   int64_t ldo;
   const int64_t* row_map; /* output row per input row (KV-cache slots), or null */
   const float* bias;      /* SIGMOID: [n], or null */
+  float limit, alpha, up_bias; /* GLU_CLAMP */
+  int32_t pad2_;
+  const void* mul;        /* GELU_MUL: [rows, n] in the product's dtype, pitch ld_mul */
+  int64_t ld_mul;
+  const int64_t* mul_map; /* GELU_MUL: row of mul per input row, or null */
 };
 
 /* z = a . w^T for one merged weight matrix, each column range leaving through its segment. a [M, K], w [N, K].
@@ -572,6 +580,73 @@ int fr_lm_norm(int dtype, float* x, int64_t ldx, const float* weight, float offs
                int n_partials, int64_t partial_stride, const int64_t* row_idx, void* out, int64_t ldo, int M, int W,
                cudaStream_t stream);
 
+/* Update of the residual stream by normalised vectors, fused with the norm that follows:
+ *     x += sum of the partials;  x += coef_p * y_p / sqrt(mean(y_p^2) + eps) * weight_p per part;  x += add (a vector);
+ *     out = x / sqrt(mean(x^2) + eps) * (offset + weight), or x itself (rounded to dtype) without a weight.
+ * x is written back unless row_idx picks rows. out may be null. Columns [W, ldo) of out are zeroed up to a multiple
+ * of 8. */
+struct fr_norm_part {
+  const void* y;       /* [M, W] in dtype, pitch ldy */
+  int64_t ldy;
+  const float* weight; /* [W] */
+  float coef;
+  int32_t pad_;
+};
+struct fr_norm_update {
+  int32_t dtype, n_parts, n_partials;
+  float eps, offset;
+  int32_t pad_;
+  float* x;
+  int64_t ldx;
+  const float* partials; /* [n_partials, M, W] */
+  int64_t partial_stride;
+  struct fr_norm_part parts[2];
+  const float* add;      /* [W] or null */
+  const int64_t* row_idx;
+  const float* weight;
+  void* out;
+  int64_t ldo;
+};
+int fr_lm_update_norm(const struct fr_norm_update* u, int M, int W, cudaStream_t stream);
+
+/* out = u / sqrt(mean(u^2) + eps) * weight over each of `groups` runs of `size` columns, with u = y * silu(gate)
+ * (FR_GATE_BEFORE) or the result times silu(gate) (FR_GATE_AFTER). weight [size], shared by the groups, or
+ * [groups * size]. */
+enum fr_gate_mode { FR_GATE_NONE = 0, FR_GATE_BEFORE = 1, FR_GATE_AFTER = 2 };
+struct fr_group_norm {
+  int32_t dtype, gate_mode, groups, size, weight_per_group;
+  float eps;
+  const void* y;
+  int64_t ldy;
+  const void* gate;
+  int64_t ldg;
+  const float* weight;
+  void* out;
+  int64_t ldo;
+};
+int fr_lm_group_norm(const struct fr_group_norm* a, int M, cudaStream_t stream);
+
+/* Norm of a token's queries (all heads at once) and keys, then rotation of the first rot_dims dimensions of every head
+ * by pos * inv_freq (dimension i with i + rot_dims / 2). q [M, heads * dim] in place; k [M, kv_heads * dim] leaves
+ * into row loc[m] of k_cache. Heads are laid out with `dim` columns of which dim_true count (the rest are zero). */
+struct fr_qk_rope {
+  int32_t dtype, heads, kv_heads, dim, dim_true, rot_dims;
+  float eps;
+  int32_t pad_;
+  void* q;
+  int64_t ldq;
+  const void* k;
+  int64_t ldk;
+  const float* q_weight; /* [heads * dim] */
+  const float* k_weight;
+  const float* inv_freq; /* [rot_dims / 2] */
+  const int64_t* pos;
+  const int64_t* loc;
+  void* k_cache;
+  int64_t ldkc;
+};
+int fr_lm_qk_norm_rope(const struct fr_qk_rope* a, int M, cudaStream_t stream);
+
 /* One channel range of fr_short_conv's output. */
 struct fr_conv_out {
   void* out;
@@ -580,11 +655,12 @@ struct fr_conv_out {
   int32_t c0, c;          /* channels [c0, c0 + c) */
 };
 
-/* Depthwise causal convolution over time of a ragged batch: y_t = sum_j w[:, j] * u_(t - taps + 1 + j), zeros
- * before position 0; values before the batch's tokens come from state [slots, taps - 1, C] (oldest first).
+/* Depthwise causal convolution over time of a ragged batch: y_t = act(bias + sum_j w[:, j] * u_(t - taps + 1 + j)),
+ * bias [C] f32 or null, zeros before position 0; values before the batch's tokens come from state [slots, taps - 1, C] (oldest first).
  * u [T, C], w [C, taps] f32, tok_req [T] = index of the token's request in qo_indptr / state_slots. The state of
  * every request is advanced past its tokens. one_token: every request has exactly one token. */
-int fr_short_conv(int dtype, const void* u, int64_t ldu, const float* w, int taps, int C, const struct fr_conv_out* outs,
+enum fr_conv_act { FR_CONV_LINEAR = 0, FR_CONV_SILU = 1 };
+int fr_short_conv(int dtype, const void* u, int64_t ldu, const float* w, const float* bias, int act, int taps, int C, const struct fr_conv_out* outs,
                   int n_outs, void* state, const int64_t* state_slots, const int32_t* tok_req, const int32_t* qo_indptr,
                   const int64_t* pos, int T, int n_req, int one_token, cudaStream_t stream);
 
@@ -592,8 +668,9 @@ int fr_short_conv(int dtype, const void* u, int64_t ldu, const float* w, int tap
  *     out_o(i) = sum_s coef[o, s] * sum_j softmax_j(scale * q_s(i) . k_s(j) - slope_s * (i - j)) v(j).
  * FR_MIX_DIFF: output head h mixes its two maps with (1, -lambda) and is divided by its root mean square over
  * vdim (eps inside the root), times out_scale. FR_MIX_TALK: output head h mixes all H heads' maps with row h of
- * the matrix coef [H, H]. */
-enum fr_mix_kind { FR_MIX_DIFF = 0, FR_MIX_TALK = 1 };
+ * the matrix coef [H, H]. FR_MIX_PLAIN: output head h takes its own map. With head_gate every output head is
+ * multiplied by sigmoid(head_gate[t, h]) (PLAIN only). */
+enum fr_mix_kind { FR_MIX_DIFF = 0, FR_MIX_TALK = 1, FR_MIX_PLAIN = 2 };
 enum fr_mask_kind {
   FR_MASK_WINDOW = 0, /* j <= i and (i - j < size or j < keep_first) */
   FR_MASK_CHUNK = 1   /* j <= i and i / size == j / size */
@@ -618,6 +695,8 @@ struct fr_mix_attn {
   const int32_t* tok_req;  /* [T] */
   const int64_t* pos;      /* [T] */
   int64_t num_slots;
+  const float* head_gate;  /* PLAIN: [T, heads], pitch ld_gate, or null */
+  int64_t ld_gate;
 };
 
 /* Any head sizes, bf16 or f32, prompts or decode: scores of every visible key, then the mixture over the values.
@@ -637,6 +716,41 @@ int fr_mix_attn_tc(const struct fr_mix_attn* a, const int32_t* tiles, int n_tile
                    int64_t scratch_bytes, cudaStream_t stream);
 int64_t fr_mix_attn_tc_scratch(const struct fr_mix_attn* a, int n_tiles, int max_pos, int64_t budget);
 int fr_mix_attn_tc_fits(int mix, int heads, int kv_heads, int dim, int vdim);
+
+/* Recurrences with a matrix state [dim, vdim] per head, fp32 throughout:
+ *     S_t = diag(a_t) S_(t-1) + k_t u_t^T,   o_t = S_t^T (scale * q_t) + skip * v_t.
+ * FR_DECAY_CHANNEL: a_t = sigmoid(up . step_t + step_bias)^inv_tau per key channel, u = v, key_heads == heads.
+ * FR_DECAY_HEAD: d_t = softplus(step_t + step_bias) per head, a_t = exp(-rate * d_t), u = d_t * v. Query / key head of
+ * head h: h / (heads / key_heads).
+ * The state of a request is row state_slots[b] of `state` ([rows, heads, fr_linear_state_floats(dim, vdim)], f32); it
+ * is zero at position 0 whatever the row holds, and is advanced past the request's tokens. */
+enum fr_decay_kind { FR_DECAY_CHANNEL = 0, FR_DECAY_HEAD = 1 };
+struct fr_linear_scan {
+  int32_t dtype, decay, heads, key_heads, dim, vdim, rank;
+  float scale, inv_tau;
+  int32_t pad_;
+  const void* q; /* [T, key_heads * dim] */
+  int64_t ldq;
+  const void* k;
+  int64_t ldk;
+  const void* v; /* [T, heads * vdim] */
+  int64_t ldv;
+  void* out;     /* [T, heads * vdim] */
+  int64_t ldo;
+  const float* step;      /* HEAD: [T, heads]; CHANNEL: [T, rank] */
+  int64_t ldstep;
+  const float* step_bias; /* HEAD: [heads]; CHANNEL: [heads * dim] */
+  const float* rate;      /* HEAD: [heads] */
+  const float* up;        /* CHANNEL: [heads * dim, rank] */
+  const float* skip;      /* [heads] or null */
+  float* state;
+  const int64_t* state_slots; /* [n_req] */
+  const int32_t* qo_indptr;   /* [n_req + 1] */
+  const int64_t* pos;         /* [T] */
+};
+int64_t fr_linear_state_floats(int dim, int vdim);
+/* Any sizes, token after token. max_tokens: the most tokens of one request; n_tokens: of the batch. */
+int fr_linear_scan_rows(const struct fr_linear_scan* a, int n_req, int max_tokens, int n_tokens, cudaStream_t stream);
 
 #ifdef __cplusplus
 }
