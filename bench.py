@@ -51,12 +51,13 @@ def parse():
     ap.add_argument("--steps", type=int, default=5)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
-    ap.add_argument("--workload", default="config4", choices=["config4", "config5", "dibepel"],
+    ap.add_argument("--workload", default="config4", choices=["config4", "config5", "dibepel", "kotipel"],
                     help="config4 (default): 32 requests x 512 beams, 3 x 8192 codes, 1M items, prompts 128-1024. "
                          "config5: the widest configuration as one replica per GPU: 2048 beams, 4 x 4096 codes, 10M "
                          "Zipf items, prompts 1024-4096 (give --requests; 64 requests over the GPUs of a box is the "
                          "stated concurrency). dibepel: prefill and decode "
-                         "throughput of the 16-bit Dibepel decoder beside the FP8 Qwen3 at equal sizes (bench_lm.py)")
+                         "throughput of the 16-bit Dibepel decoder beside the FP8 Qwen3 at equal sizes (bench_lm.py). "
+                         "kotipel: the same of the 16-bit Kotipel decoder beside Dibepel")
     ap.add_argument("--requests", type=int, default=32)
     ap.add_argument("--beam", type=int, default=512)
     ap.add_argument("--layers", type=int, default=28)
@@ -1117,6 +1118,11 @@ def main():
         import bench_lm
 
         bench_lm.run(args)
+        return
+    if args.workload == "kotipel":
+        import bench_lm
+
+        bench_lm.run_kotipel(args)
         return
     if args.attn_compare:
         import torch

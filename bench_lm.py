@@ -1,8 +1,9 @@
-"""``bench.py --workload dibepel``: prefill and decode throughput of the Dibepel decoder at sizes of real models (random
-weights), beside the FP8 Qwen3 model at equal size through the same engine, and the time of every kernel of a layer.
+"""``bench.py --workload dibepel | kotipel``: prefill and decode throughput of a 16-bit decoder at sizes of real models
+(random weights), beside the closest other model at equal size through the same engine (Dibepel beside the FP8 Qwen3,
+Kotipel beside Dibepel), and the time of every kernel of a layer.
 
-One JSON line: ``sizes[name]["dibepel" | "qwen3"]`` with ``prefill`` (tokens/s by tokens per step), ``decode`` (tokens/s by
-batch) and, for Dibepel, ``kernels`` (microseconds, achieved rate and fraction of the measured peak per kernel)."""
+One JSON line: ``sizes[name][model]`` with ``prefill`` (tokens/s by tokens per step), ``decode`` (tokens/s by batch) and
+``kernels`` (microseconds, achieved rate and fraction of the measured peak per kernel)."""
 
 from __future__ import annotations
 
@@ -28,9 +29,27 @@ def dibepel_config(width, heads, kv_heads, ff, layers):
                 layers=entries)
 
 
-def event_time(torch, fn, iters: int, warmup: int = 3, rest: float = 0.0) -> float:
-    """Median milliseconds of ``fn(i)``; the caller's working set exceeds L2 or rotates through buffers. ``rest``: seconds of
-    idling first, for single kernels that are set against the burst peak (the clocks recover from the power cap)."""
+# per width: heads of the gated linear attention (64 x 128) and of the state-space recurrence (64 wide, state 128)
+RECURRENT = {2048: (16, 64), 4096: (32, 128)}
+SIDE = 256
+
+
+def kotipel_config(width, heads, kv_heads, ff, layers):
+    gla, ssm = RECURRENT[width]
+    mlp = dict(kind="dense", ff=ff, limit=7.0)
+    mamba = dict(type="mamba2", mlp=mlp, mixer=dict(heads=ssm, vdim=64, state=128, groups=8, conv=4, norm_groups=1))
+    rot = dict(dims=128, base=5e5, scaling=dict(factor=8.0, low=1.0, high=4.0, original=8192))
+    par = dict(type="parallel", mlp=mlp, mixer=dict(
+        left=dict(heads=heads, kv_heads=kv_heads, dim=128, vdim=128, rot=rot, scale=128 ** -0.5),
+        right=dict(heads=gla, dim=64, vdim=128, tau=16.0)))
+    return dict(architecture="Kotipel", vocab=VOCAB, width=width, norm=dict(eps=1e-5), token_side=dict(dim=SIDE),
+                layers=[mamba if i % 2 == 0 else par for i in range(layers)])
+
+
+def event_time(torch, fn, iters: int, warmup: int = 3, rest: float = 0.0, flush=None) -> float:
+    """Median milliseconds of ``fn(i)``; the caller's working set exceeds L2 or rotates through buffers, or ``flush`` (a
+    buffer larger than L2) is written before every call. ``rest``: seconds of idling first, for single kernels that are set
+    against the burst peak (the clocks recover from the power cap)."""
     if rest > 0:
         torch.cuda.synchronize()
         time.sleep(rest)
@@ -39,6 +58,8 @@ def event_time(torch, fn, iters: int, warmup: int = 3, rest: float = 0.0) -> flo
     torch.cuda.synchronize()
     ev = [(torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)) for _ in range(iters)]
     for i, (a, b) in enumerate(ev):
+        if flush is not None:
+            flush.zero_()
         a.record()
         fn(i)
         b.record()
@@ -187,6 +208,141 @@ def qwen3_kernel_times(torch, lm, n_tok, peaks, iters=10):
     return res
 
 
+def kotipel_kernel_times(torch, model, n_tok, peaks, iters=10):
+    """Every kernel of a state-space and of a parallel layer alone, one prompt of ``n_tok`` tokens: the launches of one
+    forward are recorded and each is repeated on the buffers it ran on."""
+    from flashrec_b200 import lm_layers
+    from flashrec_b200.engine import LMEngine, StepEntry
+
+    cfg, w = model.cfg, model.cfg.width
+    eng = LMEngine(model, n_tok, 1, n_tok)
+    mamba, par = cfg.layers[0].mixer, cfg.layers[1].mixer
+    ff, d = cfg.layers[0].ff, cfg.side_dim
+    a, g = par.left, par.right
+    gemm = lambda n, k: ("flops", 2 * n_tok * n * k)
+    move = lambda cols: ("bytes", 2 * n_tok * cols)  # 16-bit columns in and out; the stream counts double
+    keys = n_tok * (n_tok + 1) // 2
+    mc, gk, gv = mamba.channels, g.heads * g.dim, g.heads * g.vdim
+    tail = [("norm2", move(7 * w)), ("gate_up", gemm(2 * ff, w)), ("down", gemm(w, ff)), ("copy", move(3 * w)),
+            ("side.gate", gemm(d, w)), ("side.proj", gemm(w, d))]
+    names = [("mamba.norm1", move(3 * w)), ("mamba.projections", gemm(mamba.inner + mc + mamba.heads, w)), ("mamba.conv", move(2 * mc)),
+             ("mamba.recurrence", move(mc + mamba.inner + 2 * mamba.heads)), ("mamba.norm", move(3 * mamba.inner)),
+             ("mamba.out", gemm(w, mamba.inner))]
+    names += [("mamba." + n, c) for n, c in tail]
+    names[6] = ("mamba.norm2", move(3 * w))
+    n_par = a.heads * a.dim + a.kv_heads * (a.dim + a.vdim) + 2 * gk + 2 * gv + a.heads + model.layers[1].mixer.rank
+    names += [("parallel.norm1", move(6 * w)), ("parallel.projections", gemm(n_par, w)),
+              ("parallel.qk_rope", move(2 * (a.heads + a.kv_heads) * a.dim)),
+              ("parallel.attention", ("flops", 2 * keys * a.heads * (a.dim + a.vdim))), ("parallel.left_out", gemm(w, a.heads * a.vdim)),
+              ("parallel.recurrence", move(2 * gk + 2 * gv)), ("parallel.head_norm", move(3 * gv)), ("parallel.right_out", gemm(w, gv))]
+    names += [("parallel." + n, c) for n, c in tail]
+    launches, keep = [], []
+    orig, empty = lm_layers.call, torch.empty
+
+    def record(name, *args):
+        if name != "fr_lm_embed":
+            launches.append((name, args))
+        orig(name, *args)
+
+    def kept(*args, **kw):
+        keep.append(empty(*args, **kw))
+        return keep[-1]
+
+    lm_layers.call, torch.empty = record, kept
+    try:
+        eng.step([StepEntry(0, [t % model.vocab for t in range(n_tok)])])
+    finally:
+        lm_layers.call, torch.empty = orig, empty
+    torch.cuda.synchronize()
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=model.device)
+    fused = {"parallel.recurrence": ("fr_linear_decay",)}
+    res, i = {}, 0
+    for name, (what, amount) in names:
+        group = [launches[i]]
+        i += 1
+        while group[-1][0] in fused.get(name, ()):
+            group.append(launches[i])
+            i += 1
+        ms = event_time(torch, lambda _: [orig(n, *args) for n, args in group], iters, rest=0.4, flush=flush)
+        r = {"us": round(ms * 1e3, 1), "launch": group[-1][0]}
+        if what == "flops":
+            r.update(tflops=round(amount / ms / 1e9, 1), frac_of_measured=round(amount / ms / 1e9 / peaks["bf16_tflops"], 3))
+        else:
+            r.update(gbs=round(amount / ms / 1e6), frac_of_measured=round(amount / ms / 1e6 / peaks["hbm_gbs"], 3))
+        res[name] = r
+    del keep
+    return res
+
+
+def _peaks():
+    if (ROOT / "MEASURED_PEAKS.json").exists():
+        p = json.loads((ROOT / "MEASURED_PEAKS.json").read_text())
+        return {"bf16_tflops": p["bf16_tflops"], "hbm_gbs": p["hbm_gbs"], "source": "MEASURED_PEAKS.json"}
+    return {"bf16_tflops": 1590.0, "hbm_gbs": 6650.0, "source": "fallback"}
+
+
+def _weight_bytes(tree) -> int:
+    """Bytes of the matrices that one pass over the layers reads (norms and tables of the token input aside)."""
+    from flashrec_b200.lm_layers import MergedProjection
+
+    n = 0
+    for v in vars(tree).values():
+        if isinstance(v, MergedProjection):
+            n += v.weight.numel() * v.weight.element_size()
+        elif hasattr(v, "numel") and getattr(v, "dim", lambda: 0)() == 2 and v.element_size() == 2 and v.is_contiguous():
+            n += v.numel() * 2
+        elif type(v).__module__.startswith("flashrec_b200.kotipel") and type(v).__name__.endswith("Mixer"):
+            n += _weight_bytes(v)
+    return n
+
+
+def run_kotipel(args) -> None:
+    import torch
+
+    from bench import ClockSampler
+    from flashrec_b200 import device_status
+    from flashrec_b200.dibepel import DibepelConfig, DibepelForCausalLM
+    from flashrec_b200.dibepel import random_tensors as dibepel_tensors
+    from flashrec_b200.engine import LMEngine
+    from flashrec_b200.kotipel import KotipelConfig, KotipelForCausalLM, random_tensors
+
+    peaks, dev = _peaks(), torch.device("cuda:0")
+    torch.cuda.set_device(dev)
+    prefill, decode, iters = [(1, 8192), (8, 1024)], [1, 4, 16, 64, 256], max(args.steps, 10)
+    line = {"metric": "kotipel_prefill_decode_tokens_per_s", "unit": "tokens/s", "n_gpus": 1, "data": "synthetic", "dtype": "bf16",
+            "higher_is_better": True, "peaks": peaks, "sizes": {},
+            "config": {"token_side": SIDE, "recurrent_heads": RECURRENT, "vocab": VOCAB, "context": 1024,
+                       "l2": "weights and activations of a step exceed L2"}}
+    with ClockSampler(0) as clk:
+        for name, (width, heads, kv, ff, layers) in SIZES.items():
+            cfg = KotipelConfig.from_json(kotipel_config(width, heads, kv, ff, layers))
+            model = KotipelForCausalLM(cfg, random_tensors(cfg, device=dev), torch.bfloat16, dev)
+            make = lambda tokens, reqs, seq: LMEngine(model, tokens, reqs, seq)
+            rec = {"layers": layers, "width": width, "heads": heads, "kv_heads": kv, "ff": ff,
+                   "kotipel": throughput(torch, make, cfg.vocab, prefill, decode, 1024, iters)}
+            rec["kotipel"]["kernels_8192"] = kotipel_kernel_times(torch, model, 8192, peaks)
+            w = sum(_weight_bytes(l) for l in model.layers) + model.head.weight.numel() * 2
+            for b, r in rec["kotipel"]["decode"].items():
+                r["weight_stream_frac_of_measured"] = round(w / r["graph_ms"] / 1e6 / peaks["hbm_gbs"], 3)
+            del model
+            torch.cuda.empty_cache()
+            dcfg = DibepelConfig.from_json(dibepel_config(width, heads, kv, ff, layers))
+            dib = DibepelForCausalLM(dcfg, dibepel_tensors(dcfg, device=dev), torch.bfloat16, dev)
+            make = lambda tokens, reqs, seq: LMEngine(dib, tokens, reqs, seq)
+            rec["dibepel"] = throughput(torch, make, dcfg.vocab, prefill, decode, 1024, iters)
+            rec["dibepel"]["kernels_8192"] = kernel_times(torch, dib, 8192, peaks)
+            w = sum(t.numel() for l in dib.layers for t in (l.proj.weight, l.o_w, l.down_w)) * 2 + dib.head.weight.numel() * 2
+            for b, r in rec["dibepel"]["decode"].items():
+                r["weight_stream_frac_of_measured"] = round(w / r["graph_ms"] / 1e6 / peaks["hbm_gbs"], 3)
+            del dib
+            torch.cuda.empty_cache()
+            line["sizes"][name] = rec
+    line["clocks"] = clk.summary()
+    line["value"] = line["sizes"]["1.7b"]["kotipel"]["prefill"]["1x8192"]["tokens_per_s"]
+    line["device_status"] = list(device_status())
+    print(json.dumps(line), flush=True)
+
+
 def run(args) -> None:
     import torch
 
@@ -197,10 +353,7 @@ def run(args) -> None:
     from flashrec_b200.engine import LMEngine
     from flashrec_b200.qwen3_lm import random_qwen3_lm
 
-    peaks = {"bf16_tflops": 1590.0, "hbm_gbs": 6650.0, "source": "fallback"}
-    if (ROOT / "MEASURED_PEAKS.json").exists():
-        p = json.loads((ROOT / "MEASURED_PEAKS.json").read_text())
-        peaks = {"bf16_tflops": p["bf16_tflops"], "hbm_gbs": p["hbm_gbs"], "source": "MEASURED_PEAKS.json"}
+    peaks = _peaks()
     dev = torch.device("cuda:0")
     torch.cuda.set_device(dev)
     prefill = [(1, 8192), (8, 1024)]

@@ -687,10 +687,14 @@ qk_norm_rope_kernel(const __grid_constant__ fr_qk_rope a) {
     *reinterpret_cast<float4*>(sm + c + 4) = make_float4(v[4], v[5], v[6], v[7]);
   }
   for (int i = threadIdx.x; i < half; i += kRopeThreads) {
+    // the angle as a sum of two floats: its rounding alone would show at far positions
+    const float2 f = reinterpret_cast<const float2*>(a.inv_freq)[i];
+    const float hi = p * f.x, lo = fmaf(p, f.y, fmaf(p, f.x, -hi));
     float s, c;
-    sincosf(p * a.inv_freq[i], &s, &c);
-    s_cos[i] = c;
-    s_sin[i] = s;
+    sincosf(hi, &s, &c);
+    const float c1 = 1.0f - 0.5f * lo * lo, s1 = lo - lo * lo * lo * (1.0f / 6.0f);  // lo is at most half a place of hi
+    s_cos[i] = c * c1 - s * s1;
+    s_sin[i] = s * c1 + c * s1;
   }
   sq = cta_sum<kRopeThreads>(sq, sums[0]);
   sk = cta_sum<kRopeThreads>(sk, sums[1]);

@@ -225,7 +225,7 @@ def group_norm(y: torch.Tensor, groups: int, size: int, weight: torch.Tensor, ep
 
 
 def rotary_frequencies(dims: int, base: float, scaling: Optional[dict] = None) -> torch.Tensor:
-    """Angle per position of each rotated pair (fp32 [dims / 2]). ``scaling`` (factor, low, high, original): pairs whose
+    """Angle per position of each rotated pair, as a sum of two floats (fp32 [dims / 2, 2]). ``scaling`` (factor, low, high, original): pairs whose
     wavelength exceeds original / low turn ``factor`` times slower, those below original / high as they are, and a
     linear blend in original / wavelength between."""
     f = float(base) ** (-torch.arange(0, dims, 2, dtype=torch.float64) / dims)
@@ -235,7 +235,8 @@ def rotary_frequencies(dims: int, base: float, scaling: Optional[dict] = None) -
         slow = f / float(scaling["factor"])
         s = (turns - low) / (high - low) if high != low else torch.zeros_like(f)
         f = torch.where(turns > high, f, torch.where(turns < low, slow, (1 - s) * slow + s * f))
-    return f.float()
+    hi = f.float()
+    return torch.stack([hi, (f - hi.double()).float()], dim=1).contiguous()
 
 
 def qk_norm_rope(q: torch.Tensor, k: torch.Tensor, heads: int, kv_heads: int, dim: int, q_weight: torch.Tensor,
@@ -244,7 +245,7 @@ def qk_norm_rope(q: torch.Tensor, k: torch.Tensor, heads: int, kv_heads: int, di
     Heads are padded as the weights are."""
     require_cuda(q, k, k_cache)
     a = FrQkRope(dtype=dtype_code(q.dtype), heads=heads, kv_heads=kv_heads, dim=int(q_weight.numel()) // heads, dim_true=dim,
-                 rot_dims=2 * int(inv_freq.numel()), eps=eps, q=ptr(q), ldq=q.stride(0), k=ptr(k), ldk=k.stride(0),
+                 rot_dims=2 * int(inv_freq.shape[0]), eps=eps, q=ptr(q), ldq=q.stride(0), k=ptr(k), ldk=k.stride(0),
                  q_weight=ptr(q_weight), k_weight=ptr(k_weight), inv_freq=ptr(inv_freq), pos=ptr(batch.positions),
                  loc=ptr(batch.out_cache_loc), k_cache=ptr(k_cache), ldkc=k_cache.stride(0))
     call("fr_lm_qk_norm_rope", ctypes.byref(a), int(q.shape[0]), stream_ptr(q.device))

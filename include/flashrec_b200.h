@@ -639,7 +639,7 @@ struct fr_qk_rope {
   int64_t ldk;
   const float* q_weight; /* [heads * dim] */
   const float* k_weight;
-  const float* inv_freq; /* [rot_dims / 2] */
+  const float* inv_freq; /* [rot_dims / 2, 2]: each frequency as a sum of two floats, larger one first */
   const int64_t* pos;
   const int64_t* loc;
   void* k_cache;
