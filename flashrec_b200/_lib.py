@@ -213,6 +213,9 @@ _SIGNATURES = {
     "fr_lm_qk_norm_rope": [P, _I, P],
     "fr_linear_state_floats": [_I, _I],
     "fr_linear_scan_rows": [P, _I, _I, _I, P],
+    "fr_linear_scan_chunks": [P, _I, _I, _I, _I, P, _L, P],
+    "fr_linear_scan_chunks_scratch": [P, _I, _I, _I],
+    "fr_linear_scan_chunks_fit": [_I, _I, _I],
     "fr_short_conv": [_I, P, _L, P, P, _I, _I, _I, P, _I, P, P, P, P, P, _I, _I, _I, P],
     "fr_mix_attn_rows": [P, _I, _I, _I, _I, P, _L, P, P],
     "fr_mix_attn_rows_scratch": [_I] * 6,
@@ -223,7 +226,7 @@ _SIGNATURES = {
 _RESTYPES = {"fr_version": c_char_p, "fr_decode_attn_scratch_bytes": c_int64,
              "fr_sid_head_topk_workspace_bytes": c_int64, "fr_joint_select_workspace_bytes": c_int64,
              "fr_trie_build_workspace_bytes": c_int64, "fr_mix_attn_rows_scratch": c_int64,
-             "fr_mix_attn_tc_scratch": c_int64, "fr_linear_state_floats": c_int64}
+             "fr_mix_attn_tc_scratch": c_int64, "fr_linear_state_floats": c_int64, "fr_linear_scan_chunks_scratch": c_int64}
 
 
 def lib_path() -> Path:

@@ -8,6 +8,7 @@
 //
 //   scan_rows_kernel   any sizes, either type, decode and prompts: a thread keeps 8 rows x 4 columns of S in
 //                      registers and walks the request's tokens, which are staged in shared memory in blocks
+//   linear_chunk.cu    bf16 prompts on tcgen05, a chunk of tokens at a time
 #include "fr_common.cuh"
 #include "linear_scan.cuh"
 #include "sm100_ptx.cuh"
@@ -51,7 +52,7 @@ struct RowsPlan {
 
 template <typename T, bool CHANNEL>
 __global__ void __launch_bounds__(1024)
-scan_rows_kernel(const __grid_constant__ fr_linear_scan a, const RowsPlan pl) {
+scan_rows_kernel(const __grid_constant__ fr_linear_scan a, const RowsPlan pl, int max_tokens) {
   extern __shared__ __align__(16) float sm[];
   const int np = state_rows(a.dim), vp = state_cols(a.vdim);
   const int rg_n = np / kRows, cq_n = pl.vb / kCols;
@@ -64,7 +65,7 @@ scan_rows_kernel(const __grid_constant__ fr_linear_scan a, const RowsPlan pl) {
   ptx::griddep_launch_dependents();
   const int b = blockIdx.z, h = blockIdx.y, c0 = blockIdx.x * pl.vb, tid = threadIdx.x, nt = blockDim.x;
   const int q0 = a.qo_indptr[b], q1 = a.qo_indptr[b + 1];
-  if (q0 >= q1) return;
+  if (q0 >= q1 || q1 - q0 > max_tokens) return;
   const int kh = h / (a.heads / a.key_heads);
   const int cq = tid % cq_n, rg = tid / cq_n;
   const bool active = rg < rg_n;
@@ -185,7 +186,7 @@ static int launch_rows(const fr_linear_scan& a, int n_req, int max_tokens, bool 
   static PerDeviceFlag f;
   if (ensure_dyn_smem(f, scan_rows_kernel<T, CHANNEL>, 200 * 1024) != FR_OK) return FR_ERR_CUDA;
   return launch_kernel(scan_rows_kernel<T, CHANNEL>, dim3(state_cols(a.vdim) / pl.vb, a.heads, n_req), pl.threads, pl.smem, stream, pdl,
-                       a, pl);
+                       a, pl, max_tokens);
 }
 
 }  // namespace scan

@@ -570,7 +570,8 @@ static int launch_update_norm(const fr_norm_update& u, int M, int W, cudaStream_
 // ---------------------------------------------------------------------------
 constexpr int kGroupThreads = 256;
 
-// NT threads per (row, group); eight columns at a time, NV of them per thread in registers
+// NT threads per (row, group): a part of a warp, a warp or the CTA; eight columns at a time, NV of them per thread in
+// registers
 template <typename T, int NT, int NV>
 __global__ void __launch_bounds__(kGroupThreads)
 group_norm_kernel(const __grid_constant__ fr_group_norm a, int M) {
@@ -578,9 +579,10 @@ group_norm_kernel(const __grid_constant__ fr_group_norm a, int M) {
   ptx::griddep_wait();
   ptx::griddep_launch_dependents();
   const int64_t job = static_cast<int64_t>(blockIdx.x) * (kGroupThreads / NT) + threadIdx.x / NT;
-  if (job >= static_cast<int64_t>(M) * a.groups) return;  // whole warps (NT is 32 or the CTA)
-  const int64_t t = job / a.groups;
-  const int g = static_cast<int>(job % a.groups), c0 = g * a.size, l = threadIdx.x % NT;
+  if (job - (threadIdx.x & 31) / NT >= static_cast<int64_t>(M) * a.groups) return;  // whole warps
+  const bool live = job < static_cast<int64_t>(M) * a.groups;
+  const int64_t t = live ? job / a.groups : 0;
+  const int g = live ? static_cast<int>(job % a.groups) : 0, c0 = g * a.size, l = threadIdx.x % NT;
   const T* y = static_cast<const T*>(a.y) + t * a.ldy + c0;
   const T* z = a.gate_mode != FR_GATE_NONE ? static_cast<const T*>(a.gate) + t * a.ldg + c0 : nullptr;
   const float* w = a.weight + (a.weight_per_group ? c0 : 0);
@@ -602,7 +604,13 @@ group_norm_kernel(const __grid_constant__ fr_group_norm a, int M) {
 #pragma unroll
       for (int e = 0; e < 8; ++e) ss = fmaf(v[i][e], v[i][e], ss);
     }
-    ss = NT == 32 ? warp_sum(ss) : cta_sum<kGroupThreads>(ss, sums);
+    if constexpr (NT <= 32) {
+#pragma unroll
+      for (int o = NT / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    } else {
+      ss = cta_sum<kGroupThreads>(ss, sums);
+    }
+    if (!live) return;
     const float r = 1.0f / sqrtf(ss / static_cast<float>(a.size) + a.eps);
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
@@ -648,16 +656,26 @@ static int launch_group_norm(const fr_group_norm& a, int M, cudaStream_t stream)
   const int64_t jobs = static_cast<int64_t>(M) * a.groups;
   const bool warp = a.size <= 1024;
   auto kern = warp ? group_norm_kernel<T, 32, 0> : group_norm_kernel<T, kGroupThreads, 0>;
+  int per = kGroupThreads / 32;  // groups per CTA
   if (vec && warp) kern = a.size <= 256 ? group_norm_kernel<T, 32, 1> : group_norm_kernel<T, 32, 4>;
+  if (vec && a.size <= 128) {
+    kern = a.size <= 64 ? group_norm_kernel<T, 8, 1> : group_norm_kernel<T, 16, 1>;
+    per = kGroupThreads / (a.size <= 64 ? 8 : 16);
+  }
   if (vec && !warp && a.size <= kGroupThreads * 32)
     kern = a.size <= kGroupThreads * 16 ? group_norm_kernel<T, kGroupThreads, 2> : group_norm_kernel<T, kGroupThreads, 4>;
-  return launch_kernel(kern, ceil_div(jobs, warp ? kGroupThreads / 32 : 1), kGroupThreads, 0, stream, M <= kPdlRows, a, M);
+  return launch_kernel(kern, ceil_div(jobs, warp ? per : 1), kGroupThreads, 0, stream, M <= kPdlRows, a, M);
 }
 
 // ---------------------------------------------------------------------------
 // queries and keys of one token: RMS norm over all heads at once, rotation, keys into the cache
 // ---------------------------------------------------------------------------
 constexpr int kRopeThreads = 256;
+
+__device__ __forceinline__ void ld8(const float* p, float (&v)[8]) {
+  *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(p);
+  *reinterpret_cast<float4*>(v + 4) = *reinterpret_cast<const float4*>(p + 4);
+}
 
 template <typename T>
 __global__ void __launch_bounds__(kRopeThreads)
@@ -708,6 +726,28 @@ qk_norm_rope_kernel(const __grid_constant__ fr_qk_rope a) {
     const int b = is_q ? c : c - nq, d0 = b % a.dim;
     const float rr = is_q ? rq : rk;
     float v[8];
+    if (d0 >= a.rot_dims || half % 8 == 0) {  // eight dimensions turn with eight others, or none does
+      float w8[8], i8[8];
+      ld8(src + b, v);
+      ld8(w + b, w8);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[e] *= rr * w8[e];
+      if (d0 < a.rot_dims) {
+        const int pair = d0 < half ? d0 : d0 - half, other = d0 < half ? b + half : b - half;
+        float c8[8], s8[8];
+        ld8(src + other, i8);
+        ld8(w + other, w8);
+        ld8(s_cos + pair, c8);
+        ld8(s_sin + pair, s8);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          const float it = i8[e] * rr * w8[e];
+          v[e] = d0 < half ? v[e] * c8[e] - it * s8[e] : v[e] * c8[e] + it * s8[e];
+        }
+      }
+      conv_store8<T>(is_q ? q + b : kc + b, v);
+      continue;
+    }
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
       const int d = d0 + e;
@@ -800,7 +840,7 @@ extern "C" int fr_lm_qk_norm_rope(const fr_qk_rope* a, int M, cudaStream_t strea
   if (M == 0) return FR_OK;
   FR_CHECK_ARG(a->dim_true > 0 && a->dim_true <= a->dim && a->rot_dims >= 0 && a->rot_dims % 2 == 0 && a->rot_dims <= a->dim_true);
   FR_CHECK_ARG(a->q && a->k && a->k_cache && a->q_weight && a->k_weight && a->pos && a->loc && (a->rot_dims == 0 || a->inv_freq));
-  FR_CHECK_ARG(aligned16(a->q) && aligned16(a->k) && aligned16(a->k_cache) && a->ldq % 8 == 0 && a->ldk % 8 == 0 && a->ldkc % 8 == 0);
+  FR_CHECK_ARG(aligned16(a->q) && aligned16(a->k) && aligned16(a->k_cache) && aligned16(a->q_weight) && aligned16(a->k_weight) && a->ldq % 8 == 0 && a->ldk % 8 == 0 && a->ldkc % 8 == 0);
   const int smem = ((a->heads + a->kv_heads) * a->dim + a->rot_dims) * 4;
   FR_CHECK_SUPPORTED(smem <= 200 * 1024);
   static PerDeviceFlag f0, f1;

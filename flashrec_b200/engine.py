@@ -17,10 +17,10 @@ import torch
 
 from flashrec_b200.core import ForwardBatch
 from flashrec_b200.kvcache import PAGE, SequenceManager
+from flashrec_b200.lm_layers import ROW_PORTION
 from flashrec_b200.sampling import Sampler, SamplingParams
 
 TILE_ROWS = 128          # tokens per tensor-core attention tile
-ROW_PORTION = 8          # shorter portions run their attention row by row
 
 
 @dataclass

@@ -26,6 +26,7 @@ SEG = {"store": _lib.FR_SEG_STORE, "swiglu": _lib.FR_SEG_SWIGLU, "sigmoid": _lib
        "store_f32": _lib.FR_SEG_STORE_F32, "glu_clamp": _lib.FR_SEG_GLU_CLAMP, "gelu_mul": _lib.FR_SEG_GELU_MUL}
 _PAIRED = ("swiglu", "glu_clamp")  # weight rows in [32 gate | 32 up] blocks
 MIX = {"diff": _lib.FR_MIX_DIFF, "talk": _lib.FR_MIX_TALK, "plain": _lib.FR_MIX_PLAIN}
+ROW_PORTION = 8  # shorter portions run their attention and recurrences row by row
 _SCORE_SCRATCH_BYTES = 256 << 20
 _MAP_SCRATCH_BYTES = 1 << 30  # maps of talking heads between their kernels: every token tile of a large step at once
 
@@ -378,7 +379,7 @@ class LinearScan:
         if heads % key_heads:
             raise ValueError("heads must be a multiple of key_heads")
         f32 = lambda t: None if t is None else t.to(device=device, dtype=torch.float32).contiguous()
-        self.heads, self.vdim = int(heads), int(vdim)
+        self._chunks: Optional[bool] = None
         self.step_bias, self.rate, self.up, self.skip = f32(step_bias), f32(rate), f32(up), f32(skip)
         self._args = FrLinearScan(decay=_lib.FR_DECAY_CHANNEL if decay == "channel" else _lib.FR_DECAY_HEAD, heads=heads,
                                   key_heads=key_heads, dim=dim, vdim=vdim, rank=0 if up is None else int(up.shape[1]),
@@ -387,7 +388,8 @@ class LinearScan:
 
     def forward(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, step: torch.Tensor, state: torch.Tensor,
                 batch: ForwardBatch, out: torch.Tensor) -> torch.Tensor:
-        """q, k [T, key_heads * dim], v and out [T, heads * vdim], step fp32; ``state`` [rows, state floats]."""
+        """q, k [T, key_heads * dim], v and out [T, heads * vdim], step fp32; ``state`` [rows, state floats]. bf16 prompts
+        run in chunks on the tensor cores, short portions, decode steps and fp32 token after token."""
         require_cuda(q, k, v, step, state)
         a = FrLinearScan.from_buffer_copy(self._args)
         a.dtype = dtype_code(q.dtype)
@@ -395,7 +397,17 @@ class LinearScan:
         a.out, a.ldo, a.step, a.ldstep = ptr(out), out.stride(0), ptr(step), step.stride(0)
         a.state, a.state_slots = ptr(state), ptr(batch.req_pool_indices)
         a.qo_indptr, a.pos = ptr(batch.qo_indptr), ptr(batch.positions)
+        n_req, t, s = int(batch.req_pool_indices.numel()), int(q.shape[0]), stream_ptr(q.device)
         longest = 1 if batch.one_token else max(batch.extend_seq_lens)
-        call("fr_linear_scan_rows", ctypes.byref(a), int(batch.req_pool_indices.numel()), longest, int(q.shape[0]),
-             stream_ptr(q.device))
+        lib = _lib.load()
+        if self._chunks is None:
+            self._chunks = bool(lib.fr_linear_scan_chunks_fit(a.decay, a.dim, a.vdim))
+        row_portion = longest
+        if self._chunks and a.dtype == 0 and longest > ROW_PORTION:
+            row_portion = ROW_PORTION
+            size = int(lib.fr_linear_scan_chunks_scratch(ctypes.byref(a), n_req, longest, t))
+            scratch = torch.empty(size, dtype=torch.uint8, device=q.device)
+            call("fr_linear_scan_chunks", ctypes.byref(a), n_req, longest, t, row_portion + 1, ptr(scratch), size, s)
+        if longest <= row_portion or min(batch.extend_seq_lens) <= row_portion:
+            call("fr_linear_scan_rows", ctypes.byref(a), n_req, row_portion, t, s)
         return out

@@ -51,7 +51,7 @@ FAMILIES: List[ModelFamily] = [
     ModelFamily("dibepel", lambda c: c.get("architecture") == "Dibepel", _load_dibepel, (torch.bfloat16, torch.float32),
                 ("capi", "dense_proj", "lm_rows", "attn_mix", "attn_talk")),
     ModelFamily("kotipel", lambda c: c.get("architecture") == "Kotipel", _load_kotipel, (torch.bfloat16, torch.float32),
-                ("capi", "dense_proj", "lm_rows", "attn_mix", "attn_talk", "linear_scan")),
+                ("capi", "dense_proj", "lm_rows", "attn_mix", "attn_talk", "linear_scan", "linear_chunk")),
 ]
 
 

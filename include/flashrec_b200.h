@@ -749,8 +749,15 @@ struct fr_linear_scan {
   const int64_t* pos;         /* [T] */
 };
 int64_t fr_linear_state_floats(int dim, int vdim);
-/* Any sizes, token after token. max_tokens: the most tokens of one request; n_tokens: of the batch. */
+/* Any sizes, token after token. Requests of more than max_tokens tokens are left alone; n_tokens: of the batch. */
 int fr_linear_scan_rows(const struct fr_linear_scan* a, int n_req, int max_tokens, int n_tokens, cudaStream_t stream);
+/* bf16 on the tensor cores, in chunks of up to 128 tokens: dim and vdim multiples of 16, dim <= 128
+ * (fr_linear_scan_chunks_fit tells). Requests of fewer than min_tokens tokens are left alone; longest: the most tokens
+ * of one request; scratch: fr_linear_scan_chunks_scratch(...) bytes. */
+int fr_linear_scan_chunks(const struct fr_linear_scan* a, int n_req, int longest, int n_tokens, int min_tokens, void* scratch,
+                          int64_t scratch_bytes, cudaStream_t stream);
+int64_t fr_linear_scan_chunks_scratch(const struct fr_linear_scan* a, int n_req, int longest, int n_tokens);
+int fr_linear_scan_chunks_fit(int decay, int dim, int vdim);
 
 #ifdef __cplusplus
 }

@@ -267,11 +267,20 @@ SCANS = [  # decay, heads, key heads, dim, vdim, strength of the decays
 def test_matrix_state_recurrences(dtype, case):
     """Three requests in portions of every size, on state rows that hold something else before; decays from nearly none
     to a state that is gone after two tokens."""
+    _check_scan(dtype, case, [330, 150, 41], ((400,), (70, 1, 2, 64, 63, 200), (130, 128, 3, 1, 1, 300)))
+
+
+@pytest.mark.parametrize("case", [SCANS[2], SCANS[3], SCANS[8], SCANS[10], SCANS[12]])
+def test_recurrences_in_segments(case):
+    """Prompts that are long enough for several CTAs to share one head's tokens."""
+    _check_scan(torch.bfloat16, case, [2100, 700, 1030], ((2100,), (1200, 9, 1500)))
+
+
+def _check_scan(dtype, case, lens, cuts):
     from flashrec_b200.kvcache import CacheSpec
     from flashrec_b200.lm_layers import LinearScan
 
     kind, heads, kh, dim, vdim, strength = case
-    lens = [330, 150, 41]
     rank, scale, tau = 5, 0.3, 2.0
     bias = _rand(heads * dim if kind == "channel" else heads, seed=1)
     up = _rand(heads * dim, rank, seed=2, scale=0.7) if kind == "channel" else None
@@ -298,7 +307,7 @@ def test_matrix_state_recurrences(dtype, case):
         refs.append(torch.cat(out, dim=1))
     spec = CacheSpec(0, 0, state_heads=heads, state_dim=dim, state_vdim=vdim)
     slots = [5, 0, 3]
-    for portions in ((400,), (70, 1, 2, 64, 63, 200), (130, 128, 3, 1, 1, 300)):
+    for portions in cuts:
         state = torch.full((6, spec.state_floats), float("nan"), device="cuda")
         done, got, x = [0, 0, 0], [[], [], []], 0
         while any(d < n for d, n in zip(done, lens)):
