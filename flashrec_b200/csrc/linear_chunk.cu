@@ -1,23 +1,27 @@
-// bf16 prompts of the matrix-state recurrences (fr_linear_scan in the header) on tcgen05, in chunks of up to 128 tokens.
-// With r_i the sum of the log decays of the chunk's tokens after its first (r_0 = 0) and S' = a_0 S the decayed old state,
-// u_j the value that enters the state:
+// bf16 prompts of the matrix-state recurrences (fr_linear_scan in the header) on tcgen05, in chunks of 128 tokens.
+// With r_i the sum of the log decays of the chunk's tokens after its first (r_0 = 0), u_j the value that enters the state
+// (step_j v_j, or v_j) and a_0 the decay of the first token:
 //
-//     decay per head:     P_ij = e^(r_i - r_j) q_i . k_j   (j <= i)        O = e^r (Q S') + P U
-//                         S <- e^(r_last) S' + K^T (e^(r_last - r_j) u_j)
-//     decay per channel:  q~_i = e^(r_i) q_i,  k~_j = e^(-r_j) k_j,  P = mask(Q~ K~^T),  O = Q~ S' + P U
-//                         S <- e^(r_last) (S' + K~^T U)
+//     decay per head:     P_ij = e^(r_i - r_j) q_i . k_j   (j <= i)           O = e^r (Q (a_0 S)) + P U
+//                         S <- e^(r_last) a_0 S + K^T (e^(r_last - r_j) u_j)
+//     decay per channel:  q~_i = e^(r_i - m) q_i,  k~_j = e^(m - r_j) k_j,  P = mask(Q~ K~^T),  O = Q~ S' + P U
+//                         S' = e^m a_0 S,  S <- e^(r_last - m) (S' + K~^T U),  m = r_last / 2
 //
-// Per channel a chunk ends early where the decays would leave the range that e^(-r) can hold, so any decays are exact
-// (with a single token r is 0).
+// The second form needs |r_last| below what e^(m - r) can hold. Heads of a request that leave this range anywhere are
+// flagged and left to the token-by-token kernel.
 //
 // Decays, factors, masks and the state are fp32. What is not bf16 to begin with (q~, k~, scaled values, P, S') enters the
 // tensor cores as a sum of two bf16 numbers, 16 significant bits, in two or three products.
 //
-// One CTA: one head, up to 64 columns of V and S, one segment of a request. S lives in registers (thread = row of S and
-// a quarter of the columns). Warps 0..15 work on operands, mask, state and output; warp 16 issues TMA and tcgen05.mma;
-// warp 17 computes the next chunk's factors (decay per head). Long prompts are cut into segments that run side by side:
-// a first launch finds the state that each segment adds and its total decay, the second starts every segment from the
-// combination of those before it.
+//   head_factor_kernel     decay per head: e^r and its relatives, one warp per chunk and head
+//   channel_factor_kernel  decay per channel: the low-rank decays, q~ and k~ of every chunk and head
+//   chunk_kernel           one CTA: one head, up to 64 columns of V and S, one segment of a request, chunk after chunk. S
+//                          lives in registers (thread = row of S and a quarter of the columns). Warps 0..15 work on
+//                          operands, mask, state and output; warp 16 issues TMA and tcgen05.mma. Scores, tiles and
+//                          operands are one chunk ahead of the output.
+//
+// Long prompts are cut into segments that run side by side: a first launch finds the state that each segment adds and its
+// total decay, the second starts every segment from the combination of those before it.
 #include "fr_common.cuh"
 #include "linear_scan.cuh"
 #include "sm100_ptx.cuh"
@@ -34,11 +38,10 @@ constexpr int kChunk = 128;            // tokens (UMMA M)
 constexpr int kVb = 64;                // columns of V per CTA: one swizzle span
 constexpr int kBox = kChunk * 128;     // bytes of a [128 x 64] bf16 tile
 constexpr int kCompute = 512;          // threads of the compute warps
-constexpr int kThreads = kCompute + 64;
+constexpr int kThreads = kCompute + 32;
 constexpr float kLog2e = 1.4426950408889634f;
-// largest -r (in powers of two) inside a chunk, per channel: e^(-r) k, its products and their sums stay far below 2^127,
-// and the small halves of e^r q above 2^-126
-constexpr float kMaxChannel = 86.f;
+// largest -r_last (in powers of two) per channel: e^(+-r_last / 2), its products and their sums stay far inside 2^+-126
+constexpr float kMaxChannel = 160.f;
 
 __device__ __forceinline__ float ex2(float x) {
   float y;
@@ -52,6 +55,19 @@ __device__ __forceinline__ uint32_t split2(float a, float b, uint32_t& lo) {
   return hi;
 }
 
+// Factors of one chunk and head.
+struct HeadFactors {
+  float r[kChunk];    // r_i (log2)
+  float c[kChunk];    // log2(step_j) - r_j
+  float x[kChunk];    // step_j e^(r_last - r_j)
+  float first, end;   // a_0, e^(r_last)
+  float pad_[2];
+};
+struct ChannelFactors {  // per row of S
+  float first[kChunk];   // e^m a_0
+  float end[kChunk];     // e^(r_last - m)
+};
+
 struct ChunkPlan {
   int boxes;     // 64-column boxes of a q / k row
   int seg_len;   // tokens per segment (a multiple of kChunk)
@@ -64,73 +80,44 @@ struct ChunkArgs {
   fr_linear_scan a;
   ChunkPlan pl;
   int min_tokens;      // shorter requests are left alone
-  const float* log2_decay;  // CHANNEL: [T, heads * dim]
+  void* factors;       // [chunk, head]
+  __nv_bfloat16* qk;   // CHANNEL: q~ hi, q~ lo, k~ hi, k~ lo, each [T, heads * dim]
+  int64_t qk_stride;   // elements of one of them
+  int32_t* flags;      // CHANNEL: [request, head] left to the token-by-token kernel
   float* seg_state;    // [request, segment, head][dim][state cols]
   float* seg_decay;    // [request, segment, head][dim]
   float* start_state;  // [request, head][dim][state cols]
 };
 
+// Number of a request's first chunk: requests take ceil(tokens / 128) numbers each without overlapping.
+__device__ __forceinline__ int64_t first_chunk(int q0, int b) { return q0 / kChunk + b; }
+
 // ---------------------------------------------------------------------------
-// log2 of the decays per key channel
-// ---------------------------------------------------------------------------
-constexpr int kDecayTokens = 32;
-__global__ void __launch_bounds__(256)
-log_decay_kernel(const __grid_constant__ fr_linear_scan a, int T, float* __restrict__ out) {
-  extern __shared__ float s_low[];  // [tokens][rank]
+constexpr int kFactorHeads = 8;
+__global__ void __launch_bounds__(kFactorHeads * 32)
+head_factor_kernel(const __grid_constant__ ChunkArgs g) {
   ptx::griddep_wait();
   ptx::griddep_launch_dependents();
-  const int t0 = blockIdx.x * kDecayTokens, n = min(kDecayTokens, T - t0), N = a.heads * a.dim;
-  for (int e = threadIdx.x; e < n * a.rank; e += 256) s_low[e] = a.step[static_cast<int64_t>(t0 + e / a.rank) * a.ldstep + e % a.rank];
-  __syncthreads();
-  const int ch = blockIdx.y * 256 + threadIdx.x;
-  if (ch >= N) return;
-  const float* up = a.up + static_cast<int64_t>(ch) * a.rank;
-  const float bias = a.step_bias[ch], f = -a.inv_tau * kLog2e;
-  for (int g = 0; g < n; g += 8) {
-    float z[8];
-#pragma unroll
-    for (int i = 0; i < 8; ++i) z[i] = bias;
-    for (int r = 0; r < a.rank; ++r) {
-      const float u = up[r];
-#pragma unroll
-      for (int i = 0; i < 8; ++i) z[i] = fmaf(u, s_low[min(g + i, n - 1) * a.rank + r], z[i]);
-    }
-#pragma unroll
-    for (int i = 0; i < 8; ++i)
-      if (g + i < n) out[static_cast<int64_t>(t0 + g + i) * N + ch] = softplus(-z[i]) * f;
-  }
-}
-
-// ---------------------------------------------------------------------------
-// Factors of a chunk for a decay per head, in shared memory (two sets).
-struct HeadFactors {
-  float r[kChunk];    // r_i (log2)
-  float c[kChunk];    // log2(step_j) - r_j
-  float x[kChunk];    // step_j e^(r_last - r_j)
-  float first, end;   // decay of the first token, of the others
-  float pad_[2];
-};
-
-// One warp, four tokens per lane.
-__device__ __forceinline__ void head_factors(const fr_linear_scan& a, HeadFactors* f, int64_t t, int n, int h) {
-  const int lane = threadIdx.x & 31;
-  float step[4], la[4];
+  const fr_linear_scan& a = g.a;
+  const int b = blockIdx.z, h = blockIdx.y * kFactorHeads + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int q0 = a.qo_indptr[b], q1 = a.qo_indptr[b + 1];
+  const int t = q0 + blockIdx.x * kChunk, n = min(kChunk, q1 - t);
+  if (h >= a.heads || t >= q1) return;
+  HeadFactors* f = static_cast<HeadFactors*>(g.factors) + (first_chunk(q0, b) + blockIdx.x) * a.heads + h;
+  const float rate = -a.rate[h] * kLog2e;
+  float step[4], la[4], sum = 0.f, first = 0.f;  // four tokens per lane
 #pragma unroll
   for (int e = 0; e < 4; ++e) {
     const int i = lane * 4 + e;
     step[e] = i < n ? head_step(a, t + i, h) : 0.f;
-  }
-  const float rate = -a.rate[h] * kLog2e;
-  float sum = 0.f;
-#pragma unroll
-  for (int e = 0; e < 4; ++e) {
     la[e] = rate * step[e];
-    if (lane == 0 && e == 0) {
-      f->first = ex2(la[0]);
-      la[0] = 0.f;
-    }
-    sum += la[e];
   }
+  if (lane == 0) {
+    first = ex2(la[0]);
+    la[0] = 0.f;
+  }
+#pragma unroll
+  for (int e = 0; e < 4; ++e) sum += la[e];
   float x = sum;
 #pragma unroll
   for (int o = 1; o < 32; o *= 2) {
@@ -138,29 +125,146 @@ __device__ __forceinline__ void head_factors(const fr_linear_scan& a, HeadFactor
     if (lane >= o) x += y;
   }
   const float last = __shfl_sync(0xffffffffu, x, 31);
-  float r = x - sum;
+  float r = x - sum, fr[4], fc[4], fx[4];
 #pragma unroll
   for (int e = 0; e < 4; ++e) {
-    const int i = lane * 4 + e;
     r += la[e];
-    f->r[i] = r;
-    f->c[i] = log2f(step[e]) - r;  // -inf past the end: no weight
-    f->x[i] = step[e] * ex2(last - r);
+    fr[e] = r;
+    fc[e] = log2f(step[e]) - r;  // -inf past the end: no weight
+    fx[e] = step[e] * ex2(last - r);
   }
-  if (lane == 0) f->end = ex2(last);
+  *reinterpret_cast<float4*>(f->r + lane * 4) = make_float4(fr[0], fr[1], fr[2], fr[3]);
+  *reinterpret_cast<float4*>(f->c + lane * 4) = make_float4(fc[0], fc[1], fc[2], fc[3]);
+  *reinterpret_cast<float4*>(f->x + lane * 4) = make_float4(fx[0], fx[1], fx[2], fx[3]);
+  if (lane == 0) *reinterpret_cast<float4*>(&f->first) = make_float4(first, ex2(last), 0.f, 0.f);
 }
 
-// Shared memory. HEAD: q, k tiles, two v tiles, scaled v hi and lo; CHANNEL: two v tiles, q~ hi, lo, k~ hi, lo; both: S' hi, lo.
-__host__ __device__ __forceinline__ int tile_smem(bool channel, int boxes, int dim) {
-  return (channel ? 2 * kBox + 4 * boxes * kBox : 2 * boxes * kBox + 4 * kBox) + 2 * dim * 128;
+// One chunk of one head: a thread has two channels and a share of the tokens.
+constexpr int kPrepThreads = 256;
+__global__ void __launch_bounds__(kPrepThreads)
+channel_factor_kernel(const __grid_constant__ ChunkArgs g) {
+  extern __shared__ __align__(16) float sm[];
+  const fr_linear_scan& a = g.a;
+  const int pairs = a.dim / 2;
+  int parts = 1;
+  while (parts * 2 * pairs <= kPrepThreads && parts < 32) parts *= 2;
+  const int tp = kChunk / parts;
+  float* s_la = sm;                         // [128][dim]
+  float* s_low = s_la + kChunk * a.dim;     // [128][rank]
+  float* s_part = s_low + kChunk * a.rank;  // [parts][dim]
+  ptx::griddep_wait();
+  ptx::griddep_launch_dependents();
+  const int b = blockIdx.z, h = blockIdx.y, tid = threadIdx.x;
+  const int q0 = a.qo_indptr[b], q1 = a.qo_indptr[b + 1];
+  const int t = q0 + blockIdx.x * kChunk;
+  if (t >= q1) return;
+  const int n = min(kChunk, q1 - t);
+  for (int e = tid; e < n * a.rank; e += kPrepThreads) s_low[e] = a.step[static_cast<int64_t>(t + e / a.rank) * a.ldstep + e % a.rank];
+  __syncthreads();
+  const int part = tid / pairs, ch = 2 * (tid % pairs), i0 = part * tp, i1 = min(n, i0 + tp);
+  const bool live = part < parts;
+  if (live) {
+    const int hc = h * a.dim + ch;
+    const float* up = a.up + static_cast<int64_t>(hc) * a.rank;
+    const float b0 = a.step_bias[hc], b1 = a.step_bias[hc + 1], f = -a.inv_tau * kLog2e;
+    float2 sum = make_float2(0.f, 0.f);
+    for (int i = i0; i < i1; i += 4) {
+      float z0[4], z1[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        z0[e] = b0;
+        z1[e] = b1;
+      }
+      for (int r = 0; r < a.rank; ++r) {
+        const float u0 = up[r], u1 = up[a.rank + r];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float low = s_low[min(i + e, n - 1) * a.rank + r];
+          z0[e] = fmaf(u0, low, z0[e]);
+          z1[e] = fmaf(u1, low, z1[e]);
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        if (i + e >= i1) break;
+        const float2 la = make_float2(softplus(-z0[e]) * f, softplus(-z1[e]) * f);
+        *reinterpret_cast<float2*>(s_la + (i + e) * a.dim + ch) = la;
+        if (i + e > 0) {
+          sum.x += la.x;
+          sum.y += la.y;
+        }
+      }
+    }
+    *reinterpret_cast<float2*>(s_part + part * a.dim + ch) = sum;
+  }
+  __syncthreads();
+  if (!live) return;
+  float2 r = make_float2(0.f, 0.f), last = r;
+  for (int p = 0; p < parts; ++p) {
+    const float2 d = *reinterpret_cast<const float2*>(s_part + p * a.dim + ch);
+    if (p < part) {
+      r.x += d.x;
+      r.y += d.y;
+    }
+    last.x += d.x;
+    last.y += d.y;
+  }
+  // out of range: flagged; what is written stays finite (a neighbour's tile may hold these rows, times zero)
+  const bool wide = fminf(last.x, last.y) < -kMaxChannel;
+  const float m0 = 0.5f * fmaxf(last.x, -kMaxChannel), m1 = 0.5f * fmaxf(last.y, -kMaxChannel);
+  if (part == 0) {
+    const float2 la = *reinterpret_cast<const float2*>(s_la + ch);
+    ChannelFactors* f = static_cast<ChannelFactors*>(g.factors) + (first_chunk(q0, b) + blockIdx.x) * a.heads + h;
+    *reinterpret_cast<float2*>(f->first + ch) = make_float2(ex2(la.x + m0), ex2(la.y + m1));
+    *reinterpret_cast<float2*>(f->end + ch) = make_float2(ex2(last.x - m0), ex2(last.y - m1));
+    if (wide) g.flags[b * a.heads + h] = 1;
+  }
+  const __nv_bfloat16* qp = static_cast<const __nv_bfloat16*>(a.q) + static_cast<int64_t>(t) * a.ldq + h * a.dim + ch;
+  const __nv_bfloat16* kp = static_cast<const __nv_bfloat16*>(a.k) + static_cast<int64_t>(t) * a.ldk + h * a.dim + ch;
+  const int64_t ld = static_cast<int64_t>(a.heads) * a.dim;
+  __nv_bfloat16* out = g.qk + t * ld + h * a.dim + ch;
+#pragma unroll 4
+  for (int i = i0; i < i1; ++i) {
+    if (i > 0) {
+      const float2 d = *reinterpret_cast<const float2*>(s_la + i * a.dim + ch);
+      r.x += d.x;
+      r.y += d.y;
+    }
+    const uint32_t qv = *reinterpret_cast<const uint32_t*>(qp + i * a.ldq), kv = *reinterpret_cast<const uint32_t*>(kp + i * a.ldk);
+    const float e0 = fminf(fmaxf(r.x - m0, -kMaxChannel / 2), kMaxChannel / 2), e1 = fminf(fmaxf(r.y - m1, -kMaxChannel / 2), kMaxChannel / 2);
+    uint32_t lo;
+    __nv_bfloat16* o = out + i * ld;
+    *reinterpret_cast<uint32_t*>(o) = split2(bf16lo(qv) * a.scale * ex2(e0), bf16hi(qv) * a.scale * ex2(e1), lo);
+    *reinterpret_cast<uint32_t*>(o + g.qk_stride) = lo;
+    *reinterpret_cast<uint32_t*>(o + 2 * g.qk_stride) = split2(bf16lo(kv) * ex2(-e0), bf16hi(kv) * ex2(-e1), lo);
+    *reinterpret_cast<uint32_t*>(o + 3 * g.qk_stride) = lo;
+  }
 }
-constexpr int kPartFloats = 1024;
-constexpr int kTailSmem = 2 * static_cast<int>(sizeof(HeadFactors)) + (2 * kChunk + kPartFloats) * 4 + 128;
+
+// ---------------------------------------------------------------------------
+// Shared memory: tiles of q and k (CHANNEL: hi and lo each), two of v, S' hi and lo, HEAD: scaled v hi and lo; factors.
+__host__ __device__ __forceinline__ int tile_smem(bool channel, int boxes, int dim) {
+  return (channel ? 4 : 2) * boxes * kBox + 2 * kBox + (channel ? 0 : 2 * kBox) + 2 * dim * 128;
+}
+template <bool CHANNEL>
+struct FactorsOf {
+  using type = HeadFactors;
+};
+template <>
+struct FactorsOf<true> {
+  using type = ChannelFactors;
+};
+constexpr int kTailSmem = 2 * static_cast<int>(sizeof(HeadFactors)) + 128;
+static_assert(sizeof(HeadFactors) % 16 == 0 && sizeof(ChannelFactors) % 16 == 0 && sizeof(ChannelFactors) <= sizeof(HeadFactors));
+
+struct ChunkMaps {
+  CUtensorMap v, q, k, q_lo, k_lo;
+};
 
 template <bool CHANNEL, bool STATE_ONLY>
 __global__ void __launch_bounds__(kThreads, 1)
-chunk_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tk,
-             const __grid_constant__ CUtensorMap tv, const __grid_constant__ ChunkArgs g, int* status) {
+chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ ChunkArgs g, int* status) {
+  using Factors = typename FactorsOf<CHANNEL>::type;
   extern __shared__ uint8_t smem_raw[];
   const uint32_t raw = ptx::smem_u32(smem_raw);
   const uint32_t base = (raw + 1023u) & ~1023u;
@@ -168,25 +272,20 @@ chunk_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUt
   const fr_linear_scan& a = g.a;
   const ChunkPlan& pl = g.pl;
   const int kq = pl.boxes * kBox;
-  const uint32_t off_v = CHANNEL ? 0u : 2u * kq;                       // [2] tiles of v
-  const uint32_t off_q = CHANNEL ? 2u * kBox : 0u;                     // CHANNEL: hi, lo
-  const uint32_t off_k = off_q + (CHANNEL ? 2 : 1) * kq;               // CHANNEL: hi, lo
-  const uint32_t off_x = off_v + 2u * kBox;                            // HEAD: scaled v hi, lo
-  const uint32_t off_s = CHANNEL ? off_k + 2u * kq : off_x + 2u * kBox;
+  const uint32_t off_q = 0, off_k = (CHANNEL ? 2u : 1u) * kq;  // CHANNEL: hi, lo
+  const uint32_t off_v = 2u * off_k;                           // two tiles
+  const uint32_t off_x = off_v + 2u * kBox;                    // HEAD: scaled v hi, lo
+  const uint32_t off_s = CHANNEL ? off_x : off_x + 2u * kBox;
   const uint32_t s_bytes = a.dim * 128;
-  HeadFactors* fac = reinterpret_cast<HeadFactors*>(smem + off_s + 2 * s_bytes);
-  float* s_first = reinterpret_cast<float*>(fac + 2);  // CHANNEL: [128] decay of the chunk's first token per row of S
-  float* s_end = s_first + kChunk;                     // CHANNEL: [128] decay of the others
-  float* s_part = s_end + kChunk;                      // CHANNEL: partial sums of log decays
-  uint64_t* bars = reinterpret_cast<uint64_t*>(s_part + kPartFloats);
+  Factors* fac = reinterpret_cast<Factors*>(smem + off_s + 2 * s_bytes);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(fac + 2);
   const uint32_t bar_v = ptx::smem_u32(bars);          // [2]
   const uint32_t bar_qk = bar_v + 16, bar_g = bar_v + 24, bar_su = bar_v + 32, bar_o = bar_v + 40;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 6);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
-  int* s_len = reinterpret_cast<int*>(tmem_slot + 2);  // [2] CHANNEL: tokens of this chunk and the next
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const bool compute = tid < kCompute, issuer = tid == kCompute, factor_warp = warp == kCompute / 32 + 1;
+  const bool compute = tid < kCompute, issuer = tid == kCompute;
   ptx::griddep_wait();
   const int h = blockIdx.x / pl.v_blocks, c0 = (blockIdx.x % pl.v_blocks) * kVb;
   const int b = blockIdx.z, seg = blockIdx.y;
@@ -194,6 +293,7 @@ chunk_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUt
   const int t_begin = q0 + seg * pl.seg_len;
   if (q1 - q0 < g.min_tokens || t_begin >= q1) return;
   if (STATE_ONLY && t_begin + pl.seg_len >= q1) return;  // nothing follows the last segment
+  if (CHANNEL && g.flags[b * a.heads + h] != 0) return;
   const int t_end = min(t_begin + pl.seg_len, q1);
   const int kh = h / (a.heads / a.key_heads);
   const int vb = min(kVb, a.vdim - c0);
@@ -202,44 +302,51 @@ chunk_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUt
   if (tid == 0) {
     for (int i = 0; i < 6; ++i) ptx::mbar_init(bar_v + 8 * i, 1);
     *abort_flag = 0;
-    s_len[0] = min(kChunk, t_end - t_begin);
     ptx::mbar_init_fence();
-    ptx::prefetch_tmap(&tv);
-    if (!CHANNEL) {
-      ptx::prefetch_tmap(&tq);
-      ptx::prefetch_tmap(&tk);
-    }
+    ptx::prefetch_tmap(&maps.v);
+    ptx::prefetch_tmap(&maps.q);
+    ptx::prefetch_tmap(&maps.k);
   }
   if (warp == kCompute / 32) {
     __syncwarp();
-    ptx::tmem_alloc(ptx::smem_u32(tmem_slot), CHANNEL ? 256 : 512);
+    ptx::tmem_alloc(ptx::smem_u32(tmem_slot), 512);
     ptx::tmem_relinquish();
   }
-  if (!CHANNEL && factor_warp) head_factors(a, fac, t_begin, min(kChunk, t_end - t_begin), h);
   ptx::tc_fence_before();
   __syncthreads();
   ptx::tc_fence_after();
   ptx::griddep_launch_dependents();  // not before the tensor memory is taken
   const uint32_t tmem = *tmem_slot;
-  // scores and P (HEAD: two sets), Q S' (CHANNEL: and P U), K^T U, HEAD: P U
-  const uint32_t col_in = tmem + 128, col_su = tmem + 192, col_pu = CHANNEL ? col_in : tmem + 256, col_p1 = CHANNEL ? tmem : tmem + 384;
+  // scores and P (two sets of 128 columns), Q S', K^T U, P U (CHANNEL: added to Q S')
+  const uint32_t col_in = tmem + 256, col_su = tmem + 320, col_pu = CHANNEL ? col_in : tmem + 384;
   const uint32_t lane_off = static_cast<uint32_t>((warp & 3) * 32) << 16;
+  const Factors* factors = static_cast<const Factors*>(g.factors) + (first_chunk(q0, b) + seg * (pl.seg_len / kChunk)) * a.heads + h;
 
-  auto load_v = [&](int t, int set) {  // one thread, as are the next two
-    ptx::mbar_expect_tx(bar_v + 8 * set, kBox);
-    ptx::tma_load_2d(base + off_v + set * kBox, &tv, h * a.vdim + c0, t, bar_v + 8 * set);
+  // ---- one thread: TMA and tcgen05.mma -----------------------------------------------------------------
+  auto load_v = [&](int it) {
+    const int set = it & 1;
+    ptx::mbar_expect_tx(bar_v + 8 * set, kBox + sizeof(Factors));
+    ptx::tma_load_2d(base + off_v + set * kBox, &maps.v, h * a.vdim + c0, t_begin + it * kChunk, bar_v + 8 * set);
+    ptx::bulk_load(ptx::smem_u32(fac + set), factors + static_cast<int64_t>(it) * a.heads, sizeof(Factors), bar_v + 8 * set);
   };
-  auto load_qk = [&](int t) {
-    ptx::mbar_expect_tx(bar_qk, STATE_ONLY ? kq : 2 * kq);
+  auto load_qk = [&](int it) {
+    const int t = t_begin + it * kChunk;
+    ptx::mbar_expect_tx(bar_qk, (STATE_ONLY ? 1 : 2) * off_k);
     for (int x = 0; x < pl.boxes; ++x) {
-      if (!STATE_ONLY) ptx::tma_load_2d(base + off_q + x * kBox, &tq, kh * a.dim + x * 64, t, bar_qk);
-      ptx::tma_load_2d(base + off_k + x * kBox, &tk, kh * a.dim + x * 64, t, bar_qk);
+      const int col = kh * a.dim + x * 64;
+      if (!STATE_ONLY) ptx::tma_load_2d(base + off_q + x * kBox, &maps.q, col, t, bar_qk);
+      ptx::tma_load_2d(base + off_k + x * kBox, &maps.k, col, t, bar_qk);
+      if (CHANNEL) {
+        if (!STATE_ONLY) ptx::tma_load_2d(base + off_q + kq + x * kBox, &maps.q_lo, col, t, bar_qk);
+        ptx::tma_load_2d(base + off_k + kq + x * kBox, &maps.k_lo, col, t, bar_qk);
+      }
     }
   };
-  auto issue_scores = [&](uint32_t col) {
+  auto issue_scores = [&](int it) {
     constexpr uint32_t idesc = ptx::make_idesc(1u, 1u, kChunk, kChunk);
     const uint64_t qd = ptx::smem_desc_sw128(base + off_q), kd = ptx::smem_desc_sw128(base + off_k);
     const uint64_t lo = kq >> 4;
+    const uint32_t col = tmem + (it & 1) * kChunk;
 #pragma unroll 1
     for (int k = 0; k < a.dim / 16; ++k) {
       const uint64_t o = (k >> 2) * (kBox / 16) + 2u * (k & 3);
@@ -257,7 +364,7 @@ chunk_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUt
     ptx::tc_fence_after();
   };
 
-  // S: row of the state and a quarter of the columns
+  // ---- S: row of the state and a quarter of the columns --------------------------------------------------
   const int row = tid & 127, quarter = (tid >> 7) & 3, col0 = quarter * 16;
   const bool state_thread = compute && row < a.dim;
   const bool my_cols = col0 < vb;  // vb is a multiple of 16
@@ -297,178 +404,80 @@ chunk_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUt
     }
   }
   const float skip = a.skip != nullptr ? a.skip[h] : 0.f;
-  // CHANNEL: a thread prepares two channels of every token of its share of the chunk
-  const int pairs = a.dim / 2;
-  int parts = 1;
-  while (parts * 2 * pairs <= kCompute && parts < 32) parts *= 2;
-  const int tp = kChunk / parts;
-  const int my_part = tid / pairs, ch = 2 * (tid % pairs), i0 = my_part * tp;
-  const bool prep = CHANNEL && my_part < parts;
-  const int64_t ld_la = static_cast<int64_t>(a.heads) * a.dim;
-  const uint32_t ch_off = (ch >> 6) * kBox + (ch & 7) * 2;  // of the channel pair in a tile of q~ or k~
-  auto ch_addr = [&](int i) { return smem + off_q + ch_off + i * 128 + ((((ch & 63) >> 3) ^ (i & 7)) << 4); };
 
-  if (issuer) {
-    load_v(t_begin, 0);
-    if (!CHANNEL) {
-      load_qk(t_begin);
-      if (!STATE_ONLY && ptx::mbar_wait(bar_qk, 0, abort_flag, status, 91)) issue_scores(tmem);
-    }
-  }
-  __syncwarp();
-  int it = 0;
-  for (int t = t_begin; t < t_end; ++it) {
-    const int n = min(kChunk, t_end - t);
-    const int set = it & 1;
-    const uint32_t set_ph = (it >> 1) & 1, ph = it & 1;
-    const uint32_t col_p = CHANNEL || set == 0 ? tmem : col_p1;
-    const HeadFactors* f = fac + set;
-    int len = n;
-
-    // ---- operands -----------------------------------------------------------------------------------
-    if constexpr (CHANNEL) {
-      const float* la = g.log2_decay + t * ld_la + h * a.dim + ch;
-      if (prep) {
-        float2 sum = make_float2(0.f, 0.f);
-#pragma unroll 8
-        for (int i = i0; i < i0 + tp; ++i)
-          if (i > 0 && i < n) {
-            const float2 d = *reinterpret_cast<const float2*>(la + i * ld_la);
-            sum.x += d.x;
-            sum.y += d.y;
-          }
-        *reinterpret_cast<float2*>(s_part + my_part * a.dim + ch) = sum;
-        if (my_part == 0) {
-          const float2 d = *reinterpret_cast<const float2*>(la);
-          *reinterpret_cast<float2*>(s_first + ch) = make_float2(ex2(d.x), ex2(d.y));
-        }
-      }
-      __syncthreads();
-      if (prep) {
-        float2 r = make_float2(0.f, 0.f);
-        for (int p = 0; p < my_part; ++p) {
-          const float2 d = *reinterpret_cast<const float2*>(s_part + p * a.dim + ch);
-          r.x += d.x;
-          r.y += d.y;
-        }
-        const __nv_bfloat16* qp = static_cast<const __nv_bfloat16*>(a.q) + t * a.ldq + h * a.dim + ch;
-        const __nv_bfloat16* kp = static_cast<const __nv_bfloat16*>(a.k) + t * a.ldk + h * a.dim + ch;
-        int bad = kChunk;
-        for (int g0 = i0; g0 < i0 + tp; g0 += 4) {  // four tokens' loads together (tp is a multiple of 4)
-          float2 d[4];
-          uint32_t kv[4], qv[4];
+  // Operands of a chunk: S' over the old state and its halves, scaled values; `x` keeps the raw values.
+  auto operands = [&](int it, uint32_t (&x)[8]) {
+    const int n = min(kChunk, t_end - (t_begin + it * kChunk)), set = it & 1;
+    wait_bar(bar_v + 8 * set, (it >> 1) & 1, 92);
+    const Factors* f = fac + set;
+    if (state_thread) {
+      float first;
+      if constexpr (CHANNEL) first = f->first[row];
+      else first = f->first;
+      decay_all *= first;
+      uint8_t* dst = smem + off_s + row * 128;
 #pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const int64_t i = min(g0 + e, n - 1);
-            d[e] = *reinterpret_cast<const float2*>(la + i * ld_la);
-            kv[e] = *reinterpret_cast<const uint32_t*>(kp + i * a.ldk);
-            if (!STATE_ONLY) qv[e] = *reinterpret_cast<const uint32_t*>(qp + i * a.ldq);
-          }
+      for (int c = 0; c < 16; ++c) s[c] *= first;
+      if (!STATE_ONLY) {
 #pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const int i = g0 + e;
-            uint8_t* w = ch_addr(i);
-            if (i < n) {
-              if (i > 0) {
-                r.x += d[e].x;
-                r.y += d[e].y;
-              }
-              if (fminf(r.x, r.y) < -kMaxChannel && bad == kChunk) bad = i;
-              uint32_t lo;
-              if (!STATE_ONLY) {
-                *reinterpret_cast<uint32_t*>(w) = split2(bf16lo(qv[e]) * a.scale * ex2(r.x), bf16hi(qv[e]) * a.scale * ex2(r.y), lo);
-                *reinterpret_cast<uint32_t*>(w + kq) = lo;
-              }
-              *reinterpret_cast<uint32_t*>(w + 2 * kq) = split2(bf16lo(kv[e]) * ex2(-r.x), bf16hi(kv[e]) * ex2(-r.y), lo);
-              *reinterpret_cast<uint32_t*>(w + 3 * kq) = lo;
-              if (i == n - 1) *reinterpret_cast<float2*>(s_end + ch) = make_float2(ex2(r.x), ex2(r.y));
-            } else {
-              *reinterpret_cast<uint32_t*>(w + 2 * kq) = 0u;
-              *reinterpret_cast<uint32_t*>(w + 3 * kq) = 0u;
-            }
-          }
-        }
-        if (bad < kChunk) atomicMin(s_len + set, bad);
-      }
-    }
-    const float first = !compute ? 0.f : (CHANNEL ? s_first[row] : f->first);
-    uint32_t xraw[8];
-    if (compute) {
-      if (state_thread) {
-        uint8_t* dst = smem + off_s + row * 128;
-#pragma unroll
-        for (int c = 0; c < 16; ++c) s[c] *= first;
-        if (!STATE_ONLY) {
-#pragma unroll
-          for (int x = 0; x < 2; ++x) {
-            uint32_t hi[4], lo[4];
-#pragma unroll
-            for (int e = 0; e < 4; ++e) hi[e] = split2(s[8 * x + 2 * e], s[8 * x + 2 * e + 1], lo[e]);
-            const int o = ((quarter * 2 + x) ^ (row & 7)) << 4;
-            *reinterpret_cast<uint4*>(dst + o) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-            *reinterpret_cast<uint4*>(dst + s_bytes + o) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
-          }
-        }
-      }
-      wait_bar(bar_v + 8 * set, set_ph, 92);
-      uint8_t* vrow = smem + off_v + set * kBox + row * 128;
-      if constexpr (CHANNEL) {
-        if (row >= n) {  // another request's values, or none
-#pragma unroll
-          for (int x = 0; x < 2; ++x) *reinterpret_cast<uint4*>(vrow + ((quarter * 2 + x) << 4)) = make_uint4(0, 0, 0, 0);
-        }
-      } else {
-        const float w = f->x[row];
-        const bool in = row < n;
-        uint8_t* dst = smem + off_x + row * 128;
-#pragma unroll
-        for (int x = 0; x < 2; ++x) {
-          const int o = ((quarter * 2 + x) ^ (row & 7)) << 4;
-          uint4 v = make_uint4(0, 0, 0, 0);
-          if (in) v = *reinterpret_cast<const uint4*>(vrow + o);
-          else *reinterpret_cast<uint4*>(vrow + o) = v;  // another request's values, or none
-          xraw[4 * x] = v.x; xraw[4 * x + 1] = v.y; xraw[4 * x + 2] = v.z; xraw[4 * x + 3] = v.w;
+        for (int y = 0; y < 2; ++y) {
           uint32_t hi[4], lo[4];
 #pragma unroll
-          for (int e = 0; e < 4; ++e) hi[e] = split2(bf16lo(xraw[4 * x + e]) * w, bf16hi(xraw[4 * x + e]) * w, lo[e]);
+          for (int e = 0; e < 4; ++e) hi[e] = split2(s[8 * y + 2 * e], s[8 * y + 2 * e + 1], lo[e]);
+          const int o = ((quarter * 2 + y) ^ (row & 7)) << 4;
           *reinterpret_cast<uint4*>(dst + o) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-          *reinterpret_cast<uint4*>(dst + kBox + o) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+          *reinterpret_cast<uint4*>(dst + s_bytes + o) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
         }
       }
-      ptx::fence_proxy_async_smem();
     }
+    uint8_t* vrow = smem + off_v + set * kBox + row * 128;
+    const bool in = row < n;
+    if (!in) {  // another request's values, or none
+#pragma unroll
+      for (int y = 0; y < 2; ++y) *reinterpret_cast<uint4*>(vrow + (((quarter * 2 + y) ^ (row & 7)) << 4)) = make_uint4(0, 0, 0, 0);
+    }
+    if constexpr (!CHANNEL) {
+      const float w = f->x[row];
+      uint8_t* dst = smem + off_x + row * 128;
+#pragma unroll
+      for (int y = 0; y < 2; ++y) {
+        const int o = ((quarter * 2 + y) ^ (row & 7)) << 4;
+        uint4 v = make_uint4(0, 0, 0, 0);
+        if (in) v = *reinterpret_cast<const uint4*>(vrow + o);
+        x[4 * y] = v.x; x[4 * y + 1] = v.y; x[4 * y + 2] = v.z; x[4 * y + 3] = v.w;
+        uint32_t hi[4], lo[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) hi[e] = split2(bf16lo(x[4 * y + e]) * w, bf16hi(x[4 * y + e]) * w, lo[e]);
+        *reinterpret_cast<uint4*>(dst + o) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+        *reinterpret_cast<uint4*>(dst + kBox + o) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+      }
+    }
+    ptx::fence_proxy_async_smem();
+  };
+
+  uint32_t x_now[8], x_next[8];
+  if (issuer) {
+    load_v(0);
+    load_qk(0);
+    if (!STATE_ONLY && ptx::mbar_wait(bar_qk, 0, abort_flag, status, 91)) issue_scores(0);
+  }
+  __syncwarp();
+  if (compute) operands(0, x_now);
+  const int n_chunks = (t_end - t_begin + kChunk - 1) / kChunk;
+  for (int it = 0; it < n_chunks; ++it) {
+    const int t = t_begin + it * kChunk, n = min(kChunk, t_end - t);
+    const int set = it & 1, ph = it & 1;
+    const uint32_t col_p = tmem + set * kChunk;
+    const Factors* f = fac + set;
+    const int k_tok = (n + 15) / 16;  // steps of 16 tokens
+    const bool more = it + 1 < n_chunks;
     ptx::tc_fence_before();
     __syncthreads();
-    if constexpr (CHANNEL) {
-      len = s_len[set];
-      if (len < n) {  // the chunk ends early: later tokens' keys leave, and the decay of the rest is another one
-        if (prep) {
-          for (int i = max(len, i0); i < i0 + tp; ++i) {
-            uint8_t* w = ch_addr(i);
-            *reinterpret_cast<uint32_t*>(w + 2 * kq) = 0u;
-            *reinterpret_cast<uint32_t*>(w + 3 * kq) = 0u;
-          }
-        }
-        if (tid < a.dim) {
-          float r = 0.f;
-          for (int i = 1; i < len; ++i) r += g.log2_decay[(t + i) * ld_la + h * a.dim + tid];
-          s_end[tid] = ex2(r);
-        }
-        ptx::fence_proxy_async_smem();
-        ptx::tc_fence_before();
-        __syncthreads();
-      }
-    }
-    const int next = t + len;
-    const int k_tok = (len + 15) / 16;  // steps of 16 tokens
+    if (*abort_flag) break;
     if (issuer) {
       ptx::tc_fence_after();
       const uint32_t idesc_o = ptx::make_idesc(1u, 1u, kChunk, vb) | (1u << 16);  // B is MN-major
       const uint32_t idesc_s = idesc_o | (1u << 15);                              // A too
-      if (CHANNEL) {
-        if (next < t_end) load_v(next, set ^ 1);
-        if (!STATE_ONLY) issue_scores(col_p);
-      }
       if (!STATE_ONLY) {
         const uint64_t qd = ptx::smem_desc_sw128(base + off_q), qlo = qd + (kq >> 4);
         const uint64_t sd = ptx::smem_desc_sw128(base + off_s), slo = sd + (s_bytes >> 4);  // 64 columns: no leading offset
@@ -479,7 +488,7 @@ chunk_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUt
           ptx::mma_f16(col_in, qd + o, slo + so, idesc_o, 1u);
           if (CHANNEL) ptx::mma_f16(col_in, qlo + o, sd + so, idesc_o, 1u);
         }
-      } else if (!CHANNEL) {
+      } else {
         ptx::mbar_wait(bar_qk, ph, abort_flag, status, 96);
       }
       // A = K^T: rows of S by tokens, a second box of rows for more than 64 (else the first once more, unused)
@@ -493,19 +502,18 @@ chunk_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUt
         ptx::mma_f16(col_su, CHANNEL ? kt + (kq >> 4) + o : kt + o, CHANNEL ? ud + o : ud + kBox / 16 + o, idesc_s, 1u);
       }
       ptx::tc_commit(bar_su);
-      if (!CHANNEL && next < t_end) {  // the other v tile is free, those of q and k are with these products
-        load_v(next, set ^ 1);
-        if (ptx::mbar_wait(bar_su, ph, abort_flag, status, 97)) load_qk(next);
+      if (more) {  // the other v tile is free, those of q and k are with these products
+        load_v(it + 1);
+        if (ptx::mbar_wait(bar_su, ph, abort_flag, status, 97)) load_qk(it + 1);
       }
     }
-    if (!CHANNEL && factor_warp && next < t_end) head_factors(a, fac + (set ^ 1), next, min(kChunk, t_end - next), h);
     __syncwarp();
 
     // ---- P as two bf16 halves over the scores, 32 columns per thread: [16 hi | 16 lo] ------------------
     if (!STATE_ONLY) {
       if (compute) {
         wait_bar(bar_g, ph, 93);
-        if (quarter * 32 < len) {
+        if (quarter * 32 < n) {
           uint32_t p[32];
           if (quarter > (warp & 3)) {  // keys after every query of this warp
 #pragma unroll
@@ -513,7 +521,8 @@ chunk_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUt
           } else {
             uint32_t gv[32];
             ptx::tmem_ld_32x32(col_p + lane_off + quarter * 32, gv);
-            const float ri = CHANNEL ? 0.f : f->r[row];
+            float ri = 0.f;
+            if constexpr (!CHANNEL) ri = f->r[row];
             ptx::tmem_ld_wait();
 #pragma unroll
             for (int c4 = 0; c4 < 8; ++c4) {
@@ -524,8 +533,10 @@ chunk_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUt
                 const float4 cj = *reinterpret_cast<const float4*>(f->c + j);
                 v[0] *= ex2(ri + cj.x); v[1] *= ex2(ri + cj.y); v[2] *= ex2(ri + cj.z); v[3] *= ex2(ri + cj.w);
               }
+              if (quarter == (warp & 3)) {
 #pragma unroll
-              for (int e = 0; e < 4; ++e) v[e] = j + e <= row ? v[e] : 0.f;
+                for (int e = 0; e < 4; ++e) v[e] = j + e <= row ? v[e] : 0.f;
+              }
               p[2 * c4] = split2(v[0], v[1], p[16 + 2 * c4]);
               p[2 * c4 + 1] = split2(v[2], v[3], p[16 + 2 * c4 + 1]);
             }
@@ -547,40 +558,45 @@ chunk_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUt
           ptx::mma_f16_ts(col_pu, pc + 16, vd + k * 128u, idesc_o, 1u);
         }
         ptx::tc_commit(bar_o);
-        if (!CHANNEL && next < t_end && ptx::mbar_wait(bar_qk, ph ^ 1u, abort_flag, status, 98)) issue_scores(set == 0 ? col_p1 : tmem);
+        if (more && ptx::mbar_wait(bar_qk, ph ^ 1, abort_flag, status, 98)) issue_scores(it + 1);
       }
       __syncwarp();
     }
 
-    // ---- new state, output ---------------------------------------------------------------------------
+    // ---- new state, operands of the next chunk, output ------------------------------------------------
     if (compute) {
       wait_bar(bar_su, ph, 94);
       uint32_t v[16];
       ptx::tmem_ld_32x16(col_su + lane_off + col0, v);
       ptx::tmem_ld_wait();
       if (state_thread) {
-        const float end = CHANNEL ? s_end[row] : f->end;
+        float end;
+        if constexpr (CHANNEL) end = f->end[row];
+        else end = f->end;
 #pragma unroll
         for (int c = 0; c < 16; ++c)
           s[c] = CHANNEL ? end * (s[c] + __uint_as_float(v[c])) : fmaf(end, s[c], __uint_as_float(v[c]));
-        decay_all *= first * end;
+        decay_all *= end;
       }
+      __syncwarp();
+      if (more) operands(it + 1, x_next);
       if (!STATE_ONLY) {
+        wait_bar(bar_o, ph, 95);
         uint32_t y[16];
         if (!CHANNEL) ptx::tmem_ld_32x16(col_in + lane_off + col0, y);
-        wait_bar(bar_o, ph, 95);
         ptx::tmem_ld_32x16(col_pu + lane_off + col0, v);
         ptx::tmem_ld_wait();
-        if (row < len && my_cols) {
-          __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + (t + row) * a.ldo + h * a.vdim + c0 + col0;
-          const float er = CHANNEL ? 0.f : ex2(f->r[row]);
+        if (row < n && my_cols) {
+          __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + static_cast<int64_t>(t + row) * a.ldo + h * a.vdim + c0 + col0;
+          float er = 0.f;
+          if constexpr (!CHANNEL) er = ex2(f->r[row]);
           uint32_t w[8];
 #pragma unroll
           for (int e = 0; e < 8; ++e) {
             float y0 = __uint_as_float(v[2 * e]), y1 = __uint_as_float(v[2 * e + 1]);
             if (!CHANNEL) {
-              y0 = fmaf(skip, bf16lo(xraw[e]), a.scale * fmaf(er, __uint_as_float(y[2 * e]), y0));
-              y1 = fmaf(skip, bf16hi(xraw[e]), a.scale * fmaf(er, __uint_as_float(y[2 * e + 1]), y1));
+              y0 = fmaf(skip, bf16lo(x_now[e]), a.scale * fmaf(er, __uint_as_float(y[2 * e]), y0));
+              y1 = fmaf(skip, bf16hi(x_now[e]), a.scale * fmaf(er, __uint_as_float(y[2 * e + 1]), y1));
             }
             w[e] = pack_bf16(y0, y1);
           }
@@ -588,14 +604,10 @@ chunk_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUt
           *reinterpret_cast<uint4*>(out + 8) = make_uint4(w[4], w[5], w[6], w[7]);
         }
         __syncwarp();
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x_now[e] = x_next[e];
       }
-      ptx::tc_fence_before();
     }
-    if (CHANNEL && issuer) s_len[set ^ 1] = min(kChunk, t_end - next);
-    __syncthreads();
-    ptx::tc_fence_after();
-    if (*abort_flag) break;
-    t = next;
   }
 
   if (state_thread && my_cols) {
@@ -620,7 +632,7 @@ chunk_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUt
   }
   if (warp == kCompute / 32) {
     ptx::tc_fence_after();
-    ptx::tmem_dealloc(tmem, CHANNEL ? 256 : 512);
+    ptx::tmem_dealloc(tmem, 512);
   }
 }
 
@@ -631,6 +643,7 @@ static bool plan_chunks(const fr_linear_scan& a, int n_req, int longest, ChunkPl
   pl->boxes = (a.dim + 63) / 64;
   pl->v_blocks = ceil_div(a.vdim, kVb);
   pl->smem = 1024 + tile_smem(channel, pl->boxes, a.dim) + kTailSmem;
+  if (pl->smem < 116 * 1024) pl->smem = 116 * 1024;  // one CTA per SM owns all of TMEM
   if (pl->smem > 227 * 1024) return false;
   const int64_t units = static_cast<int64_t>(a.heads) * pl->v_blocks * (n_req > 0 ? n_req : 1);
   int want = static_cast<int>(device_sm_count() / units);  // segments of the longest request that fill the GPU
@@ -642,40 +655,65 @@ static bool plan_chunks(const fr_linear_scan& a, int n_req, int longest, ChunkPl
   pl->segs = ceil_div(longest, pl->seg_len);
   return true;
 }
-static int64_t state_scratch(const fr_linear_scan& a, const ChunkPlan& pl, int n_req) {
-  if (pl.segs <= 1) return 0;
-  const int64_t per = static_cast<int64_t>(a.dim) * state_cols(a.vdim);
-  return static_cast<int64_t>(n_req) * a.heads * (pl.segs * (per + a.dim) + per) * 4;
-}
-static int64_t decay_scratch(const fr_linear_scan& a, int n_tokens) {
-  return a.decay == FR_DECAY_CHANNEL ? static_cast<int64_t>(n_tokens) * a.heads * a.dim * 4 : 0;
+
+// The scratch buffer, in this order (bytes, every part a multiple of 16).
+struct ScratchPlan {
+  int64_t factors, qk, flags, seg_state, seg_decay, start_state;
+  int64_t total() const { return factors + qk + flags + seg_state + seg_decay + start_state; }
+};
+static ScratchPlan plan_scratch(const fr_linear_scan& a, const ChunkPlan& pl, int n_req, int n_tokens) {
+  ScratchPlan s{};
+  const bool channel = a.decay == FR_DECAY_CHANNEL;
+  const int64_t chunks = n_tokens / kChunk + n_req + 1, per = static_cast<int64_t>(a.dim) * state_cols(a.vdim);
+  s.factors = chunks * a.heads * static_cast<int64_t>(channel ? sizeof(ChannelFactors) : sizeof(HeadFactors));
+  if (channel) {
+    s.qk = static_cast<int64_t>(n_tokens) * a.heads * a.dim * 8;
+    s.flags = (static_cast<int64_t>(n_req) * a.heads * 4 + 15) / 16 * 16;
+  }
+  if (pl.segs > 1) {
+    s.seg_state = static_cast<int64_t>(n_req) * pl.segs * a.heads * per * 4;
+    s.seg_decay = static_cast<int64_t>(n_req) * pl.segs * a.heads * a.dim * 4;
+    s.start_state = static_cast<int64_t>(n_req) * a.heads * per * 4;
+  }
+  return s;
 }
 
 template <bool CHANNEL, bool STATE_ONLY>
-static int launch_chunks(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const ChunkArgs& g, int n_req, int n_segs,
-                         bool pdl, int* status, cudaStream_t stream) {
+static int launch_chunks(const ChunkMaps& maps, const ChunkArgs& g, int n_req, int n_segs, bool pdl, int* status, cudaStream_t stream) {
   static PerDeviceFlag f;
   if (ensure_dyn_smem(f, chunk_kernel<CHANNEL, STATE_ONLY>, 227 * 1024) != FR_OK) return FR_ERR_CUDA;
   return launch_kernel(chunk_kernel<CHANNEL, STATE_ONLY>, dim3(g.a.heads * g.pl.v_blocks, n_segs, n_req), kThreads, g.pl.smem, stream, pdl,
-                       tq, tk, tv, g, status);
+                       maps, g, status);
 }
 
 template <bool CHANNEL>
-static int run_chunks(const ChunkArgs& g, int n_req, int n_tokens, cudaStream_t stream) {
+static int run_chunks(const ChunkArgs& g, int n_req, int longest, int n_tokens, cudaStream_t stream) {
   const fr_linear_scan& a = g.a;
-  CUtensorMap tq, tk, tv;
-  int r = make_tmap_bf16_box64(&tv, a.v, static_cast<uint64_t>(a.heads) * a.vdim, n_tokens, a.ldv, kChunk);
-  if (r == FR_OK) r = make_tmap_bf16_box64(&tq, a.q, static_cast<uint64_t>(a.key_heads) * a.dim, n_tokens, a.ldq, kChunk);
-  if (r == FR_OK) r = make_tmap_bf16_box64(&tk, a.k, static_cast<uint64_t>(a.key_heads) * a.dim, n_tokens, a.ldk, kChunk);
+  ChunkMaps m;
+  const uint64_t cols = static_cast<uint64_t>(a.key_heads) * a.dim;
+  int r = make_tmap_bf16_box64(&m.v, a.v, static_cast<uint64_t>(a.heads) * a.vdim, n_tokens, a.ldv, kChunk);
+  CUtensorMap* qk[4] = {&m.q, &m.q_lo, &m.k, &m.k_lo};
+  for (int i = 0; i < 4 && r == FR_OK; ++i) {
+    const void* p = CHANNEL ? static_cast<const void*>(g.qk + i * g.qk_stride) : (i < 2 ? a.q : a.k);
+    r = make_tmap_bf16_box64(qk[i], p, cols, n_tokens, CHANNEL ? static_cast<int64_t>(cols) : (i < 2 ? a.ldq : a.ldk), kChunk);
+  }
   if (r != FR_OK) return r;
   int* status = device_status_ptr();
   if (!status) return FR_ERR_CUDA;
   const bool pdl = n_tokens <= kPdlRows;
-  if (g.pl.segs > 1) {
-    r = launch_chunks<CHANNEL, true>(tq, tk, tv, g, n_req, g.pl.segs - 1, pdl, status, stream);
-    if (r != FR_OK) return r;
+  const int chunks = ceil_div(longest, kChunk);
+  if (CHANNEL) {
+    const int smem = (kChunk * (a.dim + a.rank) + 2 * kPrepThreads) * 4;
+    FR_CHECK_SUPPORTED(smem <= 200 * 1024);
+    static PerDeviceFlag f;
+    if (ensure_dyn_smem(f, channel_factor_kernel, 200 * 1024) != FR_OK) return FR_ERR_CUDA;
+    if (cudaMemsetAsync(g.flags, 0, static_cast<size_t>(n_req) * a.heads * 4, stream) != cudaSuccess) return FR_ERR_CUDA;
+    r = launch_kernel(channel_factor_kernel, dim3(chunks, a.heads, n_req), kPrepThreads, smem, stream, false, g);
+  } else {
+    r = launch_kernel(head_factor_kernel, dim3(chunks, ceil_div(a.heads, kFactorHeads), n_req), kFactorHeads * 32, 0, stream, pdl, g);
   }
-  return launch_chunks<CHANNEL, false>(tq, tk, tv, g, n_req, g.pl.segs, pdl, status, stream);
+  if (r == FR_OK && g.pl.segs > 1) r = launch_chunks<CHANNEL, true>(m, g, n_req, g.pl.segs - 1, pdl, status, stream);
+  return r == FR_OK ? launch_chunks<CHANNEL, false>(m, g, n_req, g.pl.segs, pdl, status, stream) : r;
 }
 
 }  // namespace scan
@@ -696,7 +734,7 @@ extern "C" int fr_linear_scan_chunks_fit(int decay, int dim, int vdim) {
 extern "C" int64_t fr_linear_scan_chunks_scratch(const fr_linear_scan* a, int n_req, int longest, int n_tokens) {
   scan::ChunkPlan pl;
   if (a == nullptr || a->heads <= 0 || n_req <= 0 || longest <= 0 || n_tokens <= 0 || !scan::plan_chunks(*a, n_req, longest, &pl)) return -1;
-  return scan::decay_scratch(*a, n_tokens) + scan::state_scratch(*a, pl, n_req) + 16;
+  return scan::plan_scratch(*a, pl, n_req, n_tokens).total();
 }
 
 extern "C" int fr_linear_scan_chunks(const fr_linear_scan* a, int n_req, int longest, int n_tokens, int min_tokens, void* scratch,
@@ -709,22 +747,25 @@ extern "C" int fr_linear_scan_chunks(const fr_linear_scan* a, int n_req, int lon
   FR_CHECK_SUPPORTED(a->dtype == 0 && scan::plan_chunks(*a, n_req, longest, &g.pl));
   FR_CHECK_ARG(aligned16(a->q) && aligned16(a->k) && aligned16(a->v) && aligned16(a->out) && a->ldq % 8 == 0 && a->ldk % 8 == 0 &&
                a->ldv % 8 == 0 && a->ldo % 8 == 0);
-  FR_CHECK_ARG(scratch && aligned16(scratch) && scratch_bytes >= fr_linear_scan_chunks_scratch(a, n_req, longest, n_tokens));
+  const scan::ScratchPlan sp = scan::plan_scratch(*a, g.pl, n_req, n_tokens);
+  FR_CHECK_ARG(scratch && aligned16(scratch) && scratch_bytes >= sp.total());
   g.a = *a;
   g.min_tokens = min_tokens;
-  float* p = static_cast<float*>(scratch);
-  if (a->decay == FR_DECAY_CHANNEL) {
-    const int smem = scan::kDecayTokens * a->rank * 4;
-    FR_CHECK_SUPPORTED(smem <= 48 * 1024);
-    g.log2_decay = p;
-    const int r = launch_kernel(scan::log_decay_kernel, dim3(ceil_div(n_tokens, scan::kDecayTokens), ceil_div(a->heads * a->dim, 256)), 256,
-                                smem, stream, n_tokens <= kPdlRows, *a, n_tokens, p);
-    if (r != FR_OK) return r;
-    p += scan::decay_scratch(*a, n_tokens) / 4;
-  }
-  const int64_t per = static_cast<int64_t>(a->dim) * scan::state_cols(a->vdim);
-  g.seg_state = p;
-  g.start_state = p + static_cast<int64_t>(n_req) * a->heads * g.pl.segs * per;
-  g.seg_decay = g.start_state + static_cast<int64_t>(n_req) * a->heads * per;
-  return a->decay == FR_DECAY_CHANNEL ? scan::run_chunks<true>(g, n_req, n_tokens, stream) : scan::run_chunks<false>(g, n_req, n_tokens, stream);
+  uint8_t* p = static_cast<uint8_t*>(scratch);
+  auto take = [&](int64_t bytes) {
+    uint8_t* at = p;
+    p += bytes;
+    return at;
+  };
+  g.factors = take(sp.factors);
+  g.qk = reinterpret_cast<__nv_bfloat16*>(take(sp.qk));
+  g.qk_stride = sp.qk / 8;
+  g.flags = reinterpret_cast<int32_t*>(take(sp.flags));
+  g.seg_state = reinterpret_cast<float*>(take(sp.seg_state));
+  g.seg_decay = reinterpret_cast<float*>(take(sp.seg_decay));
+  g.start_state = reinterpret_cast<float*>(take(sp.start_state));
+  if (a->decay == FR_DECAY_HEAD) return scan::run_chunks<false>(g, n_req, longest, n_tokens, stream);
+  const int r = scan::run_chunks<true>(g, n_req, longest, n_tokens, stream);
+  // what was flagged, token by token (nothing in the usual case: the CTAs look at the flag and leave)
+  return r == FR_OK ? scan::rows_flagged(*a, n_req, min_tokens, g.flags, stream) : r;
 }

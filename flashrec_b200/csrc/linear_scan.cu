@@ -52,7 +52,8 @@ struct RowsPlan {
 
 template <typename T, bool CHANNEL>
 __global__ void __launch_bounds__(1024)
-scan_rows_kernel(const __grid_constant__ fr_linear_scan a, const RowsPlan pl, int max_tokens) {
+scan_rows_kernel(const __grid_constant__ fr_linear_scan a, const RowsPlan pl, int min_tokens, int max_tokens,
+                 const int32_t* __restrict__ flags) {
   extern __shared__ __align__(16) float sm[];
   const int np = state_rows(a.dim), vp = state_cols(a.vdim);
   const int rg_n = np / kRows, cq_n = pl.vb / kCols;
@@ -65,7 +66,8 @@ scan_rows_kernel(const __grid_constant__ fr_linear_scan a, const RowsPlan pl, in
   ptx::griddep_launch_dependents();
   const int b = blockIdx.z, h = blockIdx.y, c0 = blockIdx.x * pl.vb, tid = threadIdx.x, nt = blockDim.x;
   const int q0 = a.qo_indptr[b], q1 = a.qo_indptr[b + 1];
-  if (q0 >= q1 || q1 - q0 > max_tokens) return;
+  if (q0 >= q1 || q1 - q0 > max_tokens || q1 - q0 < min_tokens) return;
+  if (flags != nullptr && flags[b * a.heads + h] == 0) return;
   const int kh = h / (a.heads / a.key_heads);
   const int cq = tid % cq_n, rg = tid / cq_n;
   const bool active = rg < rg_n;
@@ -180,13 +182,18 @@ static bool plan_rows(const fr_linear_scan& a, int max_tokens, RowsPlan* pl) {
 }
 
 template <typename T, bool CHANNEL>
-static int launch_rows(const fr_linear_scan& a, int n_req, int max_tokens, bool pdl, cudaStream_t stream) {
+static int launch_rows(const fr_linear_scan& a, int n_req, int min_tokens, int max_tokens, const int32_t* flags, bool pdl,
+                       cudaStream_t stream) {
   RowsPlan pl;
   FR_CHECK_SUPPORTED(plan_rows(a, max_tokens, &pl));
   static PerDeviceFlag f;
   if (ensure_dyn_smem(f, scan_rows_kernel<T, CHANNEL>, 200 * 1024) != FR_OK) return FR_ERR_CUDA;
   return launch_kernel(scan_rows_kernel<T, CHANNEL>, dim3(state_cols(a.vdim) / pl.vb, a.heads, n_req), pl.threads, pl.smem, stream, pdl,
-                       a, pl, max_tokens);
+                       a, pl, min_tokens, max_tokens, flags);
+}
+
+int rows_flagged(const fr_linear_scan& a, int n_req, int min_tokens, const int32_t* flags, cudaStream_t stream) {
+  return launch_rows<__nv_bfloat16, true>(a, n_req, min_tokens, INT32_MAX, flags, false, stream);
 }
 
 }  // namespace scan
@@ -205,8 +212,8 @@ extern "C" int fr_linear_scan_rows(const fr_linear_scan* a, int n_req, int max_t
   if (n_req == 0 || max_tokens == 0) return FR_OK;
   const bool pdl = n_tokens <= kPdlRows;
   if (a->decay == FR_DECAY_CHANNEL)
-    return a->dtype == 0 ? scan::launch_rows<__nv_bfloat16, true>(*a, n_req, max_tokens, pdl, stream)
-                         : scan::launch_rows<float, true>(*a, n_req, max_tokens, pdl, stream);
-  return a->dtype == 0 ? scan::launch_rows<__nv_bfloat16, false>(*a, n_req, max_tokens, pdl, stream)
-                       : scan::launch_rows<float, false>(*a, n_req, max_tokens, pdl, stream);
+    return a->dtype == 0 ? scan::launch_rows<__nv_bfloat16, true>(*a, n_req, 1, max_tokens, nullptr, pdl, stream)
+                         : scan::launch_rows<float, true>(*a, n_req, 1, max_tokens, nullptr, pdl, stream);
+  return a->dtype == 0 ? scan::launch_rows<__nv_bfloat16, false>(*a, n_req, 1, max_tokens, nullptr, pdl, stream)
+                       : scan::launch_rows<float, false>(*a, n_req, 1, max_tokens, nullptr, pdl, stream);
 }

@@ -30,6 +30,9 @@ __device__ __forceinline__ float head_step(const fr_linear_scan& a, int64_t t, i
   return softplus(a.step[t * a.ldstep + h] + a.step_bias[h]);
 }
 
+// linear_scan.cu: the heads [request, head] with a flag, of requests of at least min_tokens tokens (bf16, decay per channel)
+int rows_flagged(const fr_linear_scan& a, int n_req, int min_tokens, const int32_t* flags, cudaStream_t stream);
+
 static inline int check_args(const fr_linear_scan* a) {
   FR_CHECK_ARG(a && (a->dtype == 0 || a->dtype == 1) && (a->decay == FR_DECAY_CHANNEL || a->decay == FR_DECAY_HEAD));
   FR_CHECK_ARG(a->heads > 0 && a->heads <= 65535 && a->key_heads > 0 && a->heads % a->key_heads == 0 && a->dim > 0 && a->vdim > 0);

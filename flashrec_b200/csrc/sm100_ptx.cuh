@@ -103,6 +103,13 @@ __device__ __forceinline__ void tma_load_3d(uint32_t dst_smem, const CUtensorMap
       : "memory");
 }
 
+// Untiled bulk copy global -> shared; both addresses and the size are multiples of 16 bytes.
+__device__ __forceinline__ void bulk_load(uint32_t dst_smem, const void* src, uint32_t bytes, uint32_t bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst_smem),
+               "l"(reinterpret_cast<uint64_t>(src)), "r"(bytes), "r"(bar)
+               : "memory");
+}
+
 // 2-D TMA tile store shared -> global (bulk async group of the issuing thread). Out-of-range
 // parts of the box are clipped by the hardware; c0 * elemsize must be a multiple of 16 bytes and
 // neither coordinate may be negative.
