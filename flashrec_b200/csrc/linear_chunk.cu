@@ -17,7 +17,7 @@
 //   channel_factor_kernel  decay per channel: the low-rank decays, q~ and k~ of every chunk and head
 //   chunk_kernel           one CTA: one head, up to 64 columns of V and S, one segment of a request, chunk after chunk. S
 //                          lives in registers (thread = row of S and a quarter of the columns). Warps 0..15 work on
-//                          operands, mask, state and output; warp 16 issues TMA and tcgen05.mma. Scores, tiles and
+//                          operands, mask, state and output, warp 16 issues tcgen05.mma, warp 17 TMA. Scores, tiles and
 //                          operands are one chunk ahead of the output.
 //
 // Long prompts are cut into segments that run side by side: a first launch finds the state that each segment adds and its
@@ -38,7 +38,7 @@ constexpr int kChunk = 128;            // tokens (UMMA M)
 constexpr int kVb = 64;                // columns of V per CTA: one swizzle span
 constexpr int kBox = kChunk * 128;     // bytes of a [128 x 64] bf16 tile
 constexpr int kCompute = 512;          // threads of the compute warps
-constexpr int kThreads = kCompute + 32;
+constexpr int kThreads = kCompute + 64;
 constexpr float kLog2e = 1.4426950408889634f;
 // largest -r_last (in powers of two) per channel: e^(+-r_last / 2), its products and their sums stay far inside 2^+-126
 constexpr float kMaxChannel = 160.f;
@@ -54,12 +54,21 @@ __device__ __forceinline__ uint32_t split2(float a, float b, uint32_t& lo) {
   lo = pack_bf16(a - bf16lo(hi), b - bf16hi(hi));
   return hi;
 }
+__device__ __forceinline__ uint32_t split2(uint64_t v, uint32_t& lo) {
+  float a, b;
+  unpack2(v, a, b);
+  const uint32_t hi = pack_bf16(a, b);
+  unpack2(fma2(pack2(bf16lo(hi), bf16hi(hi)), dup2(-1.0f), v), a, b);
+  lo = pack_bf16(a, b);
+  return hi;
+}
 
 // Factors of one chunk and head.
 struct HeadFactors {
   float r[kChunk];    // r_i (log2)
   float c[kChunk];    // log2(step_j) - r_j
   float x[kChunk];    // step_j e^(r_last - r_j)
+  float y[kChunk];    // step_j e^(r_e - r_j), e the last of j's block of 32 tokens
   float first, end;   // a_0, e^(r_last)
   float pad_[2];
 };
@@ -125,17 +134,20 @@ head_factor_kernel(const __grid_constant__ ChunkArgs g) {
     if (lane >= o) x += y;
   }
   const float last = __shfl_sync(0xffffffffu, x, 31);
-  float r = x - sum, fr[4], fc[4], fx[4];
+  float r = x - sum, fr[4], fc[4], fx[4], fy[4];
+  const float block_end = __shfl_sync(0xffffffffu, x, lane | 7);
 #pragma unroll
   for (int e = 0; e < 4; ++e) {
     r += la[e];
     fr[e] = r;
     fc[e] = log2f(step[e]) - r;  // -inf past the end: no weight
     fx[e] = step[e] * ex2(last - r);
+    fy[e] = step[e] * ex2(block_end - r);
   }
   *reinterpret_cast<float4*>(f->r + lane * 4) = make_float4(fr[0], fr[1], fr[2], fr[3]);
   *reinterpret_cast<float4*>(f->c + lane * 4) = make_float4(fc[0], fc[1], fc[2], fc[3]);
   *reinterpret_cast<float4*>(f->x + lane * 4) = make_float4(fx[0], fx[1], fx[2], fx[3]);
+  *reinterpret_cast<float4*>(f->y + lane * 4) = make_float4(fy[0], fy[1], fy[2], fy[3]);
   if (lane == 0) *reinterpret_cast<float4*>(&f->first) = make_float4(first, ex2(last), 0.f, 0.f);
 }
 
@@ -150,8 +162,9 @@ channel_factor_kernel(const __grid_constant__ ChunkArgs g) {
   while (parts * 2 * pairs <= kPrepThreads && parts < 32) parts *= 2;
   const int tp = kChunk / parts;
   float* s_la = sm;                         // [128][dim]
-  float* s_low = s_la + kChunk * a.dim;     // [128][rank]
+  float* s_low = s_la + kChunk * a.dim;     // [rank][128]
   float* s_part = s_low + kChunk * a.rank;  // [parts][dim]
+  float* s_up = s_part + 2 * kPrepThreads;  // [rank][dim]
   ptx::griddep_wait();
   ptx::griddep_launch_dependents();
   const int b = blockIdx.z, h = blockIdx.y, tid = threadIdx.x;
@@ -159,13 +172,17 @@ channel_factor_kernel(const __grid_constant__ ChunkArgs g) {
   const int t = q0 + blockIdx.x * kChunk;
   if (t >= q1) return;
   const int n = min(kChunk, q1 - t);
-  for (int e = tid; e < n * a.rank; e += kPrepThreads) s_low[e] = a.step[static_cast<int64_t>(t + e / a.rank) * a.ldstep + e % a.rank];
+  for (int e = tid; e < kChunk * a.rank; e += kPrepThreads) {
+    const int i = e / a.rank, c = e % a.rank;
+    s_low[c * kChunk + i] = i < n ? a.step[static_cast<int64_t>(t + i) * a.ldstep + c] : 0.f;
+  }
+  for (int e = tid; e < a.dim * a.rank; e += kPrepThreads)
+    s_up[e % a.rank * a.dim + e / a.rank] = a.up[static_cast<int64_t>(h) * a.dim * a.rank + e];
   __syncthreads();
   const int part = tid / pairs, ch = 2 * (tid % pairs), i0 = part * tp, i1 = min(n, i0 + tp);
   const bool live = part < parts;
   if (live) {
     const int hc = h * a.dim + ch;
-    const float* up = a.up + static_cast<int64_t>(hc) * a.rank;
     const float b0 = a.step_bias[hc], b1 = a.step_bias[hc + 1], f = -a.inv_tau * kLog2e;
     float2 sum = make_float2(0.f, 0.f);
     for (int i = i0; i < i1; i += 4) {
@@ -176,12 +193,13 @@ channel_factor_kernel(const __grid_constant__ ChunkArgs g) {
         z1[e] = b1;
       }
       for (int r = 0; r < a.rank; ++r) {
-        const float u0 = up[r], u1 = up[a.rank + r];
+        const float2 u = *reinterpret_cast<const float2*>(s_up + r * a.dim + ch);
+        const float4 l4 = *reinterpret_cast<const float4*>(s_low + r * kChunk + i);
+        const float low[4] = {l4.x, l4.y, l4.z, l4.w};
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const float low = s_low[min(i + e, n - 1) * a.rank + r];
-          z0[e] = fmaf(u0, low, z0[e]);
-          z1[e] = fmaf(u1, low, z1[e]);
+          z0[e] = fmaf(u.x, low[e], z0[e]);
+          z1[e] = fmaf(u.y, low[e], z1[e]);
         }
       }
 #pragma unroll
@@ -242,9 +260,10 @@ channel_factor_kernel(const __grid_constant__ ChunkArgs g) {
 }
 
 // ---------------------------------------------------------------------------
-// Shared memory: tiles of q and k (CHANNEL: hi and lo each), two of v, S' hi and lo, HEAD: scaled v hi and lo; factors.
+// Shared memory: tiles of q and k (CHANNEL: hi and lo each), kSets of v, S' hi and lo, HEAD: scaled v hi and lo; factors.
+constexpr int kSets = 3;
 __host__ __device__ __forceinline__ int tile_smem(bool channel, int boxes, int dim) {
-  return (channel ? 4 : 2) * boxes * kBox + 2 * kBox + (channel ? 0 : 2 * kBox) + 2 * dim * 128;
+  return (channel ? 4 : 2) * boxes * kBox + kSets * kBox + (channel ? 0 : 2 * kBox) + 2 * dim * 128;
 }
 template <bool CHANNEL>
 struct FactorsOf {
@@ -254,11 +273,11 @@ template <>
 struct FactorsOf<true> {
   using type = ChannelFactors;
 };
-constexpr int kTailSmem = 2 * static_cast<int>(sizeof(HeadFactors)) + 128;
+constexpr int kTailSmem = kSets * static_cast<int>(sizeof(HeadFactors)) + 128;
 static_assert(sizeof(HeadFactors) % 16 == 0 && sizeof(ChannelFactors) % 16 == 0 && sizeof(ChannelFactors) <= sizeof(HeadFactors));
 
 struct ChunkMaps {
-  CUtensorMap v, q, k, q_lo, k_lo;
+  CUtensorMap v, q, k, q_lo, k_lo, out;
 };
 
 template <bool CHANNEL, bool STATE_ONLY>
@@ -273,19 +292,19 @@ chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ Chu
   const ChunkPlan& pl = g.pl;
   const int kq = pl.boxes * kBox;
   const uint32_t off_q = 0, off_k = (CHANNEL ? 2u : 1u) * kq;  // CHANNEL: hi, lo
-  const uint32_t off_v = 2u * off_k;                           // two tiles
-  const uint32_t off_x = off_v + 2u * kBox;                    // HEAD: scaled v hi, lo
+  const uint32_t off_v = 2u * off_k;                           // kSets tiles; a full chunk's output takes its v's place
+  const uint32_t off_x = off_v + kSets * kBox;                 // HEAD: scaled v hi, lo
   const uint32_t off_s = CHANNEL ? off_x : off_x + 2u * kBox;
   const uint32_t s_bytes = a.dim * 128;
   Factors* fac = reinterpret_cast<Factors*>(smem + off_s + 2 * s_bytes);
-  uint64_t* bars = reinterpret_cast<uint64_t*>(fac + 2);
-  const uint32_t bar_v = ptx::smem_u32(bars);          // [2]
-  const uint32_t bar_qk = bar_v + 16, bar_g = bar_v + 24, bar_su = bar_v + 32, bar_o = bar_v + 40;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 6);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(fac + kSets);
+  const uint32_t bar_v = ptx::smem_u32(bars);          // [kSets]
+  const uint32_t bar_qk = bar_v + 8 * kSets, bar_g = bar_qk + 8, bar_su = bar_qk + 16, bar_o = bar_qk + 24;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + kSets + 4);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const bool compute = tid < kCompute, issuer = tid == kCompute;
+  const bool compute = tid < kCompute, issuer = tid == kCompute, loader = tid == kCompute + 32;
   ptx::griddep_wait();
   const int h = blockIdx.x / pl.v_blocks, c0 = (blockIdx.x % pl.v_blocks) * kVb;
   const int b = blockIdx.z, seg = blockIdx.y;
@@ -300,7 +319,7 @@ chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ Chu
   const int vp = state_cols(a.vdim);
 
   if (tid == 0) {
-    for (int i = 0; i < 6; ++i) ptx::mbar_init(bar_v + 8 * i, 1);
+    for (int i = 0; i < kSets + 4; ++i) ptx::mbar_init(bar_v + 8 * i, 1);
     *abort_flag = 0;
     ptx::mbar_init_fence();
     ptx::prefetch_tmap(&maps.v);
@@ -322,9 +341,9 @@ chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ Chu
   const uint32_t lane_off = static_cast<uint32_t>((warp & 3) * 32) << 16;
   const Factors* factors = static_cast<const Factors*>(g.factors) + (first_chunk(q0, b) + seg * (pl.seg_len / kChunk)) * a.heads + h;
 
-  // ---- one thread: TMA and tcgen05.mma -----------------------------------------------------------------
+  // ---- TMA and tcgen05.mma, one thread each --------------------------------------------------------------
   auto load_v = [&](int it) {
-    const int set = it & 1;
+    const int set = it % kSets;
     ptx::mbar_expect_tx(bar_v + 8 * set, kBox + sizeof(Factors));
     ptx::tma_load_2d(base + off_v + set * kBox, &maps.v, h * a.vdim + c0, t_begin + it * kChunk, bar_v + 8 * set);
     ptx::bulk_load(ptx::smem_u32(fac + set), factors + static_cast<int64_t>(it) * a.heads, sizeof(Factors), bar_v + 8 * set);
@@ -407,8 +426,8 @@ chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ Chu
 
   // Operands of a chunk: S' over the old state and its halves, scaled values; `x` keeps the raw values.
   auto operands = [&](int it, uint32_t (&x)[8]) {
-    const int n = min(kChunk, t_end - (t_begin + it * kChunk)), set = it & 1;
-    wait_bar(bar_v + 8 * set, (it >> 1) & 1, 92);
+    const int n = min(kChunk, t_end - (t_begin + it * kChunk)), set = it % kSets;
+    wait_bar(bar_v + 8 * set, (it / kSets) & 1, 92);
     const Factors* f = fac + set;
     if (state_thread) {
       float first;
@@ -455,25 +474,47 @@ chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ Chu
     ptx::fence_proxy_async_smem();
   };
 
+  const int n_chunks = (t_end - t_begin + kChunk - 1) / kChunk;
+  // A full chunk's output tile leaves by TMA (a partial one must not touch the rows or columns beside it).
+  auto full_tile = [&](int it) { return !STATE_ONLY && vb == kVb && t_end - (t_begin + it * kChunk) >= kChunk; };
+  auto store_tile = [&](int it) {
+    ptx::tma_store_2d(&maps.out, base + off_v + (it % kSets) * kBox, h * a.vdim + c0, t_begin + it * kChunk);
+    ptx::bulk_commit();
+  };
   uint32_t x_now[8], x_next[8];
-  if (issuer) {
+  if (loader) {
     load_v(0);
     load_qk(0);
-    if (!STATE_ONLY && ptx::mbar_wait(bar_qk, 0, abort_flag, status, 91)) issue_scores(0);
+    if (n_chunks > 1) load_v(1);
   }
   __syncwarp();
+  if (issuer && !STATE_ONLY && ptx::mbar_wait(bar_qk, 0, abort_flag, status, 91)) issue_scores(0);
+  __syncwarp();
   if (compute) operands(0, x_now);
-  const int n_chunks = (t_end - t_begin + kChunk - 1) / kChunk;
   for (int it = 0; it < n_chunks; ++it) {
     const int t = t_begin + it * kChunk, n = min(kChunk, t_end - t);
-    const int set = it & 1, ph = it & 1;
-    const uint32_t col_p = tmem + set * kChunk;
+    const int set = it % kSets, ph = it & 1;
+    const uint32_t col_p = tmem + ph * kChunk;
     const Factors* f = fac + set;
     const int k_tok = (n + 15) / 16;  // steps of 16 tokens
     const bool more = it + 1 < n_chunks;
     ptx::tc_fence_before();
     __syncthreads();
     if (*abort_flag) break;
+    if (warp == kCompute / 32 + 1) {
+      if (loader) {
+        if (it > 0 && full_tile(it - 1)) store_tile(it - 1);
+        if (more && ptx::mbar_wait(bar_su, ph, abort_flag, status, 97)) {  // q's and k's tiles are free
+          load_qk(it + 1);
+          if (it + 2 < n_chunks) {  // and the v tile of the chunk before, once its output has left
+            ptx::bulk_wait_read<0>();
+            load_v(it + 2);
+          }
+        }
+      }
+      __syncwarp();
+      continue;
+    }
     if (issuer) {
       ptx::tc_fence_after();
       const uint32_t idesc_o = ptx::make_idesc(1u, 1u, kChunk, vb) | (1u << 16);  // B is MN-major
@@ -502,10 +543,6 @@ chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ Chu
         ptx::mma_f16(col_su, CHANNEL ? kt + (kq >> 4) + o : kt + o, CHANNEL ? ud + o : ud + kBox / 16 + o, idesc_s, 1u);
       }
       ptx::tc_commit(bar_su);
-      if (more) {  // the other v tile is free, those of q and k are with these products
-        load_v(it + 1);
-        if (ptx::mbar_wait(bar_su, ph, abort_flag, status, 97)) load_qk(it + 1);
-      }
     }
     __syncwarp();
 
@@ -518,6 +555,24 @@ chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ Chu
           if (quarter > (warp & 3)) {  // keys after every query of this warp
 #pragma unroll
             for (int c = 0; c < 32; ++c) p[c] = 0u;
+          } else if (quarter < (warp & 3)) {  // before every query: e^(r_i - r_j) in two factors, both at most one
+            uint32_t gv[32];
+            ptx::tmem_ld_32x32(col_p + lane_off + quarter * 32, gv);
+            uint64_t ai = 0;
+            if constexpr (!CHANNEL) ai = dup2(ex2(f->r[row] - f->r[quarter * 32 + 31]));
+            ptx::tmem_ld_wait();
+#pragma unroll
+            for (int c4 = 0; c4 < 8; ++c4) {
+              uint64_t v0 = pack2(__uint_as_float(gv[4 * c4]), __uint_as_float(gv[4 * c4 + 1]));
+              uint64_t v1 = pack2(__uint_as_float(gv[4 * c4 + 2]), __uint_as_float(gv[4 * c4 + 3]));
+              if constexpr (!CHANNEL) {
+                const ulonglong2 yj = *reinterpret_cast<const ulonglong2*>(f->y + quarter * 32 + 4 * c4);
+                v0 = mul2(mul2(v0, yj.x), ai);
+                v1 = mul2(mul2(v1, yj.y), ai);
+              }
+              p[2 * c4] = split2(v0, p[16 + 2 * c4]);
+              p[2 * c4 + 1] = split2(v1, p[16 + 2 * c4 + 1]);
+            }
           } else {
             uint32_t gv[32];
             ptx::tmem_ld_32x32(col_p + lane_off + quarter * 32, gv);
@@ -533,10 +588,8 @@ chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ Chu
                 const float4 cj = *reinterpret_cast<const float4*>(f->c + j);
                 v[0] *= ex2(ri + cj.x); v[1] *= ex2(ri + cj.y); v[2] *= ex2(ri + cj.z); v[3] *= ex2(ri + cj.w);
               }
-              if (quarter == (warp & 3)) {
 #pragma unroll
-                for (int e = 0; e < 4; ++e) v[e] = j + e <= row ? v[e] : 0.f;
-              }
+              for (int e = 0; e < 4; ++e) v[e] = j + e <= row ? v[e] : 0.f;
               p[2 * c4] = split2(v[0], v[1], p[16 + 2 * c4]);
               p[2 * c4 + 1] = split2(v[2], v[3], p[16 + 2 * c4 + 1]);
             }
@@ -546,7 +599,7 @@ chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ Chu
         }
         ptx::tc_fence_before();
       }
-      __syncthreads();
+      asm volatile("bar.sync 1, %0;" ::"n"(kCompute + 32) : "memory");  // all but the loader's warp
       if (issuer) {
         ptx::tc_fence_after();
         const uint32_t idesc_o = ptx::make_idesc(1u, 1u, kChunk, vb) | (1u << 16);
@@ -587,6 +640,8 @@ chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ Chu
         ptx::tmem_ld_32x16(col_pu + lane_off + col0, v);
         ptx::tmem_ld_wait();
         if (row < n && my_cols) {
+          const bool tile = full_tile(it);
+          uint8_t* stage = smem + off_v + set * kBox + row * 128;
           __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + static_cast<int64_t>(t + row) * a.ldo + h * a.vdim + c0 + col0;
           float er = 0.f;
           if constexpr (!CHANNEL) er = ex2(f->r[row]);
@@ -600,8 +655,11 @@ chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ Chu
             }
             w[e] = pack_bf16(y0, y1);
           }
-          *reinterpret_cast<uint4*>(out) = make_uint4(w[0], w[1], w[2], w[3]);
-          *reinterpret_cast<uint4*>(out + 8) = make_uint4(w[4], w[5], w[6], w[7]);
+          *reinterpret_cast<uint4*>(tile ? stage + (((quarter * 2) ^ (row & 7)) << 4) : reinterpret_cast<uint8_t*>(out)) =
+              make_uint4(w[0], w[1], w[2], w[3]);
+          *reinterpret_cast<uint4*>(tile ? stage + (((quarter * 2 + 1) ^ (row & 7)) << 4) : reinterpret_cast<uint8_t*>(out + 8)) =
+              make_uint4(w[4], w[5], w[6], w[7]);
+          ptx::fence_proxy_async_smem();
         }
         __syncwarp();
 #pragma unroll
@@ -626,6 +684,10 @@ chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ Chu
   }
   ptx::tc_fence_before();
   __syncthreads();
+  if (loader) {
+    if (!*abort_flag && full_tile(n_chunks - 1)) store_tile(n_chunks - 1);
+    ptx::bulk_wait_all();
+  }
   if (*abort_flag) {
     for (int i = 0; i < 200; ++i) __nanosleep(1000);
     __syncthreads();
@@ -692,6 +754,7 @@ static int run_chunks(const ChunkArgs& g, int n_req, int longest, int n_tokens, 
   ChunkMaps m;
   const uint64_t cols = static_cast<uint64_t>(a.key_heads) * a.dim;
   int r = make_tmap_bf16_box64(&m.v, a.v, static_cast<uint64_t>(a.heads) * a.vdim, n_tokens, a.ldv, kChunk);
+  if (r == FR_OK) r = make_tmap_bf16_box64(&m.out, a.out, static_cast<uint64_t>(a.heads) * a.vdim, n_tokens, a.ldo, kChunk);
   CUtensorMap* qk[4] = {&m.q, &m.q_lo, &m.k, &m.k_lo};
   for (int i = 0; i < 4 && r == FR_OK; ++i) {
     const void* p = CHANNEL ? static_cast<const void*>(g.qk + i * g.qk_stride) : (i < 2 ? a.q : a.k);
@@ -703,7 +766,7 @@ static int run_chunks(const ChunkArgs& g, int n_req, int longest, int n_tokens, 
   const bool pdl = n_tokens <= kPdlRows;
   const int chunks = ceil_div(longest, kChunk);
   if (CHANNEL) {
-    const int smem = (kChunk * (a.dim + a.rank) + 2 * kPrepThreads) * 4;
+    const int smem = (kChunk * (a.dim + a.rank) + 2 * kPrepThreads + a.rank * a.dim) * 4;
     FR_CHECK_SUPPORTED(smem <= 200 * 1024);
     static PerDeviceFlag f;
     if (ensure_dyn_smem(f, channel_factor_kernel, 200 * 1024) != FR_OK) return FR_ERR_CUDA;

@@ -19,30 +19,6 @@ namespace scan {
 constexpr int kRows = 8;  // rows of S per thread
 constexpr int kCols = 4;  // columns of S per thread
 
-__device__ __forceinline__ uint64_t dup2(float v) {
-  uint64_t d;
-  asm("mov.b64 %0, {%1, %1};" : "=l"(d) : "f"(v));
-  return d;
-}
-__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
-  uint64_t d;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-  return d;
-}
-__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
-  uint64_t d;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-  return d;
-}
-__device__ __forceinline__ uint64_t pack2(float lo, float hi) {
-  uint64_t d;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
-  return d;
-}
-__device__ __forceinline__ void unpack2(uint64_t v, float& lo, float& hi) {
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
-}
-
 struct RowsPlan {
   int vb;       // columns of S per CTA
   int tb;       // tokens staged at a time
