@@ -276,6 +276,26 @@ struct FactorsOf<true> {
 constexpr int kTailSmem = kSets * static_cast<int>(sizeof(HeadFactors)) + 128;
 static_assert(sizeof(HeadFactors) % 16 == 0 && sizeof(ChannelFactors) % 16 == 0 && sizeof(ChannelFactors) <= sizeof(HeadFactors));
 
+// f(0), .. f(n - 1), unrolled for the usual numbers of steps (the products are short: issuing them would pace the tensor
+// cores)
+template <class F>
+__device__ __forceinline__ void steps(int n, F&& f) {
+  if (n == 8) {
+#pragma unroll
+    for (int k = 0; k < 8; ++k) f(k);
+  } else if (n == 4) {
+#pragma unroll
+    for (int k = 0; k < 4; ++k) f(k);
+  } else {
+#pragma unroll 1
+    for (int k = 0; k < n; ++k) f(k);
+  }
+}
+// MN-major operand of 64-value blocks that are `lead` bytes apart
+__device__ __forceinline__ uint64_t desc_mn(uint32_t addr, uint32_t lead) {
+  return (ptx::smem_desc_sw128(addr) & ~(static_cast<uint64_t>(0x3fffu) << 16)) | static_cast<uint64_t>((lead >> 4) & 0x3fffu) << 16;
+}
+
 struct ChunkMaps {
   CUtensorMap v, q, k, q_lo, k_lo, out;
 };
@@ -336,8 +356,8 @@ chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ Chu
   ptx::tc_fence_after();
   ptx::griddep_launch_dependents();  // not before the tensor memory is taken
   const uint32_t tmem = *tmem_slot;
-  // scores and P (two sets of 128 columns), Q S', K^T U, P U (CHANNEL: added to Q S')
-  const uint32_t col_in = tmem + 256, col_su = tmem + 320, col_pu = CHANNEL ? col_in : tmem + 384;
+  // scores and P; Q S' with S' hi and lo side by side; K^T U (HEAD: with U hi and lo); P U (CHANNEL: added to Q S' hi)
+  const uint32_t col_p = tmem, col_in = tmem + 128, col_su = tmem + 256, col_pu = CHANNEL ? col_in : tmem + 384;
   const uint32_t lane_off = static_cast<uint32_t>((warp & 3) * 32) << 16;
   const Factors* factors = static_cast<const Factors*>(g.factors) + (first_chunk(q0, b) + seg * (pl.seg_len / kChunk)) * a.heads + h;
 
@@ -361,20 +381,18 @@ chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ Chu
       }
     }
   };
-  auto issue_scores = [&](int it) {
+  auto issue_scores = [&] {
     constexpr uint32_t idesc = ptx::make_idesc(1u, 1u, kChunk, kChunk);
     const uint64_t qd = ptx::smem_desc_sw128(base + off_q), kd = ptx::smem_desc_sw128(base + off_k);
     const uint64_t lo = kq >> 4;
-    const uint32_t col = tmem + (it & 1) * kChunk;
-#pragma unroll 1
-    for (int k = 0; k < a.dim / 16; ++k) {
+    steps(a.dim / 16, [&](int k) {
       const uint64_t o = (k >> 2) * (kBox / 16) + 2u * (k & 3);
-      ptx::mma_f16(col, qd + o, kd + o, idesc, k > 0 ? 1u : 0u);
+      ptx::mma_f16(col_p, qd + o, kd + o, idesc, k > 0 ? 1u : 0u);
       if (CHANNEL) {
-        ptx::mma_f16(col, qd + o, kd + lo + o, idesc, 1u);
-        ptx::mma_f16(col, qd + lo + o, kd + o, idesc, 1u);
+        ptx::mma_f16(col_p, qd + o, kd + lo + o, idesc, 1u);
+        ptx::mma_f16(col_p, qd + lo + o, kd + o, idesc, 1u);
       }
-    }
+    });
     ptx::tc_commit(bar_g);
   };
   auto wait_bar = [&](uint32_t bar, uint32_t parity, int site) {  // whole warps
@@ -488,13 +506,12 @@ chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ Chu
     if (n_chunks > 1) load_v(1);
   }
   __syncwarp();
-  if (issuer && !STATE_ONLY && ptx::mbar_wait(bar_qk, 0, abort_flag, status, 91)) issue_scores(0);
+  if (issuer && !STATE_ONLY && ptx::mbar_wait(bar_qk, 0, abort_flag, status, 91)) issue_scores();
   __syncwarp();
   if (compute) operands(0, x_now);
   for (int it = 0; it < n_chunks; ++it) {
     const int t = t_begin + it * kChunk, n = min(kChunk, t_end - t);
     const int set = it % kSets, ph = it & 1;
-    const uint32_t col_p = tmem + ph * kChunk;
     const Factors* f = fac + set;
     const int k_tok = (n + 15) / 16;  // steps of 16 tokens
     const bool more = it + 1 < n_chunks;
@@ -517,31 +534,27 @@ chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ Chu
     }
     if (issuer) {
       ptx::tc_fence_after();
-      const uint32_t idesc_o = ptx::make_idesc(1u, 1u, kChunk, vb) | (1u << 16);  // B is MN-major
-      const uint32_t idesc_s = idesc_o | (1u << 15);                              // A too
+      constexpr uint32_t kMnB = 1u << 16, kMnA = 1u << 15;  // operands that lie MN-major
+      constexpr uint32_t idesc_pair = ptx::make_idesc(1u, 1u, kChunk, 2 * kVb) | kMnB;
+      constexpr uint32_t idesc_one = ptx::make_idesc(1u, 1u, kChunk, kVb) | kMnB;
       if (!STATE_ONLY) {
-        const uint64_t qd = ptx::smem_desc_sw128(base + off_q), qlo = qd + (kq >> 4);
-        const uint64_t sd = ptx::smem_desc_sw128(base + off_s), slo = sd + (s_bytes >> 4);  // 64 columns: no leading offset
-#pragma unroll 1
-        for (int k = 0; k < a.dim / 16; ++k) {
+        const uint64_t qd = ptx::smem_desc_sw128(base + off_q), qlo = qd + (kq >> 4), sd = desc_mn(base + off_s, s_bytes);
+        steps(a.dim / 16, [&](int k) {
           const uint64_t o = (k >> 2) * (kBox / 16) + 2u * (k & 3), so = k * 128u;
-          ptx::mma_f16(col_in, qd + o, sd + so, idesc_o, k > 0 ? 1u : 0u);
-          ptx::mma_f16(col_in, qd + o, slo + so, idesc_o, 1u);
-          if (CHANNEL) ptx::mma_f16(col_in, qlo + o, sd + so, idesc_o, 1u);
-        }
+          ptx::mma_f16(col_in, qd + o, sd + so, idesc_pair, k > 0 ? 1u : 0u);
+          if (CHANNEL) ptx::mma_f16(col_in, qlo + o, sd + so, idesc_pair, 1u);
+        });
       } else {
         ptx::mbar_wait(bar_qk, ph, abort_flag, status, 96);
       }
       // A = K^T: rows of S by tokens, a second box of rows for more than 64 (else the first once more, unused)
-      const uint64_t lead = static_cast<uint64_t>(((pl.boxes > 1 ? kBox : 0) >> 4) & 0x3fff) << 16;
-      const uint64_t kt = (ptx::smem_desc_sw128(base + off_k) & ~(static_cast<uint64_t>(0x3fffu) << 16)) | lead;
-      const uint64_t ud = ptx::smem_desc_sw128(base + (CHANNEL ? off_v + set * kBox : off_x));
-#pragma unroll 1
-      for (int k = 0; k < k_tok; ++k) {
+      const uint64_t kt = desc_mn(base + off_k, pl.boxes > 1 ? kBox : 0);
+      const uint64_t ud = desc_mn(base + (CHANNEL ? off_v + set * kBox : off_x), kBox);
+      steps(k_tok, [&](int k) {
         const uint64_t o = k * 128u;
-        ptx::mma_f16(col_su, kt + o, ud + o, idesc_s, k > 0 ? 1u : 0u);
-        ptx::mma_f16(col_su, CHANNEL ? kt + (kq >> 4) + o : kt + o, CHANNEL ? ud + o : ud + kBox / 16 + o, idesc_s, 1u);
-      }
+        ptx::mma_f16(col_su, kt + o, ud + o, (CHANNEL ? idesc_one : idesc_pair) | kMnA, k > 0 ? 1u : 0u);
+        if (CHANNEL) ptx::mma_f16(col_su, kt + (kq >> 4) + o, ud + o, idesc_one | kMnA, 1u);
+      });
       ptx::tc_commit(bar_su);
     }
     __syncwarp();
@@ -602,16 +615,18 @@ chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ Chu
       asm volatile("bar.sync 1, %0;" ::"n"(kCompute + 32) : "memory");  // all but the loader's warp
       if (issuer) {
         ptx::tc_fence_after();
-        const uint32_t idesc_o = ptx::make_idesc(1u, 1u, kChunk, vb) | (1u << 16);
-        const uint64_t vd = ptx::smem_desc_sw128(base + off_v + set * kBox);
-#pragma unroll 1
-        for (int k = 0; k < k_tok; ++k) {
+        constexpr uint32_t idesc_one = ptx::make_idesc(1u, 1u, kChunk, kVb) | (1u << 16);
+        const uint64_t vd = desc_mn(base + off_v + set * kBox, kBox);
+        if (CHANNEL) ptx::mbar_wait(bar_su, ph, abort_flag, status, 100);  // Q S' is in place: products of another shape follow
+        steps(k_tok, [&](int k) {
           const uint32_t pc = col_p + (k >> 1) * 32 + (k & 1) * 8;
-          ptx::mma_f16_ts(col_pu, pc, vd + k * 128u, idesc_o, CHANNEL || k > 0 ? 1u : 0u);
-          ptx::mma_f16_ts(col_pu, pc + 16, vd + k * 128u, idesc_o, 1u);
-        }
+          ptx::mma_f16_ts(col_pu, pc, vd + k * 128u, idesc_one, CHANNEL || k > 0 ? 1u : 0u);
+          ptx::mma_f16_ts(col_pu, pc + 16, vd + k * 128u, idesc_one, 1u);
+        });
         ptx::tc_commit(bar_o);
-        if (more && ptx::mbar_wait(bar_qk, ph ^ 1, abort_flag, status, 98)) issue_scores(it + 1);
+        if (more && ptx::mbar_wait(bar_o, ph, abort_flag, status, 99) &&  // the next scores overwrite P
+            ptx::mbar_wait(bar_qk, ph ^ 1, abort_flag, status, 98))
+          issue_scores();
       }
       __syncwarp();
     }
@@ -619,8 +634,9 @@ chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ Chu
     // ---- new state, operands of the next chunk, output ------------------------------------------------
     if (compute) {
       wait_bar(bar_su, ph, 94);
-      uint32_t v[16];
+      uint32_t v[16], y[16];
       ptx::tmem_ld_32x16(col_su + lane_off + col0, v);
+      if (!CHANNEL) ptx::tmem_ld_32x16(col_su + kVb + lane_off + col0, y);
       ptx::tmem_ld_wait();
       if (state_thread) {
         float end;
@@ -628,15 +644,20 @@ chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ Chu
         else end = f->end;
 #pragma unroll
         for (int c = 0; c < 16; ++c)
-          s[c] = CHANNEL ? end * (s[c] + __uint_as_float(v[c])) : fmaf(end, s[c], __uint_as_float(v[c]));
+          s[c] = CHANNEL ? end * (s[c] + __uint_as_float(v[c])) : fmaf(end, s[c], __uint_as_float(v[c]) + __uint_as_float(y[c]));
         decay_all *= end;
       }
       __syncwarp();
       if (more) operands(it + 1, x_next);
       if (!STATE_ONLY) {
+        ptx::tmem_ld_32x16(col_in + kVb + lane_off + col0, y);  // Q S', with the low halves
+        if (!CHANNEL) {
+          ptx::tmem_ld_32x16(col_in + lane_off + col0, v);
+          ptx::tmem_ld_wait();
+#pragma unroll
+          for (int e = 0; e < 16; ++e) y[e] = __float_as_uint(__uint_as_float(y[e]) + __uint_as_float(v[e]));
+        }
         wait_bar(bar_o, ph, 95);
-        uint32_t y[16];
-        if (!CHANNEL) ptx::tmem_ld_32x16(col_in + lane_off + col0, y);
         ptx::tmem_ld_32x16(col_pu + lane_off + col0, v);
         ptx::tmem_ld_wait();
         if (row < n && my_cols) {
@@ -649,7 +670,10 @@ chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ Chu
 #pragma unroll
           for (int e = 0; e < 8; ++e) {
             float y0 = __uint_as_float(v[2 * e]), y1 = __uint_as_float(v[2 * e + 1]);
-            if (!CHANNEL) {
+            if (CHANNEL) {
+              y0 += __uint_as_float(y[2 * e]);
+              y1 += __uint_as_float(y[2 * e + 1]);
+            } else {
               y0 = fmaf(skip, bf16lo(x_now[e]), a.scale * fmaf(er, __uint_as_float(y[2 * e]), y0));
               y1 = fmaf(skip, bf16hi(x_now[e]), a.scale * fmaf(er, __uint_as_float(y[2 * e + 1]), y1));
             }
