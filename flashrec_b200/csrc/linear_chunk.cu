@@ -63,6 +63,13 @@ __device__ __forceinline__ uint32_t split2(uint64_t v, uint32_t& lo) {
   return hi;
 }
 
+// log2(1 + e^z): the logarithm's series where 1 + e^-|z| would lose the small term
+__device__ __forceinline__ float softplus_log2(float z) {
+  const float e = ex2(-fabsf(z) * kLog2e);
+  const float series = kLog2e * e * (1.0f - e * (0.5f - e * (1.0f / 3.0f - 0.25f * e)));
+  return fmaf(fmaxf(z, 0.f), kLog2e, e < 0.0156f ? series : __log2f(1.0f + e));
+}
+
 // Factors of one chunk and head.
 struct HeadFactors {
   float r[kChunk];    // r_i (log2)
@@ -183,7 +190,7 @@ channel_factor_kernel(const __grid_constant__ ChunkArgs g) {
   const bool live = part < parts;
   if (live) {
     const int hc = h * a.dim + ch;
-    const float b0 = a.step_bias[hc], b1 = a.step_bias[hc + 1], f = -a.inv_tau * kLog2e;
+    const float b0 = a.step_bias[hc], b1 = a.step_bias[hc + 1], f = -a.inv_tau;
     float2 sum = make_float2(0.f, 0.f);
     for (int i = i0; i < i1; i += 4) {
       float z0[4], z1[4];
@@ -205,7 +212,7 @@ channel_factor_kernel(const __grid_constant__ ChunkArgs g) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         if (i + e >= i1) break;
-        const float2 la = make_float2(softplus(-z0[e]) * f, softplus(-z1[e]) * f);
+        const float2 la = make_float2(softplus_log2(-z0[e]) * f, softplus_log2(-z1[e]) * f);
         *reinterpret_cast<float2*>(s_la + (i + e) * a.dim + ch) = la;
         if (i + e > 0) {
           sum.x += la.x;
@@ -241,7 +248,7 @@ channel_factor_kernel(const __grid_constant__ ChunkArgs g) {
   const __nv_bfloat16* kp = static_cast<const __nv_bfloat16*>(a.k) + static_cast<int64_t>(t) * a.ldk + h * a.dim + ch;
   const int64_t ld = static_cast<int64_t>(a.heads) * a.dim;
   __nv_bfloat16* out = g.qk + t * ld + h * a.dim + ch;
-#pragma unroll 4
+#pragma unroll 8
   for (int i = i0; i < i1; ++i) {
     if (i > 0) {
       const float2 d = *reinterpret_cast<const float2*>(s_la + i * a.dim + ch);
