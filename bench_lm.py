@@ -223,8 +223,7 @@ def kotipel_kernel_times(torch, model, n_tok, peaks, iters=10):
     move = lambda cols: ("bytes", 2 * n_tok * cols)  # 16-bit columns in and out; the stream counts double
     keys = n_tok * (n_tok + 1) // 2
     mc, gk, gv = mamba.channels, g.heads * g.dim, g.heads * g.vdim
-    tail = [("norm2", move(7 * w)), ("gate_up", gemm(2 * ff, w)), ("down", gemm(w, ff)), ("copy", move(3 * w)),
-            ("side.gate", gemm(d, w)), ("side.proj", gemm(w, d))]
+    tail = [("norm2", move(7 * w)), ("gate_up", gemm(2 * ff, w)), ("down", gemm(w, ff)), ("side.gate", gemm(d, w)), ("side.proj", gemm(w, d))]
     names = [("mamba.norm1", move(3 * w)), ("mamba.projections", gemm(mamba.inner + mc + mamba.heads, w)), ("mamba.conv", move(2 * mc)),
              ("mamba.recurrence", move(mc + mamba.inner + 2 * mamba.heads)), ("mamba.norm", move(3 * mamba.inner)),
              ("mamba.out", gemm(w, mamba.inner))]
@@ -240,7 +239,7 @@ def kotipel_kernel_times(torch, model, n_tok, peaks, iters=10):
     orig, empty = lm_layers.call, torch.empty
 
     def record(name, *args):
-        if name != "fr_lm_embed":
+        if name not in ("fr_lm_embed", "fr_lm_rotary_table"):  # once a step
             launches.append((name, args))
         orig(name, *args)
 
@@ -255,16 +254,10 @@ def kotipel_kernel_times(torch, model, n_tok, peaks, iters=10):
         lm_layers.call, torch.empty = orig, empty
     torch.cuda.synchronize()
     flush = torch.empty(256 << 20, dtype=torch.uint8, device=model.device)
-    fused = {"parallel.recurrence": ("fr_linear_decay",)}
-    res, i = {}, 0
-    for name, (what, amount) in names:
-        group = [launches[i]]
-        i += 1
-        while group[-1][0] in fused.get(name, ()):
-            group.append(launches[i])
-            i += 1
-        ms = event_time(torch, lambda _: [orig(n, *args) for n, args in group], iters, rest=0.4, flush=flush)
-        r = {"us": round(ms * 1e3, 1), "launch": group[-1][0]}
+    res = {}
+    for (name, (what, amount)), (entry, args) in zip(names, launches):
+        ms = event_time(torch, lambda _: orig(entry, *args), iters, rest=0.4, flush=flush)
+        r = {"us": round(ms * 1e3, 1), "entry": entry}
         if what == "flops":
             r.update(tflops=round(amount / ms / 1e9, 1), frac_of_measured=round(amount / ms / 1e9 / peaks["bf16_tflops"], 3))
         else:

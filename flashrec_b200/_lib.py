@@ -100,7 +100,7 @@ class FrMixAttn(ctypes.Structure):
 class FrNormPart(ctypes.Structure):
     """Mirror of ``struct fr_norm_part``."""
 
-    _fields_ = [("y", c_void_p), ("ldy", c_int64), ("weight", c_void_p), ("coef", c_float), ("pad_", ctypes.c_int32)]
+    _fields_ = [("y", c_void_p), ("ldy", c_int64), ("weight", c_void_p), ("coef", c_float), ("n_splits", ctypes.c_int32)]
 
 
 class FrNormUpdate(ctypes.Structure):
@@ -125,7 +125,7 @@ class FrQkRope(ctypes.Structure):
 
     _fields_ = ([(n, ctypes.c_int32) for n in ("dtype", "heads", "kv_heads", "dim", "dim_true", "rot_dims")] + [("eps", c_float),
                 ("pad_", ctypes.c_int32), ("q", c_void_p), ("ldq", c_int64), ("k", c_void_p), ("ldk", c_int64),
-                ("q_weight", c_void_p), ("k_weight", c_void_p), ("inv_freq", c_void_p), ("pos", c_void_p), ("loc", c_void_p),
+                ("q_weight", c_void_p), ("k_weight", c_void_p), ("table", c_void_p), ("loc", c_void_p),
                 ("k_cache", c_void_p), ("ldkc", c_int64)])
 
 
@@ -204,12 +204,14 @@ _SIGNATURES = {
     "fr_sid_head_topk": [P] * 6 + [P, P, _L, P, P, _L, _I] + [P] * 8 + [_L] * 3 + [_I] * 8 + [P, P, P, _L, _I, P],
     "fr_topk_merge_shards": [P] * 16 + [_L] * 2 + [_I] * 7 + [P],
     "fr_dense_proj": [_I, P, _L, P, _L, _I, _I, _I, P, _I, _I, P],
-    "fr_dense_gated_add": [_I, P, _I, P, _L, _I, _I, P, _I, _I, P],
+    "fr_dense_proj_split": [_I, P, _L, P, _L, _I, _I, _I, P, _I, P, _I, P],
+    "fr_dense_gated_add": [_I, P, _I, P, _L, _I, _I, P, _I, P, _L, _I, P],
     "fr_dense_gated_add_splits": [_I] * 5,
     "fr_lm_embed": [_I, P, _L, P, P, _L, _I, _I, _I, _F, P, _L, P, P, P, P],
     "fr_lm_norm": [_I, P, _L, P, _F, _F, P, _I, _L, P, P, _L, _I, _I, P],
     "fr_lm_update_norm": [P, _I, _I, P],
     "fr_lm_group_norm": [P, _I, P],
+    "fr_lm_rotary_table": [P, _I, P, P, _I, P],
     "fr_lm_qk_norm_rope": [P, _I, P],
     "fr_linear_state_floats": [_I, _I],
     "fr_linear_scan_rows": [P, _I, _I, _I, P],

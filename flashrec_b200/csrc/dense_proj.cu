@@ -224,7 +224,8 @@ dense_rows_proj_kernel(const T* __restrict__ a, int64_t lda, const T* __restrict
 
 template <typename T, int MB>
 __global__ void __launch_bounds__(kRowsThreads)
-dense_rows_gated_kernel(const __grid_constant__ Parts pt, float* __restrict__ x, int64_t ldx, int M, int N, int ks) {
+dense_rows_gated_kernel(const __grid_constant__ Parts pt, float* __restrict__ x, int64_t ldx, int M, int N, T* __restrict__ copy,
+                        int64_t ldc, int ks) {
   __shared__ float red[8][2][4 * MB];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int groups_per_cta = (kRowsThreads / 32) / ks;
@@ -264,6 +265,8 @@ dense_rows_gated_kernel(const __grid_constant__ Parts pt, float* __restrict__ x,
   __syncthreads();
   if (!live || kwarp != 0 || lane >= 4 * MB) return;
   const int r = lane / MB, m = lane % MB, n = grp * 4 + r;
+  if (copy != nullptr && m < M && n >= N - 8)  // the padding behind the last columns
+    for (int c = N + (n - (N - 8)); c < (N + 7) / 8 * 8 && c < ldc; c += 8) copy[m * ldc + c] = from_f<T>(0.f);
   if (m >= M || n >= N) return;
   float v = x[m * ldx + n];
   for (int p = 0; p < pt.n; ++p) {
@@ -273,6 +276,7 @@ dense_rows_gated_kernel(const __grid_constant__ Parts pt, float* __restrict__ x,
     v += (g != nullptr ? to_f<T>(g[m * pt.p[p].ldg + n]) : 1.0f) * z;
   }
   x[m * ldx + n] = v;
+  if (copy != nullptr) copy[m * ldc + n] = from_f<T>(v);
 }
 
 // ---------------------------------------------------------------------------
@@ -342,7 +346,8 @@ dense_simt_proj_kernel(const float* __restrict__ a, int64_t lda, const float* __
 }
 
 __global__ void __launch_bounds__(256)
-dense_simt_gated_kernel(const __grid_constant__ Parts pt, float* __restrict__ x, int64_t ldx, int M, int N) {
+dense_simt_gated_kernel(const __grid_constant__ Parts pt, float* __restrict__ x, int64_t ldx, int M, int N, float* __restrict__ copy,
+                        int64_t ldc) {
   __shared__ float as[kSimtK][68], ws[kSimtK][68];
   const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
@@ -362,8 +367,39 @@ dense_simt_gated_kernel(const __grid_constant__ Parts pt, float* __restrict__ x,
   for (int i = 0; i < 4; ++i)
     for (int j = 0; j < 4; ++j) {
       const int row = m0 + ty * 4 + i, col = n0 + (j >> 1) * 32 + tx * 2 + (j & 1);
-      if (row < M && col < N) x[row * ldx + col] += sum[i][j];
+      if (row < M && col < N) {
+        const float v = x[row * ldx + col] + sum[i][j];
+        x[row * ldx + col] = v;
+        if (copy != nullptr) copy[row * ldc + col] = v;
+      } else if (copy != nullptr && row < M && col < (N + 7) / 8 * 8 && col < ldc) {
+        copy[row * ldc + col] = 0.f;
+      }
     }
+}
+
+// ---------------------------------------------------------------------------
+// sum of the K shares of a split product, then the column ranges' epilogues
+// ---------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(256)
+dense_finish_kernel(const float* __restrict__ partials, int n_splits, int M, int N, const __grid_constant__ Segs sg) {
+  ptx::griddep_wait();
+  ptx::griddep_launch_dependents();
+  const int row = blockIdx.y, col = blockIdx.x * 256 + threadIdx.x;
+  if (col >= N) return;
+  const fr_out_segment& s = sg.s[seg_of(sg, col)];
+  auto sum = [&](int c) {
+    float z = 0.f;
+    for (int i = 0; i < n_splits; ++i) z += partials[(static_cast<int64_t>(i) * M + row) * N + c];
+    return z;
+  };
+  const int local = col - s.n0;
+  constexpr bool kFast = sizeof(T) == 2;
+  if (!paired(s)) {
+    seg_write<T, kFast>(s, row, local, sum(col));
+  } else if (local % 64 < 32) {
+    seg_write<T, kFast>(s, row, local / 64 * 32 + local % 64, pair_act<kFast>(s, sum(col), sum(col + 32)));
+  }
 }
 
 // ---------------------------------------------------------------------------
@@ -398,6 +434,8 @@ struct TcArgs {
   const __nv_bfloat16* gate[2];
   int64_t ldg[2];
   float* partials;   // kEpiPartial: [splits, M, N]
+  __nv_bfloat16* copy;  // kEpiAdd: the new x as bf16, or null
+  int64_t ldc;
 };
 
 // Work of a CTA in order: kEpiSegs / kEpiAdd: tile after tile, the parts of a tile back to back (its second
@@ -688,6 +726,12 @@ dense_tc_kernel(const __grid_constant__ CUtensorMap ta0, const __grid_constant__
 #pragma unroll
               for (int i = 0; i < 32; ++i) v[i] = fmaf(gt[i], __uint_as_float(r[i]), v[i]);
               if (live) store32_f32(xr, v, nvalid);
+              if (live && g.copy != nullptr && sub + 1 == subs) {
+                __nv_bfloat16* cr = g.copy + row * g.ldc + col;
+                store32_bf16(cr, v, nvalid);
+                if (nvalid < 32)
+                  for (int c = nvalid; (col + c) % 8 != 0 && col + c < g.ldc; ++c) cr[c] = __float2bfloat16_rn(0.f);
+              }
             } else {
               ptx::tmem_ld_wait();
 #pragma unroll
@@ -801,15 +845,16 @@ static int launch_rows_proj(const void* a, int64_t lda, const void* w, int64_t l
 }
 
 template <typename T>
-static int launch_rows_gated(const Parts& pt, float* x, int64_t ldx, int M, int N, cudaStream_t stream) {
+static int launch_rows_gated(const Parts& pt, float* x, int64_t ldx, int M, int N, void* copy_out, int64_t ldc, cudaStream_t stream) {
+  T* copy = static_cast<T*>(copy_out);
   int K = 0;
   for (int p = 0; p < pt.n; ++p) K = K > pt.p[p].K ? K : pt.p[p].K;
   const int ks = rows_ks(N, K);
   const int grid = ceil_div(ceil_div(N, 4), (kRowsThreads / 32) / ks);
-  if (M == 1) return launch_kernel(dense_rows_gated_kernel<T, 1>, grid, kRowsThreads, 0, stream, true, pt, x, ldx, M, N, ks);
-  if (M == 2) return launch_kernel(dense_rows_gated_kernel<T, 2>, grid, kRowsThreads, 0, stream, true, pt, x, ldx, M, N, ks);
-  if (M <= 4) return launch_kernel(dense_rows_gated_kernel<T, 4>, grid, kRowsThreads, 0, stream, true, pt, x, ldx, M, N, ks);
-  return launch_kernel(dense_rows_gated_kernel<T, 8>, grid, kRowsThreads, 0, stream, true, pt, x, ldx, M, N, ks);
+  if (M == 1) return launch_kernel(dense_rows_gated_kernel<T, 1>, grid, kRowsThreads, 0, stream, true, pt, x, ldx, M, N, copy, ldc, ks);
+  if (M == 2) return launch_kernel(dense_rows_gated_kernel<T, 2>, grid, kRowsThreads, 0, stream, true, pt, x, ldx, M, N, copy, ldc, ks);
+  if (M <= 4) return launch_kernel(dense_rows_gated_kernel<T, 4>, grid, kRowsThreads, 0, stream, true, pt, x, ldx, M, N, copy, ldc, ks);
+  return launch_kernel(dense_rows_gated_kernel<T, 8>, grid, kRowsThreads, 0, stream, true, pt, x, ldx, M, N, copy, ldc, ks);
 }
 
 static bool operand_ok(const void* p, int64_t ld, int K) {
@@ -845,13 +890,10 @@ int make_tmap_bf16_box64(CUtensorMap* map, const void* ptr, uint64_t cols, uint6
 
 using namespace fr;
 
-extern "C" int fr_dense_proj(int dtype, const void* a, int64_t lda, const void* w, int64_t ldw, int M, int N, int K,
-                             const fr_out_segment* segs, int n_segs, int algo, cudaStream_t stream) {
-  FR_CHECK_ARG((dtype == 0 || dtype == 1) && M >= 0 && N > 0 && segs && n_segs > 0 && n_segs <= dense::kMaxSegs);
-  if (M == 0) return FR_OK;
-  FR_CHECK_ARG(dense::operand_ok(a, lda, K) && dense::operand_ok(w, ldw, K) && N % 4 == 0);
-  dense::Segs sg{};
-  sg.n = n_segs;
+// Column ranges as the kernels get them; FR_ERR_BAD_ARG when they do not tile the columns as the header says.
+static int check_segs(const fr_out_segment* segs, int n_segs, int N, dense::Segs* sg) {
+  FR_CHECK_ARG(segs && n_segs > 0 && n_segs <= dense::kMaxSegs);
+  sg->n = n_segs;
   for (int i = 0; i < n_segs; ++i) {
     const fr_out_segment& s = segs[i];
     const int end = i + 1 < n_segs ? segs[i + 1].n0 : N;
@@ -862,8 +904,18 @@ extern "C" int fr_dense_proj(int dtype, const void* a, int64_t lda, const void* 
       FR_CHECK_ARG(s.n0 % 64 == 0 && (end - s.n0) % 64 == 0 && 2 * s.n <= end - s.n0);
     else
       FR_CHECK_ARG(s.n <= end - s.n0);
-    sg.s[i] = s;
+    sg->s[i] = s;
   }
+  return FR_OK;
+}
+
+extern "C" int fr_dense_proj(int dtype, const void* a, int64_t lda, const void* w, int64_t ldw, int M, int N, int K,
+                             const fr_out_segment* segs, int n_segs, int algo, cudaStream_t stream) {
+  FR_CHECK_ARG((dtype == 0 || dtype == 1) && M >= 0 && N > 0);
+  if (M == 0) return FR_OK;
+  FR_CHECK_ARG(dense::operand_ok(a, lda, K) && dense::operand_ok(w, ldw, K) && N % 4 == 0);
+  dense::Segs sg{};
+  if (check_segs(segs, n_segs, N, &sg) != FR_OK) return FR_ERR_BAD_ARG;
   if (algo == 0) algo = M <= 8 ? 1 : 2;
   if (algo == 1) {
     FR_CHECK_SUPPORTED(M <= 8);
@@ -890,6 +942,18 @@ extern "C" int fr_dense_proj(int dtype, const void* a, int64_t lda, const void* 
   }
 }
 
+extern "C" int fr_dense_proj_split(int dtype, const void* a, int64_t lda, const void* w, int64_t ldw, int M, int N, int K,
+                                   const fr_out_segment* segs, int n_segs, float* partials, int n_splits, cudaStream_t stream) {
+  FR_CHECK_ARG(M > 0 && M <= 65535 && N > 0 && partials && n_splits > 0);
+  dense::Segs sg{};
+  if (check_segs(segs, n_segs, N, &sg) != FR_OK) return FR_ERR_BAD_ARG;
+  const fr_gated_part part{a, w, nullptr, lda, ldw, 0, K, 0};
+  const int r = fr_dense_gated_add(dtype, &part, 1, partials, N, M, N, partials, n_splits, nullptr, 0, 0, stream);  // x is left alone
+  if (r != FR_OK) return r;
+  auto kern = dtype == 0 ? dense::dense_finish_kernel<__nv_bfloat16> : dense::dense_finish_kernel<float>;
+  return launch_kernel(kern, dim3(ceil_div(N, 256), M), 256, 0, stream, M <= kPdlRows, static_cast<const float*>(partials), n_splits, M, N, sg);
+}
+
 extern "C" int fr_dense_gated_add_splits(int dtype, int M, int N, int K0, int K1) {
   if (dtype != 0 || M <= 8 || N <= 0 || K0 <= 0) return 0;
   int a, b;
@@ -898,10 +962,10 @@ extern "C" int fr_dense_gated_add_splits(int dtype, int M, int N, int K0, int K1
 }
 
 extern "C" int fr_dense_gated_add(int dtype, const fr_gated_part* parts, int n_parts, float* x, int64_t ldx, int M, int N,
-                                  float* partials, int n_splits, int algo, cudaStream_t stream) {
+                                  float* partials, int n_splits, void* copy, int64_t ldc, int algo, cudaStream_t stream) {
   FR_CHECK_ARG((dtype == 0 || dtype == 1) && parts && (n_parts == 1 || n_parts == 2) && M >= 0 && N > 0);
   if (M == 0) return FR_OK;
-  FR_CHECK_ARG(x && ldx >= N);
+  FR_CHECK_ARG(x && ldx >= N && (copy == nullptr || (ldc >= N && partials == nullptr)));
   dense::Parts pt{};
   pt.n = n_parts;
   for (int p = 0; p < n_parts; ++p) {
@@ -913,13 +977,13 @@ extern "C" int fr_dense_gated_add(int dtype, const fr_gated_part* parts, int n_p
   if (algo == 0) algo = (M <= 8 && n_splits == 0) ? 1 : 2;
   if (algo == 1) {
     FR_CHECK_SUPPORTED(M <= 8 && n_splits == 0);
-    return dtype == 0 ? dense::launch_rows_gated<__nv_bfloat16>(pt, x, ldx, M, N, stream)
-                      : dense::launch_rows_gated<float>(pt, x, ldx, M, N, stream);
+    return dtype == 0 ? dense::launch_rows_gated<__nv_bfloat16>(pt, x, ldx, M, N, copy, ldc, stream)
+                      : dense::launch_rows_gated<float>(pt, x, ldx, M, N, copy, ldc, stream);
   }
   if (dtype == 1) {
     FR_CHECK_SUPPORTED(n_splits == 0);
     dim3 grid(ceil_div(N, 64), ceil_div(M, 64));
-    dense::dense_simt_gated_kernel<<<grid, 256, 0, stream>>>(pt, x, ldx, M, N);
+    dense::dense_simt_gated_kernel<<<grid, 256, 0, stream>>>(pt, x, ldx, M, N, static_cast<float*>(copy), ldc);
     return launch_status();
   }
   dense::TcArgs g{};
@@ -928,6 +992,8 @@ extern "C" int fr_dense_gated_add(int dtype, const fr_gated_part* parts, int n_p
   g.n_parts = n_parts;
   g.x = x;
   g.ldx = ldx;
+  g.copy = static_cast<__nv_bfloat16*>(copy);
+  g.ldc = ldc;
   for (int p = 0; p < n_parts; ++p) {
     g.kb[p] = ceil_div(parts[p].K, dense::kBlockK);
     g.gate[p] = static_cast<const __nv_bfloat16*>(parts[p].gate);

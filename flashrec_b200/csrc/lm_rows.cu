@@ -466,7 +466,14 @@ update_norm_kernel(const __grid_constant__ fr_norm_update u, int W) {
 #pragma unroll
       for (int p = 0; p < 2; ++p)
         if (p < u.n_parts) {
-          y[p][i] = ld4<T>(static_cast<const T*>(u.parts[p].y) + src * u.parts[p].ldy + c);
+          if (u.parts[p].n_splits == 0) {
+            y[p][i] = ld4<T>(static_cast<const T*>(u.parts[p].y) + src * u.parts[p].ldy + c);
+          } else {
+            for (int s = 0; s < u.parts[p].n_splits; ++s) {
+              const float4 q = *reinterpret_cast<const float4*>(static_cast<const float*>(u.parts[p].y) + s * u.parts[p].ldy + src * W + c);
+              y[p][i].x += q.x; y[p][i].y += q.y; y[p][i].z += q.z; y[p][i].w += q.w;
+            }
+          }
           ss[p] += sq4(y[p][i]);
         }
       if (pr != nullptr)
@@ -515,11 +522,17 @@ update_norm_kernel(const __grid_constant__ fr_norm_update u, int W) {
     }
   } else {
     float r[2] = {0.f, 0.f};
+    auto part = [&](int p, int c) {
+      const fr_norm_part& q = u.parts[p];
+      if (q.n_splits == 0) return ld_f(static_cast<const T*>(q.y) + src * q.ldy + c);
+      float f = 0.f;
+      for (int s = 0; s < q.n_splits; ++s) f += static_cast<const float*>(q.y)[s * q.ldy + src * W + c];
+      return f;
+    };
     for (int p = 0; p < u.n_parts; ++p) {
       float ss = 0.f;
-      const T* y = static_cast<const T*>(u.parts[p].y) + src * u.parts[p].ldy;
       for (int c = threadIdx.x; c < W; c += kNormThreads) {
-        const float f = ld_f(y + c);
+        const float f = part(p, c);
         ss += f * f;
       }
       r[p] = u.parts[p].coef / sqrtf(cta_sum<kNormThreads>(ss, sums[p]) / static_cast<float>(W) + u.eps);
@@ -529,7 +542,7 @@ update_norm_kernel(const __grid_constant__ fr_norm_update u, int W) {
       if (pr != nullptr)
         for (int s = 0; s < u.n_partials; ++s) f += pr[s * u.partial_stride + c];
       for (int p = 0; p < u.n_parts; ++p)
-        f += ld_f(static_cast<const T*>(u.parts[p].y) + src * u.parts[p].ldy + c) * r[p] * u.parts[p].weight[c];
+        f += part(p, c) * r[p] * u.parts[p].weight[c];
       if (u.add != nullptr) f += u.add[c];
       return f;
     };
@@ -677,6 +690,25 @@ __device__ __forceinline__ void ld8(const float* p, float (&v)[8]) {
   *reinterpret_cast<float4*>(v + 4) = *reinterpret_cast<const float4*>(p + 4);
 }
 
+__global__ void __launch_bounds__(256)
+rotary_table_kernel(const float* __restrict__ inv_freq, int pairs, const int64_t* __restrict__ pos, float* __restrict__ table, int M) {
+  ptx::griddep_wait();
+  ptx::griddep_launch_dependents();
+  const int64_t e = static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x;
+  if (e >= static_cast<int64_t>(M) * pairs) return;
+  const int64_t t = e / pairs;
+  const int i = static_cast<int>(e % pairs);
+  // the angle as a sum of two floats: its rounding alone would show at far positions
+  const float p = static_cast<float>(pos[t]);
+  const float2 f = reinterpret_cast<const float2*>(inv_freq)[i];
+  const float hi = p * f.x, lo = fmaf(p, f.y, fmaf(p, f.x, -hi));
+  float s, c;
+  sincosf(hi, &s, &c);
+  const float c1 = 1.0f - 0.5f * lo * lo, s1 = lo - lo * lo * lo * (1.0f / 6.0f);  // lo is at most half a place of hi
+  table[t * 2 * pairs + i] = c * c1 - s * s1;
+  table[t * 2 * pairs + pairs + i] = s * c1 + c * s1;
+}
+
 template <typename T>
 __global__ void __launch_bounds__(kRopeThreads)
 qk_norm_rope_kernel(const __grid_constant__ fr_qk_rope a) {
@@ -690,7 +722,6 @@ qk_norm_rope_kernel(const __grid_constant__ fr_qk_rope a) {
   ptx::griddep_wait();
   ptx::griddep_launch_dependents();
   const int64_t t = blockIdx.x;
-  const float p = static_cast<float>(a.pos[t]);
   T* q = static_cast<T*>(a.q) + t * a.ldq;
   const T* k = static_cast<const T*>(a.k) + t * a.ldk;
   float sq = 0.f, sk = 0.f;
@@ -704,16 +735,7 @@ qk_norm_rope_kernel(const __grid_constant__ fr_qk_rope a) {
     *reinterpret_cast<float4*>(sm + c) = make_float4(v[0], v[1], v[2], v[3]);
     *reinterpret_cast<float4*>(sm + c + 4) = make_float4(v[4], v[5], v[6], v[7]);
   }
-  for (int i = threadIdx.x; i < half; i += kRopeThreads) {
-    // the angle as a sum of two floats: its rounding alone would show at far positions
-    const float2 f = reinterpret_cast<const float2*>(a.inv_freq)[i];
-    const float hi = p * f.x, lo = fmaf(p, f.y, fmaf(p, f.x, -hi));
-    float s, c;
-    sincosf(hi, &s, &c);
-    const float c1 = 1.0f - 0.5f * lo * lo, s1 = lo - lo * lo * lo * (1.0f / 6.0f);  // lo is at most half a place of hi
-    s_cos[i] = c * c1 - s * s1;
-    s_sin[i] = s * c1 + c * s1;
-  }
+  for (int i = threadIdx.x; i < a.rot_dims; i += kRopeThreads) s_cos[i] = a.table[t * a.rot_dims + i];  // the sines follow
   sq = cta_sum<kRopeThreads>(sq, sums[0]);
   sk = cta_sum<kRopeThreads>(sk, sums[1]);
   const float rq = 1.0f / sqrtf(sq / static_cast<float>(a.heads * a.dim_true) + a.eps);
@@ -822,7 +844,8 @@ extern "C" int fr_lm_update_norm(const fr_norm_update* u, int M, int W, cudaStre
   FR_CHECK_ARG(u && (u->dtype == 0 || u->dtype == 1) && M >= 0 && W > 0 && u->ldx >= W && u->n_parts >= 0 && u->n_parts <= 2);
   if (M == 0) return FR_OK;
   FR_CHECK_ARG(u->x && (u->out == nullptr || u->ldo >= W) && u->n_partials >= 0 && (u->n_partials == 0 || u->partials));
-  for (int p = 0; p < u->n_parts; ++p) FR_CHECK_ARG(u->parts[p].y && u->parts[p].weight && u->parts[p].ldy >= W);
+  for (int p = 0; p < u->n_parts; ++p)
+    FR_CHECK_ARG(u->parts[p].y && u->parts[p].weight && u->parts[p].ldy >= W && u->parts[p].n_splits >= 0);
   return u->dtype == 0 ? lm::launch_update_norm<__nv_bfloat16>(*u, M, W, stream) : lm::launch_update_norm<float>(*u, M, W, stream);
 }
 
@@ -835,11 +858,19 @@ extern "C" int fr_lm_group_norm(const fr_group_norm* a, int M, cudaStream_t stre
   return a->dtype == 0 ? lm::launch_group_norm<__nv_bfloat16>(*a, M, stream) : lm::launch_group_norm<float>(*a, M, stream);
 }
 
+extern "C" int fr_lm_rotary_table(const float* inv_freq, int pairs, const int64_t* pos, float* table, int M, cudaStream_t stream) {
+  FR_CHECK_ARG(pairs >= 0 && M >= 0);
+  if (M == 0 || pairs == 0) return FR_OK;
+  FR_CHECK_ARG(inv_freq && pos && table && (reinterpret_cast<uintptr_t>(inv_freq) & 7u) == 0);
+  return launch_kernel(lm::rotary_table_kernel, ceil_div(static_cast<int64_t>(M) * pairs, 256), 256, 0, stream, M <= kPdlRows, inv_freq,
+                       pairs, pos, table, M);
+}
+
 extern "C" int fr_lm_qk_norm_rope(const fr_qk_rope* a, int M, cudaStream_t stream) {
   FR_CHECK_ARG(a && (a->dtype == 0 || a->dtype == 1) && M >= 0 && a->heads > 0 && a->kv_heads > 0 && a->dim > 0 && a->dim % 8 == 0);
   if (M == 0) return FR_OK;
   FR_CHECK_ARG(a->dim_true > 0 && a->dim_true <= a->dim && a->rot_dims >= 0 && a->rot_dims % 2 == 0 && a->rot_dims <= a->dim_true);
-  FR_CHECK_ARG(a->q && a->k && a->k_cache && a->q_weight && a->k_weight && a->pos && a->loc && (a->rot_dims == 0 || a->inv_freq));
+  FR_CHECK_ARG(a->q && a->k && a->k_cache && a->q_weight && a->k_weight && a->loc && (a->rot_dims == 0 || a->table));
   FR_CHECK_ARG(aligned16(a->q) && aligned16(a->k) && aligned16(a->k_cache) && aligned16(a->q_weight) && aligned16(a->k_weight) && a->ldq % 8 == 0 && a->ldk % 8 == 0 && a->ldkc % 8 == 0);
   const int smem = ((a->heads + a->kv_heads) * a->dim + a->rot_dims) * 4;
   FR_CHECK_SUPPORTED(smem <= 200 * 1024);

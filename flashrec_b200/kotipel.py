@@ -21,8 +21,8 @@ import torch
 from flashrec_b200.core import ForwardBatch
 from flashrec_b200.kvcache import CacheSpec, LayerCaches
 from flashrec_b200.lm_layers import (LinearScan, MergedProjection, MixAttention, Pending, ceil_to, embed, gated_add, group_norm,
-                                     interleave_rows, pad_cols, pad_heads, pad_rows, qk_norm_rope, rotary_frequencies, short_conv,
-                                     update_norm)
+                                     interleave_rows, pad_cols, pad_heads, pad_rows, qk_norm_rope, rotary_frequencies,
+                                     rotary_table, short_conv, split_product, update_norm)
 
 PARALLEL, MAMBA2 = "parallel", "mamba2"
 GLU_ALPHA, GLU_UP_BIAS = 1.702, 1.0  # fixed by the design
@@ -189,9 +189,10 @@ class KotipelConfig:
 class _Context:
     """What a layer run works with besides its weights."""
 
-    def __init__(self, batch: ForwardBatch, caches: LayerCaches, run: int, req_to_token, counters, max_keys):
+    def __init__(self, batch: ForwardBatch, caches: LayerCaches, run: int, req_to_token, counters, max_keys, tables):
         self.batch, self.caches, self.run = batch, caches, run
         self.req_to_token, self.counters, self.max_keys = req_to_token, counters, max_keys
+        self.tables = tables  # angles of the batch's positions by rotary configuration, shared by the layers
 
 
 class _Mixer:
@@ -212,6 +213,15 @@ class _Mixer:
         p.add("store", weight)
         p.finish(self.dtype, self.device)
         return p
+
+    def product(self, a: torch.Tensor, p: MergedProjection):
+        """``a`` times the one matrix of ``p``, over the model width: whole or as K shares."""
+        w = self.cfg.width
+        y = split_product(a, p.weight[:w])
+        if y is None:
+            y = self.new(int(a.shape[0]), w)
+            p(a, [y])
+        return y
 
 
 class ParallelMixer(_Mixer):
@@ -237,8 +247,8 @@ class ParallelMixer(_Mixer):
         self.proj, self.rank = proj, rank
         self.q_norm = self.f32(pad_heads(tensors("left.q.norm"), a.dim, dp))
         self.k_norm = self.f32(pad_heads(tensors("left.k.norm"), a.dim, dp))
-        scaling = dict(a.rot_scaling) if a.rot_scaling else None
-        self.inv_freq = rotary_frequencies(a.rot_dims, a.rot_base, scaling).to(self.device)
+        self.rotary = (a.rot_dims, a.rot_base, a.rot_scaling)
+        self.inv_freq = rotary_frequencies(a.rot_dims, a.rot_base, dict(a.rot_scaling) if a.rot_scaling else None).to(self.device)
         self.attn = MixAttention("plain", a.heads, a.kv_heads, a.dim, a.vdim, a.scale, self.spec)
         self.attn.bind(device)
         self.scan = LinearScan("channel", g.heads, g.heads, g.dim, g.vdim, tensors("right.a2.b"), scale=g.dim ** -0.5, tau=g.tau,
@@ -257,14 +267,14 @@ class ParallelMixer(_Mixer):
         rv, rg = self.new(t, g.heads * g.vdim), self.new(t, g.heads * g.vdim)
         gate, low = self.new(t, a.heads, f32), self.new(t, self.rank, f32)
         self.proj(h, [q, k, vc, rq, rk, rv, rg, gate, low], [None, None, b.out_cache_loc] + [None] * 6)
-        qk_norm_rope(q, k, a.heads, a.kv_heads, a.dim, self.q_norm, self.k_norm, self.cfg.eps, self.inv_freq, b, kc)
+        if self.rotary not in c.tables:
+            c.tables[self.rotary] = rotary_table(self.inv_freq, b.positions)
+        qk_norm_rope(q, k, a.heads, a.kv_heads, a.dim, self.q_norm, self.k_norm, self.cfg.eps, c.tables[self.rotary], b, kc)
         o = self.attn.forward(q, kc, vc, c.req_to_token, b, c.counters, c.max_keys, gate)
-        left = self.new(t, self.cfg.width)
-        self.left_o(o, [left])
+        left = self.product(o, self.left_o)
         y = self.scan.forward(rq, rk, rv, low, c.caches.state[c.run], b, self.new(t, g.heads * g.vdim))
         group_norm(y, g.heads, g.vdim, self.head_norm, self.cfg.eps, rv, rg)
-        right = self.new(t, self.cfg.width)
-        self.right_o(rv, [right])
+        right = self.product(rv, self.right_o)
         return Pending(parts=[(left, self.left_out, 0.5), (right, self.right_out, 0.5)])
 
 
@@ -333,14 +343,14 @@ class KotipelLayer(_Mixer):
             h = update_norm(x, eps, self.new(t, cfg.width), self.norm2, pending=pending)
             act = self.new(t, self.ff_cols)
             self.gate_up(h, [act])
-            pending = Pending(gated_add(x, [(act, self.down_w, None)]))
+            copy = self.new(t, cfg.width) if self.side_embed is not None else None
+            pending = Pending(gated_add(x, [(act, self.down_w, None)], copy=copy))
         if self.side_embed is not None:
-            copy = update_norm(x, eps, self.new(t, cfg.width), pending=pending)
+            if self.layer.ff is None or not pending.empty:
+                copy = update_norm(x, eps, self.new(t, cfg.width), pending=pending)
             g = self.new(t, int(self.side_embed.shape[1]))
             self.side_gate(copy, [g], mul=(self.side_embed, c.batch.input_ids))
-            y = self.new(t, cfg.width)
-            self.side_proj(g, [y])
-            pending = Pending(parts=[(y, self.side_norm, 1.0)])
+            pending = Pending(parts=[(self.product(g, self.side_proj), self.side_norm, 1.0)])
         return pending
 
 
@@ -381,12 +391,12 @@ class KotipelForCausalLM:
         """``static_max_pos``: bound of the positions a captured step will ever see. ``on_layer(i, x)`` is called with the
         finished residual stream after every layer run (updates are then never left pending)."""
         x = embed(self.embed_table, self.cfg.width, batch, 1.0, req_to_token)
-        pending = Pending()
+        pending, tables = Pending(), {}
         for i, run in enumerate(self.runs):
             layer = self.layers[run.layer]
             keys = layer.spec.max_keys(static_max_pos) if static_max_pos is not None else None
             add = self.loop_step[run.step] if run.step is not None else None
-            pending = layer.forward(x, _Context(batch, caches, i, req_to_token, counters, keys), pending, add)
+            pending = layer.forward(x, _Context(batch, caches, i, req_to_token, counters, keys, tables), pending, add)
             if on_layer is not None:
                 if not pending.empty:
                     update_norm(x, self.cfg.eps, None, pending=pending)

@@ -12,7 +12,7 @@ from __future__ import annotations
 import ctypes
 import math
 from dataclasses import dataclass, field
-from typing import List, Optional, Sequence, Tuple
+from typing import List, Optional, Sequence, Tuple, Union
 
 import torch
 
@@ -133,9 +133,15 @@ class MergedProjection:
             if r.kind == "gelu_mul":
                 segs[i].mul, segs[i].ld_mul, segs[i].mul_map = ptr(mul[0]), mul[0].stride(0), ptr(mul[1])
             n0 += r.rows
-        w = self.weight
-        call("fr_dense_proj", dtype_code(w.dtype), ptr(a), a.stride(0), ptr(w), w.stride(0), int(a.shape[0]), n0,
-             int(w.shape[1]), segs, len(segs), algo, stream_ptr(a.device))
+        w, m, k = self.weight, int(a.shape[0]), int(self.weight.shape[1])
+        code, s = dtype_code(w.dtype), stream_ptr(a.device)
+        # a handful of tiles: their K extent is split over the SMs
+        n_splits = _lib.load().fr_dense_gated_add_splits(code, m, n0, k, 0) if algo == 0 and n0 <= 1024 else 0
+        if n_splits >= 4:
+            buf = torch.empty((n_splits, m, n0), dtype=torch.float32, device=a.device)
+            call("fr_dense_proj_split", code, ptr(a), a.stride(0), ptr(w), w.stride(0), m, n0, k, segs, len(segs), ptr(buf), n_splits, s)
+        else:
+            call("fr_dense_proj", code, ptr(a), a.stride(0), ptr(w), w.stride(0), m, n0, k, segs, len(segs), algo, s)
 
 
 @dataclass
@@ -147,9 +153,9 @@ class Partials:
 
 
 def gated_add(x: torch.Tensor, parts: Sequence[Tuple[torch.Tensor, torch.Tensor, Optional[torch.Tensor]]],
-              algo: int = 0, split: bool = True) -> Optional[Partials]:
+              algo: int = 0, split: bool = True, copy: Optional[torch.Tensor] = None) -> Optional[Partials]:
     """``x += sum gate * (a @ w.T)`` over one or two ``(a, w, gate)`` parts; few-row products may come back as
-    partials for the following ``rms_norm`` instead."""
+    partials for the following ``rms_norm`` instead. ``copy`` gets the new x in its own type (not with partials)."""
     require_cuda(x)
     m, n = int(x.shape[0]), int(x.shape[1])
     arr = (FrGatedPart * len(parts))()
@@ -160,8 +166,10 @@ def gated_add(x: torch.Tensor, parts: Sequence[Tuple[torch.Tensor, torch.Tensor,
     k = [int(p[1].shape[1]) for p in parts] + [0]
     n_splits = _lib.load().fr_dense_gated_add_splits(code, m, n, k[0], k[1]) if split and algo == 0 else 0
     buf = torch.empty((n_splits, m, n), dtype=torch.float32, device=x.device) if n_splits > 0 else None
-    call("fr_dense_gated_add", code, arr, len(parts), ptr(x), x.stride(0), m, n, ptr(buf), n_splits, algo,
-         stream_ptr(x.device))
+    if n_splits > 0:
+        copy = None
+    call("fr_dense_gated_add", code, arr, len(parts), ptr(x), x.stride(0), m, n, ptr(buf), n_splits, ptr(copy),
+         copy.stride(0) if copy is not None else 0, algo, stream_ptr(x.device))
     return Partials(buf, n_splits) if n_splits > 0 else None
 
 
@@ -178,13 +186,26 @@ def rms_norm(x: torch.Tensor, weight: torch.Tensor, offset: float, eps: float, o
     return out
 
 
+def split_product(a: torch.Tensor, w: torch.Tensor) -> Optional[Partials]:
+    """``a @ w.T`` as K shares when it has so few tiles that they would leave SMs idle, else None."""
+    require_cuda(a)
+    m, n, code = int(a.shape[0]), int(w.shape[0]), dtype_code(w.dtype)
+    n_splits = _lib.load().fr_dense_gated_add_splits(code, m, n, int(w.shape[1]), 0)
+    if n_splits < 2:
+        return None
+    buf = torch.empty((n_splits, m, n), dtype=torch.float32, device=a.device)
+    arr = (FrGatedPart * 1)(FrGatedPart(ptr(a), ptr(w), None, a.stride(0), w.stride(0), 0, int(w.shape[1]), 0))
+    call("fr_dense_gated_add", code, arr, 1, ptr(buf), n, m, n, ptr(buf), n_splits, None, 0, 0, stream_ptr(a.device))
+    return Partials(buf, n_splits)
+
+
 @dataclass
 class Pending:
-    """What still has to be added to the residual stream: K shares of a product, and vectors that are divided by their
-    root mean square, weighted and scaled, ``(y [M, W], weight [W], coefficient)``."""
+    """What still has to be added to the residual stream: K shares of a product, and vectors (also as K shares) that are
+    divided by their root mean square, weighted and scaled, ``(y [M, W], weight [W], coefficient)``."""
 
     partials: Optional[Partials] = None
-    parts: List[Tuple[torch.Tensor, torch.Tensor, float]] = field(default_factory=list)
+    parts: List[Tuple[Union[torch.Tensor, Partials], torch.Tensor, float]] = field(default_factory=list)
 
     @property
     def empty(self) -> bool:
@@ -198,7 +219,8 @@ def update_norm(x: torch.Tensor, eps: float, out: Optional[torch.Tensor], weight
     weight). With ``row_idx`` only those rows are read and the stream itself stays."""
     require_cuda(x)
     pending = pending or Pending()
-    dtype = out.dtype if out is not None else (pending.parts[0][0].dtype if pending.parts else torch.float32)
+    whole = [y for y, _, _ in pending.parts if isinstance(y, torch.Tensor)]
+    dtype = out.dtype if out is not None else (whole[0].dtype if whole else torch.float32)
     u = FrNormUpdate(dtype=dtype_code(dtype), n_parts=len(pending.parts), eps=eps, offset=offset, x=ptr(x), ldx=x.stride(0),
                      add=ptr(add), row_idx=ptr(row_idx), weight=ptr(weight), out=ptr(out),
                      ldo=out.stride(0) if out is not None else 0)
@@ -206,7 +228,10 @@ def update_norm(x: torch.Tensor, eps: float, out: Optional[torch.Tensor], weight
         u.n_partials, u.partials = pending.partials.n, ptr(pending.partials.buf)
         u.partial_stride = pending.partials.buf.stride(0)
     for i, (y, w, coef) in enumerate(pending.parts):
-        u.parts[i] = FrNormPart(ptr(y), y.stride(0), ptr(w), coef, 0)
+        if isinstance(y, Partials):
+            u.parts[i] = FrNormPart(ptr(y.buf), y.buf.stride(0), ptr(w), coef, y.n)
+        else:
+            u.parts[i] = FrNormPart(ptr(y), y.stride(0), ptr(w), coef, 0)
     m = int(x.shape[0]) if row_idx is None else int(row_idx.numel())
     call("fr_lm_update_norm", ctypes.byref(u), m, int(x.shape[1]), stream_ptr(x.device))
     return out
@@ -240,14 +265,23 @@ def rotary_frequencies(dims: int, base: float, scaling: Optional[dict] = None) -
     return torch.stack([hi, (f - hi.double()).float()], dim=1).contiguous()
 
 
+def rotary_table(inv_freq: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
+    """Cosines, then sines of ``positions * inv_freq`` per token: [T, 2 * pairs] for :func:`qk_norm_rope`."""
+    require_cuda(positions)
+    pairs, t = int(inv_freq.shape[0]), int(positions.numel())
+    table = torch.empty((t, 2 * pairs), dtype=torch.float32, device=positions.device)
+    call("fr_lm_rotary_table", ptr(inv_freq), pairs, ptr(positions), ptr(table), t, stream_ptr(positions.device))
+    return table
+
+
 def qk_norm_rope(q: torch.Tensor, k: torch.Tensor, heads: int, kv_heads: int, dim: int, q_weight: torch.Tensor,
-                 k_weight: torch.Tensor, eps: float, inv_freq: torch.Tensor, batch: ForwardBatch, k_cache: torch.Tensor) -> None:
-    """Norms over all heads at once and rotation by ``positions * inv_freq``; ``q`` in place, ``k`` into its cache slots.
+                 k_weight: torch.Tensor, eps: float, table: torch.Tensor, batch: ForwardBatch, k_cache: torch.Tensor) -> None:
+    """Norms over all heads at once and rotation by the angles of ``table``; ``q`` in place, ``k`` into its cache slots.
     Heads are padded as the weights are."""
     require_cuda(q, k, k_cache)
     a = FrQkRope(dtype=dtype_code(q.dtype), heads=heads, kv_heads=kv_heads, dim=int(q_weight.numel()) // heads, dim_true=dim,
-                 rot_dims=2 * int(inv_freq.shape[0]), eps=eps, q=ptr(q), ldq=q.stride(0), k=ptr(k), ldk=k.stride(0),
-                 q_weight=ptr(q_weight), k_weight=ptr(k_weight), inv_freq=ptr(inv_freq), pos=ptr(batch.positions),
+                 rot_dims=int(table.shape[1]), eps=eps, q=ptr(q), ldq=q.stride(0), k=ptr(k), ldk=k.stride(0),
+                 q_weight=ptr(q_weight), k_weight=ptr(k_weight), table=ptr(table),
                  loc=ptr(batch.out_cache_loc), k_cache=ptr(k_cache), ldkc=k_cache.stride(0))
     call("fr_lm_qk_norm_rope", ctypes.byref(a), int(q.shape[0]), stream_ptr(q.device))
 

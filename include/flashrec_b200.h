@@ -549,6 +549,11 @@ struct fr_out_segment {
 int fr_dense_proj(int dtype, const void* a, int64_t lda, const void* w, int64_t ldw, int M, int N, int K,
                   const struct fr_out_segment* segs, int n_segs, int algo, cudaStream_t stream);
 
+/* The same with the K extent split over CTAs, for few rows and columns: n_splits as returned by
+ * fr_dense_gated_add_splits(dtype, M, N, K, 0), partials [n_splits, M, N] f32 scratch. */
+int fr_dense_proj_split(int dtype, const void* a, int64_t lda, const void* w, int64_t ldw, int M, int N, int K,
+                        const struct fr_out_segment* segs, int n_segs, float* partials, int n_splits, cudaStream_t stream);
+
 /* One term of fr_dense_gated_add. */
 struct fr_gated_part {
   const void* a;   /* [M, K] */
@@ -562,9 +567,10 @@ struct fr_gated_part {
 /* x[m, n] += sum_p gate_p[m, n] * (a_p . w_p^T)[m, n], one or two parts. With `partials` (f32
  * [splits, M, N]) the K extent is split instead: partial s receives its share of the sum, x is left alone
  * and fr_lm_norm adds the partials in order. n_splits: 0 without partials; else as returned by
- * fr_dense_gated_add_splits for the same shape. */
+ * fr_dense_gated_add_splits for the same shape. copy (or null, without partials): the new x rounded to dtype as well;
+ * columns [N, ldc) are zeroed up to a multiple of 8. */
 int fr_dense_gated_add(int dtype, const struct fr_gated_part* parts, int n_parts, float* x, int64_t ldx, int M, int N,
-                       float* partials, int n_splits, int algo, cudaStream_t stream);
+                       float* partials, int n_splits, void* copy, int64_t ldc, int algo, cudaStream_t stream);
 int fr_dense_gated_add_splits(int dtype, int M, int N, int K0, int K1);
 
 /* x[t, :] = table[ids[t], :] * scale, and the slot table entry of the token: req_to_token[rows[t], pos[t]] = loc[t]
@@ -586,11 +592,11 @@ int fr_lm_norm(int dtype, float* x, int64_t ldx, const float* weight, float offs
  * x is written back unless row_idx picks rows. out may be null. Columns [W, ldo) of out are zeroed up to a multiple
  * of 8. */
 struct fr_norm_part {
-  const void* y;       /* [M, W] in dtype, pitch ldy */
-  int64_t ldy;
+  const void* y;       /* [M, W] in dtype, pitch ldy; with n_splits: f32 [n_splits, M, W] whose sum it is */
+  int64_t ldy;         /* with n_splits: elements of one share */
   const float* weight; /* [W] */
   float coef;
-  int32_t pad_;
+  int32_t n_splits;
 };
 struct fr_norm_update {
   int32_t dtype, n_parts, n_partials;
@@ -626,8 +632,12 @@ struct fr_group_norm {
 };
 int fr_lm_group_norm(const struct fr_group_norm* a, int M, cudaStream_t stream);
 
+/* table[m] = cos(pos[m] * f_i), i < pairs, then the sines. inv_freq [pairs, 2]: each frequency as a sum of two floats,
+ * larger one first. */
+int fr_lm_rotary_table(const float* inv_freq, int pairs, const int64_t* pos, float* table, int M, cudaStream_t stream);
+
 /* Norm of a token's queries (all heads at once) and keys, then rotation of the first rot_dims dimensions of every head
- * by pos * inv_freq (dimension i with i + rot_dims / 2). q [M, heads * dim] in place; k [M, kv_heads * dim] leaves
+ * by the angles of the token's table row (dimension i with i + rot_dims / 2). q [M, heads * dim] in place; k [M, kv_heads * dim] leaves
  * into row loc[m] of k_cache. Heads are laid out with `dim` columns of which dim_true count (the rest are zero). */
 struct fr_qk_rope {
   int32_t dtype, heads, kv_heads, dim, dim_true, rot_dims;
@@ -639,8 +649,7 @@ struct fr_qk_rope {
   int64_t ldk;
   const float* q_weight; /* [heads * dim] */
   const float* k_weight;
-  const float* inv_freq; /* [rot_dims / 2, 2]: each frequency as a sum of two floats, larger one first */
-  const int64_t* pos;
+  const float* table;    /* [M, rot_dims] */
   const int64_t* loc;
   void* k_cache;
   int64_t ldkc;

@@ -74,6 +74,7 @@ def test_update_and_norm(dtype, w):
     from flashrec_b200.lm_layers import Partials, Pending, ceil_to, update_norm
 
     m, eps = 9, 1e-2
+    shares = _rand(4, m, w, seed=12)
     x, wt, add = _rand(m, w, seed=1), _rand(w, seed=2), _rand(w, seed=3)
     pend = _rand(3, m, w, seed=4)
     ys = [torch.nn.functional.pad(_rand(m, w, seed=5 + i, scale=0.1 + i), (0, ceil_to(w, 8) - w)).to(dtype) for i in range(2)]
@@ -102,9 +103,38 @@ def test_update_and_norm(dtype, w):
         update_norm(xd, eps, None, pending=p, add=a)
         assert rel(xd, want) < 3e-6
         rows = torch.tensor([8, 0, 0, 5], device="cuda")
+        if n_parts == 2:  # one of the vectors as shares of a split product
+            p.parts[1] = (Partials(shares.cuda(), 4), p.parts[1][1], 1.0)
+            want = want + (O.rms(shares.double().sum(0), eps) - O.rms(ys[1][:, :w].double(), eps)) * wy[1].double()
         xd = x.cuda()
         update_norm(xd, eps, out[:4], wt.cuda(), 0.0, p, a, rows)
         assert torch.equal(xd.cpu(), x) and rel(out[:4, :w], (O.rms(want, eps) * wt.double())[rows.cpu()]) < tol(dtype)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("m", [1, 7, 8, 9, 40, 200, 1500])
+@pytest.mark.parametrize("n,k", [(90, 96), (130, 1040), (2048, 512)])
+def test_products_that_update_copy_or_come_in_shares(dtype, m, n, k):
+    from flashrec_b200.lm_layers import MergedProjection, ceil_to, gated_add, split_product
+
+    a, w = _rand(m, k, seed=1).to(dtype), _rand(n, k, seed=2, scale=k ** -0.5).to(dtype)
+    x = _rand(m, n, seed=3)
+    ref = a.double() @ w.double().t()
+    xd, copy = x.cuda(), torch.full((m, ceil_to(n, 8)), 7.0, dtype=dtype, device="cuda")
+    gated_add(xd, [(a.cuda(), w.cuda(), None)], split=False, copy=copy)
+    assert rel(xd, x.double() + ref) < 3e-6
+    assert torch.equal(copy[:, :n], xd.to(dtype)) and not copy[:, n:].any()
+    p = split_product(a.cuda(), w.cuda())
+    if p is not None:
+        assert p.buf.shape == (p.n, m, n) and rel(p.buf.sum(0), ref) < 3e-6
+    proj = MergedProjection(k)
+    proj.add("store", w[:n // 2])
+    proj.add("sigmoid", w[n // 2:], bias=torch.ones(n - n // 2))
+    proj.finish(dtype, "cuda")
+    outs = [torch.empty((m, ceil_to(c, 8)), dtype=dtype, device="cuda") for c in (n // 2, n - n // 2)]
+    proj(a.cuda(), outs)
+    assert rel(outs[0][:, :n // 2], ref[:, :n // 2]) < tol(dtype)
+    assert rel(outs[1][:, :n - n // 2], torch.sigmoid(ref[:, n // 2:] + 1)) < tol(dtype)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -130,7 +160,7 @@ def test_gated_group_norm(dtype, groups, size):
 @pytest.mark.parametrize("heads,kv,dim,rot", [(6, 2, 20, 12), (2, 2, 64, 64), (1, 1, 16, 2), (16, 4, 128, 96), (3, 1, 33, 0)])
 def test_norm_and_rotation_of_queries_and_keys(dtype, heads, kv, dim, rot):
     from flashrec_b200.core import ForwardBatch
-    from flashrec_b200.lm_layers import ceil_to, pad_heads, qk_norm_rope, rotary_frequencies
+    from flashrec_b200.lm_layers import ceil_to, pad_heads, qk_norm_rope, rotary_frequencies, rotary_table
 
     spec = dict(dims=rot, base=7000.0, scaling=dict(factor=8.0, low=1.0, high=4.0, original=128))
     pos = [0, 1, 17, 1000, 31337, 200000]
@@ -142,8 +172,9 @@ def test_norm_and_rotation_of_queries_and_keys(dtype, heads, kv, dim, rot):
     loc = torch.tensor([3, 19, 0, 7, 8, 11], device="cuda")
     qd = pad(q, heads).cuda()
     freqs = rotary_frequencies(rot, 7000.0, spec["scaling"]) if rot else torch.zeros((0, 2))
-    qk_norm_rope(qd, pad(k, kv).cuda(), heads, kv, dim, pad_heads(wq, dim, dp).cuda(), pad_heads(wk, dim, dp).cuda(), eps,
-                 freqs.cuda(), ForwardBatch(None, None, None, positions=torch.tensor(pos, device="cuda"), out_cache_loc=loc), cache)
+    table = rotary_table(freqs.cuda(), torch.tensor(pos, device="cuda"))
+    qk_norm_rope(qd, pad(k, kv).cuda(), heads, kv, dim, pad_heads(wq, dim, dp).cuda(), pad_heads(wk, dim, dp).cuda(), eps, table,
+                 ForwardBatch(None, None, None, out_cache_loc=loc), cache)
     fr = O.rotary_frequencies(spec) if rot else []
     for x, w, n, got in ((q, wq, heads, qd), (k, wk, kv, cache[loc])):
         ref = (O.rms(x.double(), eps) * w.double()).view(t, n, dim)
