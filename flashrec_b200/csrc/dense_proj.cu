@@ -813,13 +813,19 @@ static int launch_tc(const TcArgs& g, const fr_gated_part* parts, cudaStream_t s
                        status);
 }
 
-// Widest tile that still gives every SM one.
+// Tile width with the least work on the busiest SM: rounds of tiles times the rows of A and B that a tile brings in.
 static int pick_block_n(int M, int N) {
-  const int sms = device_sm_count();
-  const int mb = ceil_div(M, kBlockM);
-  if (static_cast<int64_t>(mb) * ceil_div(N, 256) >= sms) return 256;
-  if (static_cast<int64_t>(mb) * ceil_div(N, 128) >= sms) return 128;
-  return 64;
+  const int64_t sms = device_sm_count(), mb = ceil_div(M, kBlockM);
+  int best = 0;
+  int64_t best_cost = 0;
+  for (int bn = 256; bn >= 64; bn /= 2) {
+    const int64_t cost = (mb * ceil_div(N, bn) + sms - 1) / sms * (kBlockM + bn);
+    if (best == 0 || cost < best_cost) {
+      best = bn;
+      best_cost = cost;
+    }
+  }
+  return best;
 }
 
 static int rows_ks(int N, int K) {

@@ -441,8 +441,9 @@ __device__ __forceinline__ float cta_sum(float v, float* sums) {
   return tot;
 }
 
-// NV: float4 values per thread; 0: any width, re-reading what does not fit into registers
-template <typename T, int NV>
+// NV: float4 values per thread; 0: any width, re-reading what does not fit into registers. SHARES: parts may come as
+// shares of a split product
+template <typename T, int NV, bool SHARES>
 __global__ void __launch_bounds__(kNormThreads)
 update_norm_kernel(const __grid_constant__ fr_norm_update u, int W) {
   __shared__ float sums[4][kNormThreads / 32];
@@ -466,7 +467,7 @@ update_norm_kernel(const __grid_constant__ fr_norm_update u, int W) {
 #pragma unroll
       for (int p = 0; p < 2; ++p)
         if (p < u.n_parts) {
-          if (u.parts[p].n_splits == 0) {
+          if (!SHARES || u.parts[p].n_splits == 0) {
             y[p][i] = ld4<T>(static_cast<const T*>(u.parts[p].y) + src * u.parts[p].ldy + c);
           } else {
             for (int s = 0; s < u.parts[p].n_splits; ++s) {
@@ -573,8 +574,15 @@ static int launch_update_norm(const fr_norm_update& u, int M, int W, cudaStream_
              (u.n_partials == 0 || (aligned16(u.partials) && u.partial_stride % 4 == 0));
   for (int p = 0; p < u.n_parts; ++p)
     vec = vec && u.parts[p].ldy % 4 == 0 && aligned16(u.parts[p].y) && aligned16(u.parts[p].weight);
-  auto kern = update_norm_kernel<T, 0>;
-  if (vec) kern = W <= kNormThreads * 8 ? update_norm_kernel<T, 2> : (W <= kNormThreads * 16 ? update_norm_kernel<T, 4> : update_norm_kernel<T, 8>);
+  bool shares = false;
+  for (int p = 0; p < u.n_parts; ++p) shares = shares || u.parts[p].n_splits > 0;
+  auto kern = update_norm_kernel<T, 0, true>;
+  if (vec && shares)
+    kern = W <= kNormThreads * 8 ? update_norm_kernel<T, 2, true>
+                                 : (W <= kNormThreads * 16 ? update_norm_kernel<T, 4, true> : update_norm_kernel<T, 8, true>);
+  else if (vec)
+    kern = W <= kNormThreads * 8 ? update_norm_kernel<T, 2, false>
+                                 : (W <= kNormThreads * 16 ? update_norm_kernel<T, 4, false> : update_norm_kernel<T, 8, false>);
   return launch_kernel(kern, M, kNormThreads, 0, stream, M <= kPdlRows, u, W);
 }
 
@@ -683,8 +691,6 @@ static int launch_group_norm(const fr_group_norm& a, int M, cudaStream_t stream)
 // ---------------------------------------------------------------------------
 // queries and keys of one token: RMS norm over all heads at once, rotation, keys into the cache
 // ---------------------------------------------------------------------------
-constexpr int kRopeThreads = 256;
-
 __device__ __forceinline__ void ld8(const float* p, float (&v)[8]) {
   *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(p);
   *reinterpret_cast<float4*>(v + 4) = *reinterpret_cast<const float4*>(p + 4);
@@ -709,24 +715,25 @@ rotary_table_kernel(const float* __restrict__ inv_freq, int pairs, const int64_t
   table[t * 2 * pairs + pairs + i] = s * c1 + c * s1;
 }
 
+// One token per CTA, eight columns per thread and turn (one turn up to 8192 columns).
+constexpr int kRopeThreads = 1024;
 template <typename T>
 __global__ void __launch_bounds__(kRopeThreads)
 qk_norm_rope_kernel(const __grid_constant__ fr_qk_rope a) {
   extern __shared__ float sm[];
   __shared__ float sums[2][kRopeThreads / 32];
-  const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim, half = a.rot_dims / 2;
-  float* s_q = sm;
-  float* s_k = s_q + nq;
+  const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim, half = a.rot_dims / 2, nt = blockDim.x;
+  float* s_k = sm + nq;
   float* s_cos = s_k + nk;
   float* s_sin = s_cos + half;
   ptx::griddep_wait();
   ptx::griddep_launch_dependents();
   const int64_t t = blockIdx.x;
+  const int64_t slot = a.loc[t];
   T* q = static_cast<T*>(a.q) + t * a.ldq;
   const T* k = static_cast<const T*>(a.k) + t * a.ldk;
-  float sq = 0.f, sk = 0.f;
-  for (int c = threadIdx.x * 8; c < nq + nk; c += kRopeThreads * 8) {
-    float v[8];
+  float v[8], sq = 0.f, sk = 0.f;
+  for (int c = threadIdx.x * 8; c < nq + nk; c += nt * 8) {
     raw_unpack(raw_load<T>(c < nq ? q + c : k + (c - nq)), v);
     float ss = 0.f;
 #pragma unroll
@@ -735,28 +742,33 @@ qk_norm_rope_kernel(const __grid_constant__ fr_qk_rope a) {
     *reinterpret_cast<float4*>(sm + c) = make_float4(v[0], v[1], v[2], v[3]);
     *reinterpret_cast<float4*>(sm + c + 4) = make_float4(v[4], v[5], v[6], v[7]);
   }
-  for (int i = threadIdx.x; i < a.rot_dims; i += kRopeThreads) s_cos[i] = a.table[t * a.rot_dims + i];  // the sines follow
-  sq = cta_sum<kRopeThreads>(sq, sums[0]);
-  sk = cta_sum<kRopeThreads>(sk, sums[1]);
-  const float rq = 1.0f / sqrtf(sq / static_cast<float>(a.heads * a.dim_true) + a.eps);
-  const float rk = 1.0f / sqrtf(sk / static_cast<float>(a.kv_heads * a.dim_true) + a.eps);
-  T* kc = static_cast<T*>(a.k_cache) + a.loc[t] * a.ldkc;
-  for (int c = threadIdx.x * 8; c < nq + nk; c += kRopeThreads * 8) {
+  for (int i = threadIdx.x; i < a.rot_dims; i += nt) s_cos[i] = a.table[t * a.rot_dims + i];  // the sines follow
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if ((threadIdx.x & 31) == 0) {
+    sums[0][threadIdx.x >> 5] = sq;
+    sums[1][threadIdx.x >> 5] = sk;
+  }
+  __syncthreads();
+  T* kc = static_cast<T*>(a.k_cache) + slot * a.ldkc;
+  for (int c = threadIdx.x * 8; c < nq + nk; c += nt * 8) {
     const bool is_q = c < nq;
-    const float* src = is_q ? s_q : s_k;
+    const float* src = is_q ? sm : s_k;
     const float* w = is_q ? a.q_weight : a.k_weight;
     const int b = is_q ? c : c - nq, d0 = b % a.dim;
-    const float rr = is_q ? rq : rk;
-    float v[8];
+    float tot = 0.f;
+    for (int i = 0; i < nt / 32; ++i) tot += sums[is_q ? 0 : 1][i];
+    const float rr = 1.0f / sqrtf(tot / static_cast<float>((is_q ? a.heads : a.kv_heads) * a.dim_true) + a.eps);
+    if (nt * 8 < nq + nk) ld8(sm + c, v);  // else the values of the one turn are still here
+    float w8[8];
+    ld8(w + b, w8);
     if (d0 >= a.rot_dims || half % 8 == 0) {  // eight dimensions turn with eight others, or none does
-      float w8[8], i8[8];
-      ld8(src + b, v);
-      ld8(w + b, w8);
 #pragma unroll
       for (int e = 0; e < 8; ++e) v[e] *= rr * w8[e];
       if (d0 < a.rot_dims) {
-        const int pair = d0 < half ? d0 : d0 - half, other = d0 < half ? b + half : b - half;
-        float c8[8], s8[8];
+        const bool low = d0 < half;
+        const int pair = low ? d0 : d0 - half, other = low ? b + half : b - half;
+        float i8[8], c8[8], s8[8];
         ld8(src + other, i8);
         ld8(w + other, w8);
         ld8(s_cos + pair, c8);
@@ -764,21 +776,20 @@ qk_norm_rope_kernel(const __grid_constant__ fr_qk_rope a) {
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
           const float it = i8[e] * rr * w8[e];
-          v[e] = d0 < half ? v[e] * c8[e] - it * s8[e] : v[e] * c8[e] + it * s8[e];
+          v[e] = low ? v[e] * c8[e] - it * s8[e] : v[e] * c8[e] + it * s8[e];
         }
       }
-      conv_store8<T>(is_q ? q + b : kc + b, v);
-      continue;
-    }
+    } else {
 #pragma unroll
-    for (int e = 0; e < 8; ++e) {
-      const int d = d0 + e;
-      const float me = src[b + e] * rr * w[b + e];
-      v[e] = me;
-      if (d < a.rot_dims) {
-        const int pair = d < half ? d : d - half, other = d < half ? b + e + half : b + e - half;
-        const float it = src[other] * rr * w[other];
-        v[e] = d < half ? me * s_cos[pair] - it * s_sin[pair] : me * s_cos[pair] + it * s_sin[pair];
+      for (int e = 0; e < 8; ++e) {
+        const int d = d0 + e;
+        const float me = v[e] * rr * w8[e];
+        v[e] = me;
+        if (d < a.rot_dims) {
+          const int pair = d < half ? d : d - half, other = d < half ? b + e + half : b + e - half;
+          const float it = src[other] * rr * w[other];
+          v[e] = d < half ? me * s_cos[pair] - it * s_sin[pair] : me * s_cos[pair] + it * s_sin[pair];
+        }
       }
     }
     conv_store8<T>(is_q ? q + b : kc + b, v);
@@ -874,11 +885,12 @@ extern "C" int fr_lm_qk_norm_rope(const fr_qk_rope* a, int M, cudaStream_t strea
   FR_CHECK_ARG(aligned16(a->q) && aligned16(a->k) && aligned16(a->k_cache) && aligned16(a->q_weight) && aligned16(a->k_weight) && a->ldq % 8 == 0 && a->ldk % 8 == 0 && a->ldkc % 8 == 0);
   const int smem = ((a->heads + a->kv_heads) * a->dim + a->rot_dims) * 4;
   FR_CHECK_SUPPORTED(smem <= 200 * 1024);
+  const int vecs = (a->heads + a->kv_heads) * a->dim / 8, threads = vecs >= lm::kRopeThreads ? lm::kRopeThreads : (vecs + 31) / 32 * 32;
   static PerDeviceFlag f0, f1;
   if (a->dtype == 0) {
     if (ensure_dyn_smem(f0, lm::qk_norm_rope_kernel<__nv_bfloat16>, 200 * 1024) != FR_OK) return FR_ERR_CUDA;
-    return launch_kernel(lm::qk_norm_rope_kernel<__nv_bfloat16>, M, lm::kRopeThreads, smem, stream, M <= kPdlRows, *a);
+    return launch_kernel(lm::qk_norm_rope_kernel<__nv_bfloat16>, M, threads, smem, stream, M <= kPdlRows, *a);
   }
   if (ensure_dyn_smem(f1, lm::qk_norm_rope_kernel<float>, 200 * 1024) != FR_OK) return FR_ERR_CUDA;
-  return launch_kernel(lm::qk_norm_rope_kernel<float>, M, lm::kRopeThreads, smem, stream, M <= kPdlRows, *a);
+  return launch_kernel(lm::qk_norm_rope_kernel<float>, M, threads, smem, stream, M <= kPdlRows, *a);
 }
