@@ -369,6 +369,7 @@ constexpr int kTcBarBytes = 288 + kPageList * 4;
 
 struct TcPlan {
   int q_boxes, v_boxes;   // 64-column boxes of a q / k row and of a v row
+  int q_bufs;             // Q tiles in shared memory: the next map's is loaded ahead, PLAIN has one map
   int v_cols;             // TMEM columns of O and of one accumulator
   int n_out;              // outputs per CTA (PLAIN: 1, which needs no accumulator)
   int out_blocks;         // CTAs along y per v head (TALK) or per head (DIFF)
@@ -385,6 +386,7 @@ static bool plan_tc(int mix, int heads, int kv_heads, int dim, int vdim, TcPlan*
   pl->v_boxes = (vdim + 63) / 64;
   pl->v_cols = (vdim + 31) / 32 * 32;
   pl->staged = 0;
+  pl->q_bufs = mix == FR_MIX_PLAIN ? 1 : 2;
   int fit = (512 - 2 * kTileN - pl->v_cols) / pl->v_cols;
   if (fit < 1) return false;
   if (fit > kMaxOut) fit = kMaxOut;
@@ -399,7 +401,7 @@ static bool plan_tc(int mix, int heads, int kv_heads, int dim, int vdim, TcPlan*
   }
   pl->tmem_cols = need <= 256 ? 256 : 512;
   for (pl->stages = 4;; --pl->stages) {
-    pl->smem = 1024 + 2 * pl->q_boxes * kM * 128 + pl->stages * (pl->q_boxes + pl->v_boxes) * kTileN * 128 + kTcBarBytes;
+    pl->smem = 1024 + pl->q_bufs * pl->q_boxes * kM * 128 + pl->stages * (pl->q_boxes + pl->v_boxes) * kTileN * 128 + kTcBarBytes;
     pl->extra = pl->staged && kM * pl->v_cols * 2 > pl->q_boxes * kM * 128 ? kM * pl->v_cols * 2 - pl->q_boxes * kM * 128 : 0;
     pl->smem += pl->extra;
     if (pl->stages == 2 || pl->smem <= (pl->tmem_cols == 256 ? 112 : 227) * 1024) break;
@@ -419,8 +421,8 @@ mix_tc_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
   uint8_t* smem = smem_raw + (base - raw);
   const int q_bytes = pl.q_boxes * kM * 128, k_bytes = pl.q_boxes * kTileN * 128, v_bytes = pl.v_boxes * kTileN * 128;
   const int n_st = pl.stages;
-  const uint32_t sm_q = base + pl.extra, sm_k = sm_q + 2 * q_bytes, sm_v = sm_k + n_st * k_bytes;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + pl.extra + 2 * q_bytes + n_st * (k_bytes + v_bytes));
+  const uint32_t sm_q = base + pl.extra, sm_k = sm_q + pl.q_bufs * q_bytes, sm_v = sm_k + n_st * k_bytes;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + pl.extra + pl.q_bufs * q_bytes + n_st * (k_bytes + v_bytes));
   const uint32_t bar0 = ptx::smem_u32(bars);
   const uint32_t bar_qfull = bar0, bar_qempty = bar0 + 16;    // [2] each
   const uint32_t bar_sfull = bar0 + 32;                       // [2]

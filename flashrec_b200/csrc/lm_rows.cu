@@ -441,12 +441,19 @@ __device__ __forceinline__ float cta_sum(float v, float* sums) {
   return tot;
 }
 
-// NV: float4 values per thread; 0: any width, re-reading what does not fit into registers. SHARES: parts may come as
-// shares of a split product
-template <typename T, int NV, bool SHARES>
-__global__ void __launch_bounds__(kNormThreads)
+// 1 / sqrt(mean + eps); the 16-bit results leave through the hardware's reciprocal root
+template <typename T>
+__device__ __forceinline__ float inv_rms(float sum, float inv_n, int n, float eps) {
+  return sizeof(T) == 2 ? rsqrtf(fmaf(sum, inv_n, eps)) : 1.0f / sqrtf(sum / static_cast<float>(n) + eps);
+}
+
+// NT threads with NV float4 values each; NV 0: any width, re-reading what does not fit into registers. NP: parts at most;
+// SHARES: they may come as shares of a split product
+template <typename T, int NT, int NV, int NP, bool SHARES>
+__global__ void __launch_bounds__(NT)
 update_norm_kernel(const __grid_constant__ fr_norm_update u, int W) {
-  __shared__ float sums[4][kNormThreads / 32];
+  __shared__ float sums[3][NT / 32];
+  const float inv_w = 1.0f / static_cast<float>(W);
   ptx::griddep_wait();
   ptx::griddep_launch_dependents();
   const int64_t t = blockIdx.x;
@@ -456,16 +463,19 @@ update_norm_kernel(const __grid_constant__ fr_norm_update u, int W) {
   const float* pr = u.n_partials > 0 ? u.partials + src * W : nullptr;
   const bool write_x = u.row_idx == nullptr && (pr != nullptr || u.n_parts > 0 || u.add != nullptr);
   if constexpr (NV > 0) {
-    float4 v[NV], y[2][NV];
-    float ss[2] = {0.f, 0.f};
+    constexpr int kP = NP > 0 ? NP : 1;
+    float4 v[NV], y[kP][NV];
+    float ss[kP] = {};
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-      const int c = (i * kNormThreads + threadIdx.x) * 4;
-      v[i] = y[0][i] = y[1][i] = make_float4(0, 0, 0, 0);
+      const int c = (i * NT + threadIdx.x) * 4;
+      v[i] = make_float4(0, 0, 0, 0);
+#pragma unroll
+      for (int p = 0; p < NP; ++p) y[p][i] = v[i];
       if (c >= W) continue;
       v[i] = *reinterpret_cast<const float4*>(xr + c);
 #pragma unroll
-      for (int p = 0; p < 2; ++p)
+      for (int p = 0; p < NP; ++p)
         if (p < u.n_parts) {
           if (!SHARES || u.parts[p].n_splits == 0) {
             y[p][i] = ld4<T>(static_cast<const T*>(u.parts[p].y) + src * u.parts[p].ldy + c);
@@ -483,18 +493,18 @@ update_norm_kernel(const __grid_constant__ fr_norm_update u, int W) {
           v[i].x += q.x; v[i].y += q.y; v[i].z += q.z; v[i].w += q.w;
         }
     }
-    float r[2] = {0.f, 0.f};
+    float r[kP] = {};
 #pragma unroll
-    for (int p = 0; p < 2; ++p)
+    for (int p = 0; p < NP; ++p)
       if (p < u.n_parts)
-        r[p] = u.parts[p].coef / sqrtf(cta_sum<kNormThreads>(ss[p], sums[p]) / static_cast<float>(W) + u.eps);
+        r[p] = u.parts[p].coef * inv_rms<T>(cta_sum<NT>(ss[p], sums[p]), inv_w, W, u.eps);
     float sx = 0.f;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-      const int c = (i * kNormThreads + threadIdx.x) * 4;
+      const int c = (i * NT + threadIdx.x) * 4;
       if (c >= W) continue;
 #pragma unroll
-      for (int p = 0; p < 2; ++p)
+      for (int p = 0; p < NP; ++p)
         if (p < u.n_parts) {
           const float4 w = *reinterpret_cast<const float4*>(u.parts[p].weight + c);
           v[i].x += y[p][i].x * r[p] * w.x; v[i].y += y[p][i].y * r[p] * w.y;
@@ -509,10 +519,10 @@ update_norm_kernel(const __grid_constant__ fr_norm_update u, int W) {
     }
     if (u.out == nullptr) return;
     float rx = 1.0f;
-    if (u.weight != nullptr) rx = 1.0f / sqrtf(cta_sum<kNormThreads>(sx, sums[2]) / static_cast<float>(W) + u.eps);
+    if (u.weight != nullptr) rx = inv_rms<T>(cta_sum<NT>(sx, sums[2]), inv_w, W, u.eps);
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-      const int c = (i * kNormThreads + threadIdx.x) * 4;
+      const int c = (i * NT + threadIdx.x) * 4;
       if (c >= W) continue;
       float4 w = make_float4(1, 1, 1, 1);
       if (u.weight != nullptr) {
@@ -532,11 +542,11 @@ update_norm_kernel(const __grid_constant__ fr_norm_update u, int W) {
     };
     for (int p = 0; p < u.n_parts; ++p) {
       float ss = 0.f;
-      for (int c = threadIdx.x; c < W; c += kNormThreads) {
+      for (int c = threadIdx.x; c < W; c += NT) {
         const float f = part(p, c);
         ss += f * f;
       }
-      r[p] = u.parts[p].coef / sqrtf(cta_sum<kNormThreads>(ss, sums[p]) / static_cast<float>(W) + u.eps);
+      r[p] = u.parts[p].coef * inv_rms<T>(cta_sum<NT>(ss, sums[p]), inv_w, W, u.eps);
     }
     auto value = [&](int c) {
       float f = xr[c];
@@ -550,13 +560,13 @@ update_norm_kernel(const __grid_constant__ fr_norm_update u, int W) {
     float rx = 1.0f;
     if (u.weight != nullptr && u.out != nullptr) {
       float sx = 0.f;
-      for (int c = threadIdx.x; c < W; c += kNormThreads) {
+      for (int c = threadIdx.x; c < W; c += NT) {
         const float f = value(c);
         sx += f * f;
       }
-      rx = 1.0f / sqrtf(cta_sum<kNormThreads>(sx, sums[2]) / static_cast<float>(W) + u.eps);
+      rx = inv_rms<T>(cta_sum<NT>(sx, sums[2]), inv_w, W, u.eps);
     }
-    for (int c = threadIdx.x; c < W; c += kNormThreads) {  // a thread writes what only it reads
+    for (int c = threadIdx.x; c < W; c += NT) {  // a thread writes what only it reads
       const float f = value(c);
       if (write_x) xr[c] = f;
       if (u.out != nullptr) st_f(o + c, u.weight != nullptr ? f * rx * (u.offset + u.weight[c]) : f);
@@ -564,26 +574,33 @@ update_norm_kernel(const __grid_constant__ fr_norm_update u, int W) {
   }
   if (u.out == nullptr) return;
   const int wpad = (W + 7) / 8 * 8;
-  for (int c = W + threadIdx.x; c < wpad && c < u.ldo; c += kNormThreads) st_f(o + c, 0.f);
+  for (int c = W + threadIdx.x; c < wpad && c < u.ldo; c += NT) st_f(o + c, 0.f);
+}
+
+template <typename T, int NP, bool SHARES>
+static int launch_update_norm_vec(const fr_norm_update& u, int M, int W, cudaStream_t stream) {
+  const bool pdl = M <= kPdlRows;
+  if (W <= 512) return launch_kernel(update_norm_kernel<T, 128, 1, NP, SHARES>, M, 128, 0, stream, pdl, u, W);
+  // few rows: latency; two parts: registers
+  if ((pdl || NP > 0) && W <= 2048) return launch_kernel(update_norm_kernel<T, 256, 2, NP, SHARES>, M, 256, 0, stream, pdl, u, W);
+  if (W <= 2048) return launch_kernel(update_norm_kernel<T, 128, 4, NP, SHARES>, M, 128, 0, stream, pdl, u, W);
+  if (NP > 0 && W <= 4096) return launch_kernel(update_norm_kernel<T, 512, 2, NP, SHARES>, M, 512, 0, stream, pdl, u, W);
+  if (W <= 4096) return launch_kernel(update_norm_kernel<T, 256, 4, NP, SHARES>, M, 256, 0, stream, pdl, u, W);
+  return launch_kernel(update_norm_kernel<T, 512, 4, NP, SHARES>, M, 512, 0, stream, pdl, u, W);
 }
 
 template <typename T>
 static int launch_update_norm(const fr_norm_update& u, int M, int W, cudaStream_t stream) {
-  bool vec = W % 4 == 0 && W <= kNormThreads * 4 * kNormVec && u.ldx % 4 == 0 && aligned16(u.x) && aligned16(u.weight) &&
-             aligned16(u.add) && u.ldo % 4 == 0 && aligned16(u.out) &&
-             (u.n_partials == 0 || (aligned16(u.partials) && u.partial_stride % 4 == 0));
-  for (int p = 0; p < u.n_parts; ++p)
-    vec = vec && u.parts[p].ldy % 4 == 0 && aligned16(u.parts[p].y) && aligned16(u.parts[p].weight);
+  bool vec = W % 4 == 0 && W <= 8192 && u.ldx % 4 == 0 && aligned16(u.x) && aligned16(u.weight) && aligned16(u.add) &&
+             u.ldo % 4 == 0 && aligned16(u.out) && (u.n_partials == 0 || (aligned16(u.partials) && u.partial_stride % 4 == 0));
   bool shares = false;
-  for (int p = 0; p < u.n_parts; ++p) shares = shares || u.parts[p].n_splits > 0;
-  auto kern = update_norm_kernel<T, 0, true>;
-  if (vec && shares)
-    kern = W <= kNormThreads * 8 ? update_norm_kernel<T, 2, true>
-                                 : (W <= kNormThreads * 16 ? update_norm_kernel<T, 4, true> : update_norm_kernel<T, 8, true>);
-  else if (vec)
-    kern = W <= kNormThreads * 8 ? update_norm_kernel<T, 2, false>
-                                 : (W <= kNormThreads * 16 ? update_norm_kernel<T, 4, false> : update_norm_kernel<T, 8, false>);
-  return launch_kernel(kern, M, kNormThreads, 0, stream, M <= kPdlRows, u, W);
+  for (int p = 0; p < u.n_parts; ++p) {
+    vec = vec && u.parts[p].ldy % 4 == 0 && aligned16(u.parts[p].y) && aligned16(u.parts[p].weight);
+    shares = shares || u.parts[p].n_splits > 0;
+  }
+  if (vec && u.n_parts == 0) return launch_update_norm_vec<T, 0, false>(u, M, W, stream);
+  if (vec) return shares ? launch_update_norm_vec<T, 2, true>(u, M, W, stream) : launch_update_norm_vec<T, 2, false>(u, M, W, stream);
+  return launch_kernel(update_norm_kernel<T, kNormThreads, 0, 2, true>, M, kNormThreads, 0, stream, M <= kPdlRows, u, W);
 }
 
 // ---------------------------------------------------------------------------
@@ -715,7 +732,83 @@ rotary_table_kernel(const float* __restrict__ inv_freq, int pairs, const int64_t
   table[t * 2 * pairs + pairs + i] = s * c1 + c * s1;
 }
 
-// One token per CTA, eight columns per thread and turn (one turn up to 8192 columns).
+// A thread owns sixteen columns of one head, eight that turn with the other eight (or sixteen that do not), keeps their
+// weights in registers and walks kRopeTokens tokens. rot_dims is a multiple of 16.
+constexpr int kRopeTokens = 8;
+template <typename T>
+__global__ void __launch_bounds__(1024)
+qk_norm_rope_units_kernel(const __grid_constant__ fr_qk_rope a, int M, int n_tokens) {
+  __shared__ float sums[2][2][32];
+  const int per_head = a.dim / 16, n_q = a.heads * per_head, n_units = (a.heads + a.kv_heads) * per_head;
+  const int half = a.rot_dims / 2, tid = threadIdx.x, warp = tid >> 5, warps = blockDim.x >> 5;
+  const bool live = tid < n_units, is_q = tid < n_q;
+  const int u = live ? (is_q ? tid : tid - n_q) : 0, head = u / per_head, x = u % per_head;
+  const bool turns = x < half / 8;
+  const int c0 = turns ? x * 8 : a.rot_dims + (x - half / 8) * 16, c1 = turns ? half + x * 8 : c0 + 8;
+  float w0[8], w1[8];
+  const float* w = (is_q ? a.q_weight : a.k_weight) + head * a.dim;
+  ld8(w + c0, w0);
+  ld8(w + c1, w1);
+  ptx::griddep_wait();
+  ptx::griddep_launch_dependents();
+  const int64_t t0 = static_cast<int64_t>(blockIdx.x) * n_tokens, t1 = t0 + n_tokens < M ? t0 + n_tokens : M;
+  T* q = static_cast<T*>(a.q) + head * a.dim;
+  const T* k = static_cast<const T*>(a.k) + head * a.dim;
+  T* kc = static_cast<T*>(a.k_cache) + head * a.dim;
+  // which sums a warp adds to, and what reads them: first and last unit of the warp
+  const bool any_q = warp * 32 < n_q, any_k = warp * 32 + 31 >= n_q;
+  const float inv_nq = 1.0f / static_cast<float>(a.heads * a.dim_true), inv_nk = 1.0f / static_cast<float>(a.kv_heads * a.dim_true);
+  Raw8<T> r0 = raw_zero<T>(), r1 = r0;
+  auto fetch = [&](int64_t t) {
+    if (!live) return;
+    const T* src = is_q ? q + t * a.ldq : k + t * a.ldk;
+    r0 = raw_load<T>(src + c0);
+    r1 = raw_load<T>(src + c1);
+  };
+  fetch(t0);
+  for (int64_t t = t0; t < t1; ++t) {
+    float v0[8], v1[8];
+    raw_unpack(r0, v0);
+    raw_unpack(r1, v1);
+    if (t + 1 < t1) fetch(t + 1);
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss = fmaf(v0[e], v0[e], fmaf(v1[e], v1[e], ss));
+    float (&s)[2][32] = sums[t & 1];
+    if (any_q) {
+      const float z = warp_sum(live && is_q ? ss : 0.f);
+      if ((tid & 31) == 0) s[0][warp] = z;
+    }
+    if (any_k) {
+      const float z = warp_sum(live && !is_q ? ss : 0.f);
+      if ((tid & 31) == 0) s[1][warp] = z;
+    }
+    float cs[8], sn[8];
+    if (live && turns) {
+      ld8(a.table + t * a.rot_dims + c0, cs);
+      ld8(a.table + t * a.rot_dims + half + c0, sn);
+    }
+    __syncthreads();
+    if (!live) continue;
+    float tot = 0.f;
+    if (is_q)
+      for (int i = 0; i * 32 < n_q; ++i) tot += s[0][i];
+    else
+      for (int i = n_q / 32; i < warps; ++i) tot += s[1][i];
+    const float rr = inv_rms<T>(tot, is_q ? inv_nq : inv_nk, (is_q ? a.heads : a.kv_heads) * a.dim_true, a.eps);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      const float y0 = v0[e] * rr * w0[e], y1 = v1[e] * rr * w1[e];
+      v0[e] = turns ? y0 * cs[e] - y1 * sn[e] : y0;
+      v1[e] = turns ? y1 * cs[e] + y0 * sn[e] : y1;
+    }
+    T* dst = is_q ? q + t * a.ldq : kc + a.loc[t] * a.ldkc;
+    conv_store8<T>(dst + c0, v0);
+    conv_store8<T>(dst + c1, v1);
+  }
+}
+
+// Any rotation: one token per CTA, eight columns per thread and turn.
 constexpr int kRopeThreads = 1024;
 template <typename T>
 __global__ void __launch_bounds__(kRopeThreads)
@@ -883,6 +976,12 @@ extern "C" int fr_lm_qk_norm_rope(const fr_qk_rope* a, int M, cudaStream_t strea
   FR_CHECK_ARG(a->dim_true > 0 && a->dim_true <= a->dim && a->rot_dims >= 0 && a->rot_dims % 2 == 0 && a->rot_dims <= a->dim_true);
   FR_CHECK_ARG(a->q && a->k && a->k_cache && a->q_weight && a->k_weight && a->loc && (a->rot_dims == 0 || a->table));
   FR_CHECK_ARG(aligned16(a->q) && aligned16(a->k) && aligned16(a->k_cache) && aligned16(a->q_weight) && aligned16(a->k_weight) && a->ldq % 8 == 0 && a->ldk % 8 == 0 && a->ldkc % 8 == 0);
+  const int units = (a->heads + a->kv_heads) * a->dim / 16;
+  if (a->dim % 16 == 0 && a->rot_dims % 16 == 0 && units <= 1024 && aligned16(a->table)) {
+    const int n = M > 148 * 16 ? lm::kRopeTokens : 1, threads = (units + 31) / 32 * 32;  // a few rows: a CTA each
+    auto kern = a->dtype == 0 ? lm::qk_norm_rope_units_kernel<__nv_bfloat16> : lm::qk_norm_rope_units_kernel<float>;
+    return launch_kernel(kern, ceil_div(M, n), threads, 0, stream, M <= kPdlRows, *a, M, n);
+  }
   const int smem = ((a->heads + a->kv_heads) * a->dim + a->rot_dims) * 4;
   FR_CHECK_SUPPORTED(smem <= 200 * 1024);
   const int vecs = (a->heads + a->kv_heads) * a->dim / 8, threads = vecs >= lm::kRopeThreads ? lm::kRopeThreads : (vecs + 31) / 32 * 32;
