@@ -217,7 +217,7 @@ _SIGNATURES = {
     "fr_linear_scan_rows": [P, _I, _I, _I, P],
     "fr_linear_scan_chunks": [P, _I, _I, _I, _I, P, _L, P],
     "fr_linear_scan_chunks_scratch": [P, _I, _I, _I],
-    "fr_linear_scan_chunks_fit": [_I, _I, _I],
+    "fr_linear_scan_chunks_fit": [P],
     "fr_short_conv": [_I, P, _L, P, P, _I, _I, _I, P, _I, P, P, P, P, P, _I, _I, _I, P],
     "fr_mix_attn_rows": [P, _I, _I, _I, _I, P, _L, P, P],
     "fr_mix_attn_rows_scratch": [_I] * 6,

@@ -73,7 +73,8 @@ __device__ __forceinline__ float softplus_log2(float z) {
 // Factors of one chunk and head.
 struct HeadFactors {
   float r[kChunk];    // r_i (log2)
-  float c[kChunk];    // log2(step_j) - r_j
+  float l[kChunk];    // r_i counted from the block of 32 tokens that i is in
+  float c[kChunk];    // log2(step_j) - l_j
   float x[kChunk];    // step_j e^(r_last - r_j)
   float y[kChunk];    // step_j e^(r_e - r_j), e the last of j's block of 32 tokens
   float first, end;   // a_0, e^(r_last)
@@ -141,17 +142,26 @@ head_factor_kernel(const __grid_constant__ ChunkArgs g) {
     if (lane >= o) x += y;
   }
   const float last = __shfl_sync(0xffffffffu, x, 31);
-  float r = x - sum, fr[4], fc[4], fx[4], fy[4];
-  const float block_end = __shfl_sync(0xffffffffu, x, lane | 7);
+  float z = sum;  // the same within a block: differences of nearby tokens keep their digits however strong the decay
+#pragma unroll
+  for (int o = 1; o < 8; o *= 2) {
+    const float y = __shfl_up_sync(0xffffffffu, z, o);
+    if ((lane & 7) >= o) z += y;
+  }
+  const float block_end = __shfl_sync(0xffffffffu, z, lane | 7);
+  float r = x - sum, l = z - sum, fr[4], fl[4], fc[4], fx[4], fy[4];
 #pragma unroll
   for (int e = 0; e < 4; ++e) {
     r += la[e];
+    l += la[e];
     fr[e] = r;
-    fc[e] = log2f(step[e]) - r;  // -inf past the end: no weight
+    fl[e] = l;
+    fc[e] = log2f(step[e]) - l;  // -inf past the end: no weight
     fx[e] = step[e] * ex2(last - r);
-    fy[e] = step[e] * ex2(block_end - r);
+    fy[e] = step[e] * ex2(block_end - l);
   }
   *reinterpret_cast<float4*>(f->r + lane * 4) = make_float4(fr[0], fr[1], fr[2], fr[3]);
+  *reinterpret_cast<float4*>(f->l + lane * 4) = make_float4(fl[0], fl[1], fl[2], fl[3]);
   *reinterpret_cast<float4*>(f->c + lane * 4) = make_float4(fc[0], fc[1], fc[2], fc[3]);
   *reinterpret_cast<float4*>(f->x + lane * 4) = make_float4(fx[0], fx[1], fx[2], fx[3]);
   *reinterpret_cast<float4*>(f->y + lane * 4) = make_float4(fy[0], fy[1], fy[2], fy[3]);
@@ -597,7 +607,7 @@ chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ Chu
             uint32_t gv[32];
             ptx::tmem_ld_32x32(col_p + lane_off + quarter * 32, gv);
             float ri = 0.f;
-            if constexpr (!CHANNEL) ri = f->r[row];
+            if constexpr (!CHANNEL) ri = f->l[row];
             ptx::tmem_ld_wait();
 #pragma unroll
             for (int c4 = 0; c4 < 8; ++c4) {
@@ -730,8 +740,11 @@ chunk_kernel(const __grid_constant__ ChunkMaps maps, const __grid_constant__ Chu
 }
 
 // ---------------------------------------------------------------------------
+static int channel_smem(const fr_linear_scan& a) { return (kChunk * (a.dim + a.rank) + 2 * kPrepThreads + a.rank * a.dim) * 4; }
+
 static bool plan_chunks(const fr_linear_scan& a, int n_req, int longest, ChunkPlan* pl) {
   if (a.dim % 16 != 0 || a.vdim % 16 != 0 || a.dim > kChunk) return false;
+  if (a.decay == FR_DECAY_CHANNEL && channel_smem(a) > 200 * 1024) return false;
   const bool channel = a.decay == FR_DECAY_CHANNEL;
   pl->boxes = (a.dim + 63) / 64;
   pl->v_blocks = ceil_div(a.vdim, kVb);
@@ -797,8 +810,7 @@ static int run_chunks(const ChunkArgs& g, int n_req, int longest, int n_tokens, 
   const bool pdl = n_tokens <= kPdlRows;
   const int chunks = ceil_div(longest, kChunk);
   if (CHANNEL) {
-    const int smem = (kChunk * (a.dim + a.rank) + 2 * kPrepThreads + a.rank * a.dim) * 4;
-    FR_CHECK_SUPPORTED(smem <= 200 * 1024);
+    const int smem = channel_smem(a);
     static PerDeviceFlag f;
     if (ensure_dyn_smem(f, channel_factor_kernel, 200 * 1024) != FR_OK) return FR_ERR_CUDA;
     if (cudaMemsetAsync(g.flags, 0, static_cast<size_t>(n_req) * a.heads * 4, stream) != cudaSuccess) return FR_ERR_CUDA;
@@ -815,14 +827,9 @@ static int run_chunks(const ChunkArgs& g, int n_req, int longest, int n_tokens, 
 
 using namespace fr;
 
-extern "C" int fr_linear_scan_chunks_fit(int decay, int dim, int vdim) {
-  fr_linear_scan a{};
-  a.decay = decay;
-  a.heads = 1;
-  a.dim = dim;
-  a.vdim = vdim;
+extern "C" int fr_linear_scan_chunks_fit(const fr_linear_scan* a) {
   scan::ChunkPlan pl;
-  return dim > 0 && vdim > 0 && scan::plan_chunks(a, 1, 1, &pl) ? 1 : 0;
+  return a != nullptr && a->heads > 0 && a->dim > 0 && a->vdim > 0 && scan::plan_chunks(*a, 1, 1, &pl) ? 1 : 0;
 }
 
 extern "C" int64_t fr_linear_scan_chunks_scratch(const fr_linear_scan* a, int n_req, int longest, int n_tokens) {

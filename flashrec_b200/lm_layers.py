@@ -435,7 +435,7 @@ class LinearScan:
         longest = 1 if batch.one_token else max(batch.extend_seq_lens)
         lib = _lib.load()
         if self._chunks is None:
-            self._chunks = bool(lib.fr_linear_scan_chunks_fit(a.decay, a.dim, a.vdim))
+            self._chunks = bool(lib.fr_linear_scan_chunks_fit(ctypes.byref(a)))
         row_portion = longest
         if self._chunks and a.dtype == 0 and longest > ROW_PORTION:
             row_portion = ROW_PORTION

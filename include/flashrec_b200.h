@@ -766,7 +766,7 @@ int fr_linear_scan_rows(const struct fr_linear_scan* a, int n_req, int max_token
 int fr_linear_scan_chunks(const struct fr_linear_scan* a, int n_req, int longest, int n_tokens, int min_tokens, void* scratch,
                           int64_t scratch_bytes, cudaStream_t stream);
 int64_t fr_linear_scan_chunks_scratch(const struct fr_linear_scan* a, int n_req, int longest, int n_tokens);
-int fr_linear_scan_chunks_fit(int decay, int dim, int vdim);
+int fr_linear_scan_chunks_fit(const struct fr_linear_scan* a);
 
 #ifdef __cplusplus
 }

@@ -289,7 +289,7 @@ SCANS = [  # decay, heads, key heads, dim, vdim, strength of the decays
     ("channel", 3, 3, 18, 22, 0.05), ("channel", 2, 2, 64, 64, 0.05), ("channel", 1, 1, 128, 128, 0.02), ("channel", 2, 2, 128, 64, 4.0),
     ("channel", 2, 2, 16, 16, 0.5), ("channel", 1, 1, 200, 96, 0.1), ("channel", 3, 3, 32, 256, 0.7),
     ("head", 6, 2, 12, 10, 0.2), ("head", 4, 1, 128, 64, 0.05), ("head", 4, 4, 64, 128, 1.0), ("head", 2, 1, 16, 16, 5.0),
-    ("head", 3, 1, 256, 40, 0.1), ("head", 2, 2, 128, 128, 0.01),
+    ("head", 3, 1, 256, 40, 0.1), ("head", 2, 2, 128, 128, 0.01), ("head", 4, 2, 64, 64, 60.0), ("channel", 3, 3, 32, 48, 1.2),
 ]
 
 
