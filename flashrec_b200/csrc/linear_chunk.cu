@@ -40,7 +40,8 @@ constexpr int kBox = kChunk * 128;     // bytes of a [128 x 64] bf16 tile
 constexpr int kCompute = 512;          // threads of the compute warps
 constexpr int kThreads = kCompute + 64;
 constexpr float kLog2e = 1.4426950408889634f;
-// largest -r_last (in powers of two) per channel: e^(+-r_last / 2), its products and their sums stay far inside 2^+-126
+// largest -r_last (in powers of two) per channel: e^(+-r_last / 2), the products of visible pairs and the state's sums stay
+// far inside 2^+-126 (scores of later keys may not: they are replaced, not multiplied, by zero)
 constexpr float kMaxChannel = 160.f;
 
 __device__ __forceinline__ float ex2(float x) {
